@@ -3,13 +3,14 @@
 Run: python hologram_b200/build.py [--force] [--verbose]   (by path: importing the package needs the built library)
 """
 import os
+import re
 import subprocess
 import sys
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libhologram_b200.so")
-SOURCES = ["api.cu", "lut.cu", "glue.cu", "attention.cu", "gemm.cu", "quant_gemv.cu", "tp.cu", "session.cu", "addressed.cpp", "pool.cpp", "archive.cpp", "blake3.cpp", "label.cpp"]
+SOURCES = ["api.cu", "lut.cu", "glue.cu", "attention.cu", "gemm.cu", "linear.cu", "causal_attention.cu", "quant_gemv.cu", "tp.cu", "session.cu", "addressed.cpp", "pool.cpp", "archive.cpp", "blake3.cpp", "label.cpp"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fno-fast-math", "--expt-relaxed-constexpr",
@@ -24,11 +25,16 @@ def _nvcc():
 
 
 def _deps(src):
-    deps = [src]
-    for name in os.listdir(CSRC):
-        if name.endswith((".h", ".cuh")):
-            deps.append(os.path.join(CSRC, name))
-    deps.append(os.path.join(HERE, "..", "include", "hologram_b200.h"))
+    """`src` and the headers it includes, directly or through other headers."""
+    deps, todo = [], [src]
+    while todo:
+        path = todo.pop()
+        if path in deps or not os.path.exists(path):
+            continue
+        deps.append(path)
+        with open(path, encoding="utf-8") as f:
+            names = re.findall(r'^#include "([^"]+)"', f.read(), re.M)
+        todo += [os.path.normpath(os.path.join(os.path.dirname(path), n)) for n in names]
     return deps
 
 

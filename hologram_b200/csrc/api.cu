@@ -928,6 +928,121 @@ int32_t do_attention_q8(holo_b200_ctx* ctx, const HoloDecodeAttentionValidQ8Call
     return holo_launch_decode_attention(ctx, a);
 }
 
+float f32_of_bits(uint32_t bits) {
+    float f;
+    memcpy(&f, &bits, 4);
+    return f;
+}
+
+// Extension: f32 rows normalised under one or two weights.
+int32_t do_rms_norm_multi(holo_b200_ctx* ctx, const HoloRmsNormMultiCall& c, holo_b200_workspace* ws) {
+    if (c.rows == 0 || c.feature == 0) return HOLO_OK;
+    if (c.dtype != HOLO_DTYPE_F32 && c.dtype != HOLO_DTYPE_BF16)
+        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: rms_norm_multi output dtype %u", c.dtype);
+    if (c.step < c.feature) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: rms_norm_multi step %u below feature %u", c.step, c.feature);
+    const float eps = f32_of_bits(c.epsilon_bits);
+    if (!(isfinite(eps) && eps > 0.0f)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: norm epsilon must be a positive finite f32");
+    const bool two = c.gamma1.slot != HOLO_NO_SLOT;
+    const uint64_t xb = (uint64_t)c.rows * c.feature * 4, gb = (uint64_t)c.feature * 4;
+    const uint64_t ob = (uint64_t)c.rows * c.step * (two ? 2 : 1) * holo_dtype_size(c.dtype);
+    uint8_t *x, *g0, *g1 = nullptr, *out;
+    HOLO_TRY(holo_resolve(ws, c.x, xb, &x, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.gamma0, gb, &g0, nullptr));
+    if (two) HOLO_TRY(holo_resolve(ws, c.gamma1, gb, &g1, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.output, ob, &out, nullptr));
+    HOLO_TRY(check_disjoint({out, ob}, c.output.slot, {{x, xb}, {g0, gb}, {g1, g1 ? gb : 0}}));
+    if ((((uintptr_t)x | (uintptr_t)g0 | (uintptr_t)g1 | (uintptr_t)out) & 3u) != 0) return holo_fail_slot(c.output.slot, "rms_norm_multi operands must be 4-byte aligned");
+    return holo_launch_rms_norm_multi(ctx, (const float*)x, (const float*)g0, (const float*)g1, out, c.rows, c.feature, c.step, eps, c.dtype);
+}
+
+// Extension: a product with up to four output segments.
+int32_t do_linear(holo_b200_ctx* ctx, const HoloLinearCall& c, holo_b200_workspace* ws) {
+    if (c.nseg < 1 || c.nseg > HOLO_LINEAR_MAX_SEGS) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear segment count %u", c.nseg);
+    if (c.m == 0 || c.k == 0 || c.n == 0) return HOLO_OK;
+    if (c.dtype != HOLO_DTYPE_F32 && c.dtype != HOLO_DTYPE_BF16) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear dtype %u", c.dtype);
+    const uint64_t es = holo_dtype_size(c.dtype);
+    HoloLinearArgs a = {};
+    uint8_t *pa, *pb, *ptr;
+    const uint64_t ab = ((uint64_t)(c.m - 1) * c.lda + c.lda) * es, bb = (uint64_t)c.k * c.n * es;
+    HOLO_TRY(holo_resolve(ws, c.a, ab, &pa, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.b, bb, &pb, nullptr));
+    const bool with_res = c.residual.slot != HOLO_NO_SLOT;
+    if (with_res && (c.nseg != 1 || c.seg[0].dtype != HOLO_DTYPE_F32))
+        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: a linear residual needs a single f32 segment");
+    for (uint32_t i = 0; i < c.nseg; ++i) {
+        const HoloLinearSeg& g = c.seg[i];
+        if (g.dtype != HOLO_DTYPE_F32 && g.dtype != HOLO_DTYPE_BF16) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear output dtype %u", g.dtype);
+        if (g.act > HOLO_LINEAR_ACT_RELU2) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear activation %u", g.act);
+        const uint32_t prev_end = i ? c.seg[i - 1].col_begin + c.seg[i - 1].width : 0;
+        if (g.width == 0 || g.col_begin % 32 != 0 || g.col_begin < prev_end || (uint64_t)g.col_begin + g.width > c.n || g.ld < g.width ||
+            (uint64_t)g.k_offset + c.k > c.lda || (i == 0 && g.col_begin != 0) ||
+            (i > 0 && g.k_offset != c.seg[i - 1].k_offset && g.col_begin % 256 != 0))
+            return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: linear segment %u (columns %u + %u of %u, k offset %u, pitch %u)", i, g.col_begin, g.width, c.n, g.k_offset, g.ld);
+        const uint64_t os = holo_dtype_size(g.dtype);
+        // with a row offset the rows land somewhere in a buffer of whole rows; the kernel drops rows past its end
+        const bool appends = g.row_pos.slot != HOLO_NO_SLOT;
+        const uint64_t ob = (appends ? g.width : (uint64_t)(c.m - 1) * g.ld + g.width) * os;
+        uint64_t extent = 0;
+        HOLO_TRY(holo_resolve(ws, g.output, ob, &ptr, &extent));
+        HOLO_TRY(check_disjoint({ptr, appends ? extent : ob}, g.output.slot, {{pa, ab}, {pb, bb}}));
+        if (((uintptr_t)ptr & (os - 1)) != 0) return holo_fail_slot(g.output.slot, "linear output must be aligned to its element");
+        HoloLinearSegArgs& o = a.seg[i];
+        o.out = ptr;
+        o.row_pos = nullptr;
+        if (appends) {
+            HOLO_TRY(holo_resolve(ws, g.row_pos, 4, &ptr, nullptr));
+            if (((uintptr_t)ptr & 3u) != 0) return holo_fail_slot(g.row_pos.slot, "row_pos operand must be 4-byte aligned on the device");
+            o.row_pos = (const uint32_t*)ptr;
+        }
+        o.row_limit = appends ? extent / ((uint64_t)g.ld * os) : c.m;
+        o.col_begin = g.col_begin; o.width = g.width; o.k_offset = g.k_offset; o.ld = g.ld; o.act = g.act; o.dtype = g.dtype;
+        if (with_res) {
+            HOLO_TRY(holo_resolve(ws, c.residual, ob, &ptr, nullptr));
+            if (((uintptr_t)ptr & 3u) != 0) return holo_fail_slot(c.residual.slot, "linear residual must be 4-byte aligned");
+            a.residual = (const float*)ptr;
+        }
+    }
+    a.a = pa; a.b = pb;
+    a.m = c.m; a.k = c.k; a.n = c.n; a.lda = c.lda; a.nseg = c.nseg;
+    a.alpha = f32_of_bits(c.alpha_bits);
+    a.dtype = c.dtype;
+    a.b_constant = c.b.slot < ws->slots.size() && ws->slots[c.b.slot].constant;
+    return holo_launch_linear(ctx, a);
+}
+
+// Extension: causal attention of new rows over the cache that already holds them.
+int32_t do_causal_attention(holo_b200_ctx* ctx, const HoloCausalAttentionCall& c, holo_b200_workspace* ws) {
+    if (c.rows == 0 || c.heads == 0) return HOLO_OK;
+    if (c.dtype != HOLO_DTYPE_F32 && c.dtype != HOLO_DTYPE_BF16) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: causal_attention dtype %u", c.dtype);
+    if (c.kv_heads == 0 || c.heads % c.kv_heads != 0)
+        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: causal_attention: heads must be a multiple of kv_heads (grouped-query)");
+    if (c.dim == 0 || c.vdim == 0 || c.dim > 512 || c.vdim > 512 || c.ld < c.heads * c.vdim || c.cache_rows == 0)
+        return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: causal_attention dim %u vdim %u pitch %u", c.dim, c.vdim, c.ld);
+    const uint64_t es = holo_dtype_size(c.dtype);
+    const uint64_t qb = (uint64_t)c.rows * c.heads * c.dim * es, kb = (uint64_t)c.cache_rows * c.kv_heads * c.dim * es;
+    const uint64_t vb = (uint64_t)c.cache_rows * c.kv_heads * c.vdim * es, ob = ((uint64_t)(c.rows - 1) * c.ld + c.heads * c.vdim) * es;
+    uint8_t *q, *k, *v, *pos, *sink = nullptr, *out;
+    HOLO_TRY(holo_resolve(ws, c.q, qb, &q, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.k, kb, &k, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.v, vb, &v, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.pos, 4, &pos, nullptr));
+    if (c.sink.slot != HOLO_NO_SLOT) HOLO_TRY(holo_resolve(ws, c.sink, (uint64_t)c.heads * 4, &sink, nullptr));
+    HOLO_TRY(holo_resolve(ws, c.output, ob, &out, nullptr));
+    HOLO_TRY(check_disjoint({out, ob}, c.output.slot, {{q, qb}, {k, kb}, {v, vb}, {pos, 4}, {sink, sink ? (uint64_t)c.heads * 4 : 0}}));
+    if ((((uintptr_t)pos | (uintptr_t)sink) & 3u) != 0) return holo_fail_slot(c.pos.slot, "pos and sink operands must be 4-byte aligned on the device");
+    HoloCausalArgs a = {};
+    a.q = q; a.k = k; a.v = v; a.pos = (const uint32_t*)pos; a.sink = (const float*)sink; a.out = out;
+    a.rows = c.rows; a.heads = c.heads; a.kv_heads = c.kv_heads; a.dim = c.dim; a.vdim = c.vdim; a.cache_rows = c.cache_rows; a.ld = c.ld;
+    a.scale = c.scale_bits ? f32_of_bits(c.scale_bits) : 1.0f / sqrtf((float)c.dim);
+    a.softcap = f32_of_bits(c.softcap_bits);
+    a.temp_coef = f32_of_bits(c.temp_coef_bits);
+    a.temp_every = f32_of_bits(c.temp_every_bits);
+    if (!(a.softcap >= 0.0f) || !(a.temp_every >= 0.0f))
+        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: causal_attention: softcap and temp_every must not be negative");
+    a.dtype = c.dtype;
+    return holo_launch_causal_attention(ctx, a);
+}
+
 int32_t do_all_reduce(holo_b200_ctx* ctx, const HoloAllReduceCall& c, holo_b200_workspace* ws) {
     size_t es = holo_dtype_size(c.dtype);
     if (c.dtype != HOLO_DTYPE_F32 && c.dtype != HOLO_DTYPE_BF16 && c.dtype != HOLO_DTYPE_F16)
@@ -985,6 +1100,9 @@ int32_t holo_dispatch_internal(holo_b200_ctx* ctx, const HoloKernelCall* call, h
         case HOLO_K_DECODE_ATTENTION_VALID_Q8: return do_attention_q8(ctx, call->u.decode_attention_valid_q8, ws);
         case HOLO_K_ALL_REDUCE: return do_all_reduce(ctx, call->u.all_reduce, ws);
         case HOLO_K_ROPE_QUANTIZE_ROWS_I8: return do_rope_quantize(ctx, call->u.rope_quantize, ws);
+        case HOLO_K_RMS_NORM_MULTI: return do_rms_norm_multi(ctx, call->u.rms_norm_multi, ws);
+        case HOLO_K_LINEAR: return do_linear(ctx, call->u.linear, ws);
+        case HOLO_K_CAUSAL_ATTENTION: return do_causal_attention(ctx, call->u.causal_attention, ws);
         default:
             if (holo_is_exact_unary(call->kind) || holo_is_exact_binary(call->kind)) return do_elementwise(ctx, call, ws);
             return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: KernelCall variant %u is not served by the B200 backend (no CPU fallback)", call->kind);
@@ -1155,6 +1273,28 @@ bool holo_collect_refs(HoloKernelCall* c, HoloRefList* l) {
             l->out(&q.scales, q.rows * 4);
             return true;
         }
+        case HOLO_K_RMS_NORM_MULTI: {
+            auto& q = c->u.rms_norm_multi;
+            l->in(&q.x); l->in(&q.gamma0); l->in(&q.gamma1);
+            l->out(&q.output, (uint64_t)q.rows * q.step * (q.gamma1.slot != HOLO_NO_SLOT ? 2 : 1) * holo_dtype_size(q.dtype));
+            return true;
+        }
+        case HOLO_K_LINEAR: {
+            auto& q = c->u.linear;
+            l->in(&q.a); l->in(&q.b); l->in(&q.residual);
+            for (uint32_t i = 0; i < q.nseg && i < HOLO_LINEAR_MAX_SEGS; ++i) {
+                l->in(&q.seg[i].row_pos);
+                const uint64_t rows = q.seg[i].row_pos.slot != HOLO_NO_SLOT ? 1 : q.m;   // an appending segment: the rows the buffer has
+                l->out(&q.seg[i].output, ((rows - 1) * q.seg[i].ld + q.seg[i].width) * holo_dtype_size(q.seg[i].dtype));
+            }
+            return true;
+        }
+        case HOLO_K_CAUSAL_ATTENTION: {
+            auto& q = c->u.causal_attention;
+            l->in(&q.q); l->in(&q.k); l->in(&q.v); l->in(&q.pos); l->in(&q.sink);
+            l->out(&q.output, ((uint64_t)(q.rows - 1) * q.ld + q.heads * q.vdim) * holo_dtype_size(q.dtype));
+            return true;
+        }
         case HOLO_K_MATMUL_DEQUANT_PLAIN: case HOLO_K_MATMUL_DEQUANT: case HOLO_K_MATMUL_DEQUANT_CODEBOOK: {
             auto& q = c->u.matmul_dequant;
             l->in(&q.a); l->in(&q.bq); l->in(&q.scales); l->in(&q.zero_points); l->in(&q.residual);
@@ -1176,7 +1316,10 @@ extern "C" int32_t holo_b200_dispatch_host(holo_b200_ctx* ctx, const HoloKernelC
     HOLO_CUDA(cudaSetDevice(ctx->device));
     HoloKernelCall local = *call;
     HoloRefList refs;
-    if (!holo_collect_refs(&local, &refs))
+    bool appends = false;   // rows of a cache at a device-side position: only a device-resident buffer has them
+    if (call->kind == HOLO_K_LINEAR)
+        for (uint32_t i = 0; i < call->u.linear.nseg && i < HOLO_LINEAR_MAX_SEGS; ++i) appends |= call->u.linear.seg[i].row_pos.slot != HOLO_NO_SLOT;
+    if (appends || !holo_collect_refs(&local, &refs))
         return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: KernelCall variant %u has no host-workspace form", call->kind);
     // Each referenced host range gets a 256-byte aligned range of one device arena; the call
     // is rewritten to index a temporary device workspace with one slot per operand. Inputs

@@ -217,6 +217,34 @@ int32_t decode_call(Reader& r, HoloKernelCall* out) {
             c.rows = r.u64(); c.row_len = r.u32(); c.dtype = r.u8();
             break;
         }
+        case HOLO_K_RMS_NORM_MULTI: {
+            HoloRmsNormMultiCall& c = out->u.rms_norm_multi;
+            c.x = r.buf(); c.gamma0 = r.buf(); c.gamma1 = r.buf(); c.output = r.buf();
+            c.rows = r.u32(); c.feature = r.u32(); c.step = r.u32(); c.epsilon_bits = r.u32(); c.dtype = r.u8();
+            break;
+        }
+        case HOLO_K_LINEAR: {
+            HoloLinearCall& c = out->u.linear;
+            c.a = r.buf(); c.b = r.buf(); c.residual = r.buf();
+            c.m = r.u32(); c.k = r.u32(); c.n = r.u32(); c.lda = r.u32(); c.alpha_bits = r.u32(); c.dtype = r.u8();
+            c.nseg = r.u8();
+            if (c.nseg < 1 || c.nseg > HOLO_LINEAR_MAX_SEGS || c.m == 0)
+                return holo_fail(HOLO_ERR_INIT, "backend init failed: linear call with %u segments over %u rows", c.nseg, c.m);
+            for (uint32_t i = 0; i < c.nseg; ++i) {
+                HoloLinearSeg& g = c.seg[i];
+                g.output = r.buf(); g.row_pos = r.buf();
+                g.col_begin = r.u32(); g.width = r.u32(); g.k_offset = r.u32(); g.ld = r.u32(); g.act = r.u8(); g.dtype = r.u8();
+            }
+            break;
+        }
+        case HOLO_K_CAUSAL_ATTENTION: {
+            HoloCausalAttentionCall& c = out->u.causal_attention;
+            c.q = r.buf(); c.k = r.buf(); c.v = r.buf(); c.pos = r.buf(); c.sink = r.buf(); c.output = r.buf();
+            c.rows = r.u32(); c.heads = r.u32(); c.kv_heads = r.u32(); c.dim = r.u32(); c.vdim = r.u32(); c.cache_rows = r.u32(); c.ld = r.u32();
+            c.scale_bits = r.u32(); c.softcap_bits = r.u32(); c.temp_coef_bits = r.u32(); c.temp_every_bits = r.u32(); c.dtype = r.u8();
+            if (c.rows == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: causal attention over no rows");
+            break;
+        }
         case HOLO_K_ALL_REDUCE: {
             HoloAllReduceCall& c = out->u.all_reduce;
             c.buffer = r.buf(); c.element_count = r.u64(); c.dtype = r.u8();

@@ -100,7 +100,7 @@ static inline bool holo_is_compute_float(uint8_t d) {
 // Every BufferRef of a call; `out_bytes` > 0 marks a written operand and gives the number of
 // bytes the kernel produces there (inputs carry 0).
 struct HoloRefList {
-    HoloBufferRef* refs[12];
+    HoloBufferRef* refs[12];      // the widest call is Linear: a, b, residual, four (output, row_pos) pairs
     uint64_t out_bytes[12];
     bool written[12];
     int n = 0;
@@ -264,6 +264,37 @@ int32_t holo_launch_matmul_add_activation(holo_b200_ctx* ctx, const void* a, con
                                           uint8_t dtype, uint8_t fused_act, const void* residual);
 int32_t holo_launch_matmul_multi(holo_b200_ctx* ctx, const void* a, const void* b, uint32_t m, uint32_t k, uint32_t n,
                                  uint8_t dtype, const HoloMatmulSeg* segs, uint32_t nseg);
+// linear.cu
+struct HoloLinearSegArgs {
+    void* out;
+    const uint32_t* row_pos;
+    uint32_t col_begin, width, k_offset, ld;
+    uint64_t row_limit;          // rows the output buffer has: rows at or past it are not stored
+    uint8_t act, dtype;
+};
+struct HoloLinearArgs {
+    const void *a, *b;
+    const float* residual;
+    HoloLinearSegArgs seg[HOLO_LINEAR_MAX_SEGS];
+    uint32_t m, k, n, lda, nseg;
+    float alpha;
+    uint8_t dtype;
+    bool b_constant;
+};
+int32_t holo_launch_linear(holo_b200_ctx* ctx, const HoloLinearArgs& a);
+int32_t holo_launch_rms_norm_multi(holo_b200_ctx* ctx, const float* x, const float* gamma0, const float* gamma1, void* out, uint32_t rows,
+                                   uint32_t feature, uint32_t step, float eps, uint8_t dtype);
+// causal_attention.cu
+struct HoloCausalArgs {
+    const void *q, *k, *v;
+    const uint32_t* pos;
+    const float* sink;           // null = no sink
+    void* out;
+    uint32_t rows, heads, kv_heads, dim, vdim, cache_rows, ld;
+    float scale, softcap, temp_coef, temp_every;   // softcap 0 = no cap, temp_every 0 = no temperature
+    uint8_t dtype;
+};
+int32_t holo_launch_causal_attention(holo_b200_ctx* ctx, const HoloCausalArgs& a);
 // quant_gemv.cu
 int32_t holo_launch_matmul_e8cb_omajor(holo_b200_ctx* ctx, const float* a, const uint8_t* bq, const int8_t* codebook, const float* scales,
                                        const int32_t* zero_points, const float* residual, float* out, uint32_t m, uint32_t k, uint32_t n, int act);

@@ -716,8 +716,31 @@ extern "C" int32_t holo_b200_session_load(holo_b200_ctx* ctx, const uint8_t* arc
     return holo_session_load_impl(ctx, archive, len, verify, nullptr, 0, out);
 }
 
+extern "C" int32_t holo_b200_session_load_shared(holo_b200_ctx* ctx, const uint8_t* archive, uint64_t len, int32_t verify,
+                                                 holo_b200_session* donor, holo_b200_session** out) {
+    if (!donor || donor->ctx != ctx) return holo_fail(HOLO_ERR_INIT, "backend init failed: the donor session belongs to another context");
+    if (donor->addressed || (verify & HOLO_SESSION_ADDRESSED)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: addressed sessions do not share their buffers");
+    return holo_session_load_impl(ctx, archive, len, verify, nullptr, 0, out, donor);
+}
+
+namespace {
+
+// The donor's device copy of a weight (null when it does not have one, or has merged it away).
+void* donor_weight(const holo_b200_session* donor, const uint8_t fingerprint[32], uint64_t* len) {
+    for (const HoloConstant& k : donor->ar.constants) {
+        if (!k.by_reference || memcmp(k.fingerprint, fingerprint, 32) != 0) continue;
+        if (k.slot < donor->ws->slots.size() && donor->ws->slots[k.slot].ptr) {
+            *len = k.len;
+            return donor->ws->slots[k.slot].ptr;
+        }
+    }
+    return nullptr;
+}
+
+}  // namespace
+
 int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint64_t len, int32_t verify, const HoloWeightProvider* provider,
-                               uint64_t budget, holo_b200_session** out) {
+                               uint64_t budget, holo_b200_session** out, holo_b200_session* donor) {
     if (!ctx || !archive || !out) return holo_fail(HOLO_ERR_INIT, "backend init failed: null argument");
     HOLO_CUDA(cudaSetDevice(ctx->device));
     holo_b200_session* s = new holo_b200_session();
@@ -728,7 +751,7 @@ int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint6
         s->ad.provider = *provider;
         s->ad.paged = true;
     }
-    int32_t rc = holo_archive_parse(archive, len, (verify & HOLO_SESSION_VERIFY) != 0, &s->ar, provider != nullptr);
+    int32_t rc = holo_archive_parse(archive, len, (verify & HOLO_SESSION_VERIFY) != 0, &s->ar, provider != nullptr || donor != nullptr);
     if (rc != HOLO_OK) {
         delete s;
         return rc;
@@ -747,9 +770,29 @@ int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint6
     std::set<uint32_t> in_slots, out_slots;
     for (const HoloPort& p : s->ar.inputs) in_slots.insert(p.slot);
     for (const HoloPort& p : s->ar.outputs) out_slots.insert(p.slot);
+    if (s->addressed) {
+        // the labels of an addressed walk do not see rows written into a resident cache
+        for (const HoloKernelCall& c : s->calls)
+            if (c.kind == HOLO_K_LINEAR)
+                for (uint32_t i = 0; i < c.u.linear.nseg; ++i)
+                    if (c.u.linear.seg[i].row_pos.slot != HOLO_NO_SLOT) {
+                        delete s;
+                        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: an addressed session cannot append to a cache in place");
+                    }
+    }
+    // weights the donor holds: slot -> its device copy
+    std::unordered_map<uint32_t, std::pair<void*, uint64_t>> borrowed;
+    if (donor)
+        for (HoloConstant& k : s->ar.constants) {
+            uint64_t n = 0;
+            void* ptr = k.by_reference ? donor_weight(donor, k.fingerprint, &n) : nullptr;
+            if (!ptr) continue;
+            k.len = n;
+            borrowed[k.slot] = {ptr, n};
+        }
     // a paged weight's length comes from the provider (session.rs:587-600)
     for (HoloConstant& k : s->ar.constants) {
-        if (k.bytes || !k.by_reference) continue;
+        if (k.bytes || !k.by_reference || borrowed.count(k.slot)) continue;
         const int64_t sz = provider && provider->size ? provider->size(provider->user, k.fingerprint) : -1;
         if (sz < 0) {
             delete s;
@@ -838,9 +881,22 @@ int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint6
             else no_static[k.slot] = 0;
         }
     }
+    if (donor)
+        for (const HoloPort& p : s->ar.inputs) {
+            if (borrowed.count(p.slot) || alias[p.slot] >= 0) continue;
+            for (const HoloPort& d : donor->ar.inputs)
+                if (d.name == p.name && d.dtype == p.dtype && d.element_count == p.element_count && donor->ws->slots[d.slot].bytes >= need[p.slot])
+                    borrowed[p.slot] = {donor->ws->slots[d.slot].ptr, donor->ws->slots[d.slot].bytes};
+        }
     rc = holo_b200_workspace_create(ctx, n_slots, &s->ws);
     for (uint32_t i = 0; rc == HOLO_OK && i < n_slots; ++i) {
         if (alias[i] >= 0 || no_static[i]) continue;
+        auto b = borrowed.find(i);
+        if (b != borrowed.end()) {
+            rc = b->second.second < need[i] ? holo_fail_slot(i, "a shared buffer is smaller than this archive needs")
+                                            : holo_b200_workspace_bind(s->ws, i, b->second.first, b->second.second);
+            continue;
+        }
         uint64_t bytes = std::max<uint64_t>(need[i], 64);
         bytes = (bytes + 63) & ~63ull;
         rc = holo_b200_workspace_alloc(s->ws, i, bytes);
@@ -855,7 +911,7 @@ int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint6
     }
     for (size_t i = 0; rc == HOLO_OK && i < s->ar.constants.size(); ++i) {
         const HoloConstant& k = s->ar.constants[i];
-        if (lazy_slot[k.slot]) continue;   // paged in on first use
+        if (lazy_slot[k.slot] || borrowed.count(k.slot)) continue;   // paged in on first use; the donor's copy
         const uint8_t* body = k.bytes;
         if (!body && provider && provider->get_range) body = (const uint8_t*)provider->get_range(provider->user, k.fingerprint, 0, k.len);
         if (!body && k.len) {

@@ -103,7 +103,7 @@ struct holo_b200_session {
 
 // session.cu
 int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint64_t len, int32_t verify, const HoloWeightProvider* provider,
-                               uint64_t budget, holo_b200_session** out);
+                               uint64_t budget, holo_b200_session** out, holo_b200_session* donor = nullptr);
 // addressed.cpp
 int32_t holo_addressed_prepare(holo_b200_session* s, const std::vector<uint64_t>& slot_need);
 void holo_addressed_destroy(holo_b200_session* s);

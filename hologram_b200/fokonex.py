@@ -1,0 +1,319 @@
+"""Fokonex: a decoder-only design with parallel attention / feed-forward layers, as `.holo` step archives.
+
+A layer adds `m * (mixer(norm1(x)) + ff(norm2(x)))` to an f32 residual stream x, both branches reading the same x
+(RMS norms whose weights are stored around zero). The mixer is grouped-query attention without rotation, with its own
+value width, a logarithmic query temperature, a score cap and one sink per query head in the softmax denominator; the
+feed-forward is relu(W_up h)^2 through W_down. A layer may reuse another layer's tensors while keeping a cache of its own.
+
+One archive is one step shape: `rows` new tokens of one sequence against a cache of `capacity` rows. Each layer is
+
+    RmsNormMulti   x -> [h1 | h2]
+    Linear         [h1 | h2] -> q, rows of the K cache, rows of the V cache (from h1), relu^2 of the up projection (from h2)
+    CausalAttention over the cache -> the left part of the activation buffer (the up projection filled the right part)
+    Linear         [attention | up] -> x += m * (...)   (W_o and W_down stacked along k)
+
+Head widths are padded with zero columns to multiples of 16 and the model width to a multiple of 8, so that every row
+pitch suits TMA whatever the configuration's sizes are; zero columns change no result.
+"""
+import json
+import os
+
+import numpy as np
+
+from . import holo
+from . import kernel_call as kc
+from . import safetensors_io
+
+BF, F32, I32 = kc.DTYPE_BF16, kc.DTYPE_F32, kc.DTYPE_I32
+STEP_IN_IDS = 4            # the token ids follow four words of which the first is the position of the step's first row
+
+
+def _up(n, multiple):
+    return (n + multiple - 1) // multiple * multiple
+
+
+class AttentionSpec:
+    """Sizes and constants of one attention mixer."""
+
+    def __init__(self, heads, kv_heads, dim, vdim, scale, softcap=0.0, temp_coef=0.0, temp_every=0.0):
+        if heads <= 0 or kv_heads <= 0 or heads % kv_heads:
+            raise ValueError(f"attention: {heads} query heads do not group over {kv_heads} key/value heads")
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.softcap, self.temp_coef, self.temp_every = scale, softcap, temp_coef, temp_every
+        self.dim_p, self.vdim_p = _up(dim, 16), _up(vdim, 16)
+
+    @classmethod
+    def from_dict(cls, d):
+        temp = d.get("q_temp") or {}
+        return cls(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), float(d["scale"]), float(d.get("softcap") or 0.0),
+                   float(temp.get("coef", 0.0)), float(temp.get("every", 0.0)))
+
+
+class LayerSpec:
+    def __init__(self, index, mixer, ff, owner):
+        self.index, self.mixer, self.ff, self.owner = index, mixer, ff, owner   # ff None = no feed-forward; owner = layer whose tensors it uses
+        self.ff_p = _up(ff, 8) if ff is not None else 0
+
+
+class FokonexConfig:
+    ARCHITECTURE = "Fokonex"
+
+    def __init__(self, vocab, width, layers, eps, residual_mult=1.0, logit_scale=1.0):
+        self.vocab, self.width, self.layers, self.eps = vocab, width, layers, eps
+        self.residual_mult, self.logit_scale = residual_mult, logit_scale
+        self.width_p = _up(width, 8)
+
+    @classmethod
+    def from_dict(cls, d):
+        if d.get("architecture") != cls.ARCHITECTURE:
+            raise ValueError(f"config.json names architecture {d.get('architecture')!r}, not {cls.ARCHITECTURE!r}")
+        layers = []
+        for i, entry in enumerate(d["layers"]):
+            if entry["type"] != "attention":
+                raise ValueError(f"layer {i}: mixer type {entry['type']!r} is not part of this design")
+            mlp = entry.get("mlp")
+            if mlp is not None and mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not part of this design")
+            owner = i
+            if entry.get("weights_of") is not None:
+                j = int(entry["weights_of"])
+                if not 0 <= j < len(d["layers"]) or j == i:
+                    raise ValueError(f"layer {i}: weights_of {j}")
+                owner, seen = j, {i}
+                while d["layers"][owner].get("weights_of") is not None:
+                    if owner in seen:
+                        raise ValueError(f"layer {i}: weights_of goes in a circle")
+                    seen.add(owner)
+                    owner = int(d["layers"][owner]["weights_of"])
+            layers.append(LayerSpec(i, AttentionSpec.from_dict(entry["mixer"]), int(mlp["ff"]) if mlp is not None else None, owner))
+        return cls(int(d["vocab"]), int(d["width"]), layers, float(d["norm"]["eps"]), float(d.get("residual_mult", 1.0)),
+                   float(d.get("logit_scale", 1.0)))
+
+    def to_dict(self):
+        out = []
+        for l in self.layers:
+            a = l.mixer
+            mixer = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale, "softcap": a.softcap,
+                     "q_temp": {"coef": a.temp_coef, "every": a.temp_every}}
+            entry = {"type": "attention", "mixer": mixer, "mlp": None if l.ff is None else {"kind": "dense", "ff": l.ff}}
+            if l.owner != l.index:
+                entry["weights_of"] = l.owner
+            out.append(entry)
+        return {"architecture": self.ARCHITECTURE, "vocab": self.vocab, "width": self.width, "layers": out, "norm": {"eps": self.eps},
+                "residual_mult": self.residual_mult, "logit_scale": self.logit_scale}
+
+    def tensor_shapes(self):
+        """Name -> shape of every tensor a checkpoint of this configuration holds."""
+        w = self.width
+        out = {"embed": (self.vocab, w)}
+        for l in self.layers:
+            if l.owner != l.index:
+                continue
+            p, a = f"l{l.index}.", l.mixer
+            out[p + "norm1"] = (w,)
+            if l.ff is not None:
+                out[p + "norm2"] = (w,)
+            out[p + "mix.q"], out[p + "mix.k"] = (a.heads * a.dim, w), (a.kv_heads * a.dim, w)
+            out[p + "mix.v"], out[p + "mix.sink"] = (a.kv_heads * a.vdim, w), (a.heads,)
+            out[p + "mix.o"] = (w, a.heads * a.vdim)
+            if l.ff is not None:
+                out[p + "mlp.up"], out[p + "mlp.down"] = (l.ff, w), (w, l.ff)
+        out["final.norm"], out["head"] = (w,), (self.vocab, w)
+        return out
+
+
+class _Slots:
+    """Slot numbers and sizes of one archive under construction."""
+
+    def __init__(self):
+        self.nbytes = []
+
+    def new(self, nbytes):
+        self.nbytes.append(int(nbytes))
+        return len(self.nbytes) - 1
+
+    def ref(self, slot, offset=0, length=None):
+        return kc.rb(slot, offset, self.nbytes[slot] - offset if length is None else length)
+
+
+class FokonexModel:
+    """Configuration and device-layout weights of one model; builds its step archives."""
+
+    def __init__(self, config, tensors, dtype=BF):
+        self.config, self.dtype = config, dtype
+        self.elem = 2 if dtype == BF else 4
+        missing = [n for n, s in config.tensor_shapes().items() if n not in tensors or tuple(tensors[n].shape) != tuple(s)]
+        if missing:
+            raise ValueError(f"checkpoint: missing or misshaped tensors: {', '.join(missing[:5])}")
+        self._constants = {}       # name -> (array, fingerprint)
+        self._pack(tensors)
+
+    @classmethod
+    def load(cls, path, dtype=BF):
+        with open(os.path.join(path, "config.json"), encoding="utf-8") as f:
+            config = FokonexConfig.from_dict(json.load(f))
+        return cls(config, safetensors_io.read(os.path.join(path, "model.safetensors")), dtype)
+
+    # ---- weights in the layout the kernels read: [in, out], columns of several products side by side ----
+    def _value(self, tensor):
+        return tensor.as_bf16() if self.dtype == BF else tensor.as_f32()
+
+    def _zeros(self, shape):
+        return np.zeros(shape, dtype=np.uint16 if self.dtype == BF else np.float32)
+
+    def _add(self, name, array):
+        array = np.ascontiguousarray(array)
+        self._constants[name] = (array, holo.fingerprint(array.view(np.uint8).reshape(-1).data))
+
+    @staticmethod
+    def _gain(tensor):
+        return (np.float32(1.0) + tensor.as_f32()).astype(np.float32)
+
+    def in_columns(self, layer):
+        """Where q, k, v and the up projection begin in a layer's input product, and its column count."""
+        a = layer.mixer
+        q = 0
+        k = _up(a.heads * a.dim_p, 32)
+        v = k + _up(a.kv_heads * a.dim_p, 32)
+        end = v + a.kv_heads * a.vdim_p
+        if layer.ff is None:
+            return (q, k, v, None), _up(end, 8)
+        up = _up(end, 256)      # the up projection reads other columns of A: it starts a tile of its own
+        return (q, k, v, up), _up(up + layer.ff, 8)
+
+    def _pack(self, t):
+        c = self.config
+        w, wp = c.width, c.width_p
+        self._add("embed", self._value(t["embed"]))
+
+        def heads_in(src, heads, d, dp):        # [heads * d, w] -> [wp, heads * dp]
+            out = self._zeros((wp, heads, dp))
+            out[:w, :, :d] = self._value(src).reshape(heads, d, w).transpose(2, 0, 1)
+            return out.reshape(wp, heads * dp)
+
+        for l in c.layers:
+            if l.owner != l.index:
+                continue
+            p, a = f"l{l.index}.", l.mixer
+            self._add(p + "norm1", self._gain(t[p + "norm1"]))
+            (q, k, v, up), cols = self.in_columns(l)
+            b = self._zeros((wp, cols))
+            for at, name, heads, d, dp in ((q, "q", a.heads, a.dim, a.dim_p), (k, "k", a.kv_heads, a.dim, a.dim_p), (v, "v", a.kv_heads, a.vdim, a.vdim_p)):
+                b[:, at:at + heads * dp] = heads_in(t[p + "mix." + name], heads, d, dp)
+            o = self._zeros((a.heads, a.vdim_p, wp))
+            o[:, :a.vdim, :w] = self._value(t[p + "mix.o"]).T.reshape(a.heads, a.vdim, w)
+            o = o.reshape(a.heads * a.vdim_p, wp)
+            if l.ff is not None:
+                self._add(p + "norm2", self._gain(t[p + "norm2"]))
+                b[:w, up:up + l.ff] = self._value(t[p + "mlp.up"]).T
+                down = self._zeros((l.ff_p, wp))
+                down[:l.ff, :w] = self._value(t[p + "mlp.down"]).T
+                o = np.concatenate([o, down])
+            self._add(p + "in", b)
+            self._add(p + "out", o)
+            self._add(p + "sink", t[p + "mix.sink"].as_f32())
+        self._add("final.norm", self._gain(t["final.norm"]))
+        head = self._zeros((wp, _up(c.vocab, 8)))
+        head[:w, :c.vocab] = self._value(t["head"]).T
+        self._add("head", head)
+
+    # ---- archives ----
+    def _begin(self):
+        return holo.HoloWriter(), _Slots(), {}
+
+    def _const(self, w, sl, made, name):
+        if name not in made:
+            array, fp = self._constants[name]
+            made[name] = sl.new(array.nbytes)
+            w.add_constant(made[name], F32 if array.dtype == np.float32 else BF, array.view(np.uint8).reshape(-1).data, known_fingerprint=fp)
+        return sl.ref(made[name])
+
+    def _hidden(self, w, sl, hidden_rows):
+        n = hidden_rows * self.config.width
+        s = sl.new(4 * n)
+        w.inputs.append(holo.Port("hidden", s, n, F32, [hidden_rows, self.config.width]))
+        return s
+
+    def _logits(self, w, sl, made, x, rows):
+        """final norm and output head over `rows` rows of x; returns the slot of the f32 logits."""
+        c, es = self.config, self.elem
+        h, logits = sl.new(rows * c.width_p * es), sl.new(4 * rows * c.vocab)
+        w.calls.append(kc.KernelCall.RmsNormMulti(kc.RmsNormMultiCall(
+            x, self._const(w, sl, made, "final.norm"), kc.NONE, sl.ref(h), rows, c.width, c.width_p, kc.f32_bits(c.eps), self.dtype)))
+        seg = kc.LinearSeg(sl.ref(logits), kc.NONE, 0, c.vocab, 0, c.vocab, kc.LINEAR_ACT_NONE, F32)
+        w.calls.append(kc.KernelCall.Linear(kc.LinearCall.make(
+            sl.ref(h), self._const(w, sl, made, "head"), [seg], rows, c.width_p, _up(c.vocab, 8), self.dtype, alpha=c.logit_scale)))
+        w.outputs.append(holo.Port("logits", logits, rows * c.vocab, F32, [rows, c.vocab]))
+
+    def build_step(self, rows, capacity, hidden_rows, with_logits, weightless=False):
+        """The archive of one step of `rows` tokens: ports `step_in` (i32: position, three unused words, the token ids),
+        `hidden` (the residual stream, [hidden_rows, width]), `l<i>.k` / `l<i>.v` (the cache of layer run i); with
+        `with_logits` also the output head over all rows (port `logits`)."""
+        c, es, dt = self.config, self.elem, self.dtype
+        w, sl, made = self._begin()
+        step_in = sl.new(4 * (STEP_IN_IDS + rows))
+        w.inputs.append(holo.Port("step_in", step_in, STEP_IN_IDS + rows, I32, [STEP_IN_IDS + rows]))
+        pos, ids = sl.ref(step_in, 0, 4), sl.ref(step_in, 4 * STEP_IN_IDS)
+        x = self._hidden(w, sl, hidden_rows)
+        xr = sl.ref(x, 0, 4 * rows * c.width)
+        # embedding rows, widened to f32
+        if dt == F32:
+            emb = xr
+        else:
+            e = sl.new(rows * c.width * 2)
+            emb = sl.ref(e)
+        w.calls.append(kc.KernelCall.Gather(kc.GatherCall(self._const(w, sl, made, "embed"), ids, emb, 1, c.vocab, c.width, rows, I32, dt)))
+        if dt != F32:
+            w.calls.append(kc.KernelCall.Cast(kc.CastCall(emb, xr, rows * c.width, BF, F32)))
+        # activations: one set per distinct layer geometry, reused by every layer that has it
+        work = {}
+        for l in c.layers:
+            a, p = l.mixer, f"l{l.owner}."
+            ka = a.heads * a.vdim_p + l.ff_p
+            key = (a.heads, a.dim_p, a.vdim_p, l.ff_p)
+            nh = 1 if l.ff is None else 2
+            if key not in work:
+                work[key] = (sl.new(rows * nh * c.width_p * es), sl.new(rows * a.heads * a.dim_p * es), sl.new(rows * ka * es))
+            h, q, act = work[key]
+            lk, lv = a.kv_heads * a.dim_p, a.kv_heads * a.vdim_p
+            kcache, vcache = sl.new(capacity * lk * es), sl.new(capacity * lv * es)
+            w.inputs.append(holo.Port(f"l{l.index}.k", kcache, capacity * lk, dt, [capacity, a.kv_heads, a.dim_p]))
+            w.inputs.append(holo.Port(f"l{l.index}.v", vcache, capacity * lv, dt, [capacity, a.kv_heads, a.vdim_p]))
+            w.calls.append(kc.KernelCall.RmsNormMulti(kc.RmsNormMultiCall(
+                xr, self._const(w, sl, made, p + "norm1"), kc.NONE if l.ff is None else self._const(w, sl, made, p + "norm2"), sl.ref(h),
+                rows, c.width, c.width_p, kc.f32_bits(c.eps), dt)))
+            (cq, ck, cv, cu), cols = self.in_columns(l)
+            segs = [kc.LinearSeg(sl.ref(q), kc.NONE, cq, a.heads * a.dim_p, 0, a.heads * a.dim_p, 0, dt),
+                    kc.LinearSeg(sl.ref(kcache), pos, ck, lk, 0, lk, 0, dt), kc.LinearSeg(sl.ref(vcache), pos, cv, lv, 0, lv, 0, dt)]
+            if l.ff is not None:
+                segs.append(kc.LinearSeg(sl.ref(act, a.heads * a.vdim_p * es), kc.NONE, cu, l.ff, c.width_p, ka, kc.LINEAR_ACT_RELU2, dt))
+            w.calls.append(kc.KernelCall.Linear(kc.LinearCall.make(
+                sl.ref(h), self._const(w, sl, made, p + "in"), segs, rows, c.width_p, cols, dt, lda=nh * c.width_p)))
+            w.calls.append(kc.KernelCall.CausalAttention(kc.CausalAttentionCall(
+                sl.ref(q), sl.ref(kcache), sl.ref(vcache), pos, self._const(w, sl, made, p + "sink"), sl.ref(act), rows, a.heads, a.kv_heads,
+                a.dim_p, a.vdim_p, capacity, ka, kc.f32_bits(a.scale), kc.f32_bits(a.softcap), kc.f32_bits(a.temp_coef),
+                kc.f32_bits(a.temp_every), dt)))
+            seg = kc.LinearSeg(xr, kc.NONE, 0, c.width, 0, c.width, 0, F32)
+            w.calls.append(kc.KernelCall.Linear(kc.LinearCall.make(
+                sl.ref(act), self._const(w, sl, made, p + "out"), [seg], rows, ka, c.width_p, dt, residual=xr, alpha=c.residual_mult)))
+        if with_logits:
+            self._logits(w, sl, made, xr, rows)
+        w.exec_plan = [[i] for i in range(len(w.calls))]
+        return w.finish(weightless=weightless)
+
+    def build_head(self, rows, hidden_rows, weightless=False):
+        """The archive that turns `rows` chosen rows of the residual stream (port `want`, i32) into logits."""
+        c = self.config
+        w, sl, made = self._begin()
+        x = self._hidden(w, sl, hidden_rows)
+        want = sl.new(4 * rows)
+        w.inputs.append(holo.Port("want", want, rows, I32, [rows]))
+        picked = sl.new(4 * rows * c.width)
+        w.calls.append(kc.KernelCall.Gather(kc.GatherCall(sl.ref(x), sl.ref(want), sl.ref(picked), 1, hidden_rows, c.width, rows, I32, F32)))
+        self._logits(w, sl, made, sl.ref(picked), rows)
+        w.exec_plan = [[i] for i in range(len(w.calls))]
+        return w.finish(weightless=weightless)
+
+    def launches(self, rows, with_logits):
+        """Kernel launches of one step, by the archive's call count."""
+        return (1 if self.dtype == F32 else 2) + 4 * len(self.config.layers) + (2 if with_logits else 0)

@@ -126,6 +126,21 @@ def encode_call(call):
         c = u.rope_quantize
         return out + b"".join(_buf(b) for b in (c.x, c.cos, c.sin, c.rope_output, c.codes, c.scales)) + struct.pack(
             "<QIB", c.rows, c.row_len, c.dtype)
+    if k == kc.K_RMS_NORM_MULTI:
+        c = u.rms_norm_multi
+        return out + b"".join(_buf(b) for b in (c.x, c.gamma0, c.gamma1, c.output)) + struct.pack(
+            "<IIIIB", c.rows, c.feature, c.step, c.epsilon_bits, c.dtype)
+    if k == kc.K_LINEAR:
+        c = u.linear
+        segs = b"".join(_buf(g.output) + _buf(g.row_pos) + struct.pack("<IIIIBB", g.col_begin, g.width, g.k_offset, g.ld, g.act, g.dtype)
+                        for g in list(c.seg)[:c.nseg])
+        return out + b"".join(_buf(b) for b in (c.a, c.b, c.residual)) + struct.pack(
+            "<IIIIIBB", c.m, c.k, c.n, c.lda, c.alpha_bits, c.dtype, c.nseg) + segs
+    if k == kc.K_CAUSAL_ATTENTION:
+        c = u.causal_attention
+        return out + b"".join(_buf(b) for b in (c.q, c.k, c.v, c.pos, c.sink, c.output)) + struct.pack(
+            "<11IB", c.rows, c.heads, c.kv_heads, c.dim, c.vdim, c.cache_rows, c.ld, c.scale_bits, c.softcap_bits, c.temp_coef_bits,
+            c.temp_every_bits, c.dtype)
     if k == kc.K_ALL_REDUCE:
         c = u.all_reduce
         return out + _buf(c.buffer) + struct.pack("<QB", c.element_count, c.dtype)
@@ -160,11 +175,14 @@ class HoloWriter:
     def __init__(self):
         self.calls, self.inputs, self.outputs, self.exec_plan = [], [], [], []
         self.inline_constants, self.weight_constants, self.extensions = [], [], []
+        self.known_fingerprints = {}            # slot -> fingerprint, for bodies hashed before
 
-    def add_constant(self, slot, dtype, array_bytes, by_reference=None):
+    def add_constant(self, slot, dtype, array_bytes, by_reference=None, known_fingerprint=None):
         body = bytes(array_bytes) if not isinstance(array_bytes, (bytes, bytearray, memoryview)) else array_bytes
         if by_reference is None:
             by_reference = len(body) > 256
+        if known_fingerprint is not None:
+            self.known_fingerprints[slot] = known_fingerprint
         (self.weight_constants if by_reference else self.inline_constants).append((slot, dtype, body))
 
     def finish(self, weightless=False):
@@ -174,7 +192,7 @@ class HoloWriter:
         for slot, dtype, body in self.inline_constants:
             const += struct.pack("<BIBI", 0, slot, dtype, len(body)) + bytes(body)
         for slot, dtype, body in self.weight_constants:
-            fp = fingerprint(body)
+            fp = self.known_fingerprints.get(slot) or fingerprint(body)
             if fp not in weights:
                 weights[fp] = body
                 order.append(fp)

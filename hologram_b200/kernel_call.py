@@ -40,6 +40,7 @@ K_DEQUANTIZE, K_MATMUL_ACTIVATION, K_MATMUL_ADD = 105, 106, 107
 K_GATHER, K_CAST, K_KV_CACHE_WRITE, K_DECODE_ATTENTION_VALID = 114, 115, 120, 121
 K_QUANTIZE_ROWS_I8, K_DECODE_ATTENTION_VALID_Q8, K_ALL_REDUCE = 0x8001, 0x8002, 0x8003
 K_ROPE_QUANTIZE_ROWS_I8 = 0x8004
+K_RMS_NORM_MULTI, K_LINEAR, K_CAUSAL_ATTENTION = 0x8005, 0x8006, 0x8007
 LUT_KIND = {LUT_SIGMOID: K_SIGMOID, LUT_TANH: K_TANH, LUT_GELU: K_GELU, LUT_SILU: K_SILU, LUT_EXP: K_EXP, LUT_ERF: K_ERF}
 
 NO_SLOT = 0xFFFFFFFF
@@ -58,6 +59,11 @@ def rb(slot, offset=0, length=0):
 
 
 NONE = BufferRef(NO_SLOT, 0, 0)
+
+
+def f32_bits(x):
+    """The bit pattern of an f32 scalar, as the calls carry their constants."""
+    return C.c_uint32.from_buffer(C.c_float(x)).value
 
 
 class UnaryCall(C.Structure):
@@ -263,6 +269,46 @@ class AllReduceCall(C.Structure):
     _fields_ = [("buffer", BufferRef), ("element_count", C.c_uint64), ("dtype", C.c_uint8)]
 
 
+class RmsNormMultiCall(C.Structure):
+    """Extension: f32 rows normalised under one or two f32 weights, side by side in the output (`step` columns each)."""
+    _fields_ = [("x", BufferRef), ("gamma0", BufferRef), ("gamma1", BufferRef), ("output", BufferRef), ("rows", C.c_uint32),
+                ("feature", C.c_uint32), ("step", C.c_uint32), ("epsilon_bits", C.c_uint32), ("dtype", C.c_uint8)]
+
+
+LINEAR_MAX_SEGS = 4
+LINEAR_ACT_NONE, LINEAR_ACT_RELU2 = 0, 1
+
+
+class LinearSeg(C.Structure):
+    _fields_ = [("output", BufferRef), ("row_pos", BufferRef), ("col_begin", C.c_uint32), ("width", C.c_uint32),
+                ("k_offset", C.c_uint32), ("ld", C.c_uint32), ("act", C.c_uint8), ("dtype", C.c_uint8)]
+
+
+class LinearCall(C.Structure):
+    """Extension: out_s[i, j] = residual + alpha * act_s(A[i, k_offset:k_offset + k] . B[:, col_begin + j]) for up to four segments."""
+    _fields_ = [("a", BufferRef), ("b", BufferRef), ("residual", BufferRef), ("seg", LinearSeg * LINEAR_MAX_SEGS), ("m", C.c_uint32),
+                ("k", C.c_uint32), ("n", C.c_uint32), ("lda", C.c_uint32), ("nseg", C.c_uint32), ("alpha_bits", C.c_uint32),
+                ("dtype", C.c_uint8)]
+
+    @classmethod
+    def make(cls, a, b, segs, m, k, n, dtype, lda=None, residual=None, alpha=1.0):
+        c = cls()
+        c.a, c.b, c.residual = a, b, NONE if residual is None else residual
+        c.m, c.k, c.n, c.lda, c.nseg, c.dtype = m, k, n, k if lda is None else lda, len(segs), dtype
+        c.alpha_bits = f32_bits(alpha)
+        for i, g in enumerate(segs):
+            c.seg[i] = g
+        return c
+
+
+class CausalAttentionCall(C.Structure):
+    """Extension: new rows of one sequence over the cache that already holds them (score cap, sink, query temperature)."""
+    _fields_ = [("q", BufferRef), ("k", BufferRef), ("v", BufferRef), ("pos", BufferRef), ("sink", BufferRef), ("output", BufferRef),
+                ("rows", C.c_uint32), ("heads", C.c_uint32), ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32),
+                ("cache_rows", C.c_uint32), ("ld", C.c_uint32), ("scale_bits", C.c_uint32), ("softcap_bits", C.c_uint32),
+                ("temp_coef_bits", C.c_uint32), ("temp_every_bits", C.c_uint32), ("dtype", C.c_uint8)]
+
+
 class _Payload(C.Union):
     _fields_ = [("unary", UnaryCall), ("binary", BinaryCall), ("matmul", MatMulCall),
                 ("matmul_activation", MatMulActivationCall), ("matmul_add", MatMulAddCall), ("matmul_add_activation", MatMulAddActivationCall), ("matmul_dequant", MatMulDequantCall), ("norm", NormCall),
@@ -271,7 +317,8 @@ class _Payload(C.Union):
                 ("decode_attention", DecodeAttentionCall),
                 ("decode_attention_valid", DecodeAttentionValidCall), ("quantize_rows_i8", QuantizeRowsI8Call),
                 ("decode_attention_valid_q8", DecodeAttentionValidQ8Call), ("all_reduce", AllReduceCall),
-                ("rope_quantize", RopeQuantizeCall)]
+                ("rope_quantize", RopeQuantizeCall), ("rms_norm_multi", RmsNormMultiCall), ("linear", LinearCall),
+                ("causal_attention", CausalAttentionCall)]
 
 
 class KernelCall(C.Structure):
@@ -383,6 +430,12 @@ class KernelCall(C.Structure):
     def AllReduce(cls, c): return cls.of(K_ALL_REDUCE, c)
     @classmethod
     def RopeQuantizeRowsI8(cls, c): return cls.of(K_ROPE_QUANTIZE_ROWS_I8, c)
+    @classmethod
+    def RmsNormMulti(cls, c): return cls.of(K_RMS_NORM_MULTI, c)
+    @classmethod
+    def Linear(cls, c): return cls.of(K_LINEAR, c)
+    @classmethod
+    def CausalAttention(cls, c): return cls.of(K_CAUSAL_ATTENTION, c)
 
 
 KernelCall._FIELD = {
@@ -391,6 +444,7 @@ KernelCall._FIELD = {
     LayoutCall: "layout", TransposeCall: "transpose", SoftmaxCall: "softmax", ExpandCall: "expand", ReduceCall: "reduce", AttentionCall: "attention", DequantActivationCall: "dequant_activation", WhereCall: "where", BroadcastBinaryCall: "broadcast_binary", DequantizeCall: "dequantize", KvCacheWriteCall: "kv_cache_write",
     DecodeAttentionCall: "decode_attention", DecodeAttentionValidCall: "decode_attention_valid", QuantizeRowsI8Call: "quantize_rows_i8",
     DecodeAttentionValidQ8Call: "decode_attention_valid_q8", AllReduceCall: "all_reduce", RopeQuantizeCall: "rope_quantize",
+    RmsNormMultiCall: "rms_norm_multi", LinearCall: "linear", CausalAttentionCall: "causal_attention",
 }
 
 

@@ -10,6 +10,7 @@ from .backend import DeviceWorkspace, WeightStore, _check, _host_ptr, lib
 vp, u32, u64, i32 = C.c_void_p, C.c_uint32, C.c_uint64, C.c_int32
 for _name, _res, _args in [
     ("holo_b200_session_load", i32, [vp, vp, u64, i32, C.POINTER(vp)]),
+    ("holo_b200_session_load_shared", i32, [vp, vp, u64, i32, vp, C.POINTER(vp)]),
     ("holo_b200_session_destroy", None, [vp]),
     ("holo_b200_session_workspace", vp, [vp]),
     ("holo_b200_session_info", i32, [vp] + [C.POINTER(u32)] * 5 + [C.POINTER(u64)]),
@@ -35,7 +36,7 @@ for _name, _res, _args in [
     _fn = getattr(lib, _name)
     _fn.restype, _fn.argtypes = _res, _args
 
-SESSION_SYMBOLS = ["holo_b200_session_load", "holo_b200_session_destroy", "holo_b200_session_workspace",
+SESSION_SYMBOLS = ["holo_b200_session_load", "holo_b200_session_load_shared", "holo_b200_session_destroy", "holo_b200_session_workspace",
                    "holo_b200_session_info", "holo_b200_session_nodes", "holo_b200_session_port", "holo_b200_session_call",
                    "holo_b200_session_execute", "holo_b200_session_capture", "holo_b200_archive_check",
                    "holo_b200_session_execute_addressed", "holo_b200_label_bytes", "holo_b200_label_derive",
@@ -114,9 +115,10 @@ class Port:
 
 
 class InferenceSession:
-    def __init__(self, backend, archive_bytes, verify=True, addressed=False, label_residual=False, weight_store=None, budget=0):
+    def __init__(self, backend, archive_bytes, verify=True, addressed=False, label_residual=False, weight_store=None, budget=0, donor=None):
         """`weight_store` (a WeightStore) makes this `load_paged` (session.rs:417): by-reference constants page in from it
-        within `budget` resident bytes (0 = never evict)."""
+        within `budget` resident bytes (0 = never evict). `donor` (a session) makes it another step shape of the donor's
+        model: weights are the donor's device copies, input ports of the same name and size share its buffers."""
         h = vp()
         buf = np.frombuffer(archive_bytes, dtype=np.uint8)
         flags = (1 if verify else 0) | (2 if addressed else 0) | (SESSION_LABEL_RESIDUAL if label_residual else 0)
@@ -124,6 +126,9 @@ class InferenceSession:
             self._store = weight_store      # the provider must outlive the session
             addressed = True
             _check(lib.holo_b200_session_load_paged(backend._h, _host_ptr(buf), buf.size, flags, C.byref(weight_store.struct), budget, C.byref(h)))
+        elif donor is not None:
+            self._donor = donor             # its buffers must outlive this session
+            _check(lib.holo_b200_session_load_shared(backend._h, _host_ptr(buf), buf.size, flags, donor._h, C.byref(h)))
         else:
             _check(lib.holo_b200_session_load(backend._h, _host_ptr(buf), buf.size, flags, C.byref(h)))
         self.addressed = addressed

@@ -137,6 +137,13 @@ extern "C" {
 /* RotaryEmbedding followed by QuantizeRowsI8 of its result, one row = one head (fused at load by the
  * session when a RoPE output feeds a row quantizer of the same row length; bit-identical to the pair). */
 #define HOLO_K_ROPE_QUANTIZE_ROWS_I8 0x8004
+/* Decoder steps with an f32 residual stream and a 16-bit (or f32) cache, over any number of rows of one sequence:
+ * RMS_NORM_MULTI normalises f32 rows under one or two weights; LINEAR is a product with up to four output segments,
+ * rounded (not truncated) stores and an optional f32 residual; CAUSAL_ATTENTION reads the cache the step has just
+ * appended to, with optional score cap, attention sink and position-dependent query temperature. */
+#define HOLO_K_RMS_NORM_MULTI 0x8005
+#define HOLO_K_LINEAR 0x8006
+#define HOLO_K_CAUSAL_ATTENTION 0x8007
 
 /* BufferRef (crates/hologram-compute/src/workspace.rs:16-24). length == 0 means "the slot's
  * full extent from offset". slot == UINT32_MAX marks an absent optional operand
@@ -396,6 +403,51 @@ typedef struct HoloRopeQuantizeCall {
     uint8_t dtype;
 } HoloRopeQuantizeCall;
 
+/* Extension. x f32 [rows, feature]; output `dtype` (f32 or bf16, rounded to nearest) [rows, n * step] where n is the
+ * number of weights given (gamma1 may be absent): columns [i * step, i * step + feature) hold
+ * x / sqrt(mean(x^2) + eps) * gamma_i (f32 [feature]), columns up to (i + 1) * step are zero. */
+typedef struct HoloRmsNormMultiCall {
+    HoloBufferRef x, gamma0, gamma1, output;
+    uint32_t rows, feature, step, epsilon_bits;
+    uint8_t dtype;
+} HoloRmsNormMultiCall;
+
+/* Extension. A [m, lda] (row pitch lda), B [k, n], both `dtype` (bf16 or f32), f32 accumulation. Segment s:
+ *   out_s[row_pos + i][j] = residual[row_pos + i][j] + alpha * act_s(sum_k A[i][k_offset + k] * B[k][col_begin + j]),  j < width
+ * stored as `dtype` f32 or bf16 (rounded to nearest) with row pitch ld. row_pos is an optional device u32 (rows of a
+ * cache). The residual (f32, same pitch as the output) needs a single f32 segment and may be the output itself.
+ * col_begin is a multiple of 32 and ascending; where k_offset changes from one segment to the next it is a multiple
+ * of 256. Columns of B between segments are padding. */
+#define HOLO_LINEAR_MAX_SEGS 4
+#define HOLO_LINEAR_ACT_NONE 0
+#define HOLO_LINEAR_ACT_RELU2 1 /* max(v, 0)^2 */
+typedef struct HoloLinearSeg {
+    HoloBufferRef output, row_pos;
+    uint32_t col_begin, width, k_offset, ld;
+    uint8_t act, dtype;
+} HoloLinearSeg;
+typedef struct HoloLinearCall {
+    HoloBufferRef a, b, residual;
+    HoloLinearSeg seg[HOLO_LINEAR_MAX_SEGS];
+    uint32_t m, k, n, lda, nseg, alpha_bits;
+    uint8_t dtype;
+} HoloLinearCall;
+
+/* Extension. Attention of `rows` new positions of one sequence over its cache, which already holds them: row i is at
+ * position p = *pos + i and sees cache rows j <= p. q [rows, heads * dim]; k [cache_rows, kv_heads * dim];
+ * v [cache_rows, kv_heads * vdim] (query head h reads kv head h / (heads / kv_heads)); output [rows, ld], head h at
+ * columns h * vdim. Scores and weights are f32:
+ *   s = (q . k) * scale * (1 + temp_coef * ln(floor((p + 1) / temp_every) + 1))   (no factor when temp_every is 0)
+ *   s = softcap * tanh(s / softcap)                                               (when softcap > 0)
+ *   out = sum_j exp(s_j) v_j / (sum_j exp(s_j) + exp(sink_h))                     (no sink term when sink is absent)
+ * A zero scale selects 1 / sqrt(dim). Rows past the end of the cache see what it holds. */
+typedef struct HoloCausalAttentionCall {
+    HoloBufferRef q, k, v, pos, sink, output;
+    uint32_t rows, heads, kv_heads, dim, vdim, cache_rows, ld;
+    uint32_t scale_bits, softcap_bits, temp_coef_bits, temp_every_bits;
+    uint8_t dtype;
+} HoloCausalAttentionCall;
+
 /* Extension. In-place sum over the context's tensor-parallel group (NCCL); a no-op when the
  * context has no group. */
 typedef struct HoloAllReduceCall {
@@ -436,6 +488,9 @@ typedef struct HoloKernelCall {
         HoloDecodeAttentionValidQ8Call decode_attention_valid_q8;
         HoloAllReduceCall all_reduce;
         HoloRopeQuantizeCall rope_quantize;
+        HoloRmsNormMultiCall rms_norm_multi;
+        HoloLinearCall linear;
+        HoloCausalAttentionCall causal_attention;
     } u;
 } HoloKernelCall;
 
@@ -517,6 +572,13 @@ typedef struct holo_b200_session holo_b200_session;
 int32_t holo_b200_session_load(holo_b200_ctx* ctx, const uint8_t* archive, uint64_t len, int32_t verify,
                                holo_b200_session** out);
 void holo_b200_session_destroy(holo_b200_session* s);
+/* Load an archive that is another step shape of a model `donor` already holds (other row counts of one decoder, its
+ * output head): a constant stored by reference whose fingerprint the donor has is bound to the donor's device copy
+ * (the archive may omit the Weights section), and an input port of the same name and size as one of the donor's shares
+ * its buffer (so the KV cache and the position are one state for all the shapes). The donor must outlive the session.
+ * Not available for addressed or paged sessions. */
+int32_t holo_b200_session_load_shared(holo_b200_ctx* ctx, const uint8_t* archive, uint64_t len, int32_t verify,
+                                      holo_b200_session* donor, holo_b200_session** out);
 /* The session's device workspace (owned by the session): upload inputs / download outputs
  * through it, or bind caller-owned device memory to a port's slot. */
 holo_b200_workspace* holo_b200_session_workspace(holo_b200_session* s);
