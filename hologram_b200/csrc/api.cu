@@ -89,6 +89,7 @@ extern "C" void holo_b200_ctx_destroy(holo_b200_ctx* ctx) {
     if (ctx->stage) cudaFree(ctx->stage);
     if (ctx->dev_status) cudaFree(ctx->dev_status);
     if (ctx->attn_arrivals) cudaFree(ctx->attn_arrivals);
+    if (ctx->causal_partials) cudaFree(ctx->causal_partials);
     if (ctx->own_stream) cudaStreamDestroy(ctx->stream);
     delete ctx;
 }

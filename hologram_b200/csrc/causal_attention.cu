@@ -1,12 +1,22 @@
 // Causal attention of new rows over a cache that already holds them (the CausalAttention call): row i of the step is
 // at position p = *pos + i and sees cache rows 0 .. p. Optional score cap (softcap * tanh(s / softcap)), one learned
 // sink per head in the softmax denominator, and a query factor that grows with the logarithm of the position.
-#include "common.h"
+//
+// bf16 with a cap of at most CAP_LIMIT needs no running maximum: every capped score lies in [-cap, cap], so exp(s) of any
+// row fits f32 (and bf16, which has f32's exponent range) as it is, partial sums over disjoint keys simply add, and the
+// accumulator is never rescaled. Two kernels use that:
+//   causal_attention_split_kernel  few rows (decode): warps stream 16-key tiles through their own cp.async rings, both
+//                                  products on mma.sync (HBM- or latency-bound), the keys split over the chip
+//   causal_attention_tile_kernel   many rows (prefill): 128-row tiles on tcgen05 with scores, weights and output in TMEM
+// Everything else (f32, no cap, larger caps, sizes TMA cannot take) runs the general kernel.
+#include "gemm_kernels.cuh"
 
-#include <cuda_bf16.h>
-#include <stdlib.h>
+#include <algorithm>
 
 namespace {
+
+constexpr float CAP_LIMIT = 64.0f;
+constexpr float LOG2E = 1.4426950408889634f;
 
 // The factor of a query at position p: 1 + coef * ln(floor((p + 1) / every) + 1). IEEE division: an exact quotient
 // stays exact, so the floor steps exactly at multiples of `every`.
@@ -95,8 +105,574 @@ int32_t launch_generic(holo_b200_ctx* ctx, const HoloCausalArgs& a) {
     return HOLO_OK;
 }
 
+
+// ---- capped scores without a maximum -----------------------------------------------------------------------------
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// exp(cap * tanh(s * factor / cap)), with c1 = 2 factor log2(e) / cap and c2 = cap log2(e):
+// tanh(y) = 1 - 2 / (exp(2y) + 1), so the exponent in log2 units is c2 - 2 c2 / (2^(s c1) + 1).
+__device__ __forceinline__ float capped_exp(float s, float c1, float c2) { return ex2(fmaf(-2.0f * c2, rcp(ex2(s * c1) + 1.0f), c2)); }
+
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+
+// ---- few rows: keys split over CTAs and warps ----------------------------------------------------------------------
+// A tile of 16 query rows packs (row, head of the group) pairs of one kv head, so every K/V row is read once for all of
+// them. Warp w of split c takes 16-key tiles w, w + W, ... of the split's range through a private ring of STAGES tiles
+// (no block-wide synchronisation in the loop). Warps merge through shared memory, splits through a partial buffer: the
+// last CTA of a (kv head, row tile) to count in adds the partials in split order; nobody waits.
+constexpr uint32_t SPLIT_SLOTS = 1024, SPLIT_SLOT_FLOATS = 16 * 257;
+
+struct SplitParams {
+    HoloCausalArgs a;
+    float* partials;
+    uint32_t* arrivals;
+    uint32_t group, splits;
+};
+
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// 16 bytes to shared memory, or 16 zero bytes when `take` is false (nothing is read then)
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool take) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(take ? 16u : 0u) : "memory");
+}
+
+template <int VT, int STAGES>   // vdim <= 16 VT
+__global__ void __launch_bounds__(256)
+causal_attention_split_kernel(const SplitParams p) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    const HoloCausalArgs& a = p.a;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+    const uint32_t split = blockIdx.x, g = blockIdx.y, z = blockIdx.z;
+    const uint32_t kp = a.dim * 2 + 16, vp = a.vdim * 2 + 16;      // shared-memory row pitches: an odd number of 16-byte units
+    const uint32_t tile_bytes = 16 * (kp + vp);
+    const uint32_t s_q = smem_u32(sm), s_ring = s_q + 16 * kp + warp * STAGES * tile_bytes;
+    const uint32_t kv_ld = a.kv_heads * a.dim, vv_ld = a.kv_heads * a.vdim;
+    holo_pdl_trigger();
+    holo_pdl_wait();
+    const uint32_t pos = *a.pos;
+    // the last position any row of this tile sees
+    const uint32_t last_row = min((z * 16 + 15) / p.group, a.rows - 1);
+    const uint32_t visible = min(pos + last_row + 1, a.cache_rows);
+    const uint32_t tiles = (visible + 15) / 16;
+    const uint32_t used = min(p.splits, (tiles + nwarps - 1) / nwarps);
+    if (split >= used) return;
+    const uint32_t t_begin = (uint32_t)((uint64_t)tiles * split / used), t_end = (uint32_t)((uint64_t)tiles * (split + 1) / used);
+    const __nv_bfloat16* kbase = (const __nv_bfloat16*)a.k + g * a.dim;
+    const __nv_bfloat16* vbase = (const __nv_bfloat16*)a.v + g * a.vdim;
+    const uint32_t kvec = a.dim / 8, vvec = a.vdim / 8;
+
+    auto load_tile = [&](uint32_t tile, uint32_t stage) {
+        const uint32_t dst = s_ring + stage * tile_bytes;
+        for (uint32_t i = lane; i < 16 * kvec; i += 32) {
+            const uint32_t r = i / kvec, c = i % kvec, key = tile * 16 + r;
+            cp_async16(dst + r * kp + c * 16, kbase + (uint64_t)min(key, a.cache_rows - 1) * kv_ld + c * 8, key < visible);
+        }
+        for (uint32_t i = lane; i < 16 * vvec; i += 32) {
+            const uint32_t r = i / vvec, c = i % vvec, key = tile * 16 + r;
+            cp_async16(dst + 16 * kp + r * vp + c * 16, vbase + (uint64_t)min(key, a.cache_rows - 1) * vv_ld + c * 8, key < visible);
+        }
+    };
+    const uint32_t first = t_begin + warp;
+#pragma unroll
+    for (int s = 0; s < STAGES - 1; ++s) {
+        const uint32_t t = first + s * nwarps;
+        if (t < t_end) load_tile(t, s);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    // the query tile (rows past the step's last one are zero)
+    for (uint32_t i = threadIdx.x; i < 16 * kvec; i += blockDim.x) {
+        const uint32_t r = i / kvec, c = i % kvec, qr = z * 16 + r, row = qr / p.group;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (row < a.rows) v = *reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.q + ((uint64_t)row * a.heads + g * p.group + qr % p.group) * a.dim + c * 8);
+        *reinterpret_cast<uint4*>(sm + r * kp + c * 16) = v;
+    }
+    __syncthreads();
+
+    const uint32_t r0 = lane >> 2;                        // this thread's rows of the tile: r0 and r0 + 8
+    const float c2 = a.softcap * LOG2E;
+    float c1[2];
+    uint32_t limit[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const uint32_t row = min((z * 16 + r0 + 8 * e) / p.group, a.rows - 1);
+        c1[e] = 2.0f * LOG2E * a.scale * query_factor(pos + row, a.temp_coef, a.temp_every) / a.softcap;
+        limit[e] = pos + row;
+    }
+    // with at most eight rows the upper half of the tile is all padding
+    const bool upper = a.rows * p.group > z * 16 + 8;
+    float o[VT][2][4];
+    float sum[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int n = 0; n < VT; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][0][e] = o[n][1][e] = 0.0f;
+    const uint32_t q_addr = s_q + (lane & 15) * kp + (lane >> 4) * 16;
+    const uint32_t k_off = ((lane & 7) + ((lane >> 4) << 3)) * kp + ((lane >> 3) & 1) * 16;
+    const uint32_t v_off = 16 * kp + ((lane & 7) + (((lane >> 3) & 1) << 3)) * vp + (lane >> 4) * 16;
+    const uint32_t ksteps = a.dim / 16, vsteps = a.vdim / 16;
+    uint32_t stage = 0;
+    for (uint32_t t = first; t < t_end; t += nwarps) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+        __syncwarp();
+        {   // refill the stage the previous iteration has emptied
+            const uint32_t nt = t + (STAGES - 1) * nwarps;
+            if (nt < t_end) load_tile(nt, stage == 0 ? STAGES - 1 : stage - 1);
+            asm volatile("cp.async.commit_group;" ::: "memory");
+        }
+        const uint32_t tile = s_ring + stage * tile_bytes;
+        float s[2][4] = {};
+#pragma unroll 4
+        for (uint32_t k = 0; k < ksteps; ++k) {
+            uint32_t qa[4], kb[4];
+            ldsm4(q_addr + k * 32, qa);
+            ldsm4(tile + k_off + k * 32, kb);
+            mma16816(s[0], qa, kb[0], kb[1]);
+            mma16816(s[1], qa, kb[2], kb[3]);
+        }
+        float w[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int half = e >> 1;
+                const uint32_t key = t * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
+                w[n][e] = 0.0f;
+                if ((half == 0 || upper) && key <= limit[half]) w[n][e] = capped_exp(s[n][e], c1[half], c2);
+                sum[half] += w[n][e];
+            }
+        const uint32_t pa[4] = {pack_bf16(w[0][0], w[0][1]), pack_bf16(w[0][2], w[0][3]), pack_bf16(w[1][0], w[1][1]), pack_bf16(w[1][2], w[1][3])};
+#pragma unroll
+        for (int n = 0; n < VT; ++n) {
+            if ((uint32_t)n < vsteps) {
+                uint32_t vb[4];
+                ldsm4t(tile + v_off + n * 32, vb);
+                mma16816(o[n][0], pa, vb[0], vb[1]);
+                mma16816(o[n][1], pa, vb[2], vb[3]);
+            }
+        }
+        stage = stage + 1 == STAGES ? 0 : stage + 1;
+        __syncwarp();
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 1);
+        sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 2);
+    }
+    __syncthreads();   // every warp is through with its ring: it becomes the merge buffer [warp][16][vdim + 1]
+    float* merge = reinterpret_cast<float*>(sm);
+    const uint32_t ml = a.vdim + 1;
+    float* mine = merge + (size_t)warp * 16 * ml;
+#pragma unroll
+    for (int n = 0; n < VT; ++n)
+        if ((uint32_t)n < vsteps)
+#pragma unroll
+            for (int h = 0; h < 2; ++h)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) mine[(r0 + 8 * (e >> 1)) * ml + n * 16 + h * 8 + (lane & 3) * 2 + (e & 1)] = o[n][h][e];
+    if ((lane & 3) == 0) {
+        mine[r0 * ml + a.vdim] = sum[0];
+        mine[(r0 + 8) * ml + a.vdim] = sum[1];
+    }
+    __syncthreads();
+    const uint32_t nrows = min(16u, a.rows * p.group - z * 16), cells = nrows * ml;
+    const uint32_t tile_id = z * a.kv_heads + g;
+    float* part = p.partials + ((uint64_t)tile_id * p.splits + split) * SPLIT_SLOT_FLOATS;
+    for (uint32_t i = threadIdx.x; i < cells; i += blockDim.x) {
+        float v = 0.0f;
+        for (uint32_t w = 0; w < nwarps; ++w) v += merge[(size_t)w * 16 * ml + i];
+        if (used == 1) merge[i] = v;     // only this thread touches cell i of every warp's part
+        else __stcg(part + i, v);
+    }
+    if (used > 1) {
+        __shared__ uint32_t s_last;
+        __threadfence();
+        __syncthreads();
+        if (threadIdx.x == 0) s_last = atomicAdd(p.arrivals + tile_id, 1u) == used - 1 ? 1u : 0u;
+        __syncthreads();
+        if (!s_last) return;
+        __threadfence();
+        if (threadIdx.x == 0) p.arrivals[tile_id] = 0;
+        const float* all = p.partials + (uint64_t)tile_id * p.splits * SPLIT_SLOT_FLOATS;
+        for (uint32_t i = threadIdx.x; i < cells; i += blockDim.x) {
+            float v = 0.0f;
+#pragma unroll 16
+            for (uint32_t c = 0; c < used; ++c) v += __ldcg(all + (uint64_t)c * SPLIT_SLOT_FLOATS + i);
+            merge[i] = v;
+        }
+    }
+    __syncthreads();
+    for (uint32_t i = threadIdx.x; i < nrows * (a.vdim / 2); i += blockDim.x) {
+        const uint32_t r = i / (a.vdim / 2), c = 2 * (i % (a.vdim / 2)), qr = z * 16 + r, head = g * p.group + qr % p.group;
+        const float denom = merge[r * ml + a.vdim] + (a.sink ? ex2(a.sink[head] * LOG2E) : 0.0f);
+        const float inv = __fdiv_rn(1.0f, denom);
+        *reinterpret_cast<uint32_t*>((__nv_bfloat16*)a.out + (uint64_t)(qr / p.group) * a.ld + head * a.vdim + c) =
+            pack_bf16(merge[r * ml + c] * inv, merge[r * ml + c + 1] * inv);
+    }
+}
+
+template <int VT, int STAGES>
+int32_t launch_split(holo_b200_ctx* ctx, const SplitParams& p, uint32_t qtiles, uint32_t warps, size_t smem) {
+    static thread_local int configured_device = -1;
+    if (configured_device != ctx->device) {
+        HOLO_CUDA(cudaFuncSetAttribute(causal_attention_split_kernel<VT, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, ctx->smem_optin - 1024));
+        configured_device = ctx->device;
+    }
+    HOLO_CUDA(holo_launch_kernel(ctx, causal_attention_split_kernel<VT, STAGES>, dim3(p.splits, p.a.kv_heads, qtiles), dim3(warps * 32), smem, 1, p));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
+// Launches the split kernel, or returns with *taken false when the shape does not suit it.
+int32_t try_split(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
+    *taken = false;
+    const uint32_t group = a.heads / a.kv_heads, qtiles = (a.rows * group + 15) / 16;
+    const uint32_t pairs = qtiles * a.kv_heads;
+    if (a.vdim > 256 || a.dim > 256 || pairs > SPLIT_SLOTS || qtiles > 65535) return HOLO_OK;
+    const int stages = a.vdim <= 64 ? 4 : a.vdim <= 128 ? 3 : 2;
+    const size_t kp = a.dim * 2 + 16, vp = a.vdim * 2 + 16, limit = (size_t)ctx->smem_optin - 1024;
+    uint32_t warps = 8;
+    auto bytes = [&](uint32_t w) { return std::max(16 * kp + w * stages * 16 * (kp + vp), (size_t)w * 16 * (a.vdim + 1) * 4); };
+    while (warps > 1 && bytes(warps) > limit) warps /= 2;
+    if (bytes(warps) > limit) return HOLO_OK;
+    if (!ctx->causal_partials) HOLO_CUDA(cudaMalloc(&ctx->causal_partials, (size_t)SPLIT_SLOTS * SPLIT_SLOT_FLOATS * 4));
+    SplitParams p;
+    p.a = a;
+    p.partials = ctx->causal_partials;
+    p.arrivals = ctx->attn_arrivals;
+    p.group = group;
+    p.splits = (uint32_t)ctx->sm_count / pairs;
+    const uint32_t most = (a.cache_rows + 16 * warps - 1) / (16 * warps);
+    if (p.splits > most) p.splits = most;
+    if (p.splits < 1) p.splits = 1;
+    *taken = true;
+    if (a.vdim <= 64) return launch_split<4, 4>(ctx, p, qtiles, warps, bytes(warps));
+    if (a.vdim <= 128) return launch_split<8, 3>(ctx, p, qtiles, warps, bytes(warps));
+    return launch_split<16, 2>(ctx, p, qtiles, warps, bytes(warps));
+}
+
+// ---- many rows: 128-row tiles on tcgen05 ------------------------------------------------------------------------------
+// One CTA per (128-row tile, kv head); a tile packs `rpt` rows times the group's heads, so the keys are read once for the
+// whole group. Keys come in tiles of 128.
+//   warp 0     TMA producer: the query tile once, K and V tiles through rings
+//   warp 1     tcgen05.mma issuer: S(t) = Q K(t)^T into one of two 128-column buffers, then O += P(t - 1) V(t - 1) with P
+//              read from TMEM (it overwrites the S it came from), so the tensor cores work on tile t while the weights of
+//              tile t - 1 are computed
+//   warps 2-5  even tiles: tcgen05.ld a row of S, cap, exponentiate, sum, tcgen05.st the bf16 weights
+//   warps 6-9  odd tiles
+// Without a running maximum O needs no correction: it stays in TMEM from the first tile to the last.
+// TMEM (all 512 columns): S/P buffers at 0 and 128, O at 256. It is allocated after the dependency wait, and dependents are
+// released only after the allocation, so no neighbouring launch can hold columns this kernel or its predecessor waits for.
+constexpr int TILE_THREADS = 320;
+constexpr uint32_t TILE_CHUNK = 128 * 128;   // 128 rows of 64 bf16 columns (one 128B-swizzled TMA box)
+
+struct TileParams {
+    HoloCausalArgs a;
+    uint32_t* status;
+    uint32_t group, rpt, qchunks, vchunks, kstages, vstages;
+};
+
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
+        ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar)
+        : "memory");
+}
+// A operand (128 x 16 bf16, two elements per 32-bit column) in TMEM
+__device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\ntcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n"
+        ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
+          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+        : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&v)[16]) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15};\n"
+        ::"r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]), "r"(v[10]),
+          "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(taddr)
+        : "memory");
+}
+
+__global__ void __launch_bounds__(TILE_THREADS, 1)
+causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                             const __grid_constant__ CUtensorMap map_v, const TileParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    const HoloCausalArgs& a = p.a;
+    const uint32_t raw = smem_u32(smem_raw);
+    const uint32_t base = (raw + 1023u) & ~1023u;
+    uint8_t* sm = smem_raw + (base - raw);
+    const uint32_t kbytes = p.qchunks * TILE_CHUNK, vbytes = p.vchunks * TILE_CHUNK;
+    const uint32_t s_q = base, s_k = s_q + kbytes, s_v = s_k + p.kstages * kbytes;
+    const uint32_t off_bars = (1 + p.kstages) * kbytes + p.vstages * vbytes;
+    const uint32_t bar_q = base + off_bars, bar_k_full = bar_q + 8, bar_k_empty = bar_k_full + 16, bar_v_full = bar_k_empty + 16,
+                   bar_v_empty = bar_v_full + 16, bar_s = bar_v_empty + 16, bar_p = bar_s + 16, bar_pv = bar_p + 16, bar_o = bar_pv + 16;
+    uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + off_bars + 128);
+    volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + off_bars + 132);
+    float* s_sum = reinterpret_cast<float*>(sm + off_bars + 256);   // [2][128]
+
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t g = blockIdx.x, qtile = gridDim.y - 1 - blockIdx.y;   // the tiles with the most keys first
+    const uint32_t row0 = qtile * p.rpt;
+    if (threadIdx.x == 0) {
+        mbar_init(bar_q, 1);
+        for (int s = 0; s < 2; ++s) {
+            mbar_init(bar_k_full + 8 * s, 1);
+            mbar_init(bar_k_empty + 8 * s, 1);
+            mbar_init(bar_v_full + 8 * s, 1);
+            mbar_init(bar_v_empty + 8 * s, 1);
+            mbar_init(bar_s + 8 * s, 1);
+            mbar_init(bar_p + 8 * s, 4);     // one arrival per weight warp
+            mbar_init(bar_pv + 8 * s, 1);
+        }
+        mbar_init(bar_o, 1);
+        *s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    holo_pdl_wait();
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(s_tmem)), "r"(512u) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    holo_pdl_trigger();
+    const uint32_t tmem_base = *s_tmem, tmem_o = tmem_base + 256;
+    const uint32_t pos = *a.pos;
+    const uint32_t visible = min(pos + min(row0 + p.rpt, a.rows), a.cache_rows);
+    const uint32_t ntiles = (visible + 127) / 128;
+
+    if (warp == 0) {
+        // ---------------- TMA producer ----------------
+        if (lane == 0) {
+            mbar_arrive_expect_tx(bar_q, p.qchunks * p.rpt * p.group * 128);
+            for (uint32_t c = 0; c < p.qchunks; ++c) tma_load_3d(s_q + c * TILE_CHUNK, &map_q, (int)(64 * c), (int)(g * p.group), (int)row0, bar_q);
+            uint32_t kt = 0, vt = 0;
+            bool ok = true;
+            for (uint32_t t = 0; t < ntiles && ok; ++t) {
+                const uint32_t ks = t % p.kstages, vs = t % p.vstages;
+                ok = t < p.kstages || mbar_wait(bar_k_empty + 8 * ks, (t / p.kstages - 1) & 1, s_abort, p.status);
+                if (!ok) break;
+                mbar_arrive_expect_tx(bar_k_full + 8 * ks, kbytes);
+                for (uint32_t c = 0; c < p.qchunks; ++c)
+                    tma_load_2d(s_k + ks * kbytes + c * TILE_CHUNK, &map_k, (int)(g * a.dim + 64 * c), (int)(t * 128), bar_k_full + 8 * ks);
+                ++kt;
+                ok = t < p.vstages || mbar_wait(bar_v_empty + 8 * vs, (t / p.vstages - 1) & 1, s_abort, p.status);
+                if (!ok) break;
+                mbar_arrive_expect_tx(bar_v_full + 8 * vs, vbytes);
+                for (uint32_t c = 0; c < p.vchunks; ++c)
+                    tma_load_2d(s_v + vs * vbytes + c * TILE_CHUNK, &map_v, (int)(g * a.vdim + 64 * c), (int)(t * 128), bar_v_full + 8 * vs);
+                ++vt;
+            }
+            if (!ok) {
+                // nothing may still be on its way into this CTA's shared memory when it ends
+                for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_q, 0); ++it) __nanosleep(64);
+                for (uint32_t t = kt > p.kstages ? kt - p.kstages : 0; t < kt; ++t)
+                    for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_k_full + 8 * (t % p.kstages), (t / p.kstages) & 1); ++it) __nanosleep(64);
+                for (uint32_t t = vt > p.vstages ? vt - p.vstages : 0; t < vt; ++t)
+                    for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_v_full + 8 * (t % p.vstages), (t / p.vstages) & 1); ++it) __nanosleep(64);
+            }
+        }
+    } else if (warp == 1) {
+        // ---------------- MMA issuer ----------------
+        if (lane == 0) {
+            // D = f32, A = B = bf16, M = 128; S: both operands K-major, N = 128; O: V is N-major, N = vdim
+            const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 3) << 17) | ((128u >> 4) << 24);
+            const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((a.vdim >> 3) << 17) | ((128u >> 4) << 24);
+            const uint32_t ksteps = a.dim / 16;
+            bool ok = mbar_wait(bar_q, 0, s_abort, p.status);
+            for (uint32_t t = 0; t <= ntiles && ok; ++t) {
+                if (t < ntiles) {
+                    const uint32_t ks = t % p.kstages, buf = t & 1u;
+                    ok = mbar_wait(bar_k_full + 8 * ks, (t / p.kstages) & 1, s_abort, p.status);
+                    // the weights of tile t - 2 share this buffer: their product must have read them
+                    if (ok && t >= 2) ok = mbar_wait(bar_pv + 8 * buf, ((t >> 1) - 1) & 1, s_abort, p.status);
+                    if (!ok) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    for (uint32_t k = 0; k < ksteps; ++k) {
+                        const uint32_t off = (k >> 2) * TILE_CHUNK + (k & 3) * 32;
+                        umma_bf16(tmem_base + buf * 128, smem_desc(s_q + off, 16, 1024), smem_desc(s_k + ks * kbytes + off, 16, 1024), idesc_s, k != 0);
+                    }
+                    umma_commit(bar_k_empty + 8 * ks);
+                    umma_commit(bar_s + 8 * buf);
+                }
+                if (t > 0) {
+                    const uint32_t u = t - 1, vs = u % p.vstages, buf = u & 1u;
+                    ok = mbar_wait(bar_p + 8 * buf, (u >> 1) & 1, s_abort, p.status) && mbar_wait(bar_v_full + 8 * vs, (u / p.vstages) & 1, s_abort, p.status);
+                    if (!ok) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+                    for (uint32_t k = 0; k < 8; ++k)
+                        umma_bf16_ts(tmem_o, tmem_base + buf * 128 + k * 8, smem_desc(s_v + vs * vbytes + k * 2048, TILE_CHUNK, 1024), idesc_o, (u | k) != 0);
+                    umma_commit(bar_v_empty + 8 * vs);
+                    umma_commit(bar_pv + 8 * buf);
+                }
+            }
+            if (ok) umma_commit(bar_o);
+        }
+    } else {
+        // ---------------- weights (TMEM lane quarter = warp % 4), then the output ----------------
+        const uint32_t quarter = warp & 3u, wg = (warp - 2) >> 2, tr = quarter * 32 + lane;
+        const uint32_t row = row0 + tr / p.group, head = g * p.group + tr % p.group;
+        const bool valid = tr < p.rpt * p.group && row < a.rows;
+        const uint32_t at = pos + min(row, a.rows - 1);
+        const uint32_t lanes = (quarter * 32u) << 16;
+        const float c2 = a.softcap * LOG2E;
+        const float c1 = 2.0f * LOG2E * a.scale * query_factor(at, a.temp_coef, a.temp_every) / a.softcap;
+        float sum = 0.0f;
+        bool ok = true;
+        for (uint32_t t = wg; t < ntiles; t += 2) {
+            ok = mbar_wait(bar_s + 8 * wg, (t >> 1) & 1, s_abort, p.status) && !*s_abort;
+            ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const uint32_t tmem_s = tmem_base + wg * 128 + lanes;
+            // every key of the tile is at or before the first row's position: no mask
+            const bool whole = t * 128 + 127 <= pos + row0;
+#pragma unroll 1
+            for (int c = 0; c < 4; ++c) {
+                uint32_t v[32], w[16];
+                tmem_ld32(tmem_s + c * 32, v);
+                const uint32_t key0 = t * 128 + c * 32;
+                float part = 0.0f;
+                if (whole) {
+#pragma unroll
+                    for (int x = 0; x < 16; ++x) {
+                        const float lo = capped_exp(__uint_as_float(v[2 * x]), c1, c2), hi = capped_exp(__uint_as_float(v[2 * x + 1]), c1, c2);
+                        part += lo + hi;
+                        w[x] = pack_bf16(lo, hi);
+                    }
+                } else {
+#pragma unroll
+                    for (int x = 0; x < 16; ++x) {
+                        const float lo = key0 + 2 * x <= at ? capped_exp(__uint_as_float(v[2 * x]), c1, c2) : 0.0f;
+                        const float hi = key0 + 2 * x + 1 <= at ? capped_exp(__uint_as_float(v[2 * x + 1]), c1, c2) : 0.0f;
+                        part += lo + hi;
+                        w[x] = pack_bf16(lo, hi);
+                    }
+                }
+                sum += part;
+                tmem_st16(tmem_s + c * 16, w);   // over scores this warp has already read
+            }
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar_p + 8 * wg) : "memory");
+        }
+        s_sum[wg * 128 + tr] = sum;
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        ok = mbar_wait(bar_o, 0, s_abort, p.status) && !*s_abort && !(*reinterpret_cast<volatile uint32_t*>(p.status) & 4u);
+        // the loads below are whole-warp instructions: the warp takes one decision
+        ok = __all_sync(0xffffffffu, ok);
+        if (ok) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const float denom = s_sum[tr] + s_sum[128 + tr] + (a.sink && valid ? ex2(a.sink[head] * LOG2E) : 0.0f);
+            const float inv = __fdiv_rn(1.0f, denom);
+            __nv_bfloat16* out = (__nv_bfloat16*)a.out + (uint64_t)row * a.ld + head * a.vdim;
+            for (uint32_t c = wg; c < a.vdim / 16; c += 2) {
+                uint32_t v[16], w[8];
+                tmem_ld16(tmem_o + lanes + c * 16, v);
+#pragma unroll
+                for (int x = 0; x < 8; ++x) w[x] = pack_bf16(__uint_as_float(v[2 * x]) * inv, __uint_as_float(v[2 * x + 1]) * inv);
+                if (valid) {
+                    reinterpret_cast<uint4*>(out + c * 16)[0] = make_uint4(w[0], w[1], w[2], w[3]);
+                    reinterpret_cast<uint4*>(out + c * 16)[1] = make_uint4(w[4], w[5], w[6], w[7]);
+                }
+            }
+        }
+    }
+    // everyone meets here, whatever happened above, so that TMEM is always released
+    __syncwarp();
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(512u) : "memory");
+    }
+}
+
+// Launches the tile kernel, or returns with *taken false when the shape does not suit it.
+int32_t try_tile(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
+    *taken = false;
+    TileParams p;
+    p.a = a;
+    p.status = ctx->dev_status;
+    p.group = a.heads / a.kv_heads;
+    if (a.dim > 256 || a.vdim > 256 || p.group > 128 || a.ld % 8 != 0 || encode_tiled_fn() == nullptr) return HOLO_OK;
+    p.rpt = 128 / p.group;
+    p.qchunks = (a.dim + 63) / 64;
+    p.vchunks = (a.vdim + 63) / 64;
+    const uint32_t extra = 256 + 1024 + 1024, limit = (uint32_t)ctx->smem_optin;   // barriers, row sums, alignment slack
+    auto bytes = [&](uint32_t ks, uint32_t vs) { return ((1 + ks) * p.qchunks + vs * p.vchunks) * TILE_CHUNK + extra; };
+    p.kstages = p.vstages = 2;
+    if (bytes(2, 2) > limit) p.kstages = 1;
+    if (bytes(p.kstages, 2) > limit) p.vstages = 1;
+    const uint32_t smem = bytes(p.kstages, p.vstages);
+    if (smem > limit) return HOLO_OK;
+    const uint32_t qtiles = (a.rows + p.rpt - 1) / p.rpt;
+    if (qtiles > 65535) return HOLO_OK;
+    CUtensorMap mq, mk, mv;
+    {   // q as [rows][heads][dim]: a box is 64 columns of the group's heads over rpt rows
+        cuuint64_t dims[3] = {a.dim, a.heads, a.rows};
+        cuuint64_t strides[2] = {(cuuint64_t)a.dim * 2, (cuuint64_t)a.heads * a.dim * 2};
+        cuuint32_t box[3] = {64, p.group, p.rpt};
+        cuuint32_t es[3] = {1, 1, 1};
+        const CUresult r = encode_tiled_fn()(&mq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(a.q), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+        if (r != CUDA_SUCCESS) return holo_fail(HOLO_ERR_DISPATCH, "dispatch failed: cuTensorMapEncodeTiled (attention) returned %d", (int)r);
+    }
+    HOLO_TRY(make_map_2d(&mk, a.k, (uint64_t)a.kv_heads * a.dim, a.cache_rows, 64, 128));
+    HOLO_TRY(make_map_2d(&mv, a.v, (uint64_t)a.kv_heads * a.vdim, a.cache_rows, 64, 128));
+    static thread_local int configured_device = -1;
+    if (configured_device != ctx->device) {
+        HOLO_CUDA(cudaFuncSetAttribute(causal_attention_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ctx->smem_optin));
+        configured_device = ctx->device;
+    }
+    *taken = true;
+    HOLO_CUDA(holo_launch_kernel(ctx, causal_attention_tile_kernel, dim3(a.kv_heads, qtiles), dim3(TILE_THREADS), smem, 1, mq, mk, mv, p));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
 }  // namespace
 
 int32_t holo_launch_causal_attention(holo_b200_ctx* ctx, const HoloCausalArgs& a) {
+    const bool capped16 = a.dtype == HOLO_DTYPE_BF16 && a.softcap > 0.0f && a.softcap <= CAP_LIMIT && a.dim % 16 == 0 && a.vdim % 16 == 0 &&
+                          a.ld % 2 == 0 && (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.out) & 15u) == 0 &&
+                          !getenv("HOLO_CAUSAL_GENERIC");
+    if (capped16) {
+        bool taken = false;
+        if (a.rows * (a.heads / a.kv_heads) <= 64) HOLO_TRY(try_split(ctx, a, &taken));
+        if (!taken) HOLO_TRY(try_tile(ctx, a, &taken));
+        if (taken) return HOLO_OK;
+    }
     return launch_generic(ctx, a);
 }

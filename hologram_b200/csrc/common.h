@@ -43,6 +43,7 @@ struct holo_b200_ctx {
     uint64_t stage_bytes = 0;
     // device-side error word (bounded waits record where they gave up)
     uint32_t* dev_status = nullptr;
+    float* causal_partials = nullptr;   // split-key partials of the causal attention, allocated once at a fixed size (graphs hold its address)
     uint32_t* attn_arrivals = nullptr;  // 65536 counters, zero between launches (decode attention)
     // launch every kernel with programmatic stream serialization (HOLO_PDL=0 turns it off)
     bool pdl = true;
