@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the B200 backend hot path.
 
-  python bench.py [--gpus N] [--steps K] [--warmup W] [--workload lut|lut_sweep|attention|matmul|gemv|w8a8|decoder]
+  python bench.py [--gpus N] [--steps K] [--warmup W] [--workload lut|lut_sweep|attention|matmul|gemv|w8a8|decoder|fokonex]
   python bench.py --impl reference ...      # the reference CPU path (oracle restatement) on host cores
 
 One JSON line on stdout (rank 0). Timed with CUDA events on the stream the kernels are
@@ -676,6 +676,185 @@ WORKLOADS = {"lut": workload_lut, "lut_sweep": workload_lut_sweep, "w8a8": workl
              "matmul": workload_matmul, "gemv": lambda *a: workload_matmul(*a, skinny=True)}
 
 
+# ------------------------------------------------------------------------------------------
+# Fokonex: throughput of whole steps and of every kernel of a layer alone, beside the like kernel of the Llama-style
+# decoder (its matmul, attention, norm) at the same size. Selected by --workload fokonex; prints one JSON line of its own.
+# ------------------------------------------------------------------------------------------
+
+FOKONEX_SIZES = {   # width, heads, kv_heads, dim, vdim, ff, vocab, layers
+    "w2048": (2048, 16, 4, 128, 128, 8192, 32000, 4),
+    "w3072": (3072, 24, 8, 96, 128, 12288, 32000, 4),
+    "w4096": (4096, 32, 8, 128, 128, 14336, 32000, 4),
+}
+
+
+def fokonex_config(size, n_layers=None):
+    from hologram_b200 import fokonex as fk
+    width, heads, kv, dim, vdim, ff, vocab, layers = FOKONEX_SIZES[size]
+    layers = n_layers or layers
+    spec = lambda: fk.AttentionSpec(heads, kv, dim, vdim, dim ** -0.5, 30.0, 0.1, 1024.0)
+    return fk.FokonexConfig(vocab, width, [fk.LayerSpec(i, spec(), ff, i) for i in range(layers)], 1e-6, 0.5, 0.25)
+
+
+def bench_fokonex(be, torch, args, stream):
+    import hologram_b200 as hb
+    from hologram_b200 import decode, decoder_holo as dh, fokonex as fk, kernel_call as kc, safetensors_io as st
+    peaks = measured_peaks()
+    rows_prefill, cached = 2048, 4096
+    iters, warm = max(args.steps, 20), max(args.warmup, 3)
+    sizes = [x for x in os.environ.get("HOLO_BENCH_FOKONEX", ",".join(FOKONEX_SIZES)).split(",") if x]
+
+    def time_ms(run, n=iters):
+        for i in range(warm):
+            run(i)
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(stream)
+        for i in range(n):
+            run(warm + i)
+        e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    def rotated(slots, make, copy_bytes):
+        """`make(ws)` over as many copies of the operands as exceed L2 together; run(i) dispatches copy i % n."""
+        n = max(1, min(64, -(-300_000_000 // copy_bytes)))
+        sets = []
+        for _ in range(n):
+            ws = hb.DeviceWorkspace(be, len(slots))
+            keep = []
+            for i, (numel, dtype, fill) in enumerate(slots):
+                t = torch.randn(numel, device="cuda").to(dtype) * 0.05 if fill == "randn" else torch.full((numel,), fill, device="cuda", dtype=dtype)
+                ws.bind(i, t.data_ptr(), t.numel() * t.element_size())
+                keep.append(t)
+            sets.append((ws, keep))
+        call = make()
+        torch.cuda.synchronize()
+        return lambda i: be.dispatch(call, sets[i % n][0]), sets
+
+    def kernel(name, slots, make, nbytes, flops):
+        copy = sum(n * (4 if d in (torch.float32, torch.int32) else 1 if d == torch.int8 else 2) for n, d, _ in slots)
+        run, keep = rotated(slots, make, copy)
+        us = time_ms(run) * 1e3
+        t_mem, t_mma = nbytes / peaks["hbm_gbs"] / 1e3, flops / peaks["bf16_tflops"] / 1e6     # us
+        del keep
+        return {"kernel": name, "us": round(us, 2), "bound": "hbm" if t_mem >= t_mma else "tensor", "roofline_us": round(max(t_mem, t_mma), 2),
+                "frac": round(max(t_mem, t_mma) / us, 3)}
+
+    bf, f32, i32, i8 = torch.bfloat16, torch.float32, torch.int32, torch.int8
+    rb = kc.rb
+    out = []
+    for size in sizes:
+        width, heads, kv, dim, vdim, ff, vocab, layers = FOKONEX_SIZES[size]
+        cfg = fokonex_config(size)
+        g = torch.Generator(device="cuda").manual_seed(0xF0)
+        tensors = {}
+        for name, shape in cfg.tensor_shapes().items():
+            t = torch.randn(shape, generator=g, device="cuda") * 0.02
+            tensors[name] = st.Tensor("BF16", t.to(bf).view(torch.int16).cpu().numpy().view(np.uint16))
+        model = fk.FokonexModel(cfg, tensors)
+        runner = decode.StepRunner(be, model, cached + rows_prefill, max_rows=rows_prefill)
+        rng = np.random.default_rng(0)
+        ids = rng.integers(0, vocab, size=rows_prefill).astype(np.int32)
+        res = {"size": size, "config": f"width {width}, {heads} q / {kv} kv heads, dim {dim}, vdim {vdim}, ff {ff}, vocab {vocab}, {layers} layers"}
+        for i in range(cached // rows_prefill):      # fill the cache through the public step
+            runner.step("bench", ids, [])
+        # device-resident steps: the captured graphs, inputs as the last step left them
+        lin = width * (heads * dim + kv * (dim + vdim) + ff) + (heads * vdim + ff) * width
+        pre = runner._steps[rows_prefill][0]
+        for base in (0, cached):
+            step_in = np.zeros(4 + rows_prefill, np.int32)
+            step_in[0], step_in[4:] = base, ids
+            pre.write("step_in", step_in)
+            ms = time_ms(lambda i: pre.execute(), 10)
+            flops = layers * (2.0 * rows_prefill * lin + 2.0 * heads * (dim + vdim) * rows_prefill * (base + (rows_prefill + 1) / 2))
+            res[f"prefill_{rows_prefill}_at_{base}"] = {"ms": round(ms, 3), "tokens_per_s": round(rows_prefill / ms * 1e3), "tflops": round(flops / ms / 1e9, 1),
+                                                        "frac": round(flops / ms / 1e9 / (peaks["bf16_tflops_sustained"] or peaks["bf16_tflops"]), 3)}
+        one = runner._steps[1][0]
+        runner.step("bench", ids[:1])
+        step_in = np.zeros(5, np.int32)
+        step_in[0], step_in[4] = cached, 1
+        one.write("step_in", step_in)
+        ms = time_ms(lambda i: one.execute(), 100)
+        nbytes = 2 * (layers * (lin + cached * kv * (dim + vdim)) + width * vocab)
+        res["decode_at_4096"] = {"ms": round(ms, 4), "tokens_per_s": round(1e3 / ms, 1), "gbs": round(nbytes / ms / 1e6), "frac": round(nbytes / ms / 1e6 / peaks["hbm_gbs"], 3)}
+        t0 = time.perf_counter()
+        for i in range(50):
+            runner.step("bench", ids[i:i + 1])
+        res["decode_e2e_tokens_per_s"] = round(50 / (time.perf_counter() - t0), 1)
+        runner.close()
+        # the Llama-style decoder at the same width, heads and feed-forward width (three FFN matrices, int8 KV), batch 1
+        dcfg = dh.DecoderConfig(d_model=width, n_heads=heads, n_kv_heads=kv, head_dim=dim, ffn=ff, vocab=vocab, n_layers=layers, batch=1, bucket=cached)
+        dsh = {"wq": (width, heads * dim), "wk": (width, kv * dim), "wv": (width, kv * dim), "wo": (heads * dim, width), "wg": (width, ff), "wu": (width, ff),
+               "wd": (ff, width), "embed": (vocab, width), "lm_head": (width, vocab)}
+
+        def dweights(name):
+            base = name.split(".")[-1]
+            return (torch.randn(dsh.get(base, (width,)), generator=g, device="cuda") * 0.02).to(bf).view(torch.int16).cpu().numpy().view(np.uint16)
+        img, info = dh.build_decoder_step(dcfg, weights=dweights)
+        sess = hb.InferenceSession(be, img, verify=False)
+        vals = {"token_ids": np.array([1], np.int32), "pos": np.array([cached - 1], np.int32), "valid_len": np.array([cached], np.int32)}
+        vals["cos_q"], vals["sin_q"] = dh.rope_tables(dcfg, 7, heads)
+        vals["cos_k"], vals["sin_k"] = dh.rope_tables(dcfg, 7, kv)
+        for n, v in vals.items():
+            sess.write(n, v)
+        sess.execute()
+        be.synchronize()
+        sess.capture()
+        ms = time_ms(lambda i: sess.execute(), 100)
+        dbytes = 2 * (layers * (width * (heads + 2 * kv) * dim + heads * dim * width + 3 * width * ff) + width * vocab) + layers * cached * kv * 2 * (dim + 4)
+        res["llama_style_decode_batch1"] = {"ms": round(ms, 4), "tokens_per_s": round(1e3 / ms, 1), "gbs": round(dbytes / ms / 1e6), "frac": round(dbytes / ms / 1e6 / peaks["hbm_gbs"], 3)}
+        sess.close()
+        del img
+        # kernels alone
+        l0 = cfg.layers[0]
+        (cq, ck, cv, cu), cols = model.in_columns(l0)
+        a = l0.mixer
+        ka = a.heads * a.vdim_p + l0.ff_p
+        table = []
+        for m in (1, rows_prefill):
+            def lin_in():
+                segs = [kc.LinearSeg(rb(2), kc.NONE, cq, heads * a.dim_p, 0, heads * a.dim_p, 0, kc.DTYPE_BF16), kc.LinearSeg(rb(3), rb(6), ck, kv * a.dim_p, 0, kv * a.dim_p, 0, kc.DTYPE_BF16),
+                        kc.LinearSeg(rb(4), rb(6), cv, kv * a.vdim_p, 0, kv * a.vdim_p, 0, kc.DTYPE_BF16), kc.LinearSeg(rb(5), kc.NONE, cu, ff, width, ff, 1, kc.DTYPE_BF16)]
+                return kc.KernelCall.Linear(kc.LinearCall.make(rb(0), rb(1), segs, m, width, cols, kc.DTYPE_BF16, lda=2 * width))
+            n_in = heads * dim + kv * (dim + vdim) + ff
+            slots = [(m * 2 * width, bf, "randn"), (width * cols, bf, "randn"), (m * heads * a.dim_p, bf, 0), (m * kv * a.dim_p, bf, 0), (m * kv * a.vdim_p, bf, 0), (m * ff, bf, 0), (1, i32, 0)]
+            table.append(kernel(f"Linear q/k/v/up, {m} rows", slots, lin_in, 2 * (width * n_in + m * (2 * width + n_in)), 2.0 * m * width * n_in))
+            mm = lambda k, n: (lambda: kc.KernelCall.MatMul(kc.MatMulCall(rb(0), rb(1), rb(2), m, k, n, kc.DTYPE_BF16, 0)))
+            table.append(kernel(f"  like: MatMul {m}x{width}x{n_in}", [(m * width, bf, "randn"), (width * n_in, bf, "randn"), (m * n_in, bf, 0)], mm(width, n_in),
+                                2 * (width * n_in + m * (width + n_in)), 2.0 * m * width * n_in))
+
+            def lin_out():
+                return kc.KernelCall.Linear(kc.LinearCall.make(rb(0), rb(1), [kc.LinearSeg(rb(2), kc.NONE, 0, width, 0, width, 0, kc.DTYPE_F32)], m, ka, width, kc.DTYPE_BF16, residual=rb(2), alpha=0.5))
+            table.append(kernel(f"Linear o/down + residual, {m} rows", [(m * ka, bf, "randn"), (ka * width, bf, "randn"), (m * width, f32, 0)], lin_out,
+                                2 * (ka * width + m * ka) + 8 * m * width, 2.0 * m * width * ka))
+            table.append(kernel(f"  like: MatMul {m}x{ka}x{width}", [(m * ka, bf, "randn"), (ka * width, bf, "randn"), (m * width, bf, 0)], mm(ka, width),
+                                2 * (ka * width + m * (width + ka)), 2.0 * m * width * ka))
+            table.append(kernel(f"RmsNormMulti, {m} rows", [(m * width, f32, "randn"), (width, f32, 1), (width, f32, 1), (m * 2 * width, bf, 0)],
+                                lambda: kc.KernelCall.RmsNormMulti(kc.RmsNormMultiCall(rb(0), rb(1), rb(2), rb(3), m, width, width, kc.f32_bits(1e-6), kc.DTYPE_BF16)), 8 * m * width, 0))
+            table.append(kernel(f"  like: RmsNorm, {m} rows", [(m * width, bf, "randn"), (width, bf, 1), (m * width, bf, 0)],
+                                lambda: kc.KernelCall.RmsNorm(kc.NormCall(rb(0), rb(1), kc.NONE, kc.NONE, rb(2), m, width, 0, 0, kc.f32_bits(1e-6), kc.DTYPE_BF16)), 4 * m * width, 0))
+            L = cached
+            base = L - m
+            keys = m * (base + (m + 1) / 2)
+            table.append(kernel(f"CausalAttention, {m} rows at {base}",
+                                [(m * heads * a.dim_p, bf, "randn"), (L * kv * a.dim_p, bf, "randn"), (L * kv * a.vdim_p, bf, "randn"), (1, i32, base), (heads, f32, 0), (m * heads * a.vdim_p, bf, 0)],
+                                lambda: kc.KernelCall.CausalAttention(kc.CausalAttentionCall(*[rb(i) for i in range(6)], m, heads, kv, a.dim_p, a.vdim_p, L, heads * a.vdim_p,
+                                                                      kc.f32_bits(dim ** -0.5), kc.f32_bits(30.0), kc.f32_bits(0.1), kc.f32_bits(1024.0), kc.DTYPE_BF16)),
+                                2 * (L * kv * (dim + vdim) + m * heads * (dim + vdim)), 2.0 * heads * (dim + vdim) * keys))
+            if m == 1:
+                slots = [(heads * dim, bf, "randn"), (kv * L * dim, i8, 1), (kv * L, f32, 0.01), (kv * L * dim, i8, 1), (kv * L, f32, 0.01), (kv * dim, i8, 1), (kv, f32, 0.01), (kv * dim, i8, 1), (kv, f32, 0.01), (1, i32, L), (heads * dim, bf, 0)]
+                table.append(kernel("  like: DecodeAttentionValidQ8, batch 1", slots,
+                                    lambda: kc.KernelCall.DecodeAttentionValidQ8(kc.DecodeAttentionValidQ8Call(*[rb(i) for i in range(11)], 1, heads, kv, 1, L, 1, dim, 0, kc.DTYPE_BF16)), 2 * L * kv * (dim + 4), 0))
+            else:
+                slots = [(heads * m * dim, bf, "randn"), (kv * m * dim, bf, "randn"), (kv * m * dim, bf, "randn"), (heads * m * dim, bf, 0)]
+                table.append(kernel(f"  like: Attention (legacy prefill), {m} rows at 0", slots,
+                                    lambda: kc.KernelCall.Attention(kc.AttentionCall(rb(0), rb(1), rb(2), rb(3), 1, heads, m, dim, kv, 1, 0, kc.DTYPE_BF16)), 2 * 2 * m * (heads + kv) * dim, 4.0 * heads * dim * m * (m + 1) / 2))
+        res["kernels"] = table
+        out.append(res)
+    return out
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -724,6 +903,18 @@ def main():
         uid = [hb.B200Backend.nccl_unique_id() if rank == 0 else None]
         dist.broadcast_object_list(uid, src=0)
         be.init_tp(uid[0], rank, world)
+    if args.workload == "fokonex":
+        sampler = ClockSampler(local_rank)
+        sampler.start()
+        results = bench_fokonex(be, torch, args, stream)
+        clocks = sampler.stop()
+        big = results[-1]["decode_at_4096"]
+        emit({"metric": "fokonex_decode_tokens_per_s", "value": big["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": 100, "warmup": args.warmup,
+              "ms_per_step": big["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 (f32 residual)",
+              "data": "synthetic (random weights)", "config": {"model": "Fokonex " + results[-1]["config"], "global_batch": 1, "seq_len": 4096,
+              "l2": "kernels alone rotate over copies that exceed L2; a step's weights exceed L2"}, "gpu_launches": be.launch_count, "clocks": clocks,
+              "peaks": measured_peaks(), "sizes": results})
+        return
     fn = WORKLOADS[args.workload]
     shard_world = args.shard_of if (args.shard_of > 1 and world == 1) else world
     wl = fn(be, torch, rank, args, shard_world) if args.workload in ("attention", "decoder") else fn(be, torch, rank, args)

@@ -121,6 +121,42 @@ __device__ __forceinline__ float rcp(float x) {
 // tanh(y) = 1 - 2 / (exp(2y) + 1), so the exponent in log2 units is c2 - 2 c2 / (2^(s c1) + 1).
 __device__ __forceinline__ float capped_exp(float s, float c1, float c2) { return ex2(fmaf(-2.0f * c2, rcp(ex2(s * c1) + 1.0f), c2)); }
 
+// The same for scores well inside the cap, |y| = |s factor / cap| <= TANH_SMALL, two at a time on the packed f32 pipe: tanh(y) / y as
+// a degree-5 polynomial in y^2 (a Chebyshev fit over the interval; |error| of tanh below 1e-7, f32 rounding included). One
+// special-function operation per score instead of three, which is what bounds the many-row kernel.
+constexpr float TANH_SMALL = 0.75f;
+__device__ __forceinline__ uint64_t pair(float lo, float hi) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(uint64_t v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+// c0 = factor / cap, c2 = cap log2(e), each twice
+__device__ __forceinline__ float2 capped_exp_small(uint64_t s, uint64_t c0, uint64_t c2) {
+    const uint64_t y = mul2(s, c0), z = mul2(y, y);
+    uint64_t t = fma2(z, pair(-0.0047239522f, -0.0047239522f), pair(0.0195937865f, 0.0195937865f));
+    t = fma2(t, z, pair(-0.0533498190f, -0.0533498190f));
+    t = fma2(t, z, pair(0.1332551539f, 0.1332551539f));
+    t = fma2(t, z, pair(-0.3333296776f, -0.3333296776f));
+    t = fma2(t, z, pair(1.0f, 1.0f));
+    const float2 e = unpair(mul2(mul2(t, y), c2));
+    return make_float2(ex2(e.x), ex2(e.y));
+}
+
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&h);
@@ -375,21 +411,22 @@ int32_t try_split(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
 // One CTA per (128-row tile, kv head); a tile packs `rpt` rows times the group's heads, so the keys are read once for the
 // whole group. Keys come in tiles of 128.
 //   warp 0     TMA producer: the query tile once, K and V tiles through rings
-//   warp 1     tcgen05.mma issuer: S(t) = Q K(t)^T into one of two 128-column buffers, then O += P(t - 1) V(t - 1) with P
-//              read from TMEM (it overwrites the S it came from), so the tensor cores work on tile t while the weights of
-//              tile t - 1 are computed
-//   warps 2-5  even tiles: tcgen05.ld a row of S, cap, exponentiate, sum, tcgen05.st the bf16 weights
-//   warps 6-9  odd tiles
+//   warp 1     tcgen05.mma issuer: S(t) = Q K(t)^T into one of two 128-column buffers, O += P(t) V(t) with P read from TMEM;
+//              as soon as the weights of tile t are stored (its scores are then dead) S(t + 2) is issued, then tile t's product
+//   warps 2-17 weights, four groups of four warps (one per TMEM lane quarter): group i takes key half i / 2 of the tiles of
+//              buffer i % 2: tcgen05.ld half a row of S, cap, exponentiate, sum, tcgen05.st the bf16 weights
 // Without a running maximum O needs no correction: it stays in TMEM from the first tile to the last.
-// TMEM (all 512 columns): S/P buffers at 0 and 128, O at 256. It is allocated after the dependency wait, and dependents are
+// TMEM (all 512 columns): S at 0 and 128, O at 256, P at 384 and 448 when vdim leaves room, else over the S it came from,
+// each key half's weights over the first half of its scores (S(t + 2) then waits for tile t's product). It is allocated after the dependency wait, and dependents are
 // released only after the allocation, so no neighbouring launch can hold columns this kernel or its predecessor waits for.
-constexpr int TILE_THREADS = 320;
+constexpr int TILE_THREADS = 576;
 constexpr uint32_t TILE_CHUNK = 128 * 128;   // 128 rows of 64 bf16 columns (one 128B-swizzled TMA box)
 
 struct TileParams {
     HoloCausalArgs a;
     uint32_t* status;
     uint32_t group, rpt, qchunks, vchunks, kstages, vstages;
+    uint32_t alias;   // P lies over S
 };
 
 __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
@@ -412,6 +449,38 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
           "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
         : "r"(taddr));
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+// The two halves of tmem_ld32: request 32 columns; wait for everything requested (the values pass through the wait, so that
+// no use of them can be scheduled before it).
+__device__ __forceinline__ void tmem_ld32_request(uint32_t taddr, uint32_t (&v)[32]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
+        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
+        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];\n"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
+          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
+          "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
+          "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
+        : "r"(taddr));
+}
+__device__ __forceinline__ void tmem_ld32_wait(uint32_t (&v)[32]) {
+    asm volatile("tcgen05.wait::ld.sync.aligned;"
+                 : "+r"(v[0]), "+r"(v[1]), "+r"(v[2]), "+r"(v[3]), "+r"(v[4]), "+r"(v[5]), "+r"(v[6]), "+r"(v[7]), "+r"(v[8]),
+                   "+r"(v[9]), "+r"(v[10]), "+r"(v[11]), "+r"(v[12]), "+r"(v[13]), "+r"(v[14]), "+r"(v[15]), "+r"(v[16]),
+                   "+r"(v[17]), "+r"(v[18]), "+r"(v[19]), "+r"(v[20]), "+r"(v[21]), "+r"(v[22]), "+r"(v[23]), "+r"(v[24]),
+                   "+r"(v[25]), "+r"(v[26]), "+r"(v[27]), "+r"(v[28]), "+r"(v[29]), "+r"(v[30]), "+r"(v[31])::"memory");
+}
+// ... and for a second array of the same request
+__device__ __forceinline__ void tmem_ld32_pass(uint32_t (&v)[32]) {
+    asm volatile("" : "+r"(v[0]), "+r"(v[1]), "+r"(v[2]), "+r"(v[3]), "+r"(v[4]), "+r"(v[5]), "+r"(v[6]), "+r"(v[7]), "+r"(v[8]),
+                   "+r"(v[9]), "+r"(v[10]), "+r"(v[11]), "+r"(v[12]), "+r"(v[13]), "+r"(v[14]), "+r"(v[15]), "+r"(v[16]),
+                   "+r"(v[17]), "+r"(v[18]), "+r"(v[19]), "+r"(v[20]), "+r"(v[21]), "+r"(v[22]), "+r"(v[23]), "+r"(v[24]),
+                   "+r"(v[25]), "+r"(v[26]), "+r"(v[27]), "+r"(v[28]), "+r"(v[29]), "+r"(v[30]), "+r"(v[31])::"memory");
+}
+__device__ __forceinline__ void tmem_st8(uint32_t taddr, const uint32_t (&v)[8]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%8], {%0, %1, %2, %3, %4, %5, %6, %7};\n"
+                 ::"r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(taddr)
+                 : "memory");
 }
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&v)[16]) {
     asm volatile(
@@ -436,7 +505,7 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
                    bar_v_empty = bar_v_full + 16, bar_s = bar_v_empty + 16, bar_p = bar_s + 16, bar_pv = bar_p + 16, bar_o = bar_pv + 16;
     uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + off_bars + 128);
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + off_bars + 132);
-    float* s_sum = reinterpret_cast<float*>(sm + off_bars + 256);   // [2][128]
+    float* s_sum = reinterpret_cast<float*>(sm + off_bars + 256);   // [4][128]
 
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t g = blockIdx.x, qtile = gridDim.y - 1 - blockIdx.y;   // the tiles with the most keys first
@@ -449,7 +518,7 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
             mbar_init(bar_v_full + 8 * s, 1);
             mbar_init(bar_v_empty + 8 * s, 1);
             mbar_init(bar_s + 8 * s, 1);
-            mbar_init(bar_p + 8 * s, 4);     // one arrival per weight warp
+            mbar_init(bar_p + 8 * s, 8);     // one arrival per weight warp
             mbar_init(bar_pv + 8 * s, 1);
         }
         mbar_init(bar_o, 1);
@@ -508,96 +577,128 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
             const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 3) << 17) | ((128u >> 4) << 24);
             const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((a.vdim >> 3) << 17) | ((128u >> 4) << 24);
             const uint32_t ksteps = a.dim / 16;
-            bool ok = mbar_wait(bar_q, 0, s_abort, p.status);
-            for (uint32_t t = 0; t <= ntiles && ok; ++t) {
-                if (t < ntiles) {
-                    const uint32_t ks = t % p.kstages, buf = t & 1u;
-                    ok = mbar_wait(bar_k_full + 8 * ks, (t / p.kstages) & 1, s_abort, p.status);
-                    // the weights of tile t - 2 share this buffer: their product must have read them
-                    if (ok && t >= 2) ok = mbar_wait(bar_pv + 8 * buf, ((t >> 1) - 1) & 1, s_abort, p.status);
-                    if (!ok) break;
-                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                    for (uint32_t k = 0; k < ksteps; ++k) {
-                        const uint32_t off = (k >> 2) * TILE_CHUNK + (k & 3) * 32;
-                        umma_bf16(tmem_base + buf * 128, smem_desc(s_q + off, 16, 1024), smem_desc(s_k + ks * kbytes + off, 16, 1024), idesc_s, k != 0);
-                    }
-                    umma_commit(bar_k_empty + 8 * ks);
-                    umma_commit(bar_s + 8 * buf);
+            auto scores = [&](uint32_t t) {       // issue S(t)
+                const uint32_t ks = t % p.kstages, buf = t & 1u;
+                if (!mbar_wait(bar_k_full + 8 * ks, (t / p.kstages) & 1, s_abort, p.status)) return false;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                for (uint32_t k = 0; k < ksteps; ++k) {
+                    const uint32_t off = (k >> 2) * TILE_CHUNK + (k & 3) * 32;
+                    umma_bf16(tmem_base + buf * 128, smem_desc(s_q + off, 16, 1024), smem_desc(s_k + ks * kbytes + off, 16, 1024), idesc_s, k != 0);
                 }
-                if (t > 0) {
-                    const uint32_t u = t - 1, vs = u % p.vstages, buf = u & 1u;
-                    ok = mbar_wait(bar_p + 8 * buf, (u >> 1) & 1, s_abort, p.status) && mbar_wait(bar_v_full + 8 * vs, (u / p.vstages) & 1, s_abort, p.status);
-                    if (!ok) break;
-                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                umma_commit(bar_k_empty + 8 * ks);
+                umma_commit(bar_s + 8 * buf);
+                return true;
+            };
+            bool ok = mbar_wait(bar_q, 0, s_abort, p.status) && scores(0) && (ntiles < 2 || scores(1));
+            for (uint32_t t = 0; t < ntiles && ok; ++t) {
+                const uint32_t vs = t % p.vstages, buf = t & 1u;
+                ok = mbar_wait(bar_p + 8 * buf, (t >> 1) & 1, s_abort, p.status);
+                if (!ok) break;
+                if (!p.alias && t + 2 < ntiles) ok = scores(t + 2);
+                ok = ok && mbar_wait(bar_v_full + 8 * vs, (t / p.vstages) & 1, s_abort, p.status);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                const uint32_t tmem_p = tmem_base + (p.alias ? buf * 128 : 384 + buf * 64);
 #pragma unroll
-                    for (uint32_t k = 0; k < 8; ++k)
-                        umma_bf16_ts(tmem_o, tmem_base + buf * 128 + k * 8, smem_desc(s_v + vs * vbytes + k * 2048, TILE_CHUNK, 1024), idesc_o, (u | k) != 0);
-                    umma_commit(bar_v_empty + 8 * vs);
-                    umma_commit(bar_pv + 8 * buf);
-                }
+                for (uint32_t k = 0; k < 8; ++k)
+                    umma_bf16_ts(tmem_o, tmem_p + k * 8 + (p.alias && k >= 4 ? 32 : 0), smem_desc(s_v + vs * vbytes + k * 2048, TILE_CHUNK, 1024), idesc_o, (t | k) != 0);
+                umma_commit(bar_v_empty + 8 * vs);
+                umma_commit(bar_pv + 8 * buf);
+                if (p.alias && t + 2 < ntiles) ok = mbar_wait(bar_pv + 8 * buf, (t >> 1) & 1, s_abort, p.status) && scores(t + 2);
             }
             if (ok) umma_commit(bar_o);
         }
     } else {
         // ---------------- weights (TMEM lane quarter = warp % 4), then the output ----------------
-        const uint32_t quarter = warp & 3u, wg = (warp - 2) >> 2, tr = quarter * 32 + lane;
+        const uint32_t quarter = warp & 3u, wg = (warp - 2) >> 2, buf = wg & 1u, half = wg >> 1, tr = quarter * 32 + lane;
         const uint32_t row = row0 + tr / p.group, head = g * p.group + tr % p.group;
         const bool valid = tr < p.rpt * p.group && row < a.rows;
         const uint32_t at = pos + min(row, a.rows - 1);
         const uint32_t lanes = (quarter * 32u) << 16;
         const float c2 = a.softcap * LOG2E;
-        const float c1 = 2.0f * LOG2E * a.scale * query_factor(at, a.temp_coef, a.temp_every) / a.softcap;
+        const float c0 = a.scale * query_factor(at, a.temp_coef, a.temp_every) / a.softcap, c1 = 2.0f * LOG2E * c0;
+        const float small = TANH_SMALL / fabsf(c0);      // scores up to here take the short form
+        const uint64_t c0_2 = pair(c0, c0), c2_2 = pair(c2, c2);
         float sum = 0.0f;
         bool ok = true;
-        for (uint32_t t = wg; t < ntiles; t += 2) {
-            ok = mbar_wait(bar_s + 8 * wg, (t >> 1) & 1, s_abort, p.status) && !*s_abort;
+        for (uint32_t t = buf; t < ntiles; t += 2) {
+            ok = mbar_wait(bar_s + 8 * buf, (t >> 1) & 1, s_abort, p.status) && !*s_abort;
             ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t tmem_s = tmem_base + wg * 128 + lanes;
+            const uint32_t tmem_s = tmem_base + buf * 128 + half * 64 + lanes;
+            const uint32_t tmem_p = (p.alias ? tmem_s : tmem_base + 384 + buf * 64 + half * 32 + lanes);
+            const uint32_t key0 = t * 128 + half * 64;
             // every key of the tile is at or before the first row's position: no mask
             const bool whole = t * 128 + 127 <= pos + row0;
-#pragma unroll 1
-            for (int c = 0; c < 4; ++c) {
-                uint32_t v[32], w[16];
-                tmem_ld32(tmem_s + c * 32, v);
-                const uint32_t key0 = t * 128 + c * 32;
-                float part = 0.0f;
-                if (whole) {
+            uint32_t v[2][32];
+            tmem_ld32_request(tmem_s, v[0]);
+            tmem_ld32_request(tmem_s + 32, v[1]);
+            tmem_ld32_wait(v[0]);
+            tmem_ld32_pass(v[1]);
+            float most[4] = {};
+#pragma unroll
+            for (int x = 0; x < 32; ++x) most[x & 3] = fmaxf(most[x & 3], fmaxf(fabsf(__uint_as_float(v[0][x])), fabsf(__uint_as_float(v[1][x]))));
+            const bool short_form = __all_sync(0xffffffffu, fmaxf(fmaxf(most[0], most[1]), fmaxf(most[2], most[3])) <= small);
+            if (!p.alias && t >= 2) {   // the product of tile t - 2 reads this P buffer
+                ok = mbar_wait(bar_pv + 8 * buf, ((t >> 1) - 1) & 1, s_abort, p.status);
+                ok = __all_sync(0xffffffffu, ok);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            }
+            if (short_form) {
+                uint64_t s2[2] = {0, 0};
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    uint32_t w[16];
 #pragma unroll
                     for (int x = 0; x < 16; ++x) {
-                        const float lo = capped_exp(__uint_as_float(v[2 * x]), c1, c2), hi = capped_exp(__uint_as_float(v[2 * x + 1]), c1, c2);
-                        part += lo + hi;
-                        w[x] = pack_bf16(lo, hi);
+                        float2 e = capped_exp_small(pair(__uint_as_float(v[c][2 * x]), __uint_as_float(v[c][2 * x + 1])), c0_2, c2_2);
+                        if (!whole) {
+                            e.x = key0 + c * 32 + 2 * x <= at ? e.x : 0.0f;
+                            e.y = key0 + c * 32 + 2 * x + 1 <= at ? e.y : 0.0f;
+                        }
+                        s2[x & 1] = fma2(pair(e.x, e.y), pair(1.0f, 1.0f), s2[x & 1]);
+                        w[x] = pack_bf16(e.x, e.y);
                     }
-                } else {
-#pragma unroll
-                    for (int x = 0; x < 16; ++x) {
-                        const float lo = key0 + 2 * x <= at ? capped_exp(__uint_as_float(v[2 * x]), c1, c2) : 0.0f;
-                        const float hi = key0 + 2 * x + 1 <= at ? capped_exp(__uint_as_float(v[2 * x + 1]), c1, c2) : 0.0f;
-                        part += lo + hi;
-                        w[x] = pack_bf16(lo, hi);
-                    }
+                    tmem_st16(tmem_p + c * 16, w);   // aliased: over scores this warp has already read
                 }
-                sum += part;
-                tmem_st16(tmem_s + c * 16, w);   // over scores this warp has already read
+                const float2 s1 = unpair(s2[0]), s3 = unpair(s2[1]);
+                sum += (s1.x + s1.y) + (s3.x + s3.y);
+            } else {
+#pragma unroll 1
+                for (uint32_t c = 0; c < 4; ++c) {   // compact: the scores are fetched again, sixteen at a time
+                    uint32_t u[16], w[8];
+                    tmem_ld16(tmem_s + c * 16, u);
+                    float part = 0.0f;
+#pragma unroll
+                    for (int x = 0; x < 8; ++x) {
+                        const uint32_t key = key0 + c * 16 + 2 * x;
+                        const float lo = key <= at ? capped_exp(__uint_as_float(u[2 * x]), c1, c2) : 0.0f;
+                        const float hi = key + 1 <= at ? capped_exp(__uint_as_float(u[2 * x + 1]), c1, c2) : 0.0f;
+                        part += lo + hi;
+                        w[x] = pack_bf16(lo, hi);
+                    }
+                    sum += part;
+                    tmem_st8(tmem_p + c * 8, w);
+                }
             }
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
-            if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar_p + 8 * wg) : "memory");
+            if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar_p + 8 * buf) : "memory");
         }
         s_sum[wg * 128 + tr] = sum;
-        asm volatile("bar.sync 1, 256;" ::: "memory");
+        asm volatile("bar.sync 1, 512;" ::: "memory");
         ok = mbar_wait(bar_o, 0, s_abort, p.status) && !*s_abort && !(*reinterpret_cast<volatile uint32_t*>(p.status) & 4u);
         // the loads below are whole-warp instructions: the warp takes one decision
         ok = __all_sync(0xffffffffu, ok);
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float denom = s_sum[tr] + s_sum[128 + tr] + (a.sink && valid ? ex2(a.sink[head] * LOG2E) : 0.0f);
+            const float denom = (s_sum[tr] + s_sum[128 + tr]) + (s_sum[256 + tr] + s_sum[384 + tr]) + (a.sink && valid ? ex2(a.sink[head] * LOG2E) : 0.0f);
             const float inv = __fdiv_rn(1.0f, denom);
             __nv_bfloat16* out = (__nv_bfloat16*)a.out + (uint64_t)row * a.ld + head * a.vdim;
-            for (uint32_t c = wg; c < a.vdim / 16; c += 2) {
+            for (uint32_t c = wg; c < a.vdim / 16; c += 4) {
                 uint32_t v[16], w[8];
                 tmem_ld16(tmem_o + lanes + c * 16, v);
 #pragma unroll
@@ -630,11 +731,15 @@ int32_t try_tile(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
     p.rpt = 128 / p.group;
     p.qchunks = (a.dim + 63) / 64;
     p.vchunks = (a.vdim + 63) / 64;
-    const uint32_t extra = 256 + 1024 + 1024, limit = (uint32_t)ctx->smem_optin;   // barriers, row sums, alignment slack
+    p.alias = a.vdim > 128 ? 1 : 0;
+    const uint32_t extra = 256 + 2048 + 1024, limit = (uint32_t)ctx->smem_optin;   // barriers, row sums, alignment slack
     auto bytes = [&](uint32_t ks, uint32_t vs) { return ((1 + ks) * p.qchunks + vs * p.vchunks) * TILE_CHUNK + extra; };
     p.kstages = p.vstages = 2;
     if (bytes(2, 2) > limit) p.kstages = 1;
-    if (bytes(p.kstages, 2) > limit) p.vstages = 1;
+    if (bytes(p.kstages, 2) > limit) {
+        p.vstages = 1;
+        p.alias = 1;   // K(t + 2) is loaded after V(t + 1): with one V stage tile t's product must come before S(t + 2)
+    }
     const uint32_t smem = bytes(p.kstages, p.vstages);
     if (smem > limit) return HOLO_OK;
     const uint32_t qtiles = (a.rows + p.rpt - 1) / p.rpt;

@@ -1289,7 +1289,7 @@ inline void tile_choice(const holo_b200_ctx* ctx, uint32_t m, uint32_t n, uint32
             bn = 128;
             splits = 2;   // three slices (288 CTAs in clusters of 3) did not all become resident: 64 x 4096 x 12288 took 32.6 us against 25.3
         } else if (tiles64 >= (uint32_t)ctx->sm_count) {
-            bn = 64;
+            bn = tiles64 > slots ? 128 : 64;   // 64-wide tiles that need a second wave lose to one wave of 128-wide ones
         } else {
             bn = tiles128 >= 16 ? 128 : 64;
             const uint32_t tiles = bn == 128 ? tiles128 : tiles64;

@@ -14,7 +14,15 @@ from .session import InferenceSession
 
 
 class CacheFull(RuntimeError):
-    pass
+    """A step or a request needs more positions than the cache has, or the cache belongs to another sequence."""
+
+
+def bucket(n):
+    """The step shape for n rows: the next power of two."""
+    b = 1
+    while b < n:
+        b *= 2
+    return b
 
 
 class SequenceCache:
@@ -63,13 +71,6 @@ class StepRunner:
         self._root.close()
         self._steps, self._heads = {}, {}
 
-    @staticmethod
-    def _bucket(n):
-        b = 1
-        while b < n:
-            b *= 2
-        return b
-
     def _session(self, table, rows, build):
         if rows not in table:
             table[rows] = [InferenceSession(self.backend, build(), verify=False, donor=self._root), False]
@@ -86,7 +87,7 @@ class StepRunner:
     def _run_rows(self, tokens, base, want):
         """One portion of at most max_rows tokens; logits of the wanted rows."""
         m = self.model
-        rows = self._bucket(len(tokens))
+        rows = bucket(len(tokens))
         entry = self._session(self._steps, rows, lambda: m.build_step(rows, self.cache.capacity, self.max_rows, False, weightless=True))
         step_in = np.zeros(4 + rows, dtype=np.int32)
         step_in[0] = base
@@ -99,7 +100,7 @@ class StepRunner:
         out = np.empty((len(want), vocab), dtype=np.float32)
         for lo in range(0, len(want), self.LOGIT_ROWS):
             part = want[lo:lo + self.LOGIT_ROWS]
-            n = self._bucket(len(part))
+            n = bucket(len(part))
             head = self._session(self._heads, n, lambda: m.build_head(n, self.max_rows, weightless=True))
             index = np.zeros(n, dtype=np.int32)
             index[:len(part)] = part

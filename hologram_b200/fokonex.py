@@ -246,6 +246,12 @@ class FokonexModel:
         w.outputs.append(holo.Port("logits", logits, rows * c.vocab, F32, [rows, c.vocab]))
 
     def build_step(self, rows, capacity, hidden_rows, with_logits, weightless=False):
+        return self.step_writer(rows, capacity, hidden_rows, with_logits).finish(weightless=weightless)
+
+    def build_head(self, rows, hidden_rows, weightless=False):
+        return self.head_writer(rows, hidden_rows).finish(weightless=weightless)
+
+    def step_writer(self, rows, capacity, hidden_rows, with_logits):
         """The archive of one step of `rows` tokens: ports `step_in` (i32: position, three unused words, the token ids),
         `hidden` (the residual stream, [hidden_rows, width]), `l<i>.k` / `l<i>.v` (the cache of layer run i); with
         `with_logits` also the output head over all rows (port `logits`)."""
@@ -299,9 +305,10 @@ class FokonexModel:
         if with_logits:
             self._logits(w, sl, made, xr, rows)
         w.exec_plan = [[i] for i in range(len(w.calls))]
-        return w.finish(weightless=weightless)
+        w.slot_bytes = list(sl.nbytes)
+        return w
 
-    def build_head(self, rows, hidden_rows, weightless=False):
+    def head_writer(self, rows, hidden_rows):
         """The archive that turns `rows` chosen rows of the residual stream (port `want`, i32) into logits."""
         c = self.config
         w, sl, made = self._begin()
@@ -312,7 +319,8 @@ class FokonexModel:
         w.calls.append(kc.KernelCall.Gather(kc.GatherCall(sl.ref(x), sl.ref(want), sl.ref(picked), 1, hidden_rows, c.width, rows, I32, F32)))
         self._logits(w, sl, made, sl.ref(picked), rows)
         w.exec_plan = [[i] for i in range(len(w.calls))]
-        return w.finish(weightless=weightless)
+        w.slot_bytes = list(sl.nbytes)
+        return w
 
     def launches(self, rows, with_logits):
         """Kernel launches of one step, by the archive's call count."""

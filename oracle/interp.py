@@ -35,6 +35,19 @@ def _put(slots, ref, arr):
     slots[ref.slot][ref.offset:ref.offset + raw.size] = raw
 
 
+def _f32(bits):
+    return float(np.array([bits], dtype=np.uint32).view(np.float32)[0])
+
+
+def _wide(a, dtype):
+    """f64 values of a bf16 or f32 array."""
+    return (orc.bf16_to_f32(a) if dtype == kc.DTYPE_BF16 else a).astype(np.float64)
+
+
+def _narrow(a, dtype):
+    return orc.f32_to_bf16_rne(np.ascontiguousarray(a).reshape(-1)) if dtype == kc.DTYPE_BF16 else np.asarray(a, dtype=np.float32)
+
+
 def run(calls, slots, all_reduce=None):
     es = lambda dt: np.dtype(_NP[dt]).itemsize
     for call in calls:
@@ -158,6 +171,58 @@ def run(calls, slots, all_reduce=None):
             rc, out = orc.kv_cache_write(cache, new, pos, c.planes, c.bucket_rows, c.new_rows, c.row_bytes)
             assert rc == 0
             _put(slots, c.output, out)
+        elif k == kc.K_CAST:
+            c = u.cast
+            _put(slots, c.output, orc.cast_float(_get(slots, c.input, c.element_count * es(c.src_dtype), c.src_dtype), c.src_dtype, c.dst_dtype))
+        elif k == kc.K_RMS_NORM_MULTI:
+            c = u.rms_norm_multi
+            x = _get(slots, c.x, c.rows * c.feature * 4, kc.DTYPE_F32).reshape(c.rows, c.feature).astype(np.float64)
+            gammas = [g for g in (c.gamma0, c.gamma1) if g.slot != kc.NO_SLOT]
+            out = np.zeros((c.rows, len(gammas), c.step), dtype=np.float32)
+            inv = 1.0 / np.sqrt((x * x).mean(axis=1, keepdims=True) + _f32(c.epsilon_bits))
+            for i, g in enumerate(gammas):
+                out[:, i, :c.feature] = x * inv * _get(slots, g, c.feature * 4, kc.DTYPE_F32)
+            _put(slots, c.output, _narrow(out, c.dtype))
+        elif k == kc.K_LINEAR:
+            c = u.linear
+            a = _wide(_get(slots, c.a, c.m * c.lda * es(c.dtype), c.dtype), c.dtype).reshape(c.m, c.lda)
+            b = _wide(_get(slots, c.b, c.k * c.n * es(c.dtype), c.dtype), c.dtype).reshape(c.k, c.n)
+            for g in list(c.seg)[:c.nseg]:
+                v = a[:, g.k_offset:g.k_offset + c.k] @ b[:, g.col_begin:g.col_begin + g.width]
+                if g.act == kc.LINEAR_ACT_RELU2:
+                    v = np.maximum(v, 0.0) ** 2
+                v = _f32(c.alpha_bits) * v
+                size = es(g.dtype)
+                first = int(_get(slots, g.row_pos, 4, kc.DTYPE_I32)[0]) if g.row_pos.slot != kc.NO_SLOT else 0
+                extent = g.output.length or slots[g.output.slot].size - g.output.offset
+                limit = extent // (g.ld * size) if g.row_pos.slot != kc.NO_SLOT else c.m
+                for i in range(min(c.m, limit - first)):
+                    at = kc.rb(g.output.slot, g.output.offset + (first + i) * g.ld * size)
+                    row = v[i]
+                    if c.residual.slot != kc.NO_SLOT:
+                        row = row + _get(slots, kc.rb(c.residual.slot, c.residual.offset + i * g.ld * 4), g.width * 4, kc.DTYPE_F32)
+                    _put(slots, at, _narrow(row.astype(np.float32), g.dtype))
+        elif k == kc.K_CAUSAL_ATTENTION:
+            c = u.causal_attention
+            size = es(c.dtype)
+            load = lambda ref, *shape: _wide(_get(slots, ref, int(np.prod(shape)) * size, c.dtype), c.dtype).reshape(shape)
+            q, kk = load(c.q, c.rows, c.heads, c.dim), load(c.k, c.cache_rows, c.kv_heads, c.dim)
+            v = load(c.v, c.cache_rows, c.kv_heads, c.vdim)
+            first = int(_get(slots, c.pos, 4, kc.DTYPE_I32)[0])
+            every, cap = _f32(c.temp_every_bits), _f32(c.softcap_bits)
+            scale = _f32(c.scale_bits) or c.dim ** -0.5
+            for i in range(c.rows):
+                n = min(first + i + 1, c.cache_rows)
+                f = scale * (1.0 + _f32(c.temp_coef_bits) * np.log(np.floor((first + i + 1) / every) + 1.0) if every else 1.0)
+                for h in range(c.heads):
+                    kv = h // (c.heads // c.kv_heads)
+                    s = kk[:n, kv] @ q[i, h] * f
+                    s = cap * np.tanh(s / cap) if cap else s
+                    sink = _get(slots, kc.rb(c.sink.slot, c.sink.offset + 4 * h), 4, kc.DTYPE_F32)[0] if c.sink.slot != kc.NO_SLOT else -np.inf
+                    top = max(s.max(), sink)
+                    e = np.exp(s - top)
+                    o = e @ v[:n, kv] / (e.sum() + np.exp(sink - top))
+                    _put(slots, kc.rb(c.output.slot, c.output.offset + (i * c.ld + h * c.vdim) * size), _narrow(o.astype(np.float32), c.dtype))
         elif k == kc.K_ALL_REDUCE:
             c = u.all_reduce
             assert c.dtype == kc.DTYPE_BF16

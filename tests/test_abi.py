@@ -34,9 +34,10 @@ def test_struct_layout_matches_the_header():
     #include <stddef.h>
     #include "hologram_b200.h"
     int main(void) {
-        printf("%zu %zu %zu %zu %zu %zu %zu %zu %zu\n", sizeof(HoloBufferRef), sizeof(HoloUnaryCall), sizeof(HoloMatMulCall),
+        printf("%zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu\n", sizeof(HoloBufferRef), sizeof(HoloUnaryCall), sizeof(HoloMatMulCall),
                sizeof(HoloMatMulAddCall), sizeof(HoloNormCall), sizeof(HoloDecodeAttentionValidQ8Call),
-               sizeof(HoloKernelCall), offsetof(HoloKernelCall, u), sizeof(HoloHostSlot));
+               sizeof(HoloKernelCall), offsetof(HoloKernelCall, u), sizeof(HoloHostSlot),
+               sizeof(HoloRmsNormMultiCall), sizeof(HoloLinearSeg), sizeof(HoloLinearCall), sizeof(HoloCausalAttentionCall));
         return 0;
     }'''
     with tempfile.TemporaryDirectory() as d:
@@ -47,7 +48,8 @@ def test_struct_layout_matches_the_header():
         got = [int(v) for v in subprocess.check_output([exe]).split()]
     want = [ctypes.sizeof(kc.BufferRef), ctypes.sizeof(kc.UnaryCall), ctypes.sizeof(kc.MatMulCall),
             ctypes.sizeof(kc.MatMulAddCall), ctypes.sizeof(kc.NormCall), ctypes.sizeof(kc.DecodeAttentionValidQ8Call),
-            ctypes.sizeof(kc.KernelCall), kc.KernelCall.u.offset, ctypes.sizeof(kc.HostSlot)]
+            ctypes.sizeof(kc.KernelCall), kc.KernelCall.u.offset, ctypes.sizeof(kc.HostSlot),
+            ctypes.sizeof(kc.RmsNormMultiCall), ctypes.sizeof(kc.LinearSeg), ctypes.sizeof(kc.LinearCall), ctypes.sizeof(kc.CausalAttentionCall)]
     assert got == want
 
 
