@@ -408,16 +408,18 @@ int32_t try_split(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
 }
 
 // ---- many rows: 128-row tiles on tcgen05 ------------------------------------------------------------------------------
-// One CTA per (128-row tile, kv head); a tile packs `rpt` rows times the group's heads, so the keys are read once for the
-// whole group. Keys come in tiles of 128.
-//   warp 0     TMA producer: the query tile once, K and V tiles through rings
-//   warp 1     tcgen05.mma issuer: S(t) = Q K(t)^T into one of two 128-column buffers, O += P(t) V(t) with P read from TMEM;
-//              as soon as the weights of tile t are stored (its scores are then dead) S(t + 2) is issued, then tile t's product
-//   warps 2-17 weights, four groups of four warps (one per TMEM lane quarter): group i takes key half i / 2 of the tiles of
-//              buffer i % 2: tcgen05.ld half a row of S, cap, exponentiate, sum, tcgen05.st the bf16 weights
+// A tile of 128 rows packs `rpt` rows times the group's heads, so the keys are read once for the whole group. One CTA works
+// on NQ such tiles of a kv head: two where there are enough rows to fill the chip and both fit (every K/V tile from L2 then
+// serves 256 rows; with one, the loop waits for L2), else one. Keys come in tiles of 128; an item is one key tile against one
+// query tile, and two items are in flight, one per S buffer.
+//   warp 0     TMA producer: the query tiles once, K and V tiles through rings
+//   warp 1     tcgen05.mma issuer: S = Q K^T, O += P V with P read from TMEM; as soon as an item's weights are stored its
+//              product is issued, and the scores of the item after next into its buffer
+//   warps 2-17 weights, four groups of four warps (one per TMEM lane quarter): group j takes key half j / 2 of the items of
+//              buffer j % 2: tcgen05.ld half a row of S, cap, exponentiate, sum, tcgen05.st the bf16 weights
 // Without a running maximum O needs no correction: it stays in TMEM from the first tile to the last.
-// TMEM (all 512 columns): S at 0 and 128, O at 256, P at 384 and 448 when vdim leaves room, else over the S it came from,
-// each key half's weights over the first half of its scores (S(t + 2) then waits for tile t's product). It is allocated after the dependency wait, and dependents are
+// TMEM (all 512 columns): S at 0 and 128, O from 256; P at 384 and 448 where vdim leaves room, else over the S it came from,
+// each key half's weights over the first half of its scores (the next scores then wait for the item's product). It is allocated after the dependency wait, and dependents are
 // released only after the allocation, so no neighbouring launch can hold columns this kernel or its predecessor waits for.
 constexpr int TILE_THREADS = 576;
 constexpr uint32_t TILE_CHUNK = 128 * 128;   // 128 rows of 64 bf16 columns (one 128B-swizzled TMA box)
@@ -426,7 +428,8 @@ struct TileParams {
     HoloCausalArgs a;
     uint32_t* status;
     uint32_t group, rpt, qchunks, vchunks, kstages, vstages;
-    uint32_t alias;   // P lies over S
+    uint32_t alias;     // P lies over S
+    uint32_t ostride;   // TMEM columns between the accumulators of two query tiles
 };
 
 __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
@@ -490,6 +493,7 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&v)[16
         : "memory");
 }
 
+template <int NQ>
 __global__ void __launch_bounds__(TILE_THREADS, 1)
 causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, const TileParams p) {
@@ -499,8 +503,8 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
     const uint32_t base = (raw + 1023u) & ~1023u;
     uint8_t* sm = smem_raw + (base - raw);
     const uint32_t kbytes = p.qchunks * TILE_CHUNK, vbytes = p.vchunks * TILE_CHUNK;
-    const uint32_t s_q = base, s_k = s_q + kbytes, s_v = s_k + p.kstages * kbytes;
-    const uint32_t off_bars = (1 + p.kstages) * kbytes + p.vstages * vbytes;
+    const uint32_t s_q = base, s_k = s_q + NQ * kbytes, s_v = s_k + p.kstages * kbytes;
+    const uint32_t off_bars = (NQ + p.kstages) * kbytes + p.vstages * vbytes;
     const uint32_t bar_q = base + off_bars, bar_k_full = bar_q + 8, bar_k_empty = bar_k_full + 16, bar_v_full = bar_k_empty + 16,
                    bar_v_empty = bar_v_full + 16, bar_s = bar_v_empty + 16, bar_p = bar_s + 16, bar_pv = bar_p + 16, bar_o = bar_pv + 16;
     uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + off_bars + 128);
@@ -509,7 +513,7 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
 
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t g = blockIdx.x, qtile = gridDim.y - 1 - blockIdx.y;   // the tiles with the most keys first
-    const uint32_t row0 = qtile * p.rpt;
+    const uint32_t row0 = qtile * NQ * p.rpt;
     if (threadIdx.x == 0) {
         mbar_init(bar_q, 1);
         for (int s = 0; s < 2; ++s) {
@@ -536,14 +540,16 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
     holo_pdl_trigger();
     const uint32_t tmem_base = *s_tmem, tmem_o = tmem_base + 256;
     const uint32_t pos = *a.pos;
-    const uint32_t visible = min(pos + min(row0 + p.rpt, a.rows), a.cache_rows);
-    const uint32_t ntiles = (visible + 127) / 128;
+    const uint32_t visible = min(pos + min(row0 + NQ * p.rpt, a.rows), a.cache_rows);
+    const uint32_t ntiles = (visible + 127) / 128, items = ntiles * NQ;
 
     if (warp == 0) {
         // ---------------- TMA producer ----------------
         if (lane == 0) {
-            mbar_arrive_expect_tx(bar_q, p.qchunks * p.rpt * p.group * 128);
-            for (uint32_t c = 0; c < p.qchunks; ++c) tma_load_3d(s_q + c * TILE_CHUNK, &map_q, (int)(64 * c), (int)(g * p.group), (int)row0, bar_q);
+            mbar_arrive_expect_tx(bar_q, NQ * p.qchunks * p.rpt * p.group * 128);
+            for (uint32_t i = 0; i < NQ; ++i)
+                for (uint32_t c = 0; c < p.qchunks; ++c)
+                    tma_load_3d(s_q + i * kbytes + c * TILE_CHUNK, &map_q, (int)(64 * c), (int)(g * p.group), (int)(row0 + i * p.rpt), bar_q);
             uint32_t kt = 0, vt = 0;
             bool ok = true;
             for (uint32_t t = 0; t < ntiles && ok; ++t) {
@@ -577,41 +583,57 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
             const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 3) << 17) | ((128u >> 4) << 24);
             const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((a.vdim >> 3) << 17) | ((128u >> 4) << 24);
             const uint32_t ksteps = a.dim / 16;
-            auto scores = [&](uint32_t t) {       // issue S(t)
-                const uint32_t ks = t % p.kstages, buf = t & 1u;
-                if (!mbar_wait(bar_k_full + 8 * ks, (t / p.kstages) & 1, s_abort, p.status)) return false;
+            // Item i is key tile i / NQ against query tile i % NQ, its scores in buffer i & 1. Between an item's weights and its
+            // buffer's next scores lies what this one thread does, so it works on ready-made descriptors (a step of 16 k-elements
+            // adds 32 bytes, four of them a chunk; a step of 16 keys adds 2048 bytes) and running stage numbers.
+            const uint64_t desc_q = smem_desc(s_q, 16, 1024), desc_k = smem_desc(s_k, 16, 1024), desc_v = smem_desc(s_v, TILE_CHUNK, 1024);
+            const uint32_t kstep = kbytes >> 4, vstep = vbytes >> 4;
+            const bool alias = p.alias != 0;
+            uint32_t ks = 0, kphase = 0, vs = 0, vphase = 0;
+            auto scores = [&](uint32_t i) {
+                const uint32_t qi = NQ == 2 ? i & 1u : 0u, buf = i & 1u;
+                if (qi == 0 && !mbar_wait(bar_k_full + 8 * ks, kphase, s_abort, p.status)) return false;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                for (uint32_t k = 0; k < ksteps; ++k) {
-                    const uint32_t off = (k >> 2) * TILE_CHUNK + (k & 3) * 32;
-                    umma_bf16(tmem_base + buf * 128, smem_desc(s_q + off, 16, 1024), smem_desc(s_k + ks * kbytes + off, 16, 1024), idesc_s, k != 0);
+                const uint64_t dq = desc_q + qi * kstep, dk = desc_k + ks * kstep;
+                const uint32_t d = tmem_base + buf * 128;
+                for (uint32_t k0 = 0, off = 0; k0 < ksteps; k0 += 4, off += TILE_CHUNK >> 4) {
+#pragma unroll
+                    for (uint32_t k = 0; k < 4; ++k)
+                        if (k0 + k < ksteps) umma_bf16(d, dq + off + 2 * k, dk + off + 2 * k, idesc_s, (k0 | k) != 0);
                 }
-                umma_commit(bar_k_empty + 8 * ks);
                 umma_commit(bar_s + 8 * buf);
+                if (qi == NQ - 1) {
+                    umma_commit(bar_k_empty + 8 * ks);
+                    if (++ks == p.kstages) ks = 0, kphase ^= 1;
+                }
                 return true;
             };
-            bool ok = mbar_wait(bar_q, 0, s_abort, p.status) && scores(0) && (ntiles < 2 || scores(1));
-            for (uint32_t t = 0; t < ntiles && ok; ++t) {
-                const uint32_t vs = t % p.vstages, buf = t & 1u;
-                ok = mbar_wait(bar_p + 8 * buf, (t >> 1) & 1, s_abort, p.status);
-                if (!ok) break;
-                if (!p.alias && t + 2 < ntiles) ok = scores(t + 2);
-                ok = ok && mbar_wait(bar_v_full + 8 * vs, (t / p.vstages) & 1, s_abort, p.status);
+            bool ok = mbar_wait(bar_q, 0, s_abort, p.status) && scores(0) && (items < 2 || scores(1));
+            for (uint32_t i = 0; i < items && ok; ++i) {
+                const uint32_t qi = NQ == 2 ? i & 1u : 0u, buf = i & 1u, phase = (i >> 1) & 1;
+                if (qi == 0) ok = mbar_wait(bar_v_full + 8 * vs, vphase, s_abort, p.status);
+                ok = ok && mbar_wait(bar_p + 8 * buf, phase, s_abort, p.status);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const uint32_t tmem_p = tmem_base + (p.alias ? buf * 128 : 384 + buf * 64);
+                if (!alias && i + 2 < items) ok = scores(i + 2);
+                if (!ok) break;
+                const uint32_t tmem_p = tmem_base + (alias ? buf * 128 : 384 + buf * 64), d = tmem_o + qi * p.ostride, gap = alias ? 32 : 0;
+                const uint64_t dv = desc_v + vs * vstep;
 #pragma unroll
-                for (uint32_t k = 0; k < 8; ++k)
-                    umma_bf16_ts(tmem_o, tmem_p + k * 8 + (p.alias && k >= 4 ? 32 : 0), smem_desc(s_v + vs * vbytes + k * 2048, TILE_CHUNK, 1024), idesc_o, (t | k) != 0);
-                umma_commit(bar_v_empty + 8 * vs);
+                for (uint32_t k = 0; k < 8; ++k) umma_bf16_ts(d, tmem_p + k * 8 + (k >= 4 ? gap : 0), dv + 128 * k, idesc_o, k != 0 || i >= NQ);
                 umma_commit(bar_pv + 8 * buf);
-                if (p.alias && t + 2 < ntiles) ok = mbar_wait(bar_pv + 8 * buf, (t >> 1) & 1, s_abort, p.status) && scores(t + 2);
+                if (qi == NQ - 1) {
+                    umma_commit(bar_v_empty + 8 * vs);
+                    if (++vs == p.vstages) vs = 0, vphase ^= 1;
+                }
+                if (alias && i + 2 < items) ok = mbar_wait(bar_pv + 8 * buf, phase, s_abort, p.status) && scores(i + 2);
             }
             if (ok) umma_commit(bar_o);
         }
     } else {
         // ---------------- weights (TMEM lane quarter = warp % 4), then the output ----------------
         const uint32_t quarter = warp & 3u, wg = (warp - 2) >> 2, buf = wg & 1u, half = wg >> 1, tr = quarter * 32 + lane;
-        const uint32_t row = row0 + tr / p.group, head = g * p.group + tr % p.group;
+        const uint32_t first = row0 + (NQ == 2 ? buf * p.rpt : 0), row = first + tr / p.group, head = g * p.group + tr % p.group;
         const bool valid = tr < p.rpt * p.group && row < a.rows;
         const uint32_t at = pos + min(row, a.rows - 1);
         const uint32_t lanes = (quarter * 32u) << 16;
@@ -621,8 +643,9 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const uint64_t c0_2 = pair(c0, c0), c2_2 = pair(c2, c2);
         float sum = 0.0f;
         bool ok = true;
-        for (uint32_t t = buf; t < ntiles; t += 2) {
-            ok = mbar_wait(bar_s + 8 * buf, (t >> 1) & 1, s_abort, p.status) && !*s_abort;
+        for (uint32_t i = buf; i < items; i += 2) {
+            const uint32_t t = i / NQ;
+            ok = mbar_wait(bar_s + 8 * buf, (i >> 1) & 1, s_abort, p.status) && !*s_abort;
             ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -630,7 +653,7 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
             const uint32_t tmem_p = (p.alias ? tmem_s : tmem_base + 384 + buf * 64 + half * 32 + lanes);
             const uint32_t key0 = t * 128 + half * 64;
             // every key of the tile is at or before the first row's position: no mask
-            const bool whole = t * 128 + 127 <= pos + row0;
+            const bool whole = t * 128 + 127 <= pos + first;
             uint32_t v[2][32];
             tmem_ld32_request(tmem_s, v[0]);
             tmem_ld32_request(tmem_s + 32, v[1]);
@@ -640,8 +663,8 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
             for (int x = 0; x < 32; ++x) most[x & 3] = fmaxf(most[x & 3], fmaxf(fabsf(__uint_as_float(v[0][x])), fabsf(__uint_as_float(v[1][x]))));
             const bool short_form = __all_sync(0xffffffffu, fmaxf(fmaxf(most[0], most[1]), fmaxf(most[2], most[3])) <= small);
-            if (!p.alias && t >= 2) {   // the product of tile t - 2 reads this P buffer
-                ok = mbar_wait(bar_pv + 8 * buf, ((t >> 1) - 1) & 1, s_abort, p.status);
+            if (!p.alias && i >= 2) {   // the product of item i - 2 reads this P buffer
+                ok = mbar_wait(bar_pv + 8 * buf, ((i >> 1) - 1) & 1, s_abort, p.status);
                 ok = __all_sync(0xffffffffu, ok);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -695,12 +718,13 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
         ok = __all_sync(0xffffffffu, ok);
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float denom = (s_sum[tr] + s_sum[128 + tr]) + (s_sum[256 + tr] + s_sum[384 + tr]) + (a.sink && valid ? ex2(a.sink[head] * LOG2E) : 0.0f);
+            const float total = NQ == 2 ? s_sum[buf * 128 + tr] + s_sum[(buf + 2) * 128 + tr] : (s_sum[tr] + s_sum[128 + tr]) + (s_sum[256 + tr] + s_sum[384 + tr]);
+            const float denom = total + (a.sink && valid ? ex2(a.sink[head] * LOG2E) : 0.0f);
             const float inv = __fdiv_rn(1.0f, denom);
             __nv_bfloat16* out = (__nv_bfloat16*)a.out + (uint64_t)row * a.ld + head * a.vdim;
-            for (uint32_t c = wg; c < a.vdim / 16; c += 4) {
+            for (uint32_t c = NQ == 2 ? half : wg; c < a.vdim / 16; c += NQ == 2 ? 2 : 4) {
                 uint32_t v[16], w[8];
-                tmem_ld16(tmem_o + lanes + c * 16, v);
+                tmem_ld16(tmem_o + (NQ == 2 ? buf * p.ostride : 0) + lanes + c * 16, v);
 #pragma unroll
                 for (int x = 0; x < 8; ++x) w[x] = pack_bf16(__uint_as_float(v[2 * x]) * inv, __uint_as_float(v[2 * x + 1]) * inv);
                 if (valid) {
@@ -720,6 +744,18 @@ causal_attention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __
     }
 }
 
+template <int NQ>
+int32_t launch_tile(holo_b200_ctx* ctx, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TileParams& p, uint32_t ctas, uint32_t smem) {
+    static thread_local int configured_device = -1;
+    if (configured_device != ctx->device) {
+        HOLO_CUDA(cudaFuncSetAttribute(causal_attention_tile_kernel<NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, ctx->smem_optin));
+        configured_device = ctx->device;
+    }
+    HOLO_CUDA(holo_launch_kernel(ctx, causal_attention_tile_kernel<NQ>, dim3(p.a.kv_heads, ctas), dim3(TILE_THREADS), smem, 1, mq, mk, mv, p));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
 // Launches the tile kernel, or returns with *taken false when the shape does not suit it.
 int32_t try_tile(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
     *taken = false;
@@ -731,19 +767,27 @@ int32_t try_tile(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
     p.rpt = 128 / p.group;
     p.qchunks = (a.dim + 63) / 64;
     p.vchunks = (a.vdim + 63) / 64;
-    p.alias = a.vdim > 128 ? 1 : 0;
     const uint32_t extra = 256 + 2048 + 1024, limit = (uint32_t)ctx->smem_optin;   // barriers, row sums, alignment slack
-    auto bytes = [&](uint32_t ks, uint32_t vs) { return ((1 + ks) * p.qchunks + vs * p.vchunks) * TILE_CHUNK + extra; };
-    p.kstages = p.vstages = 2;
-    if (bytes(2, 2) > limit) p.kstages = 1;
-    if (bytes(p.kstages, 2) > limit) {
-        p.vstages = 1;
-        p.alias = 1;   // K(t + 2) is loaded after V(t + 1): with one V stage tile t's product must come before S(t + 2)
-    }
-    const uint32_t smem = bytes(p.kstages, p.vstages);
-    if (smem > limit) return HOLO_OK;
+    auto bytes = [&](uint32_t nq, uint32_t ks, uint32_t vs) { return ((nq + ks) * p.qchunks + vs * p.vchunks) * TILE_CHUNK + extra; };
     const uint32_t qtiles = (a.rows + p.rpt - 1) / p.rpt;
     if (qtiles > 65535) return HOLO_OK;
+    p.kstages = p.vstages = 2;
+    bool two = a.vdim <= 128 && bytes(2, 2, 2) <= limit && ((qtiles + 1) / 2) * a.kv_heads >= (uint32_t)ctx->sm_count;
+    if (const char* e = getenv("HOLO_CAUSAL_QUERY_TILES")) two = atoi(e) == 2 && a.vdim <= 128 && bytes(2, 2, 2) <= limit;
+    if (two) {
+        p.ostride = a.vdim <= 64 ? 64 : 128;
+        p.alias = a.vdim > 64 ? 1 : 0;
+    } else {
+        p.ostride = 0;
+        p.alias = a.vdim > 128 ? 1 : 0;
+        if (bytes(1, 2, 2) > limit) p.kstages = 1;
+        if (bytes(1, p.kstages, 2) > limit) {
+            p.vstages = 1;
+            p.alias = 1;   // K(t + 2) is loaded after V(t + 1): with one V stage tile t's product must come before S(t + 2)
+        }
+    }
+    const uint32_t smem = bytes(two ? 2 : 1, p.kstages, p.vstages);
+    if (smem > limit) return HOLO_OK;
     CUtensorMap mq, mk, mv;
     {   // q as [rows][heads][dim]: a box is 64 columns of the group's heads over rpt rows
         cuuint64_t dims[3] = {a.dim, a.heads, a.rows};
@@ -756,15 +800,8 @@ int32_t try_tile(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
     }
     HOLO_TRY(make_map_2d(&mk, a.k, (uint64_t)a.kv_heads * a.dim, a.cache_rows, 64, 128));
     HOLO_TRY(make_map_2d(&mv, a.v, (uint64_t)a.kv_heads * a.vdim, a.cache_rows, 64, 128));
-    static thread_local int configured_device = -1;
-    if (configured_device != ctx->device) {
-        HOLO_CUDA(cudaFuncSetAttribute(causal_attention_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, ctx->smem_optin));
-        configured_device = ctx->device;
-    }
     *taken = true;
-    HOLO_CUDA(holo_launch_kernel(ctx, causal_attention_tile_kernel, dim3(a.kv_heads, qtiles), dim3(TILE_THREADS), smem, 1, mq, mk, mv, p));
-    ctx->launches++;
-    return HOLO_OK;
+    return two ? launch_tile<2>(ctx, mq, mk, mv, p, (qtiles + 1) / 2, smem) : launch_tile<1>(ctx, mq, mk, mv, p, qtiles, smem);
 }
 
 }  // namespace

@@ -175,6 +175,19 @@ def test_attention_bf16(backend, shape):
     assert np.abs(got - want).max() / np.abs(want).max() < 1e-2
 
 
+@pytest.mark.parametrize("shape", [s for s in ATTENTION_SHAPES[9:] if s[3] <= 128 and s[4] <= 128] + [(640, 4, 2, 64, 64, 700, 1400), (1000, 2, 1, 128, 128, 0, 1000)],
+                         ids=lambda s: "-".join(map(str, s)))
+@pytest.mark.parametrize("tiles", [1, 2])
+def test_attention_query_tiles_per_cta(backend, shape, tiles, monkeypatch):
+    """One and two query tiles per CTA (the choice by size needs more rows than these) give the same result."""
+    monkeypatch.setenv("HOLO_CAUSAL_QUERY_TILES", str(tiles))
+    rows, heads, groups, dim, vdim, first, cache_rows = shape
+    q, k, v, sinks = random_attention(rows, heads, groups, dim, vdim, first + rows, seed=rows + dim)
+    got = run_attention(backend, q, k, v, first, dim ** -0.5, 25.0, 0.3, 16, sinks, BF, cache_rows, stale=300.0)
+    want = ref.attention(q, k, v, first, dim ** -0.5, 25.0, 0.3, 16, sinks)
+    assert np.abs(got - want).max() / np.abs(want).max() < 1e-2
+
+
 @pytest.mark.parametrize("shape", ATTENTION_SHAPES[:9:2] + [(20, 3, 1, 20, 33, 11, 40), (5, 2, 2, 7, 130, 60, 70)], ids=lambda s: "-".join(map(str, s)))
 def test_attention_f32(backend, shape):
     rows, heads, groups, dim, vdim, first, cache_rows = shape
