@@ -19,6 +19,8 @@ from . import kernel_call as kc
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libhologram_b200.so")
+if not os.path.exists(LIB_PATH) and os.path.exists(os.path.join(_HERE, "libhologram_b200_serving.so")):
+    LIB_PATH = os.path.join(_HERE, "libhologram_b200_serving.so")      # a checkout that has only been built for serving
 
 
 class BackendError(RuntimeError):
