@@ -14,9 +14,9 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libhologram_b200.so")
-SOURCES = ["api.cu", "lut.cu", "glue.cu", "attention.cu", "gemm.cu", "linear.cu", "causal_attention.cu", "quant_gemv.cu", "tp.cu", "session.cu", "addressed.cpp", "pool.cpp", "archive.cpp", "blake3.cpp", "label.cpp"]
+SOURCES = ["api.cu", "lut.cu", "glue.cu", "attention.cu", "gemm.cu", "linear.cu", "causal_attention.cu", "window_attention.cu", "retention.cu", "moe.cu", "quant_gemv.cu", "tp.cu", "session.cu", "addressed.cpp", "pool.cpp", "archive.cpp", "blake3.cpp", "label.cpp"]
 SERVING_LIB = os.path.join(HERE, "libhologram_b200_serving.so")
-SERVING_SOURCES = ["api.cu", "glue.cu", "linear.cu", "causal_attention.cu", "session.cu", "addressed.cpp", "pool.cpp", "archive.cpp", "blake3.cpp", "label.cpp",
+SERVING_SOURCES = ["api.cu", "glue.cu", "linear.cu", "causal_attention.cu", "window_attention.cu", "retention.cu", "moe.cu", "session.cu", "addressed.cpp", "pool.cpp", "archive.cpp", "blake3.cpp", "label.cpp",
                    "absent_families.cpp"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

@@ -9,6 +9,8 @@
 
 #include <stdlib.h>
 
+#include <algorithm>
+
 #include "common.h"
 
 // ---- thread-local error state (hologram-ffi src/lib.rs:48-92 convention) --------------------
@@ -90,6 +92,7 @@ extern "C" void holo_b200_ctx_destroy(holo_b200_ctx* ctx) {
     if (ctx->dev_status) cudaFree(ctx->dev_status);
     if (ctx->attn_arrivals) cudaFree(ctx->attn_arrivals);
     if (ctx->causal_partials) cudaFree(ctx->causal_partials);
+    if (ctx->latent_partials) cudaFree(ctx->latent_partials);
     if (ctx->own_stream) cudaStreamDestroy(ctx->stream);
     delete ctx;
 }
@@ -956,6 +959,14 @@ int32_t do_rms_norm_multi(holo_b200_ctx* ctx, const HoloRmsNormMultiCall& c, hol
     return holo_launch_rms_norm_multi(ctx, (const float*)x, (const float*)g0, (const float*)g1, out, c.rows, c.feature, c.step, eps, c.dtype);
 }
 
+// A LINEAR call has no extended fields, whatever its struct holds there.
+HoloLinearCall plain_linear(HoloLinearCall c) {
+    c.rot = c.a_pos = c.tiles = HoloBufferRef{HOLO_NO_SLOT, 0, 0};
+    c.a_back = c.a_rows = c.tile_rows = c.experts = c.a_shared = 0;
+    for (HoloLinearSeg& g : c.seg) g.rot_head = g.rot_begin = g.rot_dims = 0, g.ring = 0;
+    return c;
+}
+
 // Extension: a product with up to four output segments.
 int32_t do_linear(holo_b200_ctx* ctx, const HoloLinearCall& c, holo_b200_workspace* ws) {
     if (c.nseg < 1 || c.nseg > HOLO_LINEAR_MAX_SEGS) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear segment count %u", c.nseg);
@@ -964,25 +975,56 @@ int32_t do_linear(holo_b200_ctx* ctx, const HoloLinearCall& c, holo_b200_workspa
     const uint64_t es = holo_dtype_size(c.dtype);
     HoloLinearArgs a = {};
     uint8_t *pa, *pb, *ptr;
-    const uint64_t ab = ((uint64_t)(c.m - 1) * c.lda + c.lda) * es, bb = (uint64_t)c.k * c.n * es;
+    const bool grouped = c.tiles.slot != HOLO_NO_SLOT, window = c.a_pos.slot != HOLO_NO_SLOT;
+    if (grouped) {
+        if ((c.tile_rows != 16 && c.tile_rows != 64 && c.tile_rows != 128) || c.m % c.tile_rows != 0 || c.experts == 0 || window || c.a_shared > c.tile_rows ||
+            c.lda != c.k || c.residual.slot != HOLO_NO_SLOT)
+            return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: grouped linear (%u rows in tiles of %u, %u experts, row pitch %u for k %u)", c.m, c.tile_rows,
+                             c.experts, c.lda, c.k);
+        a.tile_rows = c.tile_rows; a.experts = c.experts; a.a_shared = c.a_shared;
+    }
+    if (window && c.a_rows == 0) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: linear over a ring of no rows");
+    const uint64_t a_used = window ? c.a_rows : grouped && c.a_shared ? c.a_shared : c.m;
+    const uint64_t ab = a_used * c.lda * es, bb = (uint64_t)c.k * c.n * es * (grouped ? c.experts : 1);
     HOLO_TRY(holo_resolve(ws, c.a, ab, &pa, nullptr));
     HOLO_TRY(holo_resolve(ws, c.b, bb, &pb, nullptr));
+    if (grouped) {
+        HOLO_TRY(holo_resolve(ws, c.tiles, 4ull * (1 + c.m / c.tile_rows), &ptr, nullptr));
+        a.tiles = (const int32_t*)ptr;
+    }
+    if (window) {
+        HOLO_TRY(holo_resolve(ws, c.a_pos, 4, &ptr, nullptr));
+        a.a_pos = (const uint32_t*)ptr;
+        a.a_back = c.a_back; a.a_rows = c.a_rows;
+    }
+    if ((((uintptr_t)a.tiles | (uintptr_t)a.a_pos) & 3u) != 0) return holo_fail_slot(c.a.slot, "linear row words must be 4-byte aligned on the device");
     const bool with_res = c.residual.slot != HOLO_NO_SLOT;
     if (with_res && (c.nseg != 1 || c.seg[0].dtype != HOLO_DTYPE_F32))
         return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: a linear residual needs a single f32 segment");
     for (uint32_t i = 0; i < c.nseg; ++i) {
         const HoloLinearSeg& g = c.seg[i];
         if (g.dtype != HOLO_DTYPE_F32 && g.dtype != HOLO_DTYPE_BF16) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear output dtype %u", g.dtype);
-        if (g.act > HOLO_LINEAR_ACT_RELU2) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear activation %u", g.act);
+        if (g.act > HOLO_LINEAR_ACT_SILU_GATE) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: linear activation %u", g.act);
         const uint32_t prev_end = i ? c.seg[i - 1].col_begin + c.seg[i - 1].width : 0;
-        if (g.width == 0 || g.col_begin % 32 != 0 || g.col_begin < prev_end || (uint64_t)g.col_begin + g.width > c.n || g.ld < g.width ||
+        const uint32_t out_width = g.act == HOLO_LINEAR_ACT_SILU_GATE ? g.width / 2 : g.width;
+        if (g.act == HOLO_LINEAR_ACT_SILU_GATE && (g.width % 2 != 0 || with_res || g.rot_head))
+            return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: a gated linear segment takes pairs of columns, no residual and no rotation");
+        if (g.rot_head) {
+            if (g.rot_dims == 0 || g.rot_dims % 2 != 0 || g.rot_begin % 2 != 0 || g.rot_head % 2 != 0 || (uint64_t)g.rot_begin + g.rot_dims > g.rot_head || c.rot.slot == HOLO_NO_SLOT)
+                return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: linear segment %u rotates columns %u + %u of heads of %u", i, g.rot_begin, g.rot_dims, g.rot_head);
+            HOLO_TRY(holo_resolve(ws, c.rot, 4ull * c.m * g.rot_dims, &ptr, nullptr));
+            if (((uintptr_t)ptr & 7u) != 0) return holo_fail_slot(c.rot.slot, "the rotary table must be 8-byte aligned on the device");
+            a.rot = (const float*)ptr;
+        }
+        if (g.width == 0 || g.col_begin % 32 != 0 || g.col_begin < prev_end || (uint64_t)g.col_begin + g.width > c.n || g.ld < out_width ||
             (uint64_t)g.k_offset + c.k > c.lda || (i == 0 && g.col_begin != 0) ||
             (i > 0 && g.k_offset != c.seg[i - 1].k_offset && g.col_begin % 256 != 0))
             return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: linear segment %u (columns %u + %u of %u, k offset %u, pitch %u)", i, g.col_begin, g.width, c.n, g.k_offset, g.ld);
         const uint64_t os = holo_dtype_size(g.dtype);
         // with a row offset the rows land somewhere in a buffer of whole rows; the kernel drops rows past its end
         const bool appends = g.row_pos.slot != HOLO_NO_SLOT;
-        const uint64_t ob = (appends ? g.width : (uint64_t)(c.m - 1) * g.ld + g.width) * os;
+        if (g.ring && !appends) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: linear segment %u is a ring without its position", i);
+        const uint64_t ob = (appends ? out_width : (uint64_t)(c.m - 1) * g.ld + out_width) * os;
         uint64_t extent = 0;
         HOLO_TRY(holo_resolve(ws, g.output, ob, &ptr, &extent));
         HOLO_TRY(check_disjoint({ptr, appends ? extent : ob}, g.output.slot, {{pa, ab}, {pb, bb}}));
@@ -991,12 +1033,15 @@ int32_t do_linear(holo_b200_ctx* ctx, const HoloLinearCall& c, holo_b200_workspa
         o.out = ptr;
         o.row_pos = nullptr;
         if (appends) {
-            HOLO_TRY(holo_resolve(ws, g.row_pos, 4, &ptr, nullptr));
+            HOLO_TRY(holo_resolve(ws, g.row_pos, g.ring ? 8 : 4, &ptr, nullptr));
             if (((uintptr_t)ptr & 3u) != 0) return holo_fail_slot(g.row_pos.slot, "row_pos operand must be 4-byte aligned on the device");
             o.row_pos = (const uint32_t*)ptr;
         }
-        o.row_limit = appends ? extent / ((uint64_t)g.ld * os) : c.m;
+        // rows the buffer has (a ring's rows may be the columns of wider ones: the last is as long as what is stored)
+        o.row_limit = g.ring ? (extent - ob) / ((uint64_t)g.ld * os) + 1 : appends ? extent / ((uint64_t)g.ld * os) : c.m;
         o.col_begin = g.col_begin; o.width = g.width; o.k_offset = g.k_offset; o.ld = g.ld; o.act = g.act; o.dtype = g.dtype;
+        o.rot_head = g.rot_head; o.rot_begin = g.rot_begin; o.rot_dims = g.rot_dims; o.ring = g.ring;
+        if (o.row_limit == 0) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: linear segment %u's buffer holds no row", i);
         if (with_res) {
             HOLO_TRY(holo_resolve(ws, c.residual, ob, &ptr, nullptr));
             if (((uintptr_t)ptr & 3u) != 0) return holo_fail_slot(c.residual.slot, "linear residual must be 4-byte aligned");
@@ -1042,6 +1087,199 @@ int32_t do_causal_attention(holo_b200_ctx* ctx, const HoloCausalAttentionCall& c
         return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: causal_attention: softcap and temp_every must not be negative");
     a.dtype = c.dtype;
     return holo_launch_causal_attention(ctx, a);
+}
+
+// ---- further operations of decoder steps (all extensions) ----
+// Resolve `rows` rows of `width` elements of pitch `ld`.
+int32_t resolve_rows(holo_b200_workspace* ws, const HoloBufferRef& ref, uint64_t rows, uint64_t ld, uint64_t width, uint64_t es, uint8_t** ptr, Range* range) {
+    if (width > ld) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: rows of %llu columns at a pitch of %llu", (unsigned long long)width, (unsigned long long)ld);
+    const uint64_t bytes = ((rows - 1) * ld + width) * es;
+    HOLO_TRY(holo_resolve(ws, ref, bytes, ptr, nullptr));
+    if (((uintptr_t)*ptr & (es - 1)) != 0) return holo_fail_slot(ref.slot, "operand must be aligned to its element on the device");
+    if (range) *range = {*ptr, bytes};
+    return HOLO_OK;
+}
+int32_t resolve_words(holo_b200_workspace* ws, const HoloBufferRef& ref, uint64_t words, uint8_t** ptr) {
+    HOLO_TRY(holo_resolve(ws, ref, 4 * words, ptr, nullptr));
+    return ((uintptr_t)*ptr & 3u) != 0 ? holo_fail_slot(ref.slot, "operand must be 4-byte aligned on the device") : HOLO_OK;
+}
+bool float_or_bf16(uint8_t dtype) { return dtype == HOLO_DTYPE_F32 || dtype == HOLO_DTYPE_BF16; }
+
+int32_t do_rotary_table(holo_b200_ctx* ctx, const HoloRotaryTableCall& c, holo_b200_workspace* ws) {
+    if (c.rows == 0 || c.half == 0) return HOLO_OK;
+    uint8_t *pos, *freq, *out;
+    const uint64_t fb = 8ull * c.half, ob = 8ull * c.rows * c.half;
+    HOLO_TRY(resolve_words(ws, c.pos, 1, &pos));
+    HOLO_TRY(resolve_words(ws, c.freq, 2ull * c.half, &freq));
+    HOLO_TRY(holo_resolve(ws, c.output, ob, &out, nullptr));
+    HOLO_TRY(check_disjoint({out, ob}, c.output.slot, {{pos, 4}, {freq, fb}}));
+    if (((uintptr_t)out & 7u) != 0) return holo_fail_slot(c.output.slot, "the rotary table must be 8-byte aligned on the device");
+    return holo_launch_rotary_table(ctx, (const uint32_t*)pos, (const float*)freq, (float*)out, c.rows, c.half);
+}
+
+int32_t do_rms_norm_parts(holo_b200_ctx* ctx, const HoloRmsNormPartsCall& c, holo_b200_workspace* ws) {
+    if (c.nparts < 1 || c.nparts > HOLO_NORM_MAX_PARTS || !float_or_bf16(c.dtype))
+        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: norm of %u parts to dtype %u", c.nparts, c.dtype);
+    if (c.rows == 0) return HOLO_OK;
+    HoloNormPartsArgs a = {};
+    a.eps = f32_of_bits(c.epsilon_bits);
+    if (!(isfinite(a.eps) && a.eps > 0.0f)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: norm epsilon must be a positive finite f32");
+    const uint64_t es = holo_dtype_size(c.dtype);
+    uint8_t *x, *ptr;
+    Range xr;
+    uint64_t last = 0;
+    for (uint32_t i = 0; i < c.nparts; ++i) last = std::max<uint64_t>(last, (uint64_t)c.part[i].in_col + c.part[i].width);
+    HOLO_TRY(resolve_rows(ws, c.x, c.rows, c.ld_in, last, 4, &x, &xr));
+    if (c.step.slot != HOLO_NO_SLOT) {
+        HOLO_TRY(resolve_words(ws, c.step, 2, &ptr));
+        a.step = (const uint32_t*)ptr;
+    }
+    for (uint32_t i = 0; i < c.nparts; ++i) {
+        const HoloNormPart& p = c.part[i];
+        HoloNormPartArgs& o = a.part[i];
+        if (p.width == 0 || p.out_width < p.width || p.ld < p.out_width || (p.ring && !a.step))
+            return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: norm part %u (columns %u of %u, pitch %u)", i, p.width, p.out_width, p.ld);
+        if (p.weight.slot != HOLO_NO_SLOT) {
+            HOLO_TRY(resolve_words(ws, p.weight, p.width, &ptr));
+            o.weight = (const float*)ptr;
+        }
+        const uint64_t ob = (p.ring ? p.out_width : (uint64_t)(c.rows - 1) * p.ld + p.out_width) * es;
+        uint64_t extent = 0;
+        HOLO_TRY(holo_resolve(ws, p.output, ob, &ptr, &extent));
+        HOLO_TRY(check_disjoint({ptr, p.ring ? extent : ob}, p.output.slot, {xr, {(const uint8_t*)o.weight, o.weight ? 4ull * p.width : 0}}));
+        if (((uintptr_t)ptr & (es - 1)) != 0) return holo_fail_slot(p.output.slot, "norm output must be aligned to its element");
+        o.out = ptr;
+        o.in_col = p.in_col; o.width = p.width; o.out_width = p.out_width; o.ld = p.ld; o.norm = p.norm; o.ring = p.ring;
+        o.row_limit = p.ring ? (extent - ob) / ((uint64_t)p.ld * es) + 1 : c.rows;
+    }
+    a.x = (const float*)x;
+    a.rows = c.rows; a.ld_in = c.ld_in; a.nparts = c.nparts; a.dtype = c.dtype;
+    return holo_launch_rms_norm_parts(ctx, a);
+}
+
+int32_t do_head_linear(holo_b200_ctx* ctx, const HoloHeadLinearCall& c, holo_b200_workspace* ws) {
+    if (!float_or_bf16(c.dtype)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: head_linear dtype %u", c.dtype);
+    if (c.rows == 0 || c.heads == 0 || c.k == 0 || c.n == 0) return HOLO_OK;
+    if (c.out_step < c.n || c.b_ld < c.n) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: head_linear of %u columns (pitches %u, %u)", c.n, c.out_step, c.b_ld);
+    const uint64_t es = holo_dtype_size(c.dtype);
+    HoloHeadLinearArgs a = {};
+    uint8_t *pa, *pb, *out;
+    Range ra, ro;
+    const uint64_t bb = ((uint64_t)(c.heads - 1) * c.b_step + (uint64_t)(c.k - 1) * c.b_ld + c.n) * es;
+    HOLO_TRY(resolve_rows(ws, c.a, c.rows, c.lda, (uint64_t)(c.heads - 1) * c.a_step + c.k, es, &pa, &ra));
+    HOLO_TRY(resolve_rows(ws, c.output, c.rows, c.ld, (uint64_t)(c.heads - 1) * c.out_step + c.n, es, &out, &ro));
+    HOLO_TRY(holo_resolve(ws, c.b, bb, &pb, nullptr));
+    HOLO_TRY(check_disjoint(ro, c.output.slot, {ra, {pb, bb}}));
+    if (((uintptr_t)pb & (es - 1)) != 0) return holo_fail_slot(c.b.slot, "operand must be aligned to its element on the device");
+    a.a = pa; a.b = pb; a.out = out;
+    a.rows = c.rows; a.heads = c.heads; a.k = c.k; a.n = c.n; a.lda = c.lda; a.a_step = c.a_step; a.b_ld = c.b_ld; a.b_step = c.b_step;
+    a.ld = c.ld; a.out_step = c.out_step; a.dtype = c.dtype;
+    return holo_launch_head_linear(ctx, a);
+}
+
+int32_t do_window_attention(holo_b200_ctx* ctx, const HoloWindowAttentionCall& c, holo_b200_workspace* ws) {
+    if (!float_or_bf16(c.dtype)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: window_attention dtype %u", c.dtype);
+    if (c.rows == 0 || c.heads == 0) return HOLO_OK;
+    if (c.kv_heads == 0 || c.heads % c.kv_heads != 0)
+        return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: window_attention: heads must be a multiple of kv_heads (grouped-query)");
+    if (c.dim == 0 || c.vdim == 0 || c.dim > 1024 || c.vdim > 1024 || c.dim2 > 1024 || c.kv_rows == 0 || (c.dim2 && c.k2_rows == 0) || c.scale_bits == 0)
+        return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: window_attention dim %u + %u, vdim %u over %u rows", c.dim, c.dim2, c.vdim, c.kv_rows);
+    const uint64_t es = holo_dtype_size(c.dtype);
+    HoloWindowArgs a = {};
+    uint8_t *q, *k, *v, *q2 = nullptr, *k2 = nullptr, *pos, *sink = nullptr, *out;
+    Range rq, rk, rv, rq2 = {}, rk2 = {}, ro;
+    HOLO_TRY(resolve_rows(ws, c.q, c.rows, c.q_ld, (uint64_t)(c.heads - 1) * c.q_step + c.dim, es, &q, &rq));
+    HOLO_TRY(resolve_rows(ws, c.k, c.kv_rows, c.k_ld, (uint64_t)c.kv_heads * c.dim, es, &k, &rk));
+    HOLO_TRY(resolve_rows(ws, c.v, c.kv_rows, c.v_ld, (uint64_t)c.kv_heads * c.vdim, es, &v, &rv));
+    if (c.dim2) {
+        HOLO_TRY(resolve_rows(ws, c.q2, c.rows, c.q2_ld, (uint64_t)(c.heads - 1) * c.q2_step + c.dim2, es, &q2, &rq2));
+        HOLO_TRY(resolve_rows(ws, c.k2, c.k2_rows, c.k2_ld, c.dim2, es, &k2, &rk2));
+    }
+    HOLO_TRY(resolve_words(ws, c.pos, 1, &pos));
+    if (c.sink.slot != HOLO_NO_SLOT) HOLO_TRY(resolve_words(ws, c.sink, c.heads, &sink));
+    HOLO_TRY(resolve_rows(ws, c.output, c.rows, c.ld, (uint64_t)c.heads * c.vdim, es, &out, &ro));
+    HOLO_TRY(check_disjoint(ro, c.output.slot, {rq, rk, rv, rq2, rk2, {pos, 4}, {sink, sink ? 4ull * c.heads : 0}}));
+    a.q = q; a.k = k; a.v = v; a.q2 = q2; a.k2 = k2; a.pos = (const uint32_t*)pos; a.sink = (const float*)sink; a.out = out;
+    a.rows = c.rows; a.heads = c.heads; a.kv_heads = c.kv_heads; a.dim = c.dim; a.vdim = c.vdim; a.dim2 = c.dim2;
+    a.q_ld = c.q_ld; a.q_step = c.q_step; a.k_ld = c.k_ld; a.v_ld = c.v_ld; a.q2_ld = c.q2_ld; a.q2_step = c.q2_step; a.k2_ld = c.k2_ld; a.ld = c.ld;
+    a.kv_rows = c.kv_rows; a.kv_back = c.kv_back; a.k2_rows = c.k2_rows; a.window = c.window;
+    a.scale = f32_of_bits(c.scale_bits);
+    a.dtype = c.dtype;
+    return holo_launch_window_attention(ctx, a);
+}
+
+int32_t do_retention(holo_b200_ctx* ctx, const HoloRetentionCall& c, holo_b200_workspace* ws) {
+    if (!float_or_bf16(c.dtype)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: retention dtype %u", c.dtype);
+    if (c.rows == 0 || c.heads == 0) return HOLO_OK;
+    if (c.dim == 0 || c.vdim == 0 || c.dim > 1024 || c.vdim > 1024 || c.vmean == 0 || c.vmean > c.vdim)
+        return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: retention dim %u, vdim %u (%u in use)", c.dim, c.vdim, c.vmean);
+    const uint64_t es = holo_dtype_size(c.dtype), sb = 4ull * c.heads * c.dim * c.vdim;
+    HoloRetentionArgs a = {};
+    uint8_t *q, *k, *v, *gate, *decay, *step, *state, *out;
+    Range rq, rk, rv, rg, ro;
+    HOLO_TRY(resolve_rows(ws, c.q, c.rows, c.q_ld, (uint64_t)c.heads * c.dim, es, &q, &rq));
+    HOLO_TRY(resolve_rows(ws, c.k, c.rows, c.k_ld, (uint64_t)c.heads * c.dim, es, &k, &rk));
+    HOLO_TRY(resolve_rows(ws, c.v, c.rows, c.v_ld, (uint64_t)c.heads * c.vdim, es, &v, &rv));
+    HOLO_TRY(resolve_rows(ws, c.gate, c.rows, c.gate_ld, (uint64_t)c.heads * c.vdim, es, &gate, &rg));
+    HOLO_TRY(resolve_rows(ws, c.output, c.rows, c.ld, (uint64_t)c.heads * c.vdim, es, &out, &ro));
+    HOLO_TRY(resolve_words(ws, c.decay, c.heads, &decay));
+    HOLO_TRY(resolve_words(ws, c.step, 2, &step));
+    HOLO_TRY(holo_resolve(ws, c.state, sb, &state, nullptr));
+    if (((uintptr_t)state & 15u) != 0) return holo_fail_slot(c.state.slot, "the retention state must be 16-byte aligned on the device");
+    HOLO_TRY(check_disjoint(ro, c.output.slot, {rq, rk, rv, rg, {decay, 4ull * c.heads}, {step, 8}, {state, sb}}));
+    HOLO_TRY(check_disjoint({state, sb}, c.state.slot, {rq, rk, rv, rg, {decay, 4ull * c.heads}, {step, 8}}));
+    a.q = q; a.k = k; a.v = v; a.gate = gate; a.decay = (const float*)decay; a.step = (const uint32_t*)step; a.state = (float*)state; a.out = out;
+    a.rows = c.rows; a.heads = c.heads; a.dim = c.dim; a.vdim = c.vdim; a.vmean = c.vmean;
+    a.q_ld = c.q_ld; a.k_ld = c.k_ld; a.v_ld = c.v_ld; a.gate_ld = c.gate_ld; a.ld = c.ld;
+    a.scale = f32_of_bits(c.scale_bits);
+    a.eps = f32_of_bits(c.epsilon_bits);
+    a.dtype = c.dtype;
+    return holo_launch_retention(ctx, a);
+}
+
+int32_t do_moe_plan(holo_b200_ctx* ctx, const HoloMoePlanCall& c, holo_b200_workspace* ws) {
+    if (c.rows == 0) return HOLO_OK;
+    const uint64_t tiles = (c.rows <= c.tile_rows) ? std::min<uint64_t>(c.experts, (uint64_t)c.rows * c.top)
+                                                   : std::min<uint64_t>((uint64_t)c.rows * c.top, c.experts + (uint64_t)c.rows * c.top / c.tile_rows);
+    if (c.experts == 0 || c.experts > 1024 || c.top == 0 || c.top > c.experts || c.top > 32 || c.tile_rows == 0 || c.max_tiles < tiles)
+        return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: moe_plan of %u out of %u experts, %u tiles of %u rows", c.top, c.experts, c.max_tiles, c.tile_rows);
+    HoloMoePlanArgs a = {};
+    uint8_t *logits, *bias = nullptr, *step, *weight, *place, *tl, *source;
+    Range rl;
+    const uint64_t pairs = (uint64_t)c.rows * c.top, slots = (uint64_t)c.max_tiles * c.tile_rows;
+    HOLO_TRY(resolve_rows(ws, c.logits, c.rows, c.ld_logits, c.experts, 4, &logits, &rl));
+    if (c.bias.slot != HOLO_NO_SLOT) HOLO_TRY(resolve_words(ws, c.bias, c.experts, &bias));
+    HOLO_TRY(resolve_words(ws, c.step, 2, &step));
+    HOLO_TRY(resolve_words(ws, c.weight, pairs, &weight));
+    HOLO_TRY(resolve_words(ws, c.place, pairs, &place));
+    HOLO_TRY(resolve_words(ws, c.tiles, 1ull + c.max_tiles, &tl));
+    HOLO_TRY(resolve_words(ws, c.source, slots, &source));
+    const Range rw = {weight, 4 * pairs}, rp = {place, 4 * pairs}, rt = {tl, 4ull * (1 + c.max_tiles)}, rs = {source, 4 * slots};
+    const Range rb = {bias, bias ? 4ull * c.experts : 0}, rst = {step, 8};
+    HOLO_TRY(check_disjoint(rw, c.weight.slot, {rl, rb, rst, rp, rt, rs}));
+    HOLO_TRY(check_disjoint(rp, c.place.slot, {rl, rb, rst, rt, rs}));
+    HOLO_TRY(check_disjoint(rt, c.tiles.slot, {rl, rb, rst, rs}));
+    HOLO_TRY(check_disjoint(rs, c.source.slot, {rl, rb, rst}));
+    a.logits = (const float*)logits; a.bias = (const float*)bias; a.step = (const uint32_t*)step; a.weight = (float*)weight;
+    a.place = (int32_t*)place; a.tiles = (int32_t*)tl; a.source = (int32_t*)source;
+    a.rows = c.rows; a.experts = c.experts; a.top = c.top; a.ld_logits = c.ld_logits; a.tile_rows = c.tile_rows; a.max_tiles = c.max_tiles;
+    return holo_launch_moe_plan(ctx, a);
+}
+
+int32_t do_moe_combine(holo_b200_ctx* ctx, const HoloMoeCombineCall& c, holo_b200_workspace* ws) {
+    if (!float_or_bf16(c.dtype)) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: moe_combine dtype %u", c.dtype);
+    if (c.rows == 0 || c.width == 0) return HOLO_OK;
+    if (c.y_rows == 0) return holo_fail(HOLO_ERR_SHAPE_MISMATCH, "shape mismatch: moe_combine of no rows");
+    uint8_t *x, *y, *weight, *place, *step;
+    Range rx, ry;
+    const uint64_t pairs = (uint64_t)c.rows * c.top;
+    HOLO_TRY(resolve_rows(ws, c.x, c.rows, c.width, c.width, 4, &x, &rx));
+    HOLO_TRY(resolve_rows(ws, c.y, c.y_rows, c.ld, c.width, holo_dtype_size(c.dtype), &y, &ry));
+    HOLO_TRY(resolve_words(ws, c.weight, pairs, &weight));
+    HOLO_TRY(resolve_words(ws, c.place, pairs, &place));
+    HOLO_TRY(resolve_words(ws, c.step, 2, &step));
+    HOLO_TRY(check_disjoint(rx, c.x.slot, {ry, {weight, 4 * pairs}, {place, 4 * pairs}, {step, 8}}));
+    return holo_launch_moe_combine(ctx, (float*)x, y, (const float*)weight, (const int32_t*)place, (const uint32_t*)step, c.rows, c.width, c.top, c.ld, c.y_rows, c.dtype);
 }
 
 int32_t do_all_reduce(holo_b200_ctx* ctx, const HoloAllReduceCall& c, holo_b200_workspace* ws) {
@@ -1102,7 +1340,15 @@ int32_t holo_dispatch_internal(holo_b200_ctx* ctx, const HoloKernelCall* call, h
         case HOLO_K_ALL_REDUCE: return do_all_reduce(ctx, call->u.all_reduce, ws);
         case HOLO_K_ROPE_QUANTIZE_ROWS_I8: return do_rope_quantize(ctx, call->u.rope_quantize, ws);
         case HOLO_K_RMS_NORM_MULTI: return do_rms_norm_multi(ctx, call->u.rms_norm_multi, ws);
-        case HOLO_K_LINEAR: return do_linear(ctx, call->u.linear, ws);
+        case HOLO_K_LINEAR: return do_linear(ctx, plain_linear(call->u.linear), ws);
+        case HOLO_K_LINEAR_EX: return do_linear(ctx, call->u.linear, ws);
+        case HOLO_K_ROTARY_TABLE: return do_rotary_table(ctx, call->u.rotary_table, ws);
+        case HOLO_K_RMS_NORM_PARTS: return do_rms_norm_parts(ctx, call->u.rms_norm_parts, ws);
+        case HOLO_K_HEAD_LINEAR: return do_head_linear(ctx, call->u.head_linear, ws);
+        case HOLO_K_WINDOW_ATTENTION: return do_window_attention(ctx, call->u.window_attention, ws);
+        case HOLO_K_RETENTION: return do_retention(ctx, call->u.retention, ws);
+        case HOLO_K_MOE_PLAN: return do_moe_plan(ctx, call->u.moe_plan, ws);
+        case HOLO_K_MOE_COMBINE: return do_moe_combine(ctx, call->u.moe_combine, ws);
         case HOLO_K_CAUSAL_ATTENTION: return do_causal_attention(ctx, call->u.causal_attention, ws);
         default:
             if (holo_is_exact_unary(call->kind) || holo_is_exact_binary(call->kind)) return do_elementwise(ctx, call, ws);
@@ -1280,14 +1526,63 @@ bool holo_collect_refs(HoloKernelCall* c, HoloRefList* l) {
             l->out(&q.output, (uint64_t)q.rows * q.step * (q.gamma1.slot != HOLO_NO_SLOT ? 2 : 1) * holo_dtype_size(q.dtype));
             return true;
         }
-        case HOLO_K_LINEAR: {
+        case HOLO_K_LINEAR: case HOLO_K_LINEAR_EX: {
             auto& q = c->u.linear;
             l->in(&q.a); l->in(&q.b); l->in(&q.residual);
+            if (c->kind == HOLO_K_LINEAR_EX) { l->in(&q.rot); l->in(&q.a_pos); l->in(&q.tiles); }
             for (uint32_t i = 0; i < q.nseg && i < HOLO_LINEAR_MAX_SEGS; ++i) {
                 l->in(&q.seg[i].row_pos);
                 const uint64_t rows = q.seg[i].row_pos.slot != HOLO_NO_SLOT ? 1 : q.m;   // an appending segment: the rows the buffer has
-                l->out(&q.seg[i].output, ((rows - 1) * q.seg[i].ld + q.seg[i].width) * holo_dtype_size(q.seg[i].dtype));
+                l->out(&q.seg[i].output, ((rows - 1) * q.seg[i].ld + (q.seg[i].act == HOLO_LINEAR_ACT_SILU_GATE ? q.seg[i].width / 2 : q.seg[i].width)) *
+                                          holo_dtype_size(q.seg[i].dtype));
             }
+            return true;
+        }
+        case HOLO_K_ROTARY_TABLE: {
+            auto& q = c->u.rotary_table;
+            l->in(&q.pos); l->in(&q.freq);
+            l->out(&q.output, 8ull * q.rows * q.half);
+            return true;
+        }
+        case HOLO_K_RMS_NORM_PARTS: {
+            auto& q = c->u.rms_norm_parts;
+            l->in(&q.x); l->in(&q.step);
+            for (uint32_t i = 0; i < q.nparts && i < HOLO_NORM_MAX_PARTS; ++i) {
+                l->in(&q.part[i].weight);
+                l->out(&q.part[i].output, ((uint64_t)(q.part[i].ring ? 0 : q.rows - 1) * q.part[i].ld + q.part[i].out_width) * holo_dtype_size(q.dtype));
+            }
+            return true;
+        }
+        case HOLO_K_HEAD_LINEAR: {
+            auto& q = c->u.head_linear;
+            l->in(&q.a); l->in(&q.b);
+            l->out(&q.output, ((uint64_t)(q.rows - 1) * q.ld + (uint64_t)(q.heads - 1) * q.out_step + q.n) * holo_dtype_size(q.dtype));
+            return true;
+        }
+        case HOLO_K_WINDOW_ATTENTION: {
+            auto& q = c->u.window_attention;
+            l->in(&q.q); l->in(&q.k); l->in(&q.v); l->in(&q.q2); l->in(&q.k2); l->in(&q.pos); l->in(&q.sink);
+            l->out(&q.output, ((uint64_t)(q.rows - 1) * q.ld + (uint64_t)q.heads * q.vdim) * holo_dtype_size(q.dtype));
+            return true;
+        }
+        case HOLO_K_RETENTION: {
+            auto& q = c->u.retention;
+            l->in(&q.q); l->in(&q.k); l->in(&q.v); l->in(&q.gate); l->in(&q.decay); l->in(&q.step);
+            l->out(&q.state, 4ull * q.heads * q.dim * q.vdim);
+            l->out(&q.output, ((uint64_t)(q.rows - 1) * q.ld + (uint64_t)q.heads * q.vdim) * holo_dtype_size(q.dtype));
+            return true;
+        }
+        case HOLO_K_MOE_PLAN: {
+            auto& q = c->u.moe_plan;
+            l->in(&q.logits); l->in(&q.bias); l->in(&q.step);
+            l->out(&q.weight, 4ull * q.rows * q.top); l->out(&q.place, 4ull * q.rows * q.top);
+            l->out(&q.tiles, 4ull * (1 + q.max_tiles)); l->out(&q.source, 4ull * q.max_tiles * q.tile_rows);
+            return true;
+        }
+        case HOLO_K_MOE_COMBINE: {
+            auto& q = c->u.moe_combine;
+            l->in(&q.y); l->in(&q.weight); l->in(&q.place); l->in(&q.step);
+            l->out(&q.x, 4ull * q.rows * q.width);
             return true;
         }
         case HOLO_K_CAUSAL_ATTENTION: {
@@ -1318,6 +1613,8 @@ extern "C" int32_t holo_b200_dispatch_host(holo_b200_ctx* ctx, const HoloKernelC
     HoloKernelCall local = *call;
     HoloRefList refs;
     bool appends = false;   // rows of a cache at a device-side position: only a device-resident buffer has them
+    // the buffers these keep from call to call (caches, state, residual) are device-resident as well
+    if (call->kind >= HOLO_K_LINEAR_EX && call->kind <= HOLO_K_MOE_COMBINE) appends = true;
     if (call->kind == HOLO_K_LINEAR)
         for (uint32_t i = 0; i < call->u.linear.nseg && i < HOLO_LINEAR_MAX_SEGS; ++i) appends |= call->u.linear.seg[i].row_pos.slot != HOLO_NO_SLOT;
     if (appends || !holo_collect_refs(&local, &refs))
@@ -1327,9 +1624,9 @@ extern "C" int32_t holo_b200_dispatch_host(holo_b200_ctx* ctx, const HoloKernelC
     // are uploaded whole; written operands are not uploaded and only the bytes the kernel
     // produces are copied back.
     uint64_t total = 0;
-    uint64_t off[12], len[12];
-    uint32_t orig_slot[12];
-    uint8_t* host_ptr[12];
+    uint64_t off[HOLO_MAX_REFS], len[HOLO_MAX_REFS];
+    uint32_t orig_slot[HOLO_MAX_REFS];
+    uint8_t* host_ptr[HOLO_MAX_REFS];
     for (int i = 0; i < refs.n; ++i) {
         HoloBufferRef r = *refs.refs[i];
         off[i] = len[i] = 0;

@@ -223,8 +223,9 @@ int32_t decode_call(Reader& r, HoloKernelCall* out) {
             c.rows = r.u32(); c.feature = r.u32(); c.step = r.u32(); c.epsilon_bits = r.u32(); c.dtype = r.u8();
             break;
         }
-        case HOLO_K_LINEAR: {
+        case HOLO_K_LINEAR: case HOLO_K_LINEAR_EX: {
             HoloLinearCall& c = out->u.linear;
+            c.rot = c.a_pos = c.tiles = HoloBufferRef{HOLO_NO_SLOT, 0, 0};
             c.a = r.buf(); c.b = r.buf(); c.residual = r.buf();
             c.m = r.u32(); c.k = r.u32(); c.n = r.u32(); c.lda = r.u32(); c.alpha_bits = r.u32(); c.dtype = r.u8();
             c.nseg = r.u8();
@@ -235,6 +236,72 @@ int32_t decode_call(Reader& r, HoloKernelCall* out) {
                 g.output = r.buf(); g.row_pos = r.buf();
                 g.col_begin = r.u32(); g.width = r.u32(); g.k_offset = r.u32(); g.ld = r.u32(); g.act = r.u8(); g.dtype = r.u8();
             }
+            if (d == HOLO_K_LINEAR) break;
+            for (uint32_t i = 0; i < c.nseg; ++i) {
+                HoloLinearSeg& g = c.seg[i];
+                g.rot_head = r.u32(); g.rot_begin = r.u32(); g.rot_dims = r.u32(); g.ring = r.u8();
+            }
+            c.rot = r.buf(); c.a_pos = r.buf(); c.tiles = r.buf();
+            c.a_back = r.u32(); c.a_rows = r.u32(); c.tile_rows = r.u32(); c.experts = r.u32(); c.a_shared = r.u32();
+            break;
+        }
+        case HOLO_K_RMS_NORM_PARTS: {
+            HoloRmsNormPartsCall& c = out->u.rms_norm_parts;
+            c.x = r.buf(); c.step = r.buf(); c.rows = r.u32(); c.ld_in = r.u32(); c.epsilon_bits = r.u32(); c.dtype = r.u8();
+            c.nparts = r.u8();
+            if (c.nparts < 1 || c.nparts > HOLO_NORM_MAX_PARTS || c.rows == 0)
+                return holo_fail(HOLO_ERR_INIT, "backend init failed: norm of %u parts over %u rows", c.nparts, c.rows);
+            for (uint32_t i = 0; i < c.nparts; ++i) {
+                HoloNormPart& p = c.part[i];
+                p.weight = r.buf(); p.output = r.buf(); p.in_col = r.u32(); p.width = r.u32(); p.out_width = r.u32(); p.ld = r.u32();
+                p.norm = r.u8(); p.ring = r.u8();
+            }
+            break;
+        }
+        case HOLO_K_ROTARY_TABLE: {
+            HoloRotaryTableCall& c = out->u.rotary_table;
+            c.pos = r.buf(); c.freq = r.buf(); c.output = r.buf(); c.rows = r.u32(); c.half = r.u32();
+            break;
+        }
+        case HOLO_K_HEAD_LINEAR: {
+            HoloHeadLinearCall& c = out->u.head_linear;
+            c.a = r.buf(); c.b = r.buf(); c.output = r.buf();
+            for (uint32_t* f : {&c.rows, &c.heads, &c.k, &c.n, &c.lda, &c.a_step, &c.b_ld, &c.b_step, &c.ld, &c.out_step}) *f = r.u32();
+            c.dtype = r.u8();
+            if (c.rows == 0 || c.heads == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: head product over no rows");
+            break;
+        }
+        case HOLO_K_WINDOW_ATTENTION: {
+            HoloWindowAttentionCall& c = out->u.window_attention;
+            for (HoloBufferRef* b : {&c.q, &c.k, &c.v, &c.q2, &c.k2, &c.pos, &c.sink, &c.output}) *b = r.buf();
+            for (uint32_t* f : {&c.rows, &c.heads, &c.kv_heads, &c.dim, &c.vdim, &c.dim2, &c.q_ld, &c.q_step, &c.k_ld, &c.v_ld, &c.q2_ld, &c.q2_step,
+                                &c.k2_ld, &c.ld, &c.kv_rows, &c.kv_back, &c.k2_rows, &c.window, &c.scale_bits})
+                *f = r.u32();
+            c.dtype = r.u8();
+            if (c.rows == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: window attention over no rows");
+            break;
+        }
+        case HOLO_K_RETENTION: {
+            HoloRetentionCall& c = out->u.retention;
+            for (HoloBufferRef* b : {&c.q, &c.k, &c.v, &c.gate, &c.decay, &c.step, &c.state, &c.output}) *b = r.buf();
+            for (uint32_t* f : {&c.rows, &c.heads, &c.dim, &c.vdim, &c.vmean, &c.q_ld, &c.k_ld, &c.v_ld, &c.gate_ld, &c.ld, &c.scale_bits, &c.epsilon_bits}) *f = r.u32();
+            c.dtype = r.u8();
+            if (c.rows == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: retention over no rows");
+            break;
+        }
+        case HOLO_K_MOE_PLAN: {
+            HoloMoePlanCall& c = out->u.moe_plan;
+            for (HoloBufferRef* b : {&c.logits, &c.bias, &c.step, &c.weight, &c.place, &c.tiles, &c.source}) *b = r.buf();
+            for (uint32_t* f : {&c.rows, &c.experts, &c.top, &c.ld_logits, &c.tile_rows, &c.max_tiles}) *f = r.u32();
+            if (c.rows == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: routing of no rows");
+            break;
+        }
+        case HOLO_K_MOE_COMBINE: {
+            HoloMoeCombineCall& c = out->u.moe_combine;
+            for (HoloBufferRef* b : {&c.x, &c.y, &c.weight, &c.place, &c.step}) *b = r.buf();
+            for (uint32_t* f : {&c.rows, &c.width, &c.top, &c.ld, &c.y_rows}) *f = r.u32();
+            c.dtype = r.u8();
+            if (c.rows == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: combination over no rows");
             break;
         }
         case HOLO_K_CAUSAL_ATTENTION: {

@@ -44,6 +44,7 @@ struct holo_b200_ctx {
     // device-side error word (bounded waits record where they gave up)
     uint32_t* dev_status = nullptr;
     float* causal_partials = nullptr;   // split-key partials of the causal attention, allocated once at a fixed size (graphs hold its address)
+    float* latent_partials = nullptr;   // the same for the latent attention
     uint32_t* attn_arrivals = nullptr;  // 65536 counters, zero between launches (decode attention)
     // launch every kernel with programmatic stream serialization (HOLO_PDL=0 turns it off)
     bool pdl = true;
@@ -98,12 +99,13 @@ static inline bool holo_is_compute_float(uint8_t d) {
     return d == HOLO_DTYPE_F16 || d == HOLO_DTYPE_BF16 || d == HOLO_DTYPE_F32;
 }
 
+constexpr int HOLO_MAX_REFS = 16;   // the widest call is Linear: a, b, residual, rot, a_pos, tiles, four (output, row_pos) pairs
 // Every BufferRef of a call; `out_bytes` > 0 marks a written operand and gives the number of
 // bytes the kernel produces there (inputs carry 0).
 struct HoloRefList {
-    HoloBufferRef* refs[12];      // the widest call is Linear: a, b, residual, four (output, row_pos) pairs
-    uint64_t out_bytes[12];
-    bool written[12];
+    HoloBufferRef* refs[HOLO_MAX_REFS];
+    uint64_t out_bytes[HOLO_MAX_REFS];
+    bool written[HOLO_MAX_REFS];
     int n = 0;
     void in(HoloBufferRef* r) {
         refs[n] = r;
@@ -270,14 +272,19 @@ struct HoloLinearSegArgs {
     void* out;
     const uint32_t* row_pos;
     uint32_t col_begin, width, k_offset, ld;
-    uint64_t row_limit;          // rows the output buffer has: rows at or past it are not stored
-    uint8_t act, dtype;
+    uint64_t row_limit;          // rows the output buffer has: rows at or past it are not stored (ring: rows wrap there)
+    uint32_t rot_head, rot_begin, rot_dims;
+    uint8_t act, dtype, ring;
 };
 struct HoloLinearArgs {
     const void *a, *b;
     const float* residual;
+    const float* rot;            // cosines and sines of the rotated segments
+    const uint32_t* a_pos;       // A is a ring of a_rows rows, see HoloLinearCall
+    const int32_t* tiles;        // grouped product
     HoloLinearSegArgs seg[HOLO_LINEAR_MAX_SEGS];
     uint32_t m, k, n, lda, nseg;
+    uint32_t a_back, a_rows, tile_rows, experts, a_shared;
     float alpha;
     uint8_t dtype;
     bool b_constant;
@@ -296,6 +303,66 @@ struct HoloCausalArgs {
     uint8_t dtype;
 };
 int32_t holo_launch_causal_attention(holo_b200_ctx* ctx, const HoloCausalArgs& a);
+// linear.cu: further operations of decoder steps
+int32_t holo_launch_rotary_table(holo_b200_ctx* ctx, const uint32_t* pos, const float* freq, float* out, uint32_t rows, uint32_t half);
+struct HoloNormPartArgs {
+    const float* weight;         // null = ones
+    void* out;
+    uint32_t in_col, width, out_width, ld, norm, ring;
+    uint64_t row_limit;
+};
+struct HoloNormPartsArgs {
+    const float* x;
+    const uint32_t* step;
+    HoloNormPartArgs part[HOLO_NORM_MAX_PARTS];
+    uint32_t rows, ld_in, nparts;
+    float eps;
+    uint8_t dtype;
+};
+int32_t holo_launch_rms_norm_parts(holo_b200_ctx* ctx, const HoloNormPartsArgs& a);
+struct HoloHeadLinearArgs {
+    const void *a, *b;
+    void* out;
+    uint32_t rows, heads, k, n, lda, a_step, b_ld, b_step, ld, out_step;
+    uint8_t dtype;
+};
+int32_t holo_launch_head_linear(holo_b200_ctx* ctx, const HoloHeadLinearArgs& a);
+// window_attention.cu
+struct HoloWindowArgs {
+    const void *q, *k, *v, *q2, *k2;
+    const uint32_t* pos;
+    const float* sink;           // null = no sink
+    void* out;
+    uint32_t rows, heads, kv_heads, dim, vdim, dim2;
+    uint32_t q_ld, q_step, k_ld, v_ld, q2_ld, q2_step, k2_ld, ld;
+    uint32_t kv_rows, kv_back, k2_rows, window;
+    float scale;
+    uint8_t dtype;
+};
+int32_t holo_launch_window_attention(holo_b200_ctx* ctx, const HoloWindowArgs& a);
+// retention.cu
+struct HoloRetentionArgs {
+    const void *q, *k, *v, *gate;
+    const float* decay;
+    const uint32_t* step;
+    float* state;
+    void* out;
+    uint32_t rows, heads, dim, vdim, vmean, q_ld, k_ld, v_ld, gate_ld, ld;
+    float scale, eps;
+    uint8_t dtype;
+};
+int32_t holo_launch_retention(holo_b200_ctx* ctx, const HoloRetentionArgs& a);
+// moe.cu
+struct HoloMoePlanArgs {
+    const float *logits, *bias;
+    const uint32_t* step;
+    float* weight;
+    int32_t *place, *tiles, *source;
+    uint32_t rows, experts, top, ld_logits, tile_rows, max_tiles;
+};
+int32_t holo_launch_moe_plan(holo_b200_ctx* ctx, const HoloMoePlanArgs& a);
+int32_t holo_launch_moe_combine(holo_b200_ctx* ctx, float* x, const void* y, const float* weight, const int32_t* place, const uint32_t* step, uint32_t rows,
+                                uint32_t width, uint32_t top, uint32_t ld, uint32_t y_rows, uint8_t dtype);
 // quant_gemv.cu
 int32_t holo_launch_matmul_e8cb_omajor(holo_b200_ctx* ctx, const float* a, const uint8_t* bq, const int8_t* codebook, const float* scales,
                                        const int32_t* zero_points, const float* residual, float* out, uint32_t m, uint32_t k, uint32_t n, int act);

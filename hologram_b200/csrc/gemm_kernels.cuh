@@ -61,6 +61,8 @@ struct GemmLin {
     uint64_t row_limit;          // rows of the buffer: rows at or past it are dropped
     uint32_t col_begin, width, k_offset, ld;
     uint32_t act, f32;           // HOLO_LINEAR_ACT_*; f32 = the stored type is f32, else bf16
+    uint32_t ring;               // row_pos has two words, (first, count): rows wrap at row_limit, rows from count on are dropped
+    uint32_t rot_head, rot_begin, rot_dims;   // rotation of adjacent column pairs, see HoloLinearSeg
 };
 constexpr int MAX_LIN = 4;
 
@@ -85,6 +87,11 @@ struct GemmParams {
     GemmLin lin[MAX_LIN];
     uint32_t nlin;
     float alpha;
+    const float2* rot;           // (cos, sin) per row and pair
+    const uint32_t* a_pos;       // A is a ring of a_rows rows that starts a_back rows before *a_pos
+    uint32_t a_back, a_rows;
+    const int32_t* tiles;        // grouped: tiles in use, then the expert of each tile of tile_rows rows; B is [experts * k, n]
+    uint32_t tile_rows, a_shared;
 };
 
 // The Linear segment a column falls into (the last one that begins at or before it).
@@ -93,45 +100,96 @@ __device__ __forceinline__ uint32_t lin_segment(const GemmParams& p, uint32_t co
     while (si + 1 < p.nlin && col >= p.lin[si + 1].col_begin) ++si;
     return si;
 }
+// The A row behind row m0 of the product (m0 a multiple of the tile's rows).
+__device__ __forceinline__ uint32_t lin_a_row(const GemmParams& p, uint32_t m0) {
+    const uint32_t pos = *p.a_pos;
+    return (((pos > p.a_back ? pos - p.a_back : 0u) & ~127u) + m0) % p.a_rows;
+}
+// What a CTA's tile of a Linear product reads and stores, once the dependency wait is over.
+struct LinTile {
+    uint32_t a_row, b_row, m_end;   // first A row, first B row, end of the rows to store (m0 when the tile is not in use)
+    bool used;
+};
+__device__ __forceinline__ LinTile lin_tile(const GemmParams& p, uint32_t tile, uint32_t m0) {
+    LinTile t = {m0, 0u, p.m, true};
+    if (p.tiles) {
+        t.used = tile < (uint32_t)p.tiles[0];
+        if (t.used) t.b_row = (uint32_t)p.tiles[1 + tile] * p.k;
+        if (p.a_shared) t.a_row = 0;
+        t.m_end = !t.used ? m0 : m0 + (p.a_shared ? p.a_shared : p.tile_rows);
+    } else if (p.a_pos) {
+        t.a_row = lin_a_row(p, m0);
+    }
+    return t;
+}
+// z / (1 + exp(-t)); FAST where the result is rounded to bf16
+template <bool FAST>
+__device__ __forceinline__ float sigmoid_times(float z, float t) {
+    return FAST ? z * __fdividef(1.0f, 1.0f + __expf(-t)) : z / (1.0f + expf(-t));
+}
+template <bool FAST>
 __device__ __forceinline__ float lin_act(float v, uint32_t act) {
     if (act == HOLO_LINEAR_ACT_RELU2) {
         v = fmaxf(v, 0.0f);
         v *= v;
+    } else if (act == HOLO_LINEAR_ACT_GELU_TANH) {
+        v = sigmoid_times<FAST>(v, 1.5957691216057308f * fmaf(0.044715f * v * v, v, v));   // 0.5 (1 + tanh(y)) = 1 / (1 + exp(-2 y))
+    } else if (act == HOLO_LINEAR_ACT_SILU) {
+        v = sigmoid_times<FAST>(v, v);
     }
     return v;
 }
-// Finish and store N consecutive cells of one row (N a multiple of 4, the cells in one segment).
+// The buffer row a product row goes to; false when it is not stored.
+__device__ __forceinline__ bool lin_out_row(const GemmLin& g, uint32_t row, uint64_t* out) {
+    uint32_t r = row;
+    if (g.row_pos) {
+        r += g.row_pos[0];
+        if (g.ring) {
+            if (row >= g.row_pos[1]) return false;
+            r %= (uint32_t)g.row_limit;
+        }
+    }
+    *out = r;
+    return r < g.row_limit;
+}
+// Turn the pairs of N consecutive columns (N and the first column even) of one row.
 template <int N>
-__device__ __forceinline__ void lin_store(const GemmParams& p, uint32_t row, uint32_t col, const float (&acc)[N]) {
-    const GemmLin& g = p.lin[lin_segment(p, col)];
-    const uint32_t c = col - g.col_begin, width = g.width;
-    if (c >= width) return;
-    const uint64_t orow = (uint64_t)row + (g.row_pos ? *g.row_pos : 0u);
-    if (orow >= g.row_limit) return;
-    const uint64_t idx = orow * g.ld + c;
-    const float alpha = p.alpha;
-    const uint32_t act = g.act;
-    float v[N];
+__device__ __forceinline__ void lin_rotate(const GemmParams& p, const GemmLin& g, uint32_t row, uint32_t c, float (&v)[N]) {
+    uint32_t cc = c % g.rot_head;
+    const float2* table = p.rot + (uint64_t)row * (g.rot_dims >> 1);
 #pragma unroll
-    for (int i = 0; i < N; ++i) v[i] = alpha * lin_act(acc[i], act);
-    const bool full = c + N <= width;
+    for (int i = 0; i < N; i += 2) {
+        if (cc >= g.rot_begin && cc < g.rot_begin + g.rot_dims) {
+            const float2 t = table[(cc - g.rot_begin) >> 1];
+            const float a = v[i], b = v[i + 1];
+            v[i] = a * t.x - b * t.y;
+            v[i + 1] = b * t.x + a * t.y;
+        }
+        cc += 2;
+        if (cc >= g.rot_head) cc -= g.rot_head;
+    }
+}
+// Store N consecutive finished cells of one row, of which `left` exist.
+template <int N>
+__device__ __forceinline__ void lin_put(const GemmLin& g, uint64_t idx, uint32_t left, float (&v)[N]) {
+    const bool full = N <= left;
     if (g.f32) {
         float* out = reinterpret_cast<float*>(g.out) + idx;
         const float* res = g.residual ? g.residual + idx : nullptr;
-        if (full && ((uintptr_t)out & 15u) == 0 && ((uintptr_t)res & 15u) == 0) {
+        if (N % 4 == 0 && full && ((uintptr_t)out & 15u) == 0 && ((uintptr_t)res & 15u) == 0) {
             if (res) {
 #pragma unroll
-                for (int i = 0; i < N; i += 4) {
+                for (int i = 0; i + 3 < N; i += 4) {
                     const float4 r = *reinterpret_cast<const float4*>(res + i);
                     v[i] += r.x; v[i + 1] += r.y; v[i + 2] += r.z; v[i + 3] += r.w;
                 }
             }
 #pragma unroll
-            for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(out + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+            for (int i = 0; i + 3 < N; i += 4) *reinterpret_cast<float4*>(out + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
         } else {
 #pragma unroll
             for (int i = 0; i < N; ++i)
-                if (c + i < width) out[i] = v[i] + (res ? res[i] : 0.0f);
+                if ((uint32_t)i < left) out[i] = v[i] + (res ? res[i] : 0.0f);
         }
     } else {
         __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(g.out) + idx;
@@ -146,18 +204,43 @@ __device__ __forceinline__ void lin_store(const GemmParams& p, uint32_t row, uin
                 }
                 *reinterpret_cast<uint4*>(out + i) = make_uint4(w[0], w[1], w[2], w[3]);
             }
-        } else if (full && ((uintptr_t)out & 7u) == 0) {
+        } else if (N % 4 == 0 && full && ((uintptr_t)out & 7u) == 0) {
 #pragma unroll
-            for (int i = 0; i < N; i += 4) {
+            for (int i = 0; i + 3 < N; i += 4) {
                 const __nv_bfloat162 lo = __floats2bfloat162_rn(v[i], v[i + 1]), hi = __floats2bfloat162_rn(v[i + 2], v[i + 3]);
                 *reinterpret_cast<uint2*>(out + i) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
             }
         } else {
 #pragma unroll
             for (int i = 0; i < N; ++i)
-                if (c + i < width) out[i] = __float2bfloat16_rn(v[i]);
+                if ((uint32_t)i < left) out[i] = __float2bfloat16_rn(v[i]);
         }
     }
+}
+// Finish and store N consecutive cells of one row (N a multiple of 4, the cells in one segment).
+template <int N>
+__device__ __forceinline__ void lin_store(const GemmParams& p, uint32_t row, uint32_t col, const float (&acc)[N]) {
+    const GemmLin& g = p.lin[lin_segment(p, col)];
+    const uint32_t c = col - g.col_begin, width = g.width;
+    if (c >= width) return;
+    uint64_t orow;
+    if (!lin_out_row(g, row, &orow)) return;
+    const float alpha = p.alpha;
+    const uint32_t act = g.act;
+    if (act == HOLO_LINEAR_ACT_SILU_GATE) {
+        float v[N / 2];
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i) v[i] = alpha * (sigmoid_times<true>(acc[2 * i], acc[2 * i]) * acc[2 * i + 1]);
+        lin_put<N / 2>(g, orow * g.ld + (c >> 1), (width - c) >> 1, v);
+        return;
+    }
+    float v[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = lin_act<true>(acc[i], act);
+    if (g.rot_head) lin_rotate<N>(p, g, row, c, v);
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] *= alpha;
+    lin_put<N>(g, orow * g.ld + c, width - c, v);
 }
 // 32 accumulator columns of one row straight from TMEM registers.
 __device__ __forceinline__ void lin_store32(const GemmParams& p, uint32_t row, uint32_t col0, const uint32_t (&v)[32]) {
@@ -313,10 +396,10 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + S::BARS + 16 * STAGES + 12);
 
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t n0 = blockIdx.x * BN, m0 = blockIdx.y * BM, split = blockIdx.z;
+    const uint32_t n0 = blockIdx.x * BN, m0 = blockIdx.y * (LIN && p.tiles ? p.tile_rows : (uint32_t)BM), split = blockIdx.z;
     const uint32_t kb_begin = (uint32_t)(((uint64_t)p.kblocks * split) / p.splits);
     const uint32_t kb_end = (uint32_t)(((uint64_t)p.kblocks * (split + 1)) / p.splits);
-    const uint32_t nkb = kb_end - kb_begin;
+    uint32_t nkb = kb_end - kb_begin;
 
     holo_pdl_trigger();
     if (threadIdx.x == 0) {
@@ -353,6 +436,12 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
         }
     }
     holo_pdl_wait();  // barriers and TMEM were set up while the previous kernel drained
+    uint32_t m_end = p.m, a_row = m0, b_row = 0;
+    if (LIN) {
+        const LinTile t = lin_tile(p, blockIdx.y, m0);
+        m_end = t.m_end; a_row = t.a_row; b_row = t.b_row;
+        if (!t.used) nkb = 0;    // the whole cluster of this tile idles through
+    }
     const uint32_t ar_epoch = (AR && p.ar_world > 1) ? *reinterpret_cast<volatile uint32_t*>(p.ar_state) + 1 : 0;
     const uint64_t ar_units = ((uint64_t)p.m * p.n) >> 2;
 
@@ -370,11 +459,11 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 const uint32_t st = base + s * S::STAGE;
                 const int k0 = (int)((kb_begin + i) * BK);
                 if (i >= pre) mbar_arrive_expect_tx(bar_full + 8 * s, tx);
-                tma_load_2d(st, &map_a, k0 + a_k0, (int)m0, bar_full + 8 * s);
+                tma_load_2d(st, &map_a, k0 + a_k0, (int)a_row, bar_full + 8 * s);
                 if (i >= pre) {
 #pragma unroll
                     for (int h = 0; h < BN / 64; ++h)
-                        tma_load_2d(st + S::A_BYTES + h * (BK * 128), &map_b, (int)(n0 + 64 * h), k0, bar_full + 8 * s);
+                        tma_load_2d(st + S::A_BYTES + h * (BK * 128), &map_b, (int)(n0 + 64 * h), k0 + (int)b_row, bar_full + 8 * s);
                 }
             }
             if (*s_abort)
@@ -405,7 +494,7 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 }
                 umma_commit(bar_empty + 8 * s);  // frees the ring slot once these MMAs have read it
             }
-            if (ok) umma_commit(bar_accum);      // accumulator complete
+            if (ok && nkb != 0) umma_commit(bar_accum);      // accumulator complete
         }
     } else {
         // ---------------- epilogue warps (TMEM lane quarter = warp % 4) ----------------
@@ -423,7 +512,7 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 uint32_t v[32];
                 tmem_ld32(tmem_base + ((quarter * 32u) << 16) + (uint32_t)(c * 32), v);
                 const uint32_t col0 = n0 + c * 32;
-                if (row < p.m && col0 < p.n) lin_store32(p, row, col0, v);
+                if (row < m_end && col0 < p.n) lin_store32(p, row, col0, v);
             }
         } else if (!LIN && ok && p.splits == 1 && p.gated) {
             if constexpr (BN == 128) {
@@ -518,12 +607,12 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
             // split-K: park this CTA's f32 accumulator rows in the (now idle) ring; 16-byte units of a
             // row are XOR-swizzled with the row number so that the 32 rows of a warp do not hit one bank
             const uint32_t row_local = quarter * 32 + lane;
-            if (m0 + quarter * 32 < p.m) {  // warp-uniform: the TMEM load is a whole-warp instruction
+            if (m0 + quarter * 32 < m_end) {  // warp-uniform: the TMEM load is a whole-warp instruction
 #pragma unroll 1
                 for (int c = 0; c < BN / 32; ++c) {
                     uint32_t v[32];
                     tmem_ld32(tmem_base + ((quarter * 32u) << 16) + (uint32_t)(c * 32), v);
-                    if (row < p.m) {
+                    if (row < m_end) {
 #pragma unroll
                         for (int x = 0; x < 8; ++x) {
                             const uint32_t unit = (uint32_t)(c * 8 + x) ^ (row_local & 7u);
@@ -542,7 +631,7 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
         asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
         if (warp >= 2 && !*s_abort) {
             const uint32_t rank = split, S_ = p.splits, ew = warp - 2;
-            const uint32_t rows_valid = min(p.m - m0, (uint32_t)BM);
+            const uint32_t rows_valid = min(m_end - m0, (uint32_t)BM);
             uint32_t remote[8];
 #pragma unroll
             for (uint32_t sidx = 0; sidx < 8; ++sidx) {
@@ -772,7 +861,8 @@ matmul_umma_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const _
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + S::RING + 16 * PSTAGES + 36);
 
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t tiles_n = (p.n + PBN - 1) / PBN, tiles_m = (p.m + BM - 1) / BM, ntiles = tiles_n * tiles_m;
+    const uint32_t tiles_n = (p.n + PBN - 1) / PBN;
+    uint32_t tiles_m = (p.m + BM - 1) / BM;
 
     holo_pdl_trigger();
     if (threadIdx.x == 0) {
@@ -796,6 +886,8 @@ matmul_umma_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const _
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem_base = *s_tmem;
     holo_pdl_wait();
+    if (LIN && p.tiles) tiles_m = min(tiles_m, (uint32_t)p.tiles[0]);   // grouped: only the row tiles in use
+    const uint32_t ntiles = tiles_n * tiles_m;
 
     if (warp == 0) {
         // ---------------- TMA producer ----------------
@@ -806,15 +898,20 @@ matmul_umma_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const _
             for (uint32_t tile = blockIdx.x; tile < ntiles && ok; tile += gridDim.x) {
                 const int m0 = (int)((tile / tiles_n) * BM), n0 = (int)((tile % tiles_n) * PBN);
                 const int a_k0 = LIN ? (int)p.lin[lin_segment(p, (uint32_t)n0)].k_offset : 0;
+                int a_row = m0, b_row = 0;
+                if (LIN) {
+                    const LinTile t = lin_tile(p, tile / tiles_n, (uint32_t)m0);
+                    a_row = (int)t.a_row; b_row = (int)t.b_row;
+                }
                 for (uint32_t kb = 0; kb < p.kblocks; ++kb, ++it) {
                     const uint32_t s = it % PSTAGES, use = it / PSTAGES;
                     if (use > 0 && !mbar_wait(bar_empty + 8 * s, (use - 1) & 1, s_abort, p.status)) { ok = false; break; }
                     const uint32_t st = base + s * S::STAGE;
                     const int k0 = (int)(kb * BK);
                     mbar_arrive_expect_tx(bar_full + 8 * s, tx);
-                    tma_load_2d(st, &map_a, k0 + a_k0, m0, bar_full + 8 * s);
+                    tma_load_2d(st, &map_a, k0 + a_k0, a_row, bar_full + 8 * s);
 #pragma unroll
-                    for (int h = 0; h < PBN / 64; ++h) tma_load_2d(st + S::A_BYTES + h * (BK * 128), &map_b, n0 + 64 * h, k0, bar_full + 8 * s);
+                    for (int h = 0; h < PBN / 64; ++h) tma_load_2d(st + S::A_BYTES + h * (BK * 128), &map_b, n0 + 64 * h, k0 + b_row, bar_full + 8 * s);
                 }
             }
         }
@@ -1027,6 +1124,7 @@ matmul_umma_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 // this CTA's halves: rows [128 r, +128) of the A block, columns [bn/2 r, +bn/2) of the B block
                 const int m0 = (int)(item.m_tile * 256 + rank * 128), n0 = (int)(item.n0 + rank * (item.bn >> 1));
                 const int a_k0 = LIN ? (int)p.lin[lin_segment(p, item.n0)].k_offset : 0;
+                const int a_row = LIN && p.a_pos ? (int)lin_a_row(p, (uint32_t)m0) : m0;
                 const uint32_t tx = 2u * (S::A_BYTES + (item.bn >> 1) * BK * 2);
                 for (uint32_t kb = 0; kb < p.kblocks; ++kb, ++it) {
                     const uint32_t s = it % QSTAGES, use = it / QSTAGES;
@@ -1035,7 +1133,7 @@ matmul_umma_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                     const int k0 = (int)(kb * BK);
                     if (rank == 0) mbar_arrive_expect_tx(bar_full + 8 * s, tx);
                     const uint32_t leader_bar = map_to_cta(bar_full + 8 * s, 0);
-                    tma_load_2d_pair(st, &map_a, k0 + a_k0, m0, leader_bar);
+                    tma_load_2d_pair(st, &map_a, k0 + a_k0, a_row, leader_bar);
                     tma_load_2d_pair(st + S::A_BYTES, &map_b, n0, k0, leader_bar);
                     if (item.bn == 256) tma_load_2d_pair(st + S::A_BYTES + BK * 128, &map_b, n0 + 64, k0, leader_bar);
                 }

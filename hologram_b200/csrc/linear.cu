@@ -11,32 +11,62 @@ namespace {
 
 constexpr int CELL_ROWS = 4, CELL_THREADS = 128;
 
-// One thread: one column, up to CELL_ROWS rows (B is read once for them).
+// One thread: one column, up to CELL_ROWS rows (B is read once for them). Column pairs (rotation, gate) lie in neighbouring lanes.
 template <typename T>
 __global__ void __launch_bounds__(CELL_THREADS)
 linear_cell_kernel(const T* __restrict__ a, const T* __restrict__ b, const GemmParams p, uint32_t lda) {
     holo_pdl_trigger();
     holo_pdl_wait();
     const uint32_t col = blockIdx.x * CELL_THREADS + threadIdx.x, row0 = blockIdx.y * CELL_ROWS;
-    if (col >= p.n) return;
     const GemmLin& g = p.lin[lin_segment(p, col)];
     const uint32_t c = col - g.col_begin;
-    if (c >= g.width) return;
-    float acc[CELL_ROWS] = {};
-    const uint32_t rows = min((uint32_t)CELL_ROWS, p.m - row0);
-    for (uint32_t kk = 0; kk < p.k; ++kk) {
-        const float bv = (float)b[(uint64_t)kk * p.n + col];
-#pragma unroll
-        for (int r = 0; r < CELL_ROWS; ++r)
-            if ((uint32_t)r < rows) acc[r] = __fmaf_rn((float)a[(uint64_t)(row0 + r) * lda + g.k_offset + kk], bv, acc[r]);
+    const bool valid = col < p.n && c < g.width;
+    uint32_t rows = min((uint32_t)CELL_ROWS, p.m - row0);
+    const T* arow[CELL_ROWS];
+    if (p.tiles) {
+        const uint32_t tile = row0 / p.tile_rows, in_tile = row0 % p.tile_rows;
+        if (tile >= (uint32_t)p.tiles[0]) return;
+        b += (uint64_t)p.tiles[1 + tile] * p.k * p.n;
+        if (p.a_shared) {
+            if (in_tile >= p.a_shared) return;
+            rows = min(rows, p.a_shared - in_tile);
+        }
     }
-    const uint64_t base = g.row_pos ? *g.row_pos : 0u;
 #pragma unroll
     for (int r = 0; r < CELL_ROWS; ++r) {
-        const uint64_t orow = base + row0 + r;
-        if ((uint32_t)r >= rows || orow >= g.row_limit) continue;
-        const uint64_t idx = orow * g.ld + c;
-        const float v = p.alpha * lin_act(acc[r], g.act);
+        uint32_t ar = row0 + min((uint32_t)r, rows - 1);
+        if (p.tiles && p.a_shared) ar %= p.tile_rows;
+        else if (p.a_pos) ar = lin_a_row(p, ar);
+        arow[r] = a + (uint64_t)ar * lda + g.k_offset;
+    }
+    float acc[CELL_ROWS] = {};
+    if (valid)
+        for (uint32_t kk = 0; kk < p.k; ++kk) {
+            const float bv = (float)b[(uint64_t)kk * p.n + col];
+#pragma unroll
+            for (int r = 0; r < CELL_ROWS; ++r) acc[r] = __fmaf_rn((float)arow[r][kk], bv, acc[r]);
+        }
+#pragma unroll
+    for (int r = 0; r < CELL_ROWS; ++r) {
+        const float v0 = lin_act<false>(acc[r], g.act == HOLO_LINEAR_ACT_SILU_GATE ? HOLO_LINEAR_ACT_NONE : g.act);
+        const float v1 = __shfl_xor_sync(0xffffffffu, v0, 1);
+        uint64_t orow;
+        if (!valid || (uint32_t)r >= rows || !lin_out_row(g, row0 + r, &orow)) continue;
+        float v = v0;
+        uint32_t oc = c;
+        if (g.act == HOLO_LINEAR_ACT_SILU_GATE) {
+            if (c & 1u) continue;
+            v = sigmoid_times<false>(v0, v0) * v1;
+            oc = c >> 1;
+        } else if (g.rot_head) {
+            const uint32_t cc = c % g.rot_head;
+            if (cc >= g.rot_begin && cc < g.rot_begin + g.rot_dims) {
+                const float2 t = p.rot[(uint64_t)(row0 + r) * (g.rot_dims >> 1) + ((cc - g.rot_begin) >> 1)];
+                v = (c & 1u) ? v0 * t.x + v1 * t.y : v0 * t.x - v1 * t.y;
+            }
+        }
+        v *= p.alpha;
+        const uint64_t idx = orow * g.ld + oc;
         if (g.f32) reinterpret_cast<float*>(g.out)[idx] = v + (g.residual ? g.residual[idx] : 0.0f);
         else reinterpret_cast<__nv_bfloat16*>(g.out)[idx] = __float2bfloat16_rn(v);
     }
@@ -138,6 +168,9 @@ int32_t holo_launch_linear(holo_b200_ctx* ctx, const HoloLinearArgs& a) {
     p.alpha = a.alpha;
     p.status = ctx->dev_status;
     p.dtype = a.dtype;
+    p.rot = (const float2*)a.rot;
+    p.a_pos = a.a_pos; p.a_back = a.a_back; p.a_rows = a.a_rows;
+    p.tiles = a.tiles; p.tile_rows = a.tile_rows; p.a_shared = a.a_shared;
     bool k_offsets_ok = true;   // a TMA load starts on a 16-byte boundary
     for (uint32_t i = 0; i < a.nseg; ++i) {
         const HoloLinearSegArgs& s = a.seg[i];
@@ -149,6 +182,8 @@ int32_t holo_launch_linear(holo_b200_ctx* ctx, const HoloLinearArgs& a) {
         g.col_begin = s.col_begin; g.width = s.width; g.k_offset = s.k_offset; g.ld = s.ld;
         g.act = s.act;
         g.f32 = s.dtype == HOLO_DTYPE_F32;
+        g.ring = s.ring;
+        g.rot_head = s.rot_head; g.rot_begin = s.rot_begin; g.rot_dims = s.rot_dims;
         k_offsets_ok = k_offsets_ok && s.k_offset % 8 == 0;
     }
     const bool tma_ok = a.dtype == HOLO_DTYPE_BF16 && a.lda % 8 == 0 && a.n % 8 == 0 && k_offsets_ok && (((uintptr_t)a.a | (uintptr_t)a.b) & 15u) == 0 &&
@@ -167,34 +202,211 @@ int32_t holo_launch_linear(holo_b200_ctx* ctx, const HoloLinearArgs& a) {
     const uint32_t kblocks = (a.k + BK - 1) / BK, mtiles = (a.m + BM - 1) / BM;
     p.kblocks = kblocks;
     p.splits = 1;
-    p.b_constant = a.b_constant && !getenv("HOLO_GEMM_NO_EARLY_B") ? 1u : 0u;
+    p.b_constant = a.b_constant && !a.tiles && !getenv("HOLO_GEMM_NO_EARLY_B") ? 1u : 0u;
     CUtensorMap ma, mb;
-    HOLO_TRY(make_map_2d(&mb, a.b, a.n, a.k, 64, BK));
+    HOLO_TRY(make_map_2d(&mb, a.b, a.n, (uint64_t)a.k * (a.tiles ? a.experts : 1), 64, BK));
+    // rows A has: the matrix's own, a ring's, or the ones all tiles of a group share
+    const uint64_t a_rows = a.a_pos ? a.a_rows : a.a_shared ? a.a_shared : a.m;
     bool persistent, paired;
     persistent_choice(ctx, a.m, a.n, &persistent, &paired);
+    if (a.tiles) {
+        persistent = persistent && a.tile_rows == (uint32_t)BM && !a.a_shared;
+        paired = false;      // neighbouring row tiles may belong to different experts
+    }
     if (persistent) {
         p.box_m = BM;
-        HOLO_TRY(make_map_2d(&ma, a.a, a.lda, a.m, BK, BM));
+        HOLO_TRY(make_map_2d(&ma, a.a, a.lda, a_rows, BK, BM));
         return paired ? launch_pair<false, true>(ctx, ma, mb, p) : launch_persistent<false, true>(ctx, ma, mb, p);
     }
     int bn;
     uint32_t splits;
-    tile_choice(ctx, a.m, a.n, kblocks, &bn, &splits);
+    const uint32_t gtiles = a.tiles ? a.m / a.tile_rows : 0;
+    // a group is weight streaming like one product as wide as all its tiles together
+    if (a.tiles) tile_choice(ctx, a.tile_rows, a.n * gtiles, kblocks, &bn, &splits);
+    else tile_choice(ctx, a.m, a.n, kblocks, &bn, &splits);
     if (const char* e = getenv("HOLO_GEMM_BN")) bn = atoi(e) == 64 ? 64 : 128;
     if (const char* e = getenv("HOLO_GEMM_SPLITS")) splits = (uint32_t)atoi(e) > 0 ? (uint32_t)atoi(e) : 1;
     if (splits > kblocks) splits = kblocks;
     if (splits > 8) splits = 8;
-    if (mtiles > 65535) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: matmul grid too large");
+    if ((a.tiles ? gtiles : mtiles) > 65535) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: matmul grid too large");
     p.splits = splits;
-    p.box_m = a.m < (uint32_t)BM ? a.m : (uint32_t)BM;
-    HOLO_TRY(make_map_2d(&ma, a.a, a.lda, a.m, BK, p.box_m));
-    const dim3 grid((a.n + bn - 1) / bn, mtiles, splits);
+    const uint32_t rows = a.tiles ? (a.a_shared ? a.a_shared : a.tile_rows) : a.m;     // of one row tile, or all
+    p.box_m = rows < (uint32_t)BM ? rows : (uint32_t)BM;
+    HOLO_TRY(make_map_2d(&ma, a.a, a.lda, a_rows, BK, p.box_m));
+    const dim3 grid((a.n + bn - 1) / bn, a.tiles ? gtiles : mtiles, splits);
     if (bn == 128) {
-        if (a.m <= 16) return launch_lin<128, 5, 16>(ctx, ma, mb, p, grid);
-        if (a.m <= 64) return launch_lin<128, 4, 64>(ctx, ma, mb, p, grid);
+        if (rows <= 16) return launch_lin<128, 5, 16>(ctx, ma, mb, p, grid);
+        if (rows <= 64) return launch_lin<128, 4, 64>(ctx, ma, mb, p, grid);
         return launch_lin<128, 3, 128>(ctx, ma, mb, p, grid);
     }
-    if (a.m <= 16) return launch_lin<64, 9, 16>(ctx, ma, mb, p, grid);
-    if (a.m <= 64) return launch_lin<64, 6, 64>(ctx, ma, mb, p, grid);
+    if (rows <= 16) return launch_lin<64, 9, 16>(ctx, ma, mb, p, grid);
+    if (rows <= 64) return launch_lin<64, 6, 64>(ctx, ma, mb, p, grid);
     return launch_lin<64, 4, 128>(ctx, ma, mb, p, grid);
+}
+
+// ---- further row operations of decoder steps ----------------------------------------------------------------------
+namespace {
+
+// (cos, sin) of (*pos + row) * f_j. The frequency comes as a rounded value and its remainder, the product is split the same
+// way, and the remainder of the angle enters to first order: the error stays that of one f32 rounding at any position.
+__global__ void rotary_table_kernel(const uint32_t* __restrict__ pos, const float* __restrict__ freq, float2* __restrict__ out, uint32_t rows, uint32_t half) {
+    holo_pdl_trigger();
+    holo_pdl_wait();
+    const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= rows * half) return;
+    const uint32_t row = i / half, j = i % half, at = *pos + row;
+    const uint32_t low = at & 0xffffu;                       // positions past 2^24 are split as well
+    float s = 0.0f, c = 1.0f;
+#pragma unroll
+    for (int part = 0; part < 2; ++part) {
+        const float x = part ? (float)(at - low) : (float)low;
+        if (x == 0.0f) continue;
+        const float a = x * freq[j], e = fmaf(x, freq[j], -a) + x * freq[half + j];
+        float sa, ca;
+        sincosf(a, &sa, &ca);
+        const float s1 = fmaf(ca, e, sa), c1 = fmaf(-sa, e, ca);
+        const float sn = s * c1 + c * s1;
+        c = c * c1 - s * s1;
+        s = sn;
+    }
+    out[i] = make_float2(c, s);
+}
+
+// One warp per (row, part).
+constexpr int PARTS_WARPS = 4, PARTS_HELD = 16;
+template <typename T>
+__global__ void __launch_bounds__(PARTS_WARPS * 32)
+rms_norm_parts_kernel(const HoloNormPartsArgs a) {
+    holo_pdl_trigger();
+    const uint32_t unit = blockIdx.x * PARTS_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit >= a.rows * a.nparts) return;
+    const uint32_t row = unit / a.nparts;
+    const HoloNormPartArgs& p = a.part[unit % a.nparts];
+    holo_pdl_wait();
+    uint64_t orow = row;
+    if (p.ring) {
+        if (row >= a.step[1]) return;
+        orow = (a.step[0] + row) % (uint32_t)p.row_limit;
+    }
+    const float* x = a.x + (uint64_t)row * a.ld_in + p.in_col;
+    T* out = (T*)p.out + orow * p.ld;
+    float held[PARTS_HELD], acc = 0.0f;
+#pragma unroll
+    for (int i = 0; i < PARTS_HELD; ++i) {
+        const uint32_t j = lane + 32 * i;
+        held[i] = j < p.width ? x[j] : 0.0f;
+    }
+    float inv = 1.0f;
+    if (p.norm) {
+#pragma unroll
+        for (int i = 0; i < PARTS_HELD; ++i) acc = fmaf(held[i], held[i], acc);
+        for (uint32_t j = lane + 32 * PARTS_HELD; j < p.width; j += 32) acc = fmaf(x[j], x[j], acc);
+        for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        inv = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(acc, (float)p.width), a.eps)));
+    }
+#pragma unroll
+    for (int i = 0; i < PARTS_HELD; ++i) {
+        const uint32_t j = lane + 32 * i;
+        if (j < p.width) store_norm(out, j, held[i] * inv * (p.weight ? p.weight[j] : 1.0f));
+    }
+    for (uint32_t j = lane + 32 * PARTS_HELD; j < p.width; j += 32) store_norm(out, j, x[j] * inv * (p.weight ? p.weight[j] : 1.0f));
+    for (uint32_t j = p.width + lane; j < p.out_width; j += 32) store_norm(out, j, 0.0f);
+}
+
+// A CTA takes HEAD_COLS columns of one head for up to R rows; its threads split k and add up through shared memory.
+constexpr int HEAD_THREADS = 256;
+template <typename T> struct HeadVec;
+template <> struct HeadVec<float> { static constexpr int N = 4; };
+template <> struct HeadVec<__nv_bfloat16> { static constexpr int N = 8; };
+template <typename T>
+__device__ __forceinline__ void load_vec(const T* src, bool vec, uint32_t left, float (&v)[HeadVec<T>::N]) {
+    constexpr int N = HeadVec<T>::N;
+    if (vec) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(src);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = (float)e[i];
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = (uint32_t)i < left ? (float)src[i] : 0.0f;
+    }
+}
+template <typename T, int R>
+__global__ void __launch_bounds__(HEAD_THREADS)
+head_linear_kernel(const HoloHeadLinearArgs a, uint32_t vec) {
+    constexpr int N = HeadVec<T>::N, COLS = 4 * N, KG = HEAD_THREADS / 4;     // four column vectors, 64 slices of k
+    __shared__ float part[HEAD_THREADS / 32][R][COLS];
+    holo_pdl_trigger();
+    const uint32_t cv = threadIdx.x & 3u, kg = threadIdx.x >> 2, h = blockIdx.y, r0 = blockIdx.z * R;
+    const uint32_t col = blockIdx.x * COLS + cv * N;
+    const T* b = (const T*)a.b + (uint64_t)h * a.b_step + col;
+    const T* x = (const T*)a.a + (uint64_t)r0 * a.lda + (uint64_t)h * a.a_step;
+    const uint32_t rows = min((uint32_t)R, a.rows - r0), left = col < a.n ? a.n - col : 0u;
+    float acc[R][N] = {};
+    holo_pdl_wait();
+    if (left) {
+        const bool whole = vec && left >= (uint32_t)N;
+#pragma unroll 4
+        for (uint32_t k = kg; k < a.k; k += KG) {
+            float v[N];
+            load_vec<T>(b + (uint64_t)k * a.b_ld, whole, left, v);
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                const float xv = (uint32_t)r < rows ? (float)x[(uint64_t)r * a.lda + k] : 0.0f;
+#pragma unroll
+                for (int i = 0; i < N; ++i) acc[r][i] = fmaf(xv, v[i], acc[r][i]);
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            for (int o = 4; o < 32; o <<= 1) acc[r][i] += __shfl_xor_sync(0xffffffffu, acc[r][i], o);
+            if ((threadIdx.x & 31u) < 4) part[threadIdx.x >> 5][r][cv * N + i] = acc[r][i];
+        }
+    __syncthreads();
+    for (uint32_t i = threadIdx.x; i < rows * COLS; i += HEAD_THREADS) {
+        const uint32_t r = i / COLS, c = i % COLS, oc = blockIdx.x * COLS + c;
+        if (oc >= a.n) continue;
+        float v = 0.0f;
+#pragma unroll
+        for (int w = 0; w < HEAD_THREADS / 32; ++w) v += part[w][r][c];
+        store_norm((T*)a.out, (uint64_t)(r0 + r) * a.ld + (uint64_t)h * a.out_step + oc, v);
+    }
+}
+
+template <typename T>
+int32_t launch_head(holo_b200_ctx* ctx, const HoloHeadLinearArgs& a) {
+    constexpr int N = HeadVec<T>::N;
+    const uint32_t vec = a.b_ld % N == 0 && a.b_step % N == 0 && ((uintptr_t)a.b & 15u) == 0 ? 1u : 0u;
+    const uint32_t cols = (a.n + 4 * N - 1) / (4 * N);
+    const uint32_t per = a.rows == 1 ? 1 : 4, blocks = (a.rows + per - 1) / per;
+    if (blocks > 65535 || a.heads > 65535) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: head_linear rows %u", a.rows);
+    if (per == 1) HOLO_CUDA(holo_launch_kernel(ctx, head_linear_kernel<T, 1>, dim3(cols, a.heads, blocks), dim3(HEAD_THREADS), 0, 1, a, vec));
+    else HOLO_CUDA(holo_launch_kernel(ctx, head_linear_kernel<T, 4>, dim3(cols, a.heads, blocks), dim3(HEAD_THREADS), 0, 1, a, vec));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
+}  // namespace
+
+int32_t holo_launch_rotary_table(holo_b200_ctx* ctx, const uint32_t* pos, const float* freq, float* out, uint32_t rows, uint32_t half) {
+    const uint64_t n = (uint64_t)rows * half;
+    if (n > 0x7fffffffull) return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: rotary table of %u rows", rows);
+    HOLO_CUDA(holo_launch_kernel(ctx, rotary_table_kernel, dim3((uint32_t)((n + 127) / 128)), dim3(128), 0, 1, pos, freq, (float2*)out, rows, half));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
+int32_t holo_launch_rms_norm_parts(holo_b200_ctx* ctx, const HoloNormPartsArgs& a) {
+    const uint32_t grid = (a.rows * a.nparts + PARTS_WARPS - 1) / PARTS_WARPS;
+    if (a.dtype == HOLO_DTYPE_F32) HOLO_CUDA(holo_launch_kernel(ctx, rms_norm_parts_kernel<float>, dim3(grid), dim3(PARTS_WARPS * 32), 0, 1, a));
+    else HOLO_CUDA(holo_launch_kernel(ctx, rms_norm_parts_kernel<__nv_bfloat16>, dim3(grid), dim3(PARTS_WARPS * 32), 0, 1, a));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
+int32_t holo_launch_head_linear(holo_b200_ctx* ctx, const HoloHeadLinearArgs& a) {
+    return a.dtype == HOLO_DTYPE_F32 ? launch_head<float>(ctx, a) : launch_head<__nv_bfloat16>(ctx, a);
 }

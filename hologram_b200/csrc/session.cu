@@ -772,13 +772,18 @@ int32_t holo_session_load_impl(holo_b200_ctx* ctx, const uint8_t* archive, uint6
     for (const HoloPort& p : s->ar.outputs) out_slots.insert(p.slot);
     if (s->addressed) {
         // the labels of an addressed walk do not see rows written into a resident cache
-        for (const HoloKernelCall& c : s->calls)
+        for (const HoloKernelCall& c : s->calls) {
+            if (c.kind >= HOLO_K_LINEAR_EX && c.kind <= HOLO_K_MOE_COMBINE) {
+                delete s;
+                return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: an addressed session has no resident state (call %u)", c.kind);
+            }
             if (c.kind == HOLO_K_LINEAR)
                 for (uint32_t i = 0; i < c.u.linear.nseg; ++i)
                     if (c.u.linear.seg[i].row_pos.slot != HOLO_NO_SLOT) {
                         delete s;
                         return holo_fail(HOLO_ERR_UNSUPPORTED_OP, "unsupported op: an addressed session cannot append to a cache in place");
                     }
+        }
     }
     // weights the donor holds: slot -> its device copy
     std::unordered_map<uint32_t, std::pair<void*, uint64_t>> borrowed;

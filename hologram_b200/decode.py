@@ -2,9 +2,10 @@
 
 A model's archives are fixed step shapes; `StepRunner` keeps one session per row count in use (powers of two, the
 portion is padded up) and one per logit count. All of them share the first session's device copies of the weights
-and its cache, residual stream and position buffers, and replay as CUDA graphs after their first walk. Padding rows lie
-after the portion's last token: no real row sees them, they are dropped past the end of the cache, and a later step
-overwrites what they left there before any row can see it.
+and its cache, state, residual stream and position buffers, and replay as CUDA graphs after their first walk. Padding rows
+lie after the portion's last token: no real row sees them. What they leave in a plain cache is dropped past its end or
+overwritten by a later step before any row can see it; ring caches and recurrent states take the real rows only, by the
+row count every step carries, and a state starts from zero where the step's position is 0.
 """
 from collections import deque
 
@@ -26,7 +27,7 @@ def bucket(n):
 
 
 class SequenceCache:
-    """The positions one sequence at a time holds in the sessions' shared K/V buffers."""
+    """The positions one sequence at a time holds in the sessions' shared cache and state buffers."""
 
     def __init__(self, capacity):
         self.capacity = capacity
@@ -90,7 +91,7 @@ class StepRunner:
         rows = bucket(len(tokens))
         entry = self._session(self._steps, rows, lambda: m.build_step(rows, self.cache.capacity, self.max_rows, False, weightless=True))
         step_in = np.zeros(4 + rows, dtype=np.int32)
-        step_in[0] = base
+        step_in[0], step_in[1] = base, len(tokens)
         step_in[4:4 + len(tokens)] = tokens
         entry[0].write("step_in", step_in)
         session = self._execute(entry)

@@ -15,21 +15,11 @@ One archive is one step shape: `rows` new tokens of one sequence against a cache
 Head widths are padded with zero columns to multiples of 16 and the model width to a multiple of 8, so that every row
 pitch suits TMA whatever the configuration's sizes are; zero columns change no result.
 """
-import json
-import os
-
 import numpy as np
 
 from . import holo
 from . import kernel_call as kc
-from . import safetensors_io
-
-BF, F32, I32 = kc.DTYPE_BF16, kc.DTYPE_F32, kc.DTYPE_I32
-STEP_IN_IDS = 4            # the token ids follow four words of which the first is the position of the step's first row
-
-
-def _up(n, multiple):
-    return (n + multiple - 1) // multiple * multiple
+from .step_model import BF, F32, I32, STEP_IN_IDS, StepModel, up as _up
 
 
 class AttentionSpec:
@@ -122,48 +112,10 @@ class FokonexConfig:
         return out
 
 
-class _Slots:
-    """Slot numbers and sizes of one archive under construction."""
-
-    def __init__(self):
-        self.nbytes = []
-
-    def new(self, nbytes):
-        self.nbytes.append(int(nbytes))
-        return len(self.nbytes) - 1
-
-    def ref(self, slot, offset=0, length=None):
-        return kc.rb(slot, offset, self.nbytes[slot] - offset if length is None else length)
-
-
-class FokonexModel:
+class FokonexModel(StepModel):
     """Configuration and device-layout weights of one model; builds its step archives."""
 
-    def __init__(self, config, tensors, dtype=BF):
-        self.config, self.dtype = config, dtype
-        self.elem = 2 if dtype == BF else 4
-        missing = [n for n, s in config.tensor_shapes().items() if n not in tensors or tuple(tensors[n].shape) != tuple(s)]
-        if missing:
-            raise ValueError(f"checkpoint: missing or misshaped tensors: {', '.join(missing[:5])}")
-        self._constants = {}       # name -> (array, fingerprint)
-        self._pack(tensors)
-
-    @classmethod
-    def load(cls, path, dtype=BF):
-        with open(os.path.join(path, "config.json"), encoding="utf-8") as f:
-            config = FokonexConfig.from_dict(json.load(f))
-        return cls(config, safetensors_io.read(os.path.join(path, "model.safetensors")), dtype)
-
-    # ---- weights in the layout the kernels read: [in, out], columns of several products side by side ----
-    def _value(self, tensor):
-        return tensor.as_bf16() if self.dtype == BF else tensor.as_f32()
-
-    def _zeros(self, shape):
-        return np.zeros(shape, dtype=np.uint16 if self.dtype == BF else np.float32)
-
-    def _add(self, name, array):
-        array = np.ascontiguousarray(array)
-        self._constants[name] = (array, holo.fingerprint(array.view(np.uint8).reshape(-1).data))
+    CONFIG = FokonexConfig
 
     @staticmethod
     def _gain(tensor):
@@ -212,44 +164,7 @@ class FokonexModel:
             self._add(p + "in", b)
             self._add(p + "out", o)
             self._add(p + "sink", t[p + "mix.sink"].as_f32())
-        self._add("final.norm", self._gain(t["final.norm"]))
-        head = self._zeros((wp, _up(c.vocab, 8)))
-        head[:w, :c.vocab] = self._value(t["head"]).T
-        self._add("head", head)
-
-    # ---- archives ----
-    def _begin(self):
-        return holo.HoloWriter(), _Slots(), {}
-
-    def _const(self, w, sl, made, name):
-        if name not in made:
-            array, fp = self._constants[name]
-            made[name] = sl.new(array.nbytes)
-            w.add_constant(made[name], F32 if array.dtype == np.float32 else BF, array.view(np.uint8).reshape(-1).data, known_fingerprint=fp)
-        return sl.ref(made[name])
-
-    def _hidden(self, w, sl, hidden_rows):
-        n = hidden_rows * self.config.width
-        s = sl.new(4 * n)
-        w.inputs.append(holo.Port("hidden", s, n, F32, [hidden_rows, self.config.width]))
-        return s
-
-    def _logits(self, w, sl, made, x, rows):
-        """final norm and output head over `rows` rows of x; returns the slot of the f32 logits."""
-        c, es = self.config, self.elem
-        h, logits = sl.new(rows * c.width_p * es), sl.new(4 * rows * c.vocab)
-        w.calls.append(kc.KernelCall.RmsNormMulti(kc.RmsNormMultiCall(
-            x, self._const(w, sl, made, "final.norm"), kc.NONE, sl.ref(h), rows, c.width, c.width_p, kc.f32_bits(c.eps), self.dtype)))
-        seg = kc.LinearSeg(sl.ref(logits), kc.NONE, 0, c.vocab, 0, c.vocab, kc.LINEAR_ACT_NONE, F32)
-        w.calls.append(kc.KernelCall.Linear(kc.LinearCall.make(
-            sl.ref(h), self._const(w, sl, made, "head"), [seg], rows, c.width_p, _up(c.vocab, 8), self.dtype, alpha=c.logit_scale)))
-        w.outputs.append(holo.Port("logits", logits, rows * c.vocab, F32, [rows, c.vocab]))
-
-    def build_step(self, rows, capacity, hidden_rows, with_logits, weightless=False):
-        return self.step_writer(rows, capacity, hidden_rows, with_logits).finish(weightless=weightless)
-
-    def build_head(self, rows, hidden_rows, weightless=False):
-        return self.head_writer(rows, hidden_rows).finish(weightless=weightless)
+        self._pack_head(t, self._gain(t["final.norm"]), c.logit_scale)
 
     def step_writer(self, rows, capacity, hidden_rows, with_logits):
         """The archive of one step of `rows` tokens: ports `step_in` (i32: position, three unused words, the token ids),
@@ -262,15 +177,7 @@ class FokonexModel:
         pos, ids = sl.ref(step_in, 0, 4), sl.ref(step_in, 4 * STEP_IN_IDS)
         x = self._hidden(w, sl, hidden_rows)
         xr = sl.ref(x, 0, 4 * rows * c.width)
-        # embedding rows, widened to f32
-        if dt == F32:
-            emb = xr
-        else:
-            e = sl.new(rows * c.width * 2)
-            emb = sl.ref(e)
-        w.calls.append(kc.KernelCall.Gather(kc.GatherCall(self._const(w, sl, made, "embed"), ids, emb, 1, c.vocab, c.width, rows, I32, dt)))
-        if dt != F32:
-            w.calls.append(kc.KernelCall.Cast(kc.CastCall(emb, xr, rows * c.width, BF, F32)))
+        self._embed(w, sl, made, ids, xr, rows)
         # activations: one set per distinct layer geometry, reused by every layer that has it
         work = {}
         for l in c.layers:
@@ -289,38 +196,22 @@ class FokonexModel:
                 xr, self._const(w, sl, made, p + "norm1"), kc.NONE if l.ff is None else self._const(w, sl, made, p + "norm2"), sl.ref(h),
                 rows, c.width, c.width_p, kc.f32_bits(c.eps), dt)))
             (cq, ck, cv, cu), cols = self.in_columns(l)
-            segs = [kc.LinearSeg(sl.ref(q), kc.NONE, cq, a.heads * a.dim_p, 0, a.heads * a.dim_p, 0, dt),
-                    kc.LinearSeg(sl.ref(kcache), pos, ck, lk, 0, lk, 0, dt), kc.LinearSeg(sl.ref(vcache), pos, cv, lv, 0, lv, 0, dt)]
+            segs = [kc.LinearSeg.make(sl.ref(q), a.heads * a.dim_p, a.heads * a.dim_p, dt, cq),
+                    kc.LinearSeg.make(sl.ref(kcache), lk, lk, dt, ck, row_pos=pos), kc.LinearSeg.make(sl.ref(vcache), lv, lv, dt, cv, row_pos=pos)]
             if l.ff is not None:
-                segs.append(kc.LinearSeg(sl.ref(act, a.heads * a.vdim_p * es), kc.NONE, cu, l.ff, c.width_p, ka, kc.LINEAR_ACT_RELU2, dt))
+                segs.append(kc.LinearSeg.make(sl.ref(act, a.heads * a.vdim_p * es), l.ff, ka, dt, cu, c.width_p, kc.LINEAR_ACT_RELU2))
             w.calls.append(kc.KernelCall.Linear(kc.LinearCall.make(
                 sl.ref(h), self._const(w, sl, made, p + "in"), segs, rows, c.width_p, cols, dt, lda=nh * c.width_p)))
             w.calls.append(kc.KernelCall.CausalAttention(kc.CausalAttentionCall(
                 sl.ref(q), sl.ref(kcache), sl.ref(vcache), pos, self._const(w, sl, made, p + "sink"), sl.ref(act), rows, a.heads, a.kv_heads,
                 a.dim_p, a.vdim_p, capacity, ka, kc.f32_bits(a.scale), kc.f32_bits(a.softcap), kc.f32_bits(a.temp_coef),
                 kc.f32_bits(a.temp_every), dt)))
-            seg = kc.LinearSeg(xr, kc.NONE, 0, c.width, 0, c.width, 0, F32)
+            seg = kc.LinearSeg.make(xr, c.width, c.width, F32)
             w.calls.append(kc.KernelCall.Linear(kc.LinearCall.make(
                 sl.ref(act), self._const(w, sl, made, p + "out"), [seg], rows, ka, c.width_p, dt, residual=xr, alpha=c.residual_mult)))
         if with_logits:
             self._logits(w, sl, made, xr, rows)
-        w.exec_plan = [[i] for i in range(len(w.calls))]
-        w.slot_bytes = list(sl.nbytes)
-        return w
-
-    def head_writer(self, rows, hidden_rows):
-        """The archive that turns `rows` chosen rows of the residual stream (port `want`, i32) into logits."""
-        c = self.config
-        w, sl, made = self._begin()
-        x = self._hidden(w, sl, hidden_rows)
-        want = sl.new(4 * rows)
-        w.inputs.append(holo.Port("want", want, rows, I32, [rows]))
-        picked = sl.new(4 * rows * c.width)
-        w.calls.append(kc.KernelCall.Gather(kc.GatherCall(sl.ref(x), sl.ref(want), sl.ref(picked), 1, hidden_rows, c.width, rows, I32, F32)))
-        self._logits(w, sl, made, sl.ref(picked), rows)
-        w.exec_plan = [[i] for i in range(len(w.calls))]
-        w.slot_bytes = list(sl.nbytes)
-        return w
+        return self._end(w, sl)
 
     def launches(self, rows, with_logits):
         """Kernel launches of one step, by the archive's call count."""

@@ -3,6 +3,7 @@ Rust toolchain). Byte layout follows crates/hologram-archive: framing writer.rs:
 calls kernel_codec.rs:130-137 + put_* :569-873, ports writer.rs:246-263, constants
 constant_codec.rs:66-95, weights writer.rs:388-440, exec plan writer.rs:325-336.
 """
+import ctypes
 import struct
 
 import blake3
@@ -27,6 +28,19 @@ def _binary(c):
 
 def _matmul(c):
     return _buf(c.a) + _buf(c.b) + _buf(c.output) + struct.pack("<IIIBB", c.m, c.k, c.n, c.dtype, c.b_packed)
+
+
+# calls whose payload is written field by field as the struct lists them
+_FLAT = {kc.K_ROTARY_TABLE: "rotary_table", kc.K_HEAD_LINEAR: "head_linear", kc.K_WINDOW_ATTENTION: "window_attention", kc.K_RETENTION: "retention",
+         kc.K_MOE_PLAN: "moe_plan", kc.K_MOE_COMBINE: "moe_combine"}
+
+
+def _flat(c):
+    out = b""
+    for name, kind in c._fields_:
+        v = getattr(c, name)
+        out += _buf(v) if kind is kc.BufferRef else struct.pack("<B" if kind is ctypes.c_uint8 else "<I", v)
+    return out
 
 
 def encode_call(call):
@@ -130,12 +144,24 @@ def encode_call(call):
         c = u.rms_norm_multi
         return out + b"".join(_buf(b) for b in (c.x, c.gamma0, c.gamma1, c.output)) + struct.pack(
             "<IIIIB", c.rows, c.feature, c.step, c.epsilon_bits, c.dtype)
-    if k == kc.K_LINEAR:
+    if k in (kc.K_LINEAR, kc.K_LINEAR_EX):
         c = u.linear
         segs = b"".join(_buf(g.output) + _buf(g.row_pos) + struct.pack("<IIIIBB", g.col_begin, g.width, g.k_offset, g.ld, g.act, g.dtype)
                         for g in list(c.seg)[:c.nseg])
-        return out + b"".join(_buf(b) for b in (c.a, c.b, c.residual)) + struct.pack(
+        base = out + b"".join(_buf(b) for b in (c.a, c.b, c.residual)) + struct.pack(
             "<IIIIIBB", c.m, c.k, c.n, c.lda, c.alpha_bits, c.dtype, c.nseg) + segs
+        if k == kc.K_LINEAR:
+            return base
+        rows = b"".join(struct.pack("<IIIB", g.rot_head, g.rot_begin, g.rot_dims, g.ring) for g in list(c.seg)[:c.nseg])
+        return base + rows + b"".join(_buf(b) for b in (c.rot, c.a_pos, c.tiles)) + struct.pack(
+            "<IIIII", c.a_back, c.a_rows, c.tile_rows, c.experts, c.a_shared)
+    if k == kc.K_RMS_NORM_PARTS:
+        c = u.rms_norm_parts
+        parts = b"".join(_buf(p.weight) + _buf(p.output) + struct.pack("<IIIIBB", p.in_col, p.width, p.out_width, p.ld, p.norm, p.ring)
+                         for p in list(c.part)[:c.nparts])
+        return out + _buf(c.x) + _buf(c.step) + struct.pack("<IIIBB", c.rows, c.ld_in, c.epsilon_bits, c.dtype, c.nparts) + parts
+    if k in _FLAT:
+        return out + _flat(getattr(u, _FLAT[k]))
     if k == kc.K_CAUSAL_ATTENTION:
         c = u.causal_attention
         return out + b"".join(_buf(b) for b in (c.q, c.k, c.v, c.pos, c.sink, c.output)) + struct.pack(

@@ -41,6 +41,8 @@ K_GATHER, K_CAST, K_KV_CACHE_WRITE, K_DECODE_ATTENTION_VALID = 114, 115, 120, 12
 K_QUANTIZE_ROWS_I8, K_DECODE_ATTENTION_VALID_Q8, K_ALL_REDUCE = 0x8001, 0x8002, 0x8003
 K_ROPE_QUANTIZE_ROWS_I8 = 0x8004
 K_RMS_NORM_MULTI, K_LINEAR, K_CAUSAL_ATTENTION = 0x8005, 0x8006, 0x8007
+K_LINEAR_EX, K_ROTARY_TABLE, K_RMS_NORM_PARTS, K_HEAD_LINEAR = 0x8008, 0x8009, 0x800a, 0x800b
+K_WINDOW_ATTENTION, K_RETENTION, K_MOE_PLAN, K_MOE_COMBINE = 0x800c, 0x800d, 0x800e, 0x800f
 LUT_KIND = {LUT_SIGMOID: K_SIGMOID, LUT_TANH: K_TANH, LUT_GELU: K_GELU, LUT_SILU: K_SILU, LUT_EXP: K_EXP, LUT_ERF: K_ERF}
 
 NO_SLOT = 0xFFFFFFFF
@@ -276,29 +278,46 @@ class RmsNormMultiCall(C.Structure):
 
 
 LINEAR_MAX_SEGS = 4
-LINEAR_ACT_NONE, LINEAR_ACT_RELU2 = 0, 1
+LINEAR_ACT_NONE, LINEAR_ACT_RELU2, LINEAR_ACT_GELU_TANH, LINEAR_ACT_SILU, LINEAR_ACT_SILU_GATE = range(5)
 
 
 class LinearSeg(C.Structure):
     _fields_ = [("output", BufferRef), ("row_pos", BufferRef), ("col_begin", C.c_uint32), ("width", C.c_uint32),
-                ("k_offset", C.c_uint32), ("ld", C.c_uint32), ("act", C.c_uint8), ("dtype", C.c_uint8)]
+                ("k_offset", C.c_uint32), ("ld", C.c_uint32), ("act", C.c_uint8), ("dtype", C.c_uint8), ("ring", C.c_uint8),
+                ("rot_head", C.c_uint32), ("rot_begin", C.c_uint32), ("rot_dims", C.c_uint32)]
+
+    @classmethod
+    def make(cls, output, width, ld, dtype, col_begin=0, k_offset=0, act=LINEAR_ACT_NONE, row_pos=None, ring=False, rotate=None):
+        """`rotate` = (columns per head, first rotated column, rotated columns)."""
+        head, begin, dims = rotate or (0, 0, 0)
+        return cls(output, NONE if row_pos is None else row_pos, col_begin, width, k_offset, ld, act, dtype, int(ring), head, begin, dims)
 
 
 class LinearCall(C.Structure):
-    """Extension: out_s[i, j] = residual + alpha * act_s(A[i, k_offset:k_offset + k] . B[:, col_begin + j]) for up to four segments."""
-    _fields_ = [("a", BufferRef), ("b", BufferRef), ("residual", BufferRef), ("seg", LinearSeg * LINEAR_MAX_SEGS), ("m", C.c_uint32),
-                ("k", C.c_uint32), ("n", C.c_uint32), ("lda", C.c_uint32), ("nseg", C.c_uint32), ("alpha_bits", C.c_uint32),
-                ("dtype", C.c_uint8)]
+    """Extension: out_s[i, j] = residual + alpha * act_s(A[i, k_offset:k_offset + k] . B[:, col_begin + j]) for up to four segments;
+    the extended fields add rotation, ring rows, a row window of A and groups."""
+    _fields_ = [("a", BufferRef), ("b", BufferRef), ("residual", BufferRef), ("rot", BufferRef), ("a_pos", BufferRef), ("tiles", BufferRef),
+                ("seg", LinearSeg * LINEAR_MAX_SEGS), ("m", C.c_uint32), ("k", C.c_uint32), ("n", C.c_uint32), ("lda", C.c_uint32),
+                ("nseg", C.c_uint32), ("alpha_bits", C.c_uint32), ("a_back", C.c_uint32), ("a_rows", C.c_uint32), ("tile_rows", C.c_uint32),
+                ("experts", C.c_uint32), ("a_shared", C.c_uint32), ("dtype", C.c_uint8)]
 
     @classmethod
-    def make(cls, a, b, segs, m, k, n, dtype, lda=None, residual=None, alpha=1.0):
+    def make(cls, a, b, segs, m, k, n, dtype, lda=None, residual=None, alpha=1.0, rot=None, a_pos=None, a_back=0, a_rows=0, tiles=None,
+             tile_rows=0, experts=0, a_shared=0):
         c = cls()
         c.a, c.b, c.residual = a, b, NONE if residual is None else residual
+        c.rot, c.a_pos, c.tiles = (NONE if r is None else r for r in (rot, a_pos, tiles))
         c.m, c.k, c.n, c.lda, c.nseg, c.dtype = m, k, n, k if lda is None else lda, len(segs), dtype
+        c.a_back, c.a_rows, c.tile_rows, c.experts, c.a_shared = a_back, a_rows, tile_rows, experts, a_shared
         c.alpha_bits = f32_bits(alpha)
         for i, g in enumerate(segs):
             c.seg[i] = g
         return c
+
+    @property
+    def extended(self):
+        refs = (self.rot, self.a_pos, self.tiles)
+        return any(r.slot != NO_SLOT for r in refs) or any(g.ring or g.rot_head for g in list(self.seg)[:self.nseg])
 
 
 class CausalAttentionCall(C.Structure):
@@ -307,6 +326,67 @@ class CausalAttentionCall(C.Structure):
                 ("rows", C.c_uint32), ("heads", C.c_uint32), ("kv_heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32),
                 ("cache_rows", C.c_uint32), ("ld", C.c_uint32), ("scale_bits", C.c_uint32), ("softcap_bits", C.c_uint32),
                 ("temp_coef_bits", C.c_uint32), ("temp_every_bits", C.c_uint32), ("dtype", C.c_uint8)]
+
+
+class RotaryTableCall(C.Structure):
+    """Extension: (cos, sin) of every row's angles."""
+    _fields_ = [("pos", BufferRef), ("freq", BufferRef), ("output", BufferRef), ("rows", C.c_uint32), ("half", C.c_uint32)]
+
+
+NORM_MAX_PARTS = 3
+
+
+class NormPart(C.Structure):
+    _fields_ = [("weight", BufferRef), ("output", BufferRef), ("in_col", C.c_uint32), ("width", C.c_uint32), ("out_width", C.c_uint32),
+                ("ld", C.c_uint32), ("norm", C.c_uint8), ("ring", C.c_uint8)]
+
+
+class RmsNormPartsCall(C.Structure):
+    """Extension: column ranges of f32 rows, each normalised (or copied) into a buffer of its own."""
+    _fields_ = [("x", BufferRef), ("step", BufferRef), ("part", NormPart * NORM_MAX_PARTS), ("rows", C.c_uint32), ("ld_in", C.c_uint32),
+                ("nparts", C.c_uint32), ("epsilon_bits", C.c_uint32), ("dtype", C.c_uint8)]
+
+    @classmethod
+    def make(cls, x, parts, rows, ld_in, eps, dtype, step=None):
+        c = cls()
+        c.x, c.step, c.rows, c.ld_in, c.nparts, c.epsilon_bits, c.dtype = x, NONE if step is None else step, rows, ld_in, len(parts), f32_bits(eps), dtype
+        for i, p in enumerate(parts):
+            c.part[i] = p
+        return c
+
+
+class HeadLinearCall(C.Structure):
+    """Extension: every head's columns times a matrix of its own."""
+    _fields_ = [("a", BufferRef), ("b", BufferRef), ("output", BufferRef)] + [(n, C.c_uint32) for n in (
+        "rows", "heads", "k", "n", "lda", "a_step", "b_ld", "b_step", "ld", "out_step")] + [("dtype", C.c_uint8)]
+
+
+WHOLE_CACHE = 0xFFFFFFFF     # kv_back of keys whose row 0 is position 0
+
+
+class WindowAttentionCall(C.Structure):
+    """Extension: sliding-window attention with a sink and an optional key part all heads share."""
+    _fields_ = [(n, BufferRef) for n in ("q", "k", "v", "q2", "k2", "pos", "sink", "output")] + [(n, C.c_uint32) for n in (
+        "rows", "heads", "kv_heads", "dim", "vdim", "dim2", "q_ld", "q_step", "k_ld", "v_ld", "q2_ld", "q2_step", "k2_ld", "ld",
+        "kv_rows", "kv_back", "k2_rows", "window", "scale_bits")] + [("dtype", C.c_uint8)]
+
+
+class RetentionCall(C.Structure):
+    """Extension: linear attention with one decay per head, an f32 state, and a normed, gated output."""
+    _fields_ = [(n, BufferRef) for n in ("q", "k", "v", "gate", "decay", "step", "state", "output")] + [(n, C.c_uint32) for n in (
+        "rows", "heads", "dim", "vdim", "vmean", "q_ld", "k_ld", "v_ld", "gate_ld", "ld", "scale_bits", "epsilon_bits")] + [("dtype", C.c_uint8)]
+
+
+class MoePlanCall(C.Structure):
+    """Extension: router logits -> chosen experts, weights and the row tiles of the grouped products."""
+    _fields_ = [(n, BufferRef) for n in ("logits", "bias", "step", "weight", "place", "tiles", "source")] + [(n, C.c_uint32) for n in (
+        "rows", "experts", "top", "ld_logits", "tile_rows", "max_tiles")]
+
+
+class MoeCombineCall(C.Structure):
+    """Extension: x += the weighted sum of the chosen experts' outputs."""
+    _fields_ = [(n, BufferRef) for n in ("x", "y", "weight", "place", "step")] + [(n, C.c_uint32) for n in (
+        "rows", "width", "top", "ld", "y_rows")] + [("dtype", C.c_uint8)]
 
 
 class _Payload(C.Union):
@@ -318,7 +398,9 @@ class _Payload(C.Union):
                 ("decode_attention_valid", DecodeAttentionValidCall), ("quantize_rows_i8", QuantizeRowsI8Call),
                 ("decode_attention_valid_q8", DecodeAttentionValidQ8Call), ("all_reduce", AllReduceCall),
                 ("rope_quantize", RopeQuantizeCall), ("rms_norm_multi", RmsNormMultiCall), ("linear", LinearCall),
-                ("causal_attention", CausalAttentionCall)]
+                ("causal_attention", CausalAttentionCall), ("rotary_table", RotaryTableCall), ("rms_norm_parts", RmsNormPartsCall),
+                ("head_linear", HeadLinearCall), ("window_attention", WindowAttentionCall), ("retention", RetentionCall),
+                ("moe_plan", MoePlanCall), ("moe_combine", MoeCombineCall)]
 
 
 class KernelCall(C.Structure):
@@ -433,9 +515,23 @@ class KernelCall(C.Structure):
     @classmethod
     def RmsNormMulti(cls, c): return cls.of(K_RMS_NORM_MULTI, c)
     @classmethod
-    def Linear(cls, c): return cls.of(K_LINEAR, c)
+    def Linear(cls, c): return cls.of(K_LINEAR_EX if c.extended else K_LINEAR, c)    # the wire form follows the call
     @classmethod
     def CausalAttention(cls, c): return cls.of(K_CAUSAL_ATTENTION, c)
+    @classmethod
+    def RotaryTable(cls, c): return cls.of(K_ROTARY_TABLE, c)
+    @classmethod
+    def RmsNormParts(cls, c): return cls.of(K_RMS_NORM_PARTS, c)
+    @classmethod
+    def HeadLinear(cls, c): return cls.of(K_HEAD_LINEAR, c)
+    @classmethod
+    def WindowAttention(cls, c): return cls.of(K_WINDOW_ATTENTION, c)
+    @classmethod
+    def Retention(cls, c): return cls.of(K_RETENTION, c)
+    @classmethod
+    def MoePlan(cls, c): return cls.of(K_MOE_PLAN, c)
+    @classmethod
+    def MoeCombine(cls, c): return cls.of(K_MOE_COMBINE, c)
 
 
 KernelCall._FIELD = {
@@ -445,6 +541,8 @@ KernelCall._FIELD = {
     DecodeAttentionCall: "decode_attention", DecodeAttentionValidCall: "decode_attention_valid", QuantizeRowsI8Call: "quantize_rows_i8",
     DecodeAttentionValidQ8Call: "decode_attention_valid_q8", AllReduceCall: "all_reduce", RopeQuantizeCall: "rope_quantize",
     RmsNormMultiCall: "rms_norm_multi", LinearCall: "linear", CausalAttentionCall: "causal_attention",
+    RotaryTableCall: "rotary_table", RmsNormPartsCall: "rms_norm_parts", HeadLinearCall: "head_linear", WindowAttentionCall: "window_attention",
+    RetentionCall: "retention", MoePlanCall: "moe_plan", MoeCombineCall: "moe_combine",
 }
 
 

@@ -4,8 +4,9 @@ import os
 
 from . import kernel_call as kc
 from .fokonex import FokonexModel
+from .zisevik import ZisevikModel
 
-ARCHITECTURES = {"Fokonex": FokonexModel}
+ARCHITECTURES = {m.CONFIG.ARCHITECTURE: m for m in (FokonexModel, ZisevikModel)}
 DTYPES = {"bfloat16": kc.DTYPE_BF16, "float32": kc.DTYPE_F32}
 
 

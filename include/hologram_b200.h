@@ -144,6 +144,22 @@ extern "C" {
 #define HOLO_K_RMS_NORM_MULTI 0x8005
 #define HOLO_K_LINEAR 0x8006
 #define HOLO_K_CAUSAL_ATTENTION 0x8007
+/* Steps with rotary positions, ring caches, recurrent state and routed experts:
+ * LINEAR_EX is the wire form of a LINEAR whose extended fields are in use (rotation, ring rows, a row window of A, groups);
+ * ROTARY_TABLE holds the step's cosines and sines, which LINEAR_EX applies as it stores;
+ * RMS_NORM_PARTS normalises (or copies) column ranges of an f32 row into separate buffers;
+ * HEAD_LINEAR multiplies every head's columns by a matrix of its own;
+ * WINDOW_ATTENTION has a sliding window, an optional key part all heads share, and pitches of its own for every operand;
+ * RETENTION is linear attention with one fixed decay per head and an f32 state;
+ * MOE_PLAN turns router logits into chosen experts, weights and row tiles; MOE_COMBINE adds the weighted expert outputs. */
+#define HOLO_K_LINEAR_EX 0x8008
+#define HOLO_K_ROTARY_TABLE 0x8009
+#define HOLO_K_RMS_NORM_PARTS 0x800a
+#define HOLO_K_HEAD_LINEAR 0x800b
+#define HOLO_K_WINDOW_ATTENTION 0x800c
+#define HOLO_K_RETENTION 0x800d
+#define HOLO_K_MOE_PLAN 0x800e
+#define HOLO_K_MOE_COMBINE 0x800f
 
 /* BufferRef (crates/hologram-compute/src/workspace.rs:16-24). length == 0 means "the slot's
  * full extent from offset". slot == UINT32_MAX marks an absent optional operand
@@ -421,15 +437,31 @@ typedef struct HoloRmsNormMultiCall {
 #define HOLO_LINEAR_MAX_SEGS 4
 #define HOLO_LINEAR_ACT_NONE 0
 #define HOLO_LINEAR_ACT_RELU2 1 /* max(v, 0)^2 */
+#define HOLO_LINEAR_ACT_GELU_TANH 2 /* v / (1 + exp(-2 sqrt(2/pi) (v + 0.044715 v^3))), the tanh form of gelu */
+#define HOLO_LINEAR_ACT_SILU 3 /* v / (1 + exp(-v)) */
+#define HOLO_LINEAR_ACT_SILU_GATE 4 /* columns in pairs: silu(v[2j]) * v[2j + 1] is output column j (width counts columns of B) */
+/* Extended fields (all zero / absent = the plain form):
+ *  rot_head > 0: the segment's columns are heads of rot_head columns; in each, the pairs (v[2j], v[2j + 1]) of the rot_dims
+ *    columns from rot_begin on become (v0 cos - v1 sin, v1 cos + v0 sin) with row i's j-th angle from `rot` (f32
+ *    [m, rot_dims / 2, (cos, sin)]). After the activation, before alpha.
+ *  ring: row_pos names two words, (first, count): row i < count of the step goes to buffer row (first + i) mod the rows the
+ *    buffer has; rows from count on are not stored.
+ *  a_pos: A is a ring of a_rows rows as well; row i of the product reads its row (start + i) mod a_rows,
+ *    start = max(0, *a_pos - a_back) rounded down to a multiple of 128 (a_rows is one, or never wraps).
+ *  tiles: the product is grouped. B is [experts, k, n]; `tiles` (i32: the number of tiles in use, then each one's expert)
+ *    says which matrix rows [t * tile_rows, (t + 1) * tile_rows) meet; m = most tiles * tile_rows; rows of unused tiles are
+ *    not stored. a_shared: every tile reads the same first rows of A (a_shared of them, at most tile_rows). */
 typedef struct HoloLinearSeg {
     HoloBufferRef output, row_pos;
     uint32_t col_begin, width, k_offset, ld;
-    uint8_t act, dtype;
+    uint8_t act, dtype, ring;
+    uint32_t rot_head, rot_begin, rot_dims;
 } HoloLinearSeg;
 typedef struct HoloLinearCall {
-    HoloBufferRef a, b, residual;
+    HoloBufferRef a, b, residual, rot, a_pos, tiles;
     HoloLinearSeg seg[HOLO_LINEAR_MAX_SEGS];
     uint32_t m, k, n, lda, nseg, alpha_bits;
+    uint32_t a_back, a_rows, tile_rows, experts, a_shared;
     uint8_t dtype;
 } HoloLinearCall;
 
@@ -447,6 +479,83 @@ typedef struct HoloCausalAttentionCall {
     uint32_t scale_bits, softcap_bits, temp_coef_bits, temp_every_bits;
     uint8_t dtype;
 } HoloCausalAttentionCall;
+
+/* Extension. Angles of a step's rows: output f32 [rows, half, 2] = (cos, sin) of (*pos + i) * f_j. freq holds f_j as two f32
+ * arrays, [half] rounded values and [half] remainders, so that the angle is good to f32 at any position. */
+typedef struct HoloRotaryTableCall {
+    HoloBufferRef pos, freq, output;
+    uint32_t rows, half;
+} HoloRotaryTableCall;
+
+/* Extension. Column ranges of f32 rows (pitch ld_in): part p takes columns [in_col, in_col + width) and stores
+ *   x / sqrt(mean(x^2) + eps) * weight     (norm = 1; weight f32 [width], absent = all ones)   or x itself (norm = 0)
+ * as `dtype` into columns [0, width) of its output (pitch ld), zeros up to out_width. ring: as in LINEAR_EX, with `step` as
+ * the two words (first, count). */
+#define HOLO_NORM_MAX_PARTS 3
+typedef struct HoloNormPart {
+    HoloBufferRef weight, output;
+    uint32_t in_col, width, out_width, ld;
+    uint8_t norm, ring;
+} HoloNormPart;
+typedef struct HoloRmsNormPartsCall {
+    HoloBufferRef x, step;
+    HoloNormPart part[HOLO_NORM_MAX_PARTS];
+    uint32_t rows, ld_in, nparts, epsilon_bits;
+    uint8_t dtype;
+} HoloRmsNormPartsCall;
+
+/* Extension. For every head h: output[i, h * out_step + j] = sum_k a[i, h * a_step + k] * b_h[k, j], b_h starting b_step
+ * elements after b_(h-1) with row pitch b_ld; f32 accumulation, `dtype` operands and result (rounded to nearest). */
+typedef struct HoloHeadLinearCall {
+    HoloBufferRef a, b, output;
+    uint32_t rows, heads, k, n, lda, a_step, b_ld, b_step, ld, out_step;
+    uint8_t dtype;
+} HoloHeadLinearCall;
+
+/* Extension. Attention of `rows` new positions of one sequence with a sliding window. Row i is at p = *pos + i and sees
+ * 0 <= p - j < window (window 0: every j <= p). Head h reads q at columns h * q_step of pitch q_ld, k and v at columns
+ * g * dim and g * vdim (g = h / (heads / kv_heads)) of pitches k_ld and v_ld, and, when dim2 > 0, q2 at columns
+ * h * q2_step and one k2 for all heads. Scores and weights are f32:
+ *   s = (q . k + q2 . k2) * scale;  out = sum_j exp(s_j) v_j / (sum_j exp(s_j) + exp(sink_h))
+ * k and v have kv_rows rows; position j is row (j - start) mod kv_rows, start = 0 when kv_back is 0xFFFFFFFF, else
+ * max(0, *pos - kv_back) rounded down to a multiple of 128. k2 has k2_rows rows, position j is row j mod k2_rows.
+ * Positions a row sees are distinct rows of every buffer (the caller's buffers are long enough). */
+typedef struct HoloWindowAttentionCall {
+    HoloBufferRef q, k, v, q2, k2, pos, sink, output;
+    uint32_t rows, heads, kv_heads, dim, vdim, dim2;
+    uint32_t q_ld, q_step, k_ld, v_ld, q2_ld, q2_step, k2_ld, ld;
+    uint32_t kv_rows, kv_back, k2_rows, window, scale_bits;
+    uint8_t dtype;
+} HoloWindowAttentionCall;
+
+/* Extension. step = (first, count); rows i < count advance the f32 state [heads, dim, vdim] of one sequence, which is zero
+ * where first is 0:   S = decay_h S + k_i v_i^T,   o_i = scale * S^T q_i
+ *   output[i, h * vdim + e] = o_i[e] / sqrt(mean_{e < vmean}(o_i^2) + eps) * gate[i, h * vdim + e]
+ * q, k [rows, heads * dim], v, gate [rows, heads * vdim] with pitches of their own; vmean <= vdim columns carry values (the
+ * rest are zero). Rows from count on are not stored. */
+typedef struct HoloRetentionCall {
+    HoloBufferRef q, k, v, gate, decay, step, state, output;
+    uint32_t rows, heads, dim, vdim, vmean, q_ld, k_ld, v_ld, gate_ld, ld, scale_bits, epsilon_bits;
+    uint8_t dtype;
+} HoloRetentionCall;
+
+/* Extension. logits f32 [rows, ld_logits] (+ bias f32 [experts]): for every row i < count (step = (first, count)) the `top`
+ * largest, weight[i, t] = softmax over those, and the row tiles of the grouped products that follow:
+ *   rows <= tile_rows: one tile per expert chosen by any row, row i of a tile is row i of the step;
+ *   else: the (row, choice) pairs sorted by expert, every expert's rows starting a tile.
+ * tiles i32 [1 + max_tiles] = count, experts; place i32 [rows, top] = the pair's row among all tiles' rows;
+ * source i32 [max_tiles * tile_rows] = the step row behind each (0 where there is none; unused in the first form). */
+typedef struct HoloMoePlanCall {
+    HoloBufferRef logits, bias, step, weight, place, tiles, source;
+    uint32_t rows, experts, top, ld_logits, tile_rows, max_tiles;
+} HoloMoePlanCall;
+
+/* Extension. x f32 [rows, width] += sum_t weight[i, t] * y[place[i, t], :] for rows i < count; y `dtype` with pitch ld. */
+typedef struct HoloMoeCombineCall {
+    HoloBufferRef x, y, weight, place, step;
+    uint32_t rows, width, top, ld, y_rows;
+    uint8_t dtype;
+} HoloMoeCombineCall;
 
 /* Extension. In-place sum over the context's tensor-parallel group (NCCL); a no-op when the
  * context has no group. */
@@ -489,8 +598,15 @@ typedef struct HoloKernelCall {
         HoloAllReduceCall all_reduce;
         HoloRopeQuantizeCall rope_quantize;
         HoloRmsNormMultiCall rms_norm_multi;
-        HoloLinearCall linear;
+        HoloLinearCall linear;          /* LINEAR, LINEAR_EX */
         HoloCausalAttentionCall causal_attention;
+        HoloRotaryTableCall rotary_table;
+        HoloRmsNormPartsCall rms_norm_parts;
+        HoloHeadLinearCall head_linear;
+        HoloWindowAttentionCall window_attention;
+        HoloRetentionCall retention;
+        HoloMoePlanCall moe_plan;
+        HoloMoeCombineCall moe_combine;
     } u;
 } HoloKernelCall;
 

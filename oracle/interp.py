@@ -48,6 +48,86 @@ def _narrow(a, dtype):
     return orc.f32_to_bf16_rne(np.ascontiguousarray(a).reshape(-1)) if dtype == kc.DTYPE_BF16 else np.asarray(a, dtype=np.float32)
 
 
+def _word(slots, ref, index=0):
+    return int(_get(slots, kc.rb(ref.slot, ref.offset + 4 * index), 4, kc.DTYPE_I32).view(np.uint32)[0])
+
+
+def _extent(slots, ref):
+    return ref.length or slots[ref.slot].size - ref.offset
+
+
+def _matrix(slots, ref, rows, cols, ld, dtype):
+    """f64 values of `rows` rows of `cols` columns at pitch `ld`."""
+    size = np.dtype(_NP[dtype]).itemsize
+    flat = _wide(_get(slots, ref, ((rows - 1) * ld + cols) * size, dtype), dtype)
+    return np.lib.stride_tricks.as_strided(flat, (rows, cols), (8 * ld, 8)).copy()
+
+
+def _put_matrix(slots, ref, values, ld, dtype):
+    size = np.dtype(_NP[dtype]).itemsize
+    for i, row in enumerate(values):
+        _put(slots, kc.rb(ref.slot, ref.offset + i * ld * size), _narrow(row.astype(np.float32), dtype))
+
+
+def _linear_act(v, act):
+    if act == kc.LINEAR_ACT_RELU2:
+        return np.maximum(v, 0.0) ** 2
+    if act == kc.LINEAR_ACT_GELU_TANH:
+        return 0.5 * v * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (v + 0.044715 * v ** 3)))
+    if act == kc.LINEAR_ACT_SILU:
+        return v / (1.0 + np.exp(-v))
+    if act == kc.LINEAR_ACT_SILU_GATE:
+        return v[:, 0::2] / (1.0 + np.exp(-v[:, 0::2])) * v[:, 1::2]
+    return v
+
+
+def _linear(slots, c, extended):
+    size = np.dtype(_NP[c.dtype]).itemsize
+    grouped, window = extended and c.tiles.slot != kc.NO_SLOT, extended and c.a_pos.slot != kc.NO_SLOT
+    if window:
+        start = max(0, _word(slots, c.a_pos) - c.a_back) // 128 * 128
+        a = _matrix(slots, c.a, c.a_rows, c.lda, c.lda, c.dtype)[(start + np.arange(c.m)) % c.a_rows]
+    elif grouped and c.a_shared:
+        a = np.zeros((c.m, c.lda))
+        shared = _matrix(slots, c.a, c.a_shared, c.lda, c.lda, c.dtype)
+        for t in range(c.m // c.tile_rows):
+            a[t * c.tile_rows:t * c.tile_rows + c.a_shared] = shared
+    else:
+        a = _matrix(slots, c.a, c.m, c.lda, c.lda, c.dtype)
+    b = _wide(_get(slots, c.b, c.k * c.n * size * (c.experts if grouped else 1), c.dtype), c.dtype).reshape(-1, c.k, c.n)
+    if grouped:
+        tiles = _get(slots, c.tiles, 4 * (1 + c.m // c.tile_rows), kc.DTYPE_I32)
+        tiles = tiles[1:1 + tiles[0]]
+    for g in list(c.seg)[:c.nseg]:
+        cols = slice(g.col_begin, g.col_begin + g.width)
+        if grouped:
+            part = [a[t * c.tile_rows:(t + 1) * c.tile_rows, g.k_offset:g.k_offset + c.k] @ b[e][:, cols] for t, e in enumerate(tiles)]
+            v = np.concatenate(part) if part else np.zeros((0, g.width))
+        else:
+            v = a[:, g.k_offset:g.k_offset + c.k] @ b[0][:, cols]
+        v = _linear_act(v, g.act)
+        if extended and g.rot_head:
+            table = _matrix(slots, c.rot, c.m, g.rot_dims, g.rot_dims, kc.DTYPE_F32).reshape(c.m, -1, 2)
+            for head in range(0, g.width, g.rot_head):
+                lo = head + g.rot_begin
+                e, o = v[:, lo:lo + g.rot_dims:2].copy(), v[:, lo + 1:lo + g.rot_dims:2].copy()
+                v[:, lo:lo + g.rot_dims:2] = e * table[..., 0] - o * table[..., 1]
+                v[:, lo + 1:lo + g.rot_dims:2] = o * table[..., 0] + e * table[..., 1]
+        v = _f32(c.alpha_bits) * v
+        out_size = np.dtype(_NP[g.dtype]).itemsize
+        appends, ring = g.row_pos.slot != kc.NO_SLOT, extended and g.ring
+        first = _word(slots, g.row_pos) if appends else 0
+        limit = _extent(slots, g.output) // (g.ld * out_size) if appends else c.m
+        if ring:
+            limit = (_extent(slots, g.output) - g.width * out_size) // (g.ld * out_size) + 1
+        count = min(len(v), _word(slots, g.row_pos, 1)) if ring else min(len(v), limit - first)
+        for i in range(count):
+            row, cells = ((first + i) % limit if ring else first + i), v[i]
+            if c.residual.slot != kc.NO_SLOT:
+                cells = cells + _get(slots, kc.rb(c.residual.slot, c.residual.offset + i * g.ld * 4), g.width * 4, kc.DTYPE_F32)
+            _put(slots, kc.rb(g.output.slot, g.output.offset + row * g.ld * out_size), _narrow(cells.astype(np.float32), g.dtype))
+
+
 def run(calls, slots, all_reduce=None):
     es = lambda dt: np.dtype(_NP[dt]).itemsize
     for call in calls:
@@ -183,25 +263,103 @@ def run(calls, slots, all_reduce=None):
             for i, g in enumerate(gammas):
                 out[:, i, :c.feature] = x * inv * _get(slots, g, c.feature * 4, kc.DTYPE_F32)
             _put(slots, c.output, _narrow(out, c.dtype))
-        elif k == kc.K_LINEAR:
-            c = u.linear
-            a = _wide(_get(slots, c.a, c.m * c.lda * es(c.dtype), c.dtype), c.dtype).reshape(c.m, c.lda)
-            b = _wide(_get(slots, c.b, c.k * c.n * es(c.dtype), c.dtype), c.dtype).reshape(c.k, c.n)
-            for g in list(c.seg)[:c.nseg]:
-                v = a[:, g.k_offset:g.k_offset + c.k] @ b[:, g.col_begin:g.col_begin + g.width]
-                if g.act == kc.LINEAR_ACT_RELU2:
-                    v = np.maximum(v, 0.0) ** 2
-                v = _f32(c.alpha_bits) * v
-                size = es(g.dtype)
-                first = int(_get(slots, g.row_pos, 4, kc.DTYPE_I32)[0]) if g.row_pos.slot != kc.NO_SLOT else 0
-                extent = g.output.length or slots[g.output.slot].size - g.output.offset
-                limit = extent // (g.ld * size) if g.row_pos.slot != kc.NO_SLOT else c.m
-                for i in range(min(c.m, limit - first)):
-                    at = kc.rb(g.output.slot, g.output.offset + (first + i) * g.ld * size)
-                    row = v[i]
-                    if c.residual.slot != kc.NO_SLOT:
-                        row = row + _get(slots, kc.rb(c.residual.slot, c.residual.offset + i * g.ld * 4), g.width * 4, kc.DTYPE_F32)
-                    _put(slots, at, _narrow(row.astype(np.float32), g.dtype))
+        elif k in (kc.K_LINEAR, kc.K_LINEAR_EX):
+            _linear(slots, u.linear, k == kc.K_LINEAR_EX)
+        elif k == kc.K_ROTARY_TABLE:
+            c = u.rotary_table
+            f = _get(slots, c.freq, 8 * c.half, kc.DTYPE_F32).astype(np.float64).reshape(2, c.half).sum(axis=0)
+            a = (_word(slots, c.pos) + np.arange(c.rows))[:, None] * f
+            _put(slots, c.output, np.stack([np.cos(a), np.sin(a)], axis=-1).astype(np.float32))
+        elif k == kc.K_RMS_NORM_PARTS:
+            c = u.rms_norm_parts
+            for p in list(c.part)[:c.nparts]:
+                x = _matrix(slots, kc.rb(c.x.slot, c.x.offset + 4 * p.in_col), c.rows, p.width, c.ld_in, kc.DTYPE_F32)
+                if p.norm:
+                    x = x / np.sqrt((x * x).mean(axis=1, keepdims=True) + _f32(c.epsilon_bits))
+                if p.weight.slot != kc.NO_SLOT:
+                    x = x * _get(slots, p.weight, 4 * p.width, kc.DTYPE_F32)
+                x = np.concatenate([x, np.zeros((c.rows, p.out_width - p.width))], axis=1)
+                size = es(c.dtype)
+                for i in range(min(c.rows, _word(slots, c.step, 1)) if p.ring else c.rows):
+                    row = (_word(slots, c.step) + i) % ((_extent(slots, p.output) - p.out_width * size) // (p.ld * size) + 1) if p.ring else i
+                    _put(slots, kc.rb(p.output.slot, p.output.offset + row * p.ld * size), _narrow(x[i].astype(np.float32), c.dtype))
+        elif k == kc.K_HEAD_LINEAR:
+            c = u.head_linear
+            size = es(c.dtype)
+            for h in range(c.heads):
+                a = _matrix(slots, kc.rb(c.a.slot, c.a.offset + h * c.a_step * size), c.rows, c.k, c.lda, c.dtype)
+                b = _matrix(slots, kc.rb(c.b.slot, c.b.offset + h * c.b_step * size), c.k, c.n, c.b_ld, c.dtype)
+                _put_matrix(slots, kc.rb(c.output.slot, c.output.offset + h * c.out_step * size), a @ b, c.ld, c.dtype)
+        elif k == kc.K_WINDOW_ATTENTION:
+            c = u.window_attention
+            size, first, scale = es(c.dtype), _word(slots, c.pos), _f32(c.scale_bits)
+            start = 0 if c.kv_back == kc.WHOLE_CACHE else max(0, first - c.kv_back) // 128 * 128
+            kk, vv = (_matrix(slots, r, c.kv_rows, c.kv_heads * d, ld, c.dtype) for r, d, ld in ((c.k, c.dim, c.k_ld), (c.v, c.vdim, c.v_ld)))
+            k2 = _matrix(slots, c.k2, c.k2_rows, c.dim2, c.k2_ld, c.dtype) if c.dim2 else None
+            for h in range(c.heads):
+                g = h // (c.heads // c.kv_heads)
+                q = _matrix(slots, kc.rb(c.q.slot, c.q.offset + h * c.q_step * size), c.rows, c.dim, c.q_ld, c.dtype)
+                q2 = _matrix(slots, kc.rb(c.q2.slot, c.q2.offset + h * c.q2_step * size), c.rows, c.dim2, c.q2_ld, c.dtype) if c.dim2 else None
+                sink = _get(slots, kc.rb(c.sink.slot, c.sink.offset + 4 * h), 4, kc.DTYPE_F32)[0] if c.sink.slot != kc.NO_SLOT else -np.inf
+                out = np.zeros((c.rows, c.vdim))
+                for i in range(c.rows):
+                    p = first + i
+                    j = np.arange(max(0, p + 1 - c.window) if c.window else 0, p + 1)
+                    rows = (j - start) % c.kv_rows
+                    s = kk[rows, g * c.dim:(g + 1) * c.dim] @ q[i]
+                    if c.dim2:
+                        s = s + k2[j % c.k2_rows] @ q2[i]
+                    s = s * scale
+                    top = max(s.max(), sink)
+                    e = np.exp(s - top)
+                    out[i] = e @ vv[rows, g * c.vdim:(g + 1) * c.vdim] / (e.sum() + np.exp(sink - top))
+                _put_matrix(slots, kc.rb(c.output.slot, c.output.offset + h * c.vdim * size), out, c.ld, c.dtype)
+        elif k == kc.K_RETENTION:
+            c = u.retention
+            q, kk = (_matrix(slots, r, c.rows, c.heads * c.dim, ld, c.dtype).reshape(c.rows, c.heads, c.dim) for r, ld in ((c.q, c.q_ld), (c.k, c.k_ld)))
+            v, gate = (_matrix(slots, r, c.rows, c.heads * c.vdim, ld, c.dtype).reshape(c.rows, c.heads, c.vdim) for r, ld in ((c.v, c.v_ld), (c.gate, c.gate_ld)))
+            decay = _get(slots, c.decay, 4 * c.heads, kc.DTYPE_F32).astype(np.float64)
+            state = _get(slots, c.state, 4 * c.heads * c.dim * c.vdim, kc.DTYPE_F32).astype(np.float64).reshape(c.heads, c.dim, c.vdim)
+            state = state * (_word(slots, c.step) != 0)
+            size = es(c.dtype)
+            for i in range(min(c.rows, _word(slots, c.step, 1))):
+                state = decay[:, None, None] * state + kk[i][:, :, None] * v[i][:, None, :]
+                o = _f32(c.scale_bits) * np.einsum("hde,hd->he", state, q[i])
+                o = o / np.sqrt((o[:, :c.vmean] ** 2).mean(axis=1, keepdims=True) + _f32(c.epsilon_bits)) * gate[i]
+                _put(slots, kc.rb(c.output.slot, c.output.offset + i * c.ld * size), _narrow(o.reshape(-1).astype(np.float32), c.dtype))
+            _put(slots, c.state, state.astype(np.float32))
+        elif k == kc.K_MOE_PLAN:
+            c = u.moe_plan
+            z = _matrix(slots, c.logits, c.rows, c.experts, c.ld_logits, kc.DTYPE_F32)
+            if c.bias.slot != kc.NO_SLOT:
+                z = z + _get(slots, c.bias, 4 * c.experts, kc.DTYPE_F32)
+            n = min(c.rows, _word(slots, c.step, 1))
+            chosen = np.argsort(-z[:n], axis=1, kind="stable")[:, :c.top]
+            e = np.take_along_axis(z[:n], chosen, axis=1)
+            e = np.exp(e - e[:, :1])
+            weight, place = np.zeros((c.rows, c.top), dtype=np.float32), np.zeros((c.rows, c.top), dtype=np.int32)
+            weight[:n] = e / e.sum(axis=1, keepdims=True)
+            tiles, source = [], np.zeros(c.max_tiles * c.tile_rows, dtype=np.int32)
+            for x in range(c.experts):
+                pairs = np.argwhere(chosen == x)
+                for at, (i, t) in enumerate(pairs):
+                    place[i, t] = len(tiles) * c.tile_rows + (i if c.rows <= c.tile_rows else at)
+                    source[place[i, t]] = i
+                tiles += [x] * (min(1, len(pairs)) if c.rows <= c.tile_rows else -(-len(pairs) // c.tile_rows))
+            assert len(tiles) <= c.max_tiles
+            _put(slots, c.weight, weight)
+            _put(slots, c.place, place)
+            _put(slots, c.source, source)
+            _put(slots, c.tiles, np.array([len(tiles)] + tiles, dtype=np.int32))
+        elif k == kc.K_MOE_COMBINE:
+            c = u.moe_combine
+            x = _matrix(slots, c.x, c.rows, c.width, c.width, kc.DTYPE_F32)
+            y = _matrix(slots, c.y, c.y_rows, c.width, c.ld, c.dtype)
+            weight = _get(slots, c.weight, 4 * c.rows * c.top, kc.DTYPE_F32).reshape(c.rows, c.top)
+            place = _get(slots, c.place, 4 * c.rows * c.top, kc.DTYPE_I32).reshape(c.rows, c.top)
+            for i in range(min(c.rows, _word(slots, c.step, 1))):
+                x[i] += weight[i].astype(np.float64) @ y[place[i]]
+            _put(slots, c.x, x.astype(np.float32))
         elif k == kc.K_CAUSAL_ATTENTION:
             c = u.causal_attention
             size = es(c.dtype)

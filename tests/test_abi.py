@@ -34,10 +34,12 @@ def test_struct_layout_matches_the_header():
     #include <stddef.h>
     #include "hologram_b200.h"
     int main(void) {
-        printf("%zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu\n", sizeof(HoloBufferRef), sizeof(HoloUnaryCall), sizeof(HoloMatMulCall),
+        printf("%zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu %zu\n", sizeof(HoloBufferRef), sizeof(HoloUnaryCall), sizeof(HoloMatMulCall),
                sizeof(HoloMatMulAddCall), sizeof(HoloNormCall), sizeof(HoloDecodeAttentionValidQ8Call),
                sizeof(HoloKernelCall), offsetof(HoloKernelCall, u), sizeof(HoloHostSlot),
-               sizeof(HoloRmsNormMultiCall), sizeof(HoloLinearSeg), sizeof(HoloLinearCall), sizeof(HoloCausalAttentionCall));
+               sizeof(HoloRmsNormMultiCall), sizeof(HoloLinearSeg), sizeof(HoloLinearCall), sizeof(HoloCausalAttentionCall),
+               offsetof(HoloLinearSeg, rot_head), sizeof(HoloRotaryTableCall), sizeof(HoloNormPart), sizeof(HoloRmsNormPartsCall), sizeof(HoloHeadLinearCall),
+               sizeof(HoloWindowAttentionCall), sizeof(HoloRetentionCall), sizeof(HoloMoePlanCall), sizeof(HoloMoeCombineCall));
         return 0;
     }'''
     with tempfile.TemporaryDirectory() as d:
@@ -49,7 +51,10 @@ def test_struct_layout_matches_the_header():
     want = [ctypes.sizeof(kc.BufferRef), ctypes.sizeof(kc.UnaryCall), ctypes.sizeof(kc.MatMulCall),
             ctypes.sizeof(kc.MatMulAddCall), ctypes.sizeof(kc.NormCall), ctypes.sizeof(kc.DecodeAttentionValidQ8Call),
             ctypes.sizeof(kc.KernelCall), kc.KernelCall.u.offset, ctypes.sizeof(kc.HostSlot),
-            ctypes.sizeof(kc.RmsNormMultiCall), ctypes.sizeof(kc.LinearSeg), ctypes.sizeof(kc.LinearCall), ctypes.sizeof(kc.CausalAttentionCall)]
+            ctypes.sizeof(kc.RmsNormMultiCall), ctypes.sizeof(kc.LinearSeg), ctypes.sizeof(kc.LinearCall), ctypes.sizeof(kc.CausalAttentionCall),
+            kc.LinearSeg.rot_head.offset, ctypes.sizeof(kc.RotaryTableCall), ctypes.sizeof(kc.NormPart), ctypes.sizeof(kc.RmsNormPartsCall),
+            ctypes.sizeof(kc.HeadLinearCall), ctypes.sizeof(kc.WindowAttentionCall), ctypes.sizeof(kc.RetentionCall), ctypes.sizeof(kc.MoePlanCall),
+            ctypes.sizeof(kc.MoeCombineCall)]
     assert got == want
 
 
