@@ -9,14 +9,13 @@
 //                                  products on mma.sync (HBM- or latency-bound), the keys split over the chip
 //   causal_attention_tile_kernel   many rows (prefill): 128-row tiles on tcgen05 with scores, weights and output in TMEM
 // Everything else (f32, no cap, larger caps, sizes TMA cannot take) runs the general kernel.
-#include "gemm_kernels.cuh"
+#include "attention_tile.cuh"
 
 #include <algorithm>
 
 namespace {
 
 constexpr float CAP_LIMIT = 64.0f;
-constexpr float LOG2E = 1.4426950408889634f;
 
 // The factor of a query at position p: 1 + coef * ln(floor((p + 1) / every) + 1). IEEE division: an exact quotient
 // stays exact, so the floor steps exactly at multiples of `every`.
@@ -107,16 +106,6 @@ int32_t launch_generic(holo_b200_ctx* ctx, const HoloCausalArgs& a) {
 
 
 // ---- capped scores without a maximum -----------------------------------------------------------------------------
-__device__ __forceinline__ float ex2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float rcp(float x) {
-    float y;
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 // exp(cap * tanh(s * factor / cap)), with c1 = 2 factor log2(e) / cap and c2 = cap log2(e):
 // tanh(y) = 1 - 2 / (exp(2y) + 1), so the exponent in log2 units is c2 - 2 c2 / (2^(s c1) + 1).
 __device__ __forceinline__ float capped_exp(float s, float c1, float c2) { return ex2(fmaf(-2.0f * c2, rcp(ex2(s * c1) + 1.0f), c2)); }
@@ -125,26 +114,6 @@ __device__ __forceinline__ float capped_exp(float s, float c1, float c2) { retur
 // a degree-5 polynomial in y^2 (a Chebyshev fit over the interval; |error| of tanh below 1e-7, f32 rounding included). One
 // special-function operation per score instead of three, which is what bounds the many-row kernel.
 constexpr float TANH_SMALL = 0.75f;
-__device__ __forceinline__ uint64_t pair(float lo, float hi) {
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
-    return r;
-}
-__device__ __forceinline__ float2 unpair(uint64_t v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-    uint64_t r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
 // c0 = factor / cap, c2 = cap log2(e), each twice
 __device__ __forceinline__ float2 capped_exp_small(uint64_t s, uint64_t c0, uint64_t c2) {
     const uint64_t y = mul2(s, c0), z = mul2(y, y);
@@ -155,11 +124,6 @@ __device__ __forceinline__ float2 capped_exp_small(uint64_t s, uint64_t c0, uint
     t = fma2(t, z, pair(1.0f, 1.0f));
     const float2 e = unpair(mul2(mul2(t, y), c2));
     return make_float2(ex2(e.x), ex2(e.y));
-}
-
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&h);
 }
 
 // ---- few rows: keys split over CTAs and warps ----------------------------------------------------------------------
@@ -175,22 +139,6 @@ struct SplitParams {
     uint32_t* arrivals;
     uint32_t group, splits;
 };
-
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// 16 bytes to shared memory, or 16 zero bytes when `take` is false (nothing is read then)
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool take) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(take ? 16u : 0u) : "memory");
-}
 
 template <int VT, int STAGES>   // vdim <= 16 VT
 __global__ void __launch_bounds__(256)
@@ -422,7 +370,6 @@ int32_t try_split(holo_b200_ctx* ctx, const HoloCausalArgs& a, bool* taken) {
 // each key half's weights over the first half of its scores (the next scores then wait for the item's product). It is allocated after the dependency wait, and dependents are
 // released only after the allocation, so no neighbouring launch can hold columns this kernel or its predecessor waits for.
 constexpr int TILE_THREADS = 576;
-constexpr uint32_t TILE_CHUNK = 128 * 128;   // 128 rows of 64 bf16 columns (one 128B-swizzled TMA box)
 
 struct TileParams {
     HoloCausalArgs a;
@@ -431,67 +378,6 @@ struct TileParams {
     uint32_t alias;     // P lies over S
     uint32_t ostride;   // TMEM columns between the accumulators of two query tiles
 };
-
-__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-        ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar)
-        : "memory");
-}
-// A operand (128 x 16 bf16, two elements per 32-bit column) in TMEM
-__device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n.reg .pred p;\nsetp.ne.b32 p, %4, 0;\ntcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}\n"
-        ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
-        : "r"(taddr));
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
-// The two halves of tmem_ld32: request 32 columns; wait for everything requested (the values pass through the wait, so that
-// no use of them can be scheduled before it).
-__device__ __forceinline__ void tmem_ld32_request(uint32_t taddr, uint32_t (&v)[32]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];\n"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]),
-          "=r"(v[17]), "=r"(v[18]), "=r"(v[19]), "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]),
-          "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]), "=r"(v[30]), "=r"(v[31])
-        : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_ld32_wait(uint32_t (&v)[32]) {
-    asm volatile("tcgen05.wait::ld.sync.aligned;"
-                 : "+r"(v[0]), "+r"(v[1]), "+r"(v[2]), "+r"(v[3]), "+r"(v[4]), "+r"(v[5]), "+r"(v[6]), "+r"(v[7]), "+r"(v[8]),
-                   "+r"(v[9]), "+r"(v[10]), "+r"(v[11]), "+r"(v[12]), "+r"(v[13]), "+r"(v[14]), "+r"(v[15]), "+r"(v[16]),
-                   "+r"(v[17]), "+r"(v[18]), "+r"(v[19]), "+r"(v[20]), "+r"(v[21]), "+r"(v[22]), "+r"(v[23]), "+r"(v[24]),
-                   "+r"(v[25]), "+r"(v[26]), "+r"(v[27]), "+r"(v[28]), "+r"(v[29]), "+r"(v[30]), "+r"(v[31])::"memory");
-}
-// ... and for a second array of the same request
-__device__ __forceinline__ void tmem_ld32_pass(uint32_t (&v)[32]) {
-    asm volatile("" : "+r"(v[0]), "+r"(v[1]), "+r"(v[2]), "+r"(v[3]), "+r"(v[4]), "+r"(v[5]), "+r"(v[6]), "+r"(v[7]), "+r"(v[8]),
-                   "+r"(v[9]), "+r"(v[10]), "+r"(v[11]), "+r"(v[12]), "+r"(v[13]), "+r"(v[14]), "+r"(v[15]), "+r"(v[16]),
-                   "+r"(v[17]), "+r"(v[18]), "+r"(v[19]), "+r"(v[20]), "+r"(v[21]), "+r"(v[22]), "+r"(v[23]), "+r"(v[24]),
-                   "+r"(v[25]), "+r"(v[26]), "+r"(v[27]), "+r"(v[28]), "+r"(v[29]), "+r"(v[30]), "+r"(v[31])::"memory");
-}
-__device__ __forceinline__ void tmem_st8(uint32_t taddr, const uint32_t (&v)[8]) {
-    asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%8], {%0, %1, %2, %3, %4, %5, %6, %7};\n"
-                 ::"r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(taddr)
-                 : "memory");
-}
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&v)[16]) {
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15};\n"
-        ::"r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]), "r"(v[10]),
-          "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(taddr)
-        : "memory");
-}
 
 template <int NQ>
 __global__ void __launch_bounds__(TILE_THREADS, 1)

@@ -247,28 +247,26 @@ int32_t holo_launch_linear(holo_b200_ctx* ctx, const HoloLinearArgs& a) {
 // ---- further row operations of decoder steps ----------------------------------------------------------------------
 namespace {
 
-// (cos, sin) of (*pos + row) * f_j. The frequency comes as a rounded value and its remainder, the product is split the same
-// way, and the remainder of the angle enters to first order: the error stays that of one f32 rounding at any position.
+// (cos, sin) of (*pos + row) times frequency j. The frequency is in turns, as a rounded value and its remainder; the product is
+// split the same way and its whole turns dropped, which is exact: the angle's error is one f32 rounding below half a turn
+// at any position.
+__device__ __forceinline__ float turns(float x, float hi, float lo) {
+    const float t = x * hi;
+    return (t - rintf(t)) + fmaf(x, lo, fmaf(x, hi, -t));
+}
 __global__ void rotary_table_kernel(const uint32_t* __restrict__ pos, const float* __restrict__ freq, float2* __restrict__ out, uint32_t rows, uint32_t half) {
     holo_pdl_trigger();
     holo_pdl_wait();
     const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= rows * half) return;
-    const uint32_t row = i / half, j = i % half, at = *pos + row;
-    const uint32_t low = at & 0xffffu;                       // positions past 2^24 are split as well
-    float s = 0.0f, c = 1.0f;
-#pragma unroll
-    for (int part = 0; part < 2; ++part) {
-        const float x = part ? (float)(at - low) : (float)low;
-        if (x == 0.0f) continue;
-        const float a = x * freq[j], e = fmaf(x, freq[j], -a) + x * freq[half + j];
-        float sa, ca;
-        sincosf(a, &sa, &ca);
-        const float s1 = fmaf(ca, e, sa), c1 = fmaf(-sa, e, ca);
-        const float sn = s * c1 + c * s1;
-        c = c * c1 - s * s1;
-        s = sn;
+    const uint32_t row = i / half, j = i % half, at = *pos + row, low = at & 0xfffffu;      // both parts are exact in f32
+    float r = turns((float)low, freq[j], freq[half + j]);
+    if (at != low) {
+        r += turns((float)(at - low), freq[j], freq[half + j]);
+        r -= rintf(r);
     }
+    float s, c;
+    sincospif(2.0f * r, &s, &c);
     out[i] = make_float2(c, s);
 }
 

@@ -1,9 +1,13 @@
 // Retention (linear attention with one fixed decay per head): S = decay S + k v^T, o = scale S^T q, every head's o divided by its
 // root mean square and multiplied by the gate. The state is f32 and stays in place between steps.
-#include "common.h"
-
-#include <cuda_bf16.h>
-#include <stdlib.h>
+//
+//   retention_chunk_kernel      bf16, several rows: chunks of 128 tokens on mma.sync, the state in registers from the first
+//                               chunk to the last
+//   retention_token_kernel      one row
+//   retention_sequence_kernel   everything else: token by token, one CTA per head
+//
+// In the first two a cluster of CTAs shares a head, each with a slice of the value columns; they exchange the sums of squares.
+#include "attention_tile.cuh"
 
 #include <algorithm>
 
@@ -11,6 +15,426 @@ namespace {
 
 __device__ __forceinline__ void store_out(float* out, uint64_t i, float v) { out[i] = v; }
 __device__ __forceinline__ void store_out(__nv_bfloat16* out, uint64_t i, float v) { out[i] = __float2bfloat16_rn(v); }
+
+// ---- value slices of a head in a cluster ----------------------------------------------------------------------------------
+constexpr uint32_t MAX_SLICES = 8;
+__device__ __forceinline__ void store_remote(uint32_t addr, uint32_t rank, float v) {
+    uint32_t r;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(addr), "r"(rank));
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(r), "f"(v) : "memory");
+}
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
+// ---- one row --------------------------------------------------------------------------------------------------------------
+// Grid (slices, heads). A thread owns four columns of the slice and every GROUPS-th key dimension; the state is read, advanced
+// and written once.
+constexpr int TOK_THREADS = 256;
+template <typename T>
+__global__ void __launch_bounds__(TOK_THREADS)
+retention_token_kernel(const HoloRetentionArgs a, uint32_t width) {
+    extern __shared__ __align__(16) float t_mem[];      // q [dim], k [dim], parts [groups][width], o [width]
+    __shared__ float s_sq[MAX_SLICES], s_part[TOK_THREADS / 32];
+    const uint32_t slice = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vecs = width / 4, groups = TOK_THREADS / vecs;
+    float *s_q = t_mem, *s_k = s_q + a.dim, *s_parts = s_k + a.dim, *s_o = s_parts + groups * width;
+    holo_pdl_trigger();
+    cluster_arrive();       // everyone has started: their shared memory may be written
+    holo_pdl_wait();
+    cluster_wait();
+    const bool run = a.step[1] != 0, fresh = a.step[0] == 0;     // the same for every thread of the cluster
+    const uint32_t cv = tid % vecs, group = tid / vecs, e0 = slice * width + cv * 4;
+    if (run) {
+        for (uint32_t i = tid; i < a.dim; i += TOK_THREADS) {
+            s_q[i] = (float)((const T*)a.q)[(uint64_t)h * a.dim + i];
+            s_k[i] = (float)((const T*)a.k)[(uint64_t)h * a.dim + i];
+        }
+        __syncthreads();
+        if (group < groups) {
+            const float decay = a.decay[h];
+            float v[4], acc[4] = {};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) v[i] = (float)((const T*)a.v)[(uint64_t)h * a.vdim + e0 + i];
+            float* state = a.state + (uint64_t)h * a.dim * a.vdim + e0;
+#pragma unroll 8
+            for (uint32_t d = group; d < a.dim; d += groups) {
+                float4* at = reinterpret_cast<float4*>(state + (uint64_t)d * a.vdim);
+                float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *at;
+                const float k = s_k[d], q = s_q[d];
+                s.x = fmaf(decay, s.x, k * v[0]); s.y = fmaf(decay, s.y, k * v[1]);
+                s.z = fmaf(decay, s.z, k * v[2]); s.w = fmaf(decay, s.w, k * v[3]);
+                *at = s;
+                acc[0] = fmaf(s.x, q, acc[0]); acc[1] = fmaf(s.y, q, acc[1]);
+                acc[2] = fmaf(s.z, q, acc[2]); acc[3] = fmaf(s.w, q, acc[3]);
+            }
+            *reinterpret_cast<float4*>(s_parts + group * width + cv * 4) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        }
+        __syncthreads();
+        float sq = 0.0f;
+        for (uint32_t c = tid; c < width; c += TOK_THREADS) {
+            float o = 0.0f;
+            for (uint32_t g = 0; g < groups; ++g) o += s_parts[g * width + c];
+            o *= a.scale;
+            s_o[c] = o;
+            if (slice * width + c < a.vmean) sq = fmaf(o, o, sq);
+        }
+        for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        if ((tid & 31u) == 0) s_part[tid >> 5] = sq;
+        __syncthreads();
+        if (tid < gridDim.x) {
+            float total = 0.0f;
+#pragma unroll
+            for (int w = 0; w < TOK_THREADS / 32; ++w) total += s_part[w];
+            store_remote(smem_u32(&s_sq[slice]), tid, total);
+        }
+    }
+    __syncwarp();
+    cluster_arrive();
+    cluster_wait();
+    if (!run) return;
+    float total = 0.0f;
+    for (uint32_t i = 0; i < gridDim.x; ++i) total += s_sq[i];
+    const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
+    for (uint32_t c = tid; c < width; c += TOK_THREADS) {
+        const uint64_t e = (uint64_t)h * a.vdim + slice * width + c;
+        store_out((T*)a.out, e, s_o[c] * inv * (float)((const T*)a.gate)[e]);
+    }
+}
+
+template <typename T>
+int32_t launch_token(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
+    *taken = false;
+    uint32_t slices = MAX_SLICES;
+    while (slices > 1 && (a.vdim % (4 * slices) != 0 || a.vdim / slices < 16)) slices /= 2;
+    const uint32_t width = a.vdim / slices;
+    if (a.dim % 4 || a.vdim % 4 || width > 4 * TOK_THREADS) return HOLO_OK;
+    const size_t smem = (2 * a.dim + (TOK_THREADS / (width / 4)) * width + width) * sizeof(float);    // at most 16 KiB
+    HOLO_CUDA(holo_launch_kernel_cluster(ctx, retention_token_kernel<T>, dim3(slices, a.heads), dim3(TOK_THREADS), smem, slices, 1u, a, width));
+    ctx->launches++;
+    *taken = true;
+    return HOLO_OK;
+}
+
+// ---- several rows -----------------------------------------------------------------------------------------------------------
+// Grid (slices, heads), a slice has W value columns. Per chunk of up to 128 tokens (64 where those do not fit), with p(n) = decay^n, L tokens in the chunk:
+//   o_i  = p(i + 1) S^T q_i + sum_{j <= i} p(i - j) (q_i . k_j) v_j          warp w: tokens 16 w .. 16 w + 15
+//   S    = p(L) S + sum_j p(L - 1 - j) k_j v_j^T                             warp w: key dimensions 8 (w + 8 n) .. + 7
+// S is held transposed in the accumulator registers of the second product. What enters a product besides q, k and v (S, the
+// decayed scores, the decayed values) is f32 and goes in as the sum of two bf16 values, so that it keeps 16 significant bits;
+// everything is added up in f32.
+constexpr int CHUNK_WARPS = 8;
+
+__device__ __forceinline__ void split_bf16(float lo, float hi, uint32_t& big, uint32_t& small) {
+    big = pack_bf16(lo, hi);
+    const __nv_bfloat162 b = *reinterpret_cast<const __nv_bfloat162*>(&big);
+    small = pack_bf16(lo - __low2float(b), hi - __high2float(b));
+}
+
+template <int W, int CHUNK>
+struct ChunkSmem {
+    static constexpr uint32_t VP = W * 2 + 16;      // row pitches: an odd number of 16-byte units
+    uint32_t qk, stage, stages, sbig, vbig, power, sums, total;
+    __host__ __device__ ChunkSmem(uint32_t dim, uint32_t nstages) {
+        qk = dim * 2 + 16;
+        stages = nstages;
+        stage = CHUNK * (2 * qk + VP);               // q, k, v rows
+        sbig = nstages * stage;                      // S^T as [W][dim], twice
+        vbig = sbig + 2 * W * qk;                    // decayed values [CHUNK][W], twice
+        power = vbig + 2 * CHUNK * VP;               // p(0) .. p(CHUNK)
+        sums = power + (CHUNK + 4) * 4;              // sums of squares [2][MAX_SLICES][CHUNK]
+        total = sums + 2 * MAX_SLICES * CHUNK * 4;
+    }
+};
+
+template <int W, int NT, int CHUNK>   // dim <= 64 NT, CHUNK at most 16 tokens per warp
+__global__ void __launch_bounds__(CHUNK_WARPS * 32)
+retention_chunk_kernel(const HoloRetentionArgs a, uint32_t nstages) {
+    extern __shared__ __align__(16) uint8_t sm[];
+    constexpr int MT = W / 16, OT = W / 8;
+    const ChunkSmem<W, CHUNK> s(a.dim, nstages);
+    constexpr uint32_t VP = ChunkSmem<W, CHUNK>::VP;
+    const uint32_t slice = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r0 = lane >> 2, c0 = (lane & 3) * 2;
+    const uint32_t base = smem_u32(sm), ntiles = a.dim / 8, ksteps = a.dim / 16;
+    float* s_power = reinterpret_cast<float*>(sm + s.power);
+    float* s_sums = reinterpret_cast<float*>(sm + s.sums);
+    holo_pdl_trigger();
+    cluster_arrive();       // everyone has started: their shared memory may be written
+    holo_pdl_wait();
+    cluster_wait();
+    const uint32_t count = min(a.rows, a.step[1]), chunks = (count + CHUNK - 1) / CHUNK;
+    const bool fresh = a.step[0] == 0;
+    if (chunks == 0) return;                         // the same for the whole cluster
+    const float decay = a.decay[h];
+    for (uint32_t i = tid; i <= CHUNK; i += blockDim.x) s_power[i] = i == 0 ? 1.0f : powf(decay, (float)i);
+    const __nv_bfloat16* q = (const __nv_bfloat16*)a.q + (uint64_t)h * a.dim;
+    const __nv_bfloat16* k = (const __nv_bfloat16*)a.k + (uint64_t)h * a.dim;
+    const uint64_t col = (uint64_t)h * a.vdim + slice * W;
+    const __nv_bfloat16* v = (const __nv_bfloat16*)a.v + col;
+
+    auto load_chunk = [&](uint32_t chunk, uint32_t stage) {
+        const uint32_t dst = base + stage * s.stage, vecs = a.dim / 8;
+        for (uint32_t i = tid; i < CHUNK * vecs; i += blockDim.x) {
+            const uint32_t r = i / vecs, c = i % vecs, row = chunk * CHUNK + r;
+            const uint64_t from = min(row, count - 1);
+            cp_async16(dst + r * s.qk + c * 16, q + from * a.q_ld + c * 8, row < count);
+            cp_async16(dst + (CHUNK + r) * s.qk + c * 16, k + from * a.k_ld + c * 8, row < count);
+        }
+        for (uint32_t i = tid; i < CHUNK * (W / 8); i += blockDim.x) {
+            const uint32_t r = i / (W / 8), c = i % (W / 8), row = chunk * CHUNK + r;
+            cp_async16(dst + 2 * CHUNK * s.qk + r * VP + c * 16, v + (uint64_t)min(row, count - 1) * a.v_ld + c * 8, row < count);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    load_chunk(0, 0);
+    // S^T: rows = value columns 16 m + r0 (+ 8), columns = key dimensions 8 (warp + 8 n) + c0 (+ 1)
+    float st[NT][MT][4];
+    float* home = a.state + (uint64_t)h * a.dim * a.vdim + slice * W;
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const uint32_t d = (warp + 8 * n) * 8 + c0 + (e & 1), x = 16 * m + r0 + 8 * (e >> 1);
+                st[n][m][e] = !fresh && d < a.dim ? home[(uint64_t)d * a.vdim + x] : 0.0f;
+            }
+    for (uint32_t chunk = 0; chunk < chunks; ++chunk) {
+        const uint32_t stage = s.stages == 2 ? chunk & 1u : 0u, tokens = min((uint32_t)CHUNK, count - chunk * CHUNK);
+        const uint32_t s_q = base + stage * s.stage, s_k = s_q + CHUNK * s.qk, s_v = s_k + CHUNK * s.qk;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                             // the chunk is here; everyone is through with the one before
+        if (s.stages == 2 && chunk + 1 < chunks) load_chunk(chunk + 1, stage ^ 1u);
+        // S and the decayed values as pairs of bf16
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+            if ((warp + 8 * n) < ntiles)
+#pragma unroll
+                for (int m = 0; m < MT; ++m)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        uint32_t big, small;
+                        split_bf16(st[n][m][2 * e], st[n][m][2 * e + 1], big, small);
+                        uint8_t* at = sm + s.sbig + (16 * m + r0 + 8 * e) * s.qk + ((warp + 8 * n) * 8 + c0) * 2;
+                        *reinterpret_cast<uint32_t*>(at) = big;
+                        *reinterpret_cast<uint32_t*>(at + W * s.qk) = small;
+                    }
+        }
+        for (uint32_t i = tid; i < CHUNK * (W / 2); i += blockDim.x) {
+            const uint32_t r = i / (W / 2), c = i % (W / 2);
+            const float f = r < tokens ? s_power[tokens - 1 - r] : 0.0f;
+            const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(sm + (s_v - base) + r * VP + c * 4);
+            uint32_t big, small;
+            split_bf16(__low2float(x) * f, __high2float(x) * f, big, small);
+            uint8_t* at = sm + s.vbig + r * VP + c * 4;
+            *reinterpret_cast<uint32_t*>(at) = big;
+            *reinterpret_cast<uint32_t*>(at + CHUNK * VP) = small;
+        }
+        __syncthreads();
+        // outputs of this warp's 16 tokens
+        const uint32_t row = warp * 16;
+        float o[OT][4];
+#pragma unroll
+        for (int n = 0; n < OT; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[n][e] = 0.0f;
+        const bool active = row < tokens;
+        if (active) {
+            const uint32_t q_addr = s_q + (row + (lane & 15)) * s.qk + (lane >> 4) * 16;
+            // operands whose rows are the output's columns: 16 rows, one step of 16
+            const uint32_t n_off = ((lane & 7) + ((lane >> 4) << 3)) * s.qk + ((lane >> 3) & 1) * 16;
+            for (uint32_t x = 0; x < ksteps; ++x) {
+                uint32_t qa[4], sb[4];
+                ldsm4(q_addr + x * 32, qa);
+#pragma unroll
+                for (int n = 0; n < OT; n += 2) {
+                    const uint32_t at = base + s.sbig + n * 8 * s.qk + n_off + x * 32;
+                    ldsm4(at, sb);
+                    mma16816(o[n], qa, sb[0], sb[1]);
+                    mma16816(o[n + 1], qa, sb[2], sb[3]);
+                    ldsm4(at + W * s.qk, sb);
+                    mma16816(o[n], qa, sb[0], sb[1]);
+                    mma16816(o[n + 1], qa, sb[2], sb[3]);
+                }
+            }
+            const float f0 = s_power[row + r0 + 1], f1 = s_power[row + r0 + 9];
+#pragma unroll
+            for (int n = 0; n < OT; ++n) {
+                o[n][0] *= f0; o[n][1] *= f0;
+                o[n][2] *= f1; o[n][3] *= f1;
+            }
+            const uint32_t v_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * VP + (lane >> 4) * 16;
+            for (uint32_t j = 0; j <= warp; ++j) {
+                float sc[2][4] = {};
+                const uint32_t k_addr = s_k + j * 16 * s.qk + n_off;
+#pragma unroll 4
+                for (uint32_t x = 0; x < ksteps; ++x) {
+                    uint32_t qa[4], kb[4];
+                    ldsm4(q_addr + x * 32, qa);
+                    ldsm4(k_addr + x * 32, kb);
+                    mma16816(sc[0], qa, kb[0], kb[1]);
+                    mma16816(sc[1], qa, kb[2], kb[3]);
+                }
+#pragma unroll
+                for (int n = 0; n < 2; ++n)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int back = (int)(row + r0 + 8 * (e >> 1)) - (int)(j * 16 + n * 8 + c0 + (e & 1));
+                        sc[n][e] = back >= 0 ? sc[n][e] * s_power[back] : 0.0f;
+                    }
+                uint32_t big[4], small[4];
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    split_bf16(sc[n][0], sc[n][1], big[2 * n], small[2 * n]);
+                    split_bf16(sc[n][2], sc[n][3], big[2 * n + 1], small[2 * n + 1]);
+                }
+#pragma unroll
+                for (int n = 0; n < OT; n += 2) {
+                    uint32_t vb[4];
+                    ldsm4t(s_v + j * 16 * VP + v_off + n * 16, vb);
+                    mma16816(o[n], big, vb[0], vb[1]);
+                    mma16816(o[n + 1], big, vb[2], vb[3]);
+                    mma16816(o[n], small, vb[0], vb[1]);
+                    mma16816(o[n + 1], small, vb[2], vb[3]);
+                }
+            }
+        }
+        // sums of squares of this slice, to every CTA of the head
+        float sq[2] = {};
+#pragma unroll
+        for (int n = 0; n < OT; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                o[n][e] *= a.scale;
+                if (slice * W + n * 8 + c0 + (e & 1) < a.vmean) sq[e >> 1] = fmaf(o[n][e], o[n][e], sq[e >> 1]);
+            }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            sq[e] += __shfl_xor_sync(0xffffffffu, sq[e], 1);
+            sq[e] += __shfl_xor_sync(0xffffffffu, sq[e], 2);
+        }
+        const uint32_t sums = (chunk & 1u) * MAX_SLICES * CHUNK;
+        if (row < CHUNK)
+            for (uint32_t to = lane & 3; to < gridDim.x; to += 4)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) store_remote(base + s.sums + (sums + slice * CHUNK + row + r0 + 8 * e) * 4, to, sq[e]);
+        __syncwarp();
+        cluster_arrive();
+        // while the sums travel: the gates of this warp's tokens, and the state
+        __nv_bfloat162 gate[2][OT];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const uint32_t i = chunk * CHUNK + row + r0 + 8 * e;
+#pragma unroll
+            for (int n = 0; n < OT; ++n)
+                if (row < CHUNK && i < count) gate[e][n] = *reinterpret_cast<const __nv_bfloat162*>((const __nv_bfloat16*)a.gate + (uint64_t)i * a.gate_ld + col + n * 8 + c0);
+        }
+        const float keep = s_power[tokens];
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) st[n][m][e] *= keep;
+        {
+            // A: rows = value columns (the stored rows are tokens: transposed), B: rows = tokens, columns = key dimensions
+            const uint32_t a_off = ((lane & 7) + ((lane >> 4) << 3)) * VP + ((lane >> 3) & 1) * 16;
+            const uint32_t b_off = ((lane & 7) + (((lane >> 3) & 1) << 3)) * s.qk;
+            const uint32_t steps = (tokens + 15) / 16;
+            for (uint32_t x = 0; x < steps; ++x) {
+                uint32_t big[MT][4], small[MT][4];
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    const uint32_t at = base + s.vbig + x * 16 * VP + a_off + m * 32;
+                    ldsm4t(at, big[m]);
+                    ldsm4t(at + CHUNK * VP, small[m]);
+                }
+#pragma unroll
+                for (int n = 0; n < NT; n += 2) {
+                    // two tiles of eight key dimensions at once: lanes 16 .. 31 address the second one
+                    const uint32_t t0 = warp + 8 * n, t1 = t0 + 8;
+                    if (t0 < ntiles) {
+                        uint32_t kb[4];
+                        ldsm4t(s_k + x * 16 * s.qk + b_off + ((lane >> 4) && t1 < ntiles ? t1 : t0) * 16, kb);
+#pragma unroll
+                        for (int m = 0; m < MT; ++m) {
+                            mma16816(st[n][m], big[m], kb[0], kb[1]);
+                            mma16816(st[n][m], small[m], kb[0], kb[1]);
+                            if (n + 1 < NT && t1 < ntiles) {
+                                mma16816(st[n + 1 < NT ? n + 1 : n][m], big[m], kb[2], kb[3]);
+                                mma16816(st[n + 1 < NT ? n + 1 : n][m], small[m], kb[2], kb[3]);
+                            }
+                        }
+                    }
+                }
+            }
+        }
+        __syncwarp();
+        cluster_wait();
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const uint32_t i = chunk * CHUNK + row + r0 + 8 * e;
+            if (row >= CHUNK || i >= count) continue;
+            float total = 0.0f;
+            for (uint32_t x = 0; x < gridDim.x; ++x) total += s_sums[sums + x * CHUNK + row + r0 + 8 * e];
+            const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
+            __nv_bfloat16* out = (__nv_bfloat16*)a.out + (uint64_t)i * a.ld + col;
+#pragma unroll
+            for (int n = 0; n < OT; ++n)
+                *reinterpret_cast<__nv_bfloat162*>(out + n * 8 + c0) =
+                    __floats2bfloat162_rn(o[n][2 * e] * inv * __low2float(gate[e][n]), o[n][2 * e + 1] * inv * __high2float(gate[e][n]));
+        }
+        if (s.stages == 1 && chunk + 1 < chunks) {
+            __syncthreads();
+            load_chunk(chunk + 1, 0);
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const uint32_t d = (warp + 8 * n) * 8 + c0 + (e & 1), x = 16 * m + r0 + 8 * (e >> 1);
+                if (d < a.dim) home[(uint64_t)d * a.vdim + x] = st[n][m][e];
+            }
+}
+
+template <int W, int NT, int CHUNK>
+int32_t launch_chunk_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
+    const uint32_t limit = (uint32_t)ctx->smem_optin - 1024;
+    uint32_t stages = a.rows > (uint32_t)CHUNK ? 2 : 1;
+    if (ChunkSmem<W, CHUNK>(a.dim, stages).total > limit) stages = 1;
+    const uint32_t smem = ChunkSmem<W, CHUNK>(a.dim, stages).total;
+    if (smem > limit) return HOLO_OK;
+    static thread_local int configured_device = -1;
+    if (configured_device != ctx->device) {
+        HOLO_CUDA(cudaFuncSetAttribute(retention_chunk_kernel<W, NT, CHUNK>, cudaFuncAttributeMaxDynamicSharedMemorySize, limit));
+        configured_device = ctx->device;
+    }
+    const uint32_t slices = a.vdim / W;
+    HOLO_CUDA(holo_launch_kernel_cluster(ctx, retention_chunk_kernel<W, NT, CHUNK>, dim3(slices, a.heads), dim3(CHUNK_WARPS * 32), smem, slices, 1u, a, stages));
+    ctx->launches++;
+    *taken = true;
+    return HOLO_OK;
+}
+template <int W>
+int32_t launch_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
+    if (a.dim <= 128) return launch_chunk_as<W, 2, 128>(ctx, a, taken);
+    HOLO_TRY((launch_chunk_as<W, 4, 128>(ctx, a, taken)));
+    return *taken ? HOLO_OK : launch_chunk_as<W, 4, 64>(ctx, a, taken);      // wide keys and values: shorter chunks
+}
+// Launches the chunk kernel, or returns with *taken false when the shape does not suit it.
+int32_t try_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
+    *taken = false;
+    if (a.dtype != HOLO_DTYPE_BF16 || a.dim % 16 || a.vdim % 16 || a.dim > 256 || (a.q_ld | a.k_ld | a.v_ld) % 8 || (a.gate_ld | a.ld) % 2 ||
+        (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) & 15u) || (((uintptr_t)a.gate | (uintptr_t)a.out) & 3u))
+        return HOLO_OK;
+    const auto fits = [&](uint32_t w) { return a.vdim % w == 0 && a.vdim / w <= MAX_SLICES; };
+    if (fits(32)) return launch_chunk<32>(ctx, a, taken);
+    if (fits(16)) return launch_chunk<16>(ctx, a, taken);
+    if (fits(48)) return launch_chunk<48>(ctx, a, taken);
+    if (fits(64)) return launch_chunk<64>(ctx, a, taken);
+    return HOLO_OK;
+}
 
 // ---- general form: one CTA per head, token by token ---------------------------------------------------------------------
 // 64 value columns at a time, four threads per column over the key dimensions. The state sits in shared memory where it fits.
@@ -93,5 +517,11 @@ int32_t launch_sequence(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
 }  // namespace
 
 int32_t holo_launch_retention(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
+    if (!getenv("HOLO_RETENTION_GENERAL")) {
+        bool taken = false;
+        if (a.rows == 1) HOLO_TRY(a.dtype == HOLO_DTYPE_F32 ? launch_token<float>(ctx, a, &taken) : launch_token<__nv_bfloat16>(ctx, a, &taken));
+        else HOLO_TRY(try_chunk(ctx, a, &taken));
+        if (taken) return HOLO_OK;
+    }
     return a.dtype == HOLO_DTYPE_F32 ? launch_sequence<float>(ctx, a) : launch_sequence<__nv_bfloat16>(ctx, a);
 }

@@ -5,14 +5,14 @@
 //   latent_attention_kernel   bf16, one key head whose values are the first columns of its keys (latent attention with the
 //                             up projections absorbed into query and output): key tiles in shared memory serve 16 (row, head)
 //                             pairs for both products (mma.sync), the window split over the chip
+//   window_tile_kernel        bf16, many rows: 128-row query tiles on tcgen05 with scores, weights and output in TMEM, a running
+//                             maximum per row and an accumulator that is rescaled only when the maximum has grown by a lot
 //   window_attention_kernel   everything else, f32 included: one CTA per (row, head)
-#include "gemm_kernels.cuh"
+#include "attention_tile.cuh"
 
 #include <algorithm>
 
 namespace {
-
-constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ void store_out(float* out, uint64_t i, float v) { out[i] = v; }
 __device__ __forceinline__ void store_out(__nv_bfloat16* out, uint64_t i, float v) { out[i] = __float2bfloat16_rn(v); }
@@ -122,21 +122,6 @@ struct LatentParams {
     float* partials;     // [pair tile][split][16][vdim + 2]
     uint32_t splits;
 };
-
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool take) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(take ? 16u : 0u) : "memory");
-}
 
 // The keys a pair tile sees: positions [lo, hi].
 struct LatentRange {
@@ -410,12 +395,349 @@ int32_t try_latent(holo_b200_ctx* ctx, const HoloWindowArgs& a, bool* taken) {
     return wide ? launch_latent_kt<64>(ctx, p, (uint32_t)pair_tiles) : launch_latent_kt<32>(ctx, p, (uint32_t)pair_tiles);
 }
 
+// ---- many rows: 128-row tiles on tcgen05 ------------------------------------------------------------------------------
+// A tile of 128 rows packs `rpt` rows times the heads of a group. One CTA works on NQ tiles of a key head, the keys in tiles
+// of 128; while the weight warps of one query tile exponentiate, the tensor core works for the other.
+//   warp 0      TMA producer: the query tiles once; key chunks (128 keys x 64 columns; the shared key part follows the head's
+//               own) and value tiles through rings
+//   warp 1      tcgen05.mma issuer. Per key tile and query tile q: O_q += P_q V as soon as the weights are stored, then
+//               S_q = Q_q K^T of the next key tile into the same columns (one thread's products execute in order)
+//   warps 2-9   weights and output, four warps per query tile, one thread per row
+// The weights are exp2(s - m) with m a reference that follows the row's maximum only when it has grown by more than RAISE
+// (log2 units): weights stay below 2^RAISE, and O is rarely rescaled. TMEM: S_q (P_q over its first half) at 128 q, O_q at
+// 256 + 128 q (NQ 2) or 256 (NQ 1, up to 256 columns). Allocated after the dependency wait, dependents released after that.
+constexpr int WT_THREADS = 320;
+constexpr float RAISE = 8.0f;
+
+struct WindowTileParams {
+    HoloWindowArgs a;
+    uint32_t* status;
+    uint32_t group, rpt, chunks1, chunks2, vchunks, kslots, vslots;
+};
+
+template <int NQ>
+__global__ void __launch_bounds__(WT_THREADS, 1)
+window_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_q2, const __grid_constant__ CUtensorMap map_k,
+                   const __grid_constant__ CUtensorMap map_k2, const __grid_constant__ CUtensorMap map_v, const WindowTileParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    const HoloWindowArgs& a = p.a;
+    const uint32_t raw = smem_u32(smem_raw);
+    const uint32_t base = (raw + 1023u) & ~1023u;
+    uint8_t* sm = smem_raw + (base - raw);
+    const uint32_t kchunks = p.chunks1 + p.chunks2, qbytes = kchunks * TILE_CHUNK, vbytes = p.vchunks * TILE_CHUNK;
+    const uint32_t s_q = base, s_k = s_q + NQ * qbytes, s_v = s_k + p.kslots * TILE_CHUNK;
+    const uint32_t off_bars = NQ * qbytes + p.kslots * TILE_CHUNK + p.vslots * vbytes;
+    // at most 16 key slots and 2 value slots
+    const uint32_t bar_q = base + off_bars, bar_k_full = bar_q + 8, bar_k_empty = bar_k_full + 128, bar_v_full = bar_k_empty + 128, bar_v_empty = bar_v_full + 16,
+                   bar_s = bar_v_empty + 16, bar_p = bar_s + 16, bar_pv = bar_p + 16;
+    uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + off_bars + 384);
+    volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + off_bars + 388);
+
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t g = blockIdx.x, row0 = (gridDim.y - 1 - blockIdx.y) * NQ * p.rpt;   // the tiles with the most keys first
+    if (threadIdx.x == 0) {
+        mbar_init(bar_q, 1);
+        for (uint32_t i = 0; i < p.kslots; ++i) {
+            mbar_init(bar_k_full + 8 * i, 1);
+            mbar_init(bar_k_empty + 8 * i, 1);
+        }
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(bar_v_full + 8 * i, 1);
+            mbar_init(bar_v_empty + 8 * i, 1);
+            mbar_init(bar_s + 8 * i, 1);
+            mbar_init(bar_p + 8 * i, 4);     // one arrival per weight warp
+            mbar_init(bar_pv + 8 * i, 1);
+        }
+        *s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    holo_pdl_wait();
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(s_tmem)), "r"(512u) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    holo_pdl_trigger();
+    const uint32_t tmem_base = *s_tmem;
+    const uint32_t pos = *a.pos, start = kv_start(a, pos);
+    const uint32_t t_lo = first_seen(a, pos + row0) / 128, t_hi = (pos + min(row0 + NQ * p.rpt, a.rows) - 1) / 128, ntiles = t_hi - t_lo + 1;
+
+    if (warp == 0) {
+        // ---------------- TMA producer ----------------
+        if (lane == 0) {
+            mbar_arrive_expect_tx(bar_q, NQ * kchunks * p.rpt * p.group * 128);
+            for (uint32_t i = 0; i < NQ; ++i) {
+                const int row = (int)(row0 + i * p.rpt), head = (int)(g * p.group);
+                for (uint32_t c = 0; c < p.chunks1; ++c) tma_load_3d(s_q + i * qbytes + c * TILE_CHUNK, &map_q, (int)(64 * c), head, row, bar_q);
+                for (uint32_t c = 0; c < p.chunks2; ++c) tma_load_3d(s_q + i * qbytes + (p.chunks1 + c) * TILE_CHUNK, &map_q2, (int)(64 * c), head, row, bar_q);
+            }
+            uint32_t ks = 0, kuse = 0, vs = 0, vuse = 0;      // slot, and how often the ring has gone round
+            bool ok = true;
+            for (uint32_t t = t_lo; t <= t_hi && ok; ++t) {
+                const int krow = (int)((t * 128 - start) % a.kv_rows), k2row = a.dim2 ? (int)(t * 128 % a.k2_rows) : 0;
+                for (uint32_t c = 0; c < kchunks && ok; ++c) {
+                    ok = kuse == 0 || mbar_wait(bar_k_empty + 8 * ks, (kuse - 1) & 1, s_abort, p.status);
+                    if (!ok) break;
+                    mbar_arrive_expect_tx(bar_k_full + 8 * ks, TILE_CHUNK);
+                    if (c < p.chunks1) tma_load_2d(s_k + ks * TILE_CHUNK, &map_k, (int)(g * a.dim + 64 * c), krow, bar_k_full + 8 * ks);
+                    else tma_load_2d(s_k + ks * TILE_CHUNK, &map_k2, (int)(64 * (c - p.chunks1)), k2row, bar_k_full + 8 * ks);
+                    if (++ks == p.kslots) ks = 0, ++kuse;
+                }
+                ok = ok && (vuse == 0 || mbar_wait(bar_v_empty + 8 * vs, (vuse - 1) & 1, s_abort, p.status));
+                if (!ok) break;
+                mbar_arrive_expect_tx(bar_v_full + 8 * vs, vbytes);
+                for (uint32_t c = 0; c < p.vchunks; ++c) tma_load_2d(s_v + vs * vbytes + c * TILE_CHUNK, &map_v, (int)(g * a.vdim + 64 * c), krow, bar_v_full + 8 * vs);
+                if (++vs == p.vslots) vs = 0, ++vuse;
+            }
+            if (!ok) {
+                // nothing may still be on its way into this CTA's shared memory when it ends: the last load of every slot
+                for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_q, 0); ++it) __nanosleep(64);
+                for (uint32_t i = 0; i < p.kslots; ++i) {
+                    const uint32_t loads = kuse + (i < ks ? 1u : 0u);
+                    for (uint32_t it = 0; loads && it < WAIT_LIMIT && !mbar_try_wait(bar_k_full + 8 * i, (loads - 1) & 1); ++it) __nanosleep(64);
+                }
+                for (uint32_t i = 0; i < p.vslots; ++i) {
+                    const uint32_t loads = vuse + (i < vs ? 1u : 0u);
+                    for (uint32_t it = 0; loads && it < WAIT_LIMIT && !mbar_try_wait(bar_v_full + 8 * i, (loads - 1) & 1); ++it) __nanosleep(64);
+                }
+            }
+        }
+    } else if (warp == 1) {
+        // ---------------- MMA issuer ----------------
+        if (lane == 0) {
+            // D = f32, A = B = bf16, M = 128; S: both operands K-major, N = 128; O: V is N-major, N = vdim
+            const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 3) << 17) | ((128u >> 4) << 24);
+            const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((a.vdim >> 3) << 17) | ((128u >> 4) << 24);
+            const uint64_t desc_q = smem_desc(s_q, 16, 1024), desc_k = smem_desc(s_k, 16, 1024), desc_v = smem_desc(s_v, TILE_CHUNK, 1024);
+            uint32_t ks = 0, kphase = 0, vs = 0, vphase = 0;
+            // S_q of the key tile whose chunks begin at slot ks; the last query tile gives every chunk back
+            auto scores = [&](uint32_t q) {
+                uint32_t slot = ks, phase = kphase;
+                for (uint32_t c = 0; c < kchunks; ++c) {
+                    if (q == 0 && !mbar_wait(bar_k_full + 8 * slot, phase, s_abort, p.status)) return false;
+                    if (q == 0) asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    const uint32_t width = c < p.chunks1 ? a.dim - 64 * c : a.dim2 - 64 * (c - p.chunks1);
+                    const uint64_t dq = desc_q + ((q * qbytes + c * TILE_CHUNK) >> 4), dk = desc_k + ((slot * TILE_CHUNK) >> 4);
+#pragma unroll
+                    for (uint32_t k = 0; k < 4; ++k)
+                        if (16 * k < width) umma_bf16(tmem_base + q * 128, dq + 2 * k, dk + 2 * k, idesc_s, (c | k) != 0);
+                    if (q == NQ - 1) umma_commit(bar_k_empty + 8 * slot);
+                    if (++slot == p.kslots) slot = 0, phase ^= 1;
+                }
+                umma_commit(bar_s + 8 * q);
+                if (q == NQ - 1) ks = slot, kphase = phase;
+                return true;
+            };
+            bool ok = mbar_wait(bar_q, 0, s_abort, p.status);
+            for (uint32_t q = 0; q < NQ && ok; ++q) ok = scores(q);
+            for (uint32_t i = 0; i < ntiles && ok; ++i) {
+                for (uint32_t q = 0; q < NQ && ok; ++q) {
+                    if (q == 0) ok = mbar_wait(bar_v_full + 8 * vs, vphase, s_abort, p.status);
+                    ok = ok && mbar_wait(bar_p + 8 * q, i & 1, s_abort, p.status);
+                    if (!ok) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    const uint64_t dv = desc_v + ((vs * vbytes) >> 4);
+#pragma unroll
+                    for (uint32_t k = 0; k < 8; ++k)
+                        umma_bf16_ts(tmem_base + 256 + q * 128, tmem_base + q * 128 + k * 8, dv + 128 * k, idesc_o, k != 0 || i != 0);
+                    umma_commit(bar_pv + 8 * q);
+                    if (q == NQ - 1) {
+                        umma_commit(bar_v_empty + 8 * vs);
+                        if (++vs == p.vslots) vs = 0, vphase ^= 1;
+                    }
+                    if (i + 1 < ntiles) ok = scores(q);
+                }
+            }
+        }
+    } else if ((warp - 2) >> 2 < NQ) {
+        // ---------------- weights (TMEM lane quarter = warp % 4), then the output ----------------
+        const uint32_t q = (warp - 2) >> 2, quarter = warp & 3u, tr = quarter * 32 + lane;
+        const uint32_t first = row0 + q * p.rpt, row = first + tr / p.group, head = g * p.group + tr % p.group;
+        const bool valid = tr < p.rpt * p.group && row < a.rows;
+        const uint32_t at = pos + min(row, a.rows - 1), seen = first_seen(a, at);
+        const uint32_t last_seen = first_seen(a, pos + min(first + p.rpt, a.rows) - 1);   // the first key the tile's last row sees
+        const uint32_t lanes = (quarter * 32u) << 16, tmem_s = tmem_base + q * 128 + lanes, tmem_o = tmem_base + 256 + q * 128 + lanes;
+        const float c = a.scale * LOG2E;
+        const uint64_t c2 = pair(c, c);
+        float ref = -1e30f, sum = 0.0f;
+        bool ok = true;
+        for (uint32_t i = 0; i < ntiles; ++i) {
+            ok = mbar_wait(bar_s + 8 * q, i & 1, s_abort, p.status) && !*s_abort;
+            // the product before these scores (it has finished: they were issued after it)
+            if (ok && i > 0) ok = mbar_wait(bar_pv + 8 * q, (i - 1) & 1, s_abort, p.status);
+            ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const uint32_t key0 = (t_lo + i) * 128;
+            uint32_t v[4][32];
+#pragma unroll
+            for (int x = 0; x < 4; ++x) tmem_ld32_request(tmem_s + 32 * x, v[x]);
+            tmem_ld32_wait(v[0]);
+#pragma unroll
+            for (int x = 1; x < 4; ++x) tmem_ld32_pass(v[x]);
+            if (key0 + 127 > pos + first || key0 < last_seen) {      // some row does not see some key
+#pragma unroll
+                for (int x = 0; x < 4; ++x)
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) {
+                        const uint32_t key = key0 + 32 * x + e;
+                        if (key > at || key < seen) v[x][e] = 0xff800000u;   // -infinity
+                    }
+            }
+            float top[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+            for (int x = 0; x < 4; ++x)
+#pragma unroll
+                for (int e = 0; e < 32; ++e) top[e & 3] = fmaxf(top[e & 3], __uint_as_float(v[x][e]));
+            const float most = fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) * c;
+            const bool raise = most > ref + RAISE;
+            if (__any_sync(0xffffffffu, raise)) {
+                const float f = raise ? ex2(ref - most) : 1.0f;
+                if (raise) ref = most;
+                sum *= f;
+                if (i > 0) {     // the products so far are in O, the next one waits for this warp's weights
+                    for (uint32_t x = 0; x < a.vdim / 16; ++x) {
+                        uint32_t o[16];
+                        tmem_ld16(tmem_o + 16 * x, o);
+#pragma unroll
+                        for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * f);
+                        tmem_st16(tmem_o + 16 * x, o);
+                    }
+                }
+            }
+            const uint64_t minus = pair(-ref, -ref);
+            uint64_t part[2] = {0, 0};
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                uint32_t w[16];
+#pragma unroll
+                for (int e = 0; e < 16; ++e) {
+                    const float2 s = unpair(fma2(pair(__uint_as_float(v[x][2 * e]), __uint_as_float(v[x][2 * e + 1])), c2, minus));
+                    const float lo = ex2(s.x), hi = ex2(s.y);
+                    part[e & 1] = add2(part[e & 1], pair(lo, hi));
+                    w[e] = pack_bf16(lo, hi);
+                }
+                tmem_st16(tmem_s + 16 * x, w);      // over scores this warp has already read
+            }
+            const float2 a0 = unpair(part[0]), a1 = unpair(part[1]);
+            sum += (a0.x + a0.y) + (a1.x + a1.y);
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar_p + 8 * q) : "memory");
+        }
+        ok = ok && mbar_wait(bar_pv + 8 * q, (ntiles - 1) & 1, s_abort, p.status) && !*s_abort && !(*reinterpret_cast<volatile uint32_t*>(p.status) & 4u);
+        ok = __all_sync(0xffffffffu, ok);
+        if (ok) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const float denom = sum + (a.sink && valid ? ex2(fmaf(a.sink[head], LOG2E, -ref)) : 0.0f);
+            const float inv = __fdiv_rn(1.0f, denom);
+            __nv_bfloat16* out = (__nv_bfloat16*)a.out + (uint64_t)row * a.ld + (uint64_t)head * a.vdim;
+            for (uint32_t x = 0; x < a.vdim / 16; ++x) {
+                uint32_t v[16], w[8];
+                tmem_ld16(tmem_o + 16 * x, v);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) w[e] = pack_bf16(__uint_as_float(v[2 * e]) * inv, __uint_as_float(v[2 * e + 1]) * inv);
+                if (valid) {
+                    reinterpret_cast<uint4*>(out + 16 * x)[0] = make_uint4(w[0], w[1], w[2], w[3]);
+                    reinterpret_cast<uint4*>(out + 16 * x)[1] = make_uint4(w[4], w[5], w[6], w[7]);
+                }
+            }
+        }
+    }
+    // everyone meets here, whatever happened above, so that TMEM is always released
+    __syncwarp();
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(512u) : "memory");
+    }
+}
+
+// `cols` columns of every head over all rows, a box of 64 columns of a group's heads over the tile's rows.
+int32_t make_map_heads(CUtensorMap* map, const void* ptr, uint32_t cols, uint32_t heads, uint32_t rows, uint64_t step, uint64_t ld, uint32_t group, uint32_t rpt) {
+    cuuint64_t dims[3] = {cols, heads, rows};
+    cuuint64_t strides[2] = {step * 2, ld * 2};
+    cuuint32_t box[3] = {64, group, rpt};
+    cuuint32_t es[3] = {1, 1, 1};
+    const CUresult r = encode_tiled_fn()(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? HOLO_OK : holo_fail(HOLO_ERR_DISPATCH, "dispatch failed: cuTensorMapEncodeTiled (attention) returned %d", (int)r);
+}
+// `cols` columns of rows of pitch ld, boxes of 64 columns and 128 rows.
+int32_t make_map_keys(CUtensorMap* map, const void* ptr, uint64_t cols, uint64_t rows, uint64_t ld) {
+    cuuint64_t dims[2] = {cols, rows};
+    cuuint64_t strides[1] = {ld * 2};
+    cuuint32_t box[2] = {64, 128};
+    cuuint32_t es[2] = {1, 1};
+    const CUresult r = encode_tiled_fn()(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? HOLO_OK : holo_fail(HOLO_ERR_DISPATCH, "dispatch failed: cuTensorMapEncodeTiled (attention) returned %d", (int)r);
+}
+
+template <int NQ>
+int32_t launch_window_tile(holo_b200_ctx* ctx, const CUtensorMap (&m)[5], const WindowTileParams& p, uint32_t ctas, uint32_t smem) {
+    static thread_local int configured_device = -1;
+    if (configured_device != ctx->device) {
+        HOLO_CUDA(cudaFuncSetAttribute(window_tile_kernel<NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, ctx->smem_optin));
+        configured_device = ctx->device;
+    }
+    HOLO_CUDA(holo_launch_kernel(ctx, window_tile_kernel<NQ>, dim3(p.a.kv_heads, ctas), dim3(WT_THREADS), smem, 1, m[0], m[1], m[2], m[3], m[4], p));
+    ctx->launches++;
+    return HOLO_OK;
+}
+
+// Launches the tile kernel, or returns with *taken false when the shape does not suit it.
+int32_t try_window_tile(holo_b200_ctx* ctx, const HoloWindowArgs& a, bool* taken) {
+    *taken = false;
+    WindowTileParams p;
+    p.a = a;
+    p.status = ctx->dev_status;
+    p.group = a.heads / a.kv_heads;
+    if (a.dtype != HOLO_DTYPE_BF16 || !(a.scale > 0.0f) || a.dim % 16 || a.dim2 % 16 || a.vdim % 16 || a.dim > 512 || a.dim2 > 512 || a.vdim > 256 || p.group > 128 ||
+        a.kv_rows % 128 || a.k2_rows % 128 || (a.q_ld | a.q_step | a.k_ld | a.v_ld | a.q2_ld | a.q2_step | a.k2_ld | a.ld) % 8 ||
+        (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.q2 | (uintptr_t)a.k2 | (uintptr_t)a.out) & 15u) || encode_tiled_fn() == nullptr)
+        return HOLO_OK;
+    p.rpt = 128 / p.group;
+    p.chunks1 = (a.dim + 63) / 64;
+    p.chunks2 = (a.dim2 + 63) / 64;
+    p.vchunks = (a.vdim + 63) / 64;
+    const uint32_t kchunks = p.chunks1 + p.chunks2, extra = 512 + 1024, slots = ((uint32_t)ctx->smem_optin - extra) / TILE_CHUNK;
+    const uint32_t qtiles = (a.rows + p.rpt - 1) / p.rpt;
+    if (qtiles > 65535) return HOLO_OK;
+    // two query tiles per CTA where they fit beside a whole key tile and a value tile; two value slots where one more key chunk fits as well
+    uint32_t nq = a.vdim <= 128 && qtiles > 1 && 3 * kchunks + p.vchunks <= slots ? 2 : 1;
+    if (const char* e = getenv("HOLO_WINDOW_QUERY_TILES")) nq = atoi(e) == 1 ? 1 : nq;
+    if ((nq + 1) * kchunks + p.vchunks > slots) return HOLO_OK;
+    p.vslots = (nq + 1) * kchunks + 1 + 2 * p.vchunks <= slots ? 2 : 1;
+    p.kslots = std::min<uint32_t>(slots - nq * kchunks - p.vslots * p.vchunks, 2 * kchunks);
+    p.kslots = std::min<uint32_t>(p.kslots, 16);
+    if (p.kslots < kchunks) return HOLO_OK;
+    const uint32_t smem = (nq * kchunks + p.kslots + p.vslots * p.vchunks) * TILE_CHUNK + extra;
+    CUtensorMap m[5];
+    HOLO_TRY(make_map_heads(&m[0], a.q, a.dim, a.heads, a.rows, a.q_step, a.q_ld, p.group, p.rpt));
+    HOLO_TRY(make_map_keys(&m[2], a.k, (uint64_t)a.kv_heads * a.dim, a.kv_rows, a.k_ld));
+    HOLO_TRY(make_map_keys(&m[4], a.v, (uint64_t)a.kv_heads * a.vdim, a.kv_rows, a.v_ld));
+    m[1] = m[0];
+    m[3] = m[2];
+    if (a.dim2) {
+        HOLO_TRY(make_map_heads(&m[1], a.q2, a.dim2, a.heads, a.rows, a.q2_step, a.q2_ld, p.group, p.rpt));
+        HOLO_TRY(make_map_keys(&m[3], a.k2, a.dim2, a.k2_rows, a.k2_ld));
+    }
+    *taken = true;
+    return nq == 2 ? launch_window_tile<2>(ctx, m, p, (qtiles + 1) / 2, smem) : launch_window_tile<1>(ctx, m, p, qtiles, smem);
+}
+
 }  // namespace
 
 int32_t holo_launch_window_attention(holo_b200_ctx* ctx, const HoloWindowArgs& a) {
     if (!getenv("HOLO_WINDOW_GENERAL")) {
         bool taken = false;
         HOLO_TRY(try_latent(ctx, a, &taken));
+        if (!taken) HOLO_TRY(try_window_tile(ctx, a, &taken));
         if (taken) return HOLO_OK;
     }
     return a.dtype == HOLO_DTYPE_F32 ? launch_general<float>(ctx, a) : launch_general<__nv_bfloat16>(ctx, a);

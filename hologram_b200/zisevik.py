@@ -46,8 +46,8 @@ class Rotation:
         return {"dims": self.dims, "base": self.base}
 
     def frequencies(self):
-        """f32 [2, dims / 2]: the rounded frequencies and their remainders."""
-        f = self.base ** (-2.0 * np.arange(self.dims // 2, dtype=np.float64) / max(self.dims, 1))
+        """f32 [2, dims / 2]: the frequencies in turns per position, rounded, and their remainders."""
+        f = self.base ** (-2.0 * np.arange(self.dims // 2, dtype=np.float64) / max(self.dims, 1)) / (2.0 * np.pi)
         hi = f.astype(np.float32)
         return np.stack([hi, (f - hi).astype(np.float32)])
 

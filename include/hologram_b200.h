@@ -480,8 +480,9 @@ typedef struct HoloCausalAttentionCall {
     uint8_t dtype;
 } HoloCausalAttentionCall;
 
-/* Extension. Angles of a step's rows: output f32 [rows, half, 2] = (cos, sin) of (*pos + i) * f_j. freq holds f_j as two f32
- * arrays, [half] rounded values and [half] remainders, so that the angle is good to f32 at any position. */
+/* Extension. Angles of a step's rows: output f32 [rows, half, 2] = (cos, sin) of 2 pi (*pos + i) f_j. freq holds f_j, in turns
+ * per position, as two f32 arrays, [half] rounded values and [half] remainders, so that the angle is good to f32 at any
+ * position. */
 typedef struct HoloRotaryTableCall {
     HoloBufferRef pos, freq, output;
     uint32_t rows, half;

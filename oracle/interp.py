@@ -268,7 +268,7 @@ def run(calls, slots, all_reduce=None):
         elif k == kc.K_ROTARY_TABLE:
             c = u.rotary_table
             f = _get(slots, c.freq, 8 * c.half, kc.DTYPE_F32).astype(np.float64).reshape(2, c.half).sum(axis=0)
-            a = (_word(slots, c.pos) + np.arange(c.rows))[:, None] * f
+            a = 2.0 * np.pi * (_word(slots, c.pos) + np.arange(c.rows))[:, None] * f
             _put(slots, c.output, np.stack([np.cos(a), np.sin(a)], axis=-1).astype(np.float32))
         elif k == kc.K_RMS_NORM_PARTS:
             c = u.rms_norm_parts

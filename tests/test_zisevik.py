@@ -149,7 +149,7 @@ def test_rotated_pairs_are_stored_side_by_side():
     rot = zk.Rotation(6, 100.0)
     assert rot.order(8).tolist() == [0, 3, 1, 4, 2, 5, 6, 7]
     hi, lo = rot.frequencies()
-    exact = 100.0 ** (-2.0 * np.arange(3) / 6)
+    exact = 100.0 ** (-2.0 * np.arange(3) / 6) / (2.0 * np.pi)
     assert np.abs(hi.astype(np.float64) + lo - exact).max() < 1e-15 * 2
     model, _ = make_model("odd")
     t = ref.random_tensors(ref.CONFIGS["odd"])
