@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the B200 backend hot path.
 
-  python bench.py [--gpus N] [--steps K] [--warmup W] [--workload lut|lut_sweep|attention|matmul|gemv|w8a8|decoder|fokonex]
+  python bench.py [--gpus N] [--steps K] [--warmup W] [--workload lut|lut_sweep|attention|matmul|gemv|w8a8|decoder|fokonex|zisevik]
   python bench.py --impl reference ...      # the reference CPU path (oracle restatement) on host cores
 
 One JSON line on stdout (rank 0). Timed with CUDA events on the stream the kernels are
@@ -855,6 +855,243 @@ def bench_fokonex(be, torch, args, stream):
     return out
 
 
+# ------------------------------------------------------------------------------------------
+# Zisevik: throughput of whole steps and of every kernel of its layers alone, beside Fokonex (the closest model) at the same
+# width and number of layer runs, measured the same way. Selected by --workload zisevik; prints one JSON line of its own.
+# ------------------------------------------------------------------------------------------
+
+ZISEVIK_SIZES = {   # width, (heads, dim, rot, vdim, kv rank, q rank, window), (heads, dim, vdim), dense ff, (experts, top, ff), vocab
+    "w2048": (2048, (16, 128, 64, 128, 512, 768, 1024), (8, 256, 512), 8192, (64, 6, 1408), 32000),
+    "w3072": (3072, (24, 96, 32, 96, 384, 1024, 2048), (24, 128, 256), 12288, (32, 4, 1536), 32000),
+    "w4096": (4096, (32, 128, 64, 128, 512, 1536, 4096), (16, 256, 512), 14336, (16, 2, 4096), 32000),
+}
+
+
+def zisevik_config(size):
+    from hologram_b200 import zisevik as zk
+    width, (h, d, r, v, kv, q, window), (rh, rd, rv), ff, (n, top, eff), vocab = ZISEVIK_SIZES[size]
+    latent = lambda: zk.LatentSpec(h, d, r, v, kv, q, (d + r) ** -0.5, window, zk.Rotation(r, 10000.0))
+    keep = lambda: zk.RetentionSpec(rh, rd, rv, [1.0 - 2.0 ** -(5 + 4.0 * i / rh) for i in range(rh)], zk.Rotation(rd, 10000.0))
+    layers = [zk.LayerSpec(0, latent(), zk.DenseSpec(ff)), zk.LayerSpec(1, keep(), zk.RoutedSpec(n, top, eff)), zk.LayerSpec(2, latent(), zk.DenseSpec(ff))]
+    return zk.ZisevikConfig(vocab, width, layers, 1e-6, (1, 3, 2))
+
+
+class DeviceBytes:
+    """A raw device range as something torch can view."""
+
+    def __init__(self, ptr, nbytes):
+        self.__cuda_array_interface__ = {"shape": (nbytes,), "typestr": "|u1", "data": (ptr, False), "version": 3}
+
+
+def call_work(kc, call, pos, words):
+    """(name, algorithmic bytes, FLOPs, key) of one call of a step at position `pos`; `words(ref)` reads an i32 operand."""
+    k, u = call.kind, call.u
+    es = lambda dt: 4 if dt == kc.DTYPE_F32 else 2
+    if k in (kc.K_LINEAR, kc.K_LINEAR_EX):
+        c = u.linear
+        segs = list(c.seg)[:c.nseg]
+        n, m, b, name = sum(g.width for g in segs), c.m, es(c.dtype), f"Linear {c.k} x {sum(g.width for g in segs)}"
+        outs = sum(m * (g.width // 2 if g.act == kc.LINEAR_ACT_SILU_GATE else g.width) * es(g.dtype) for g in segs)
+        res = 4 * m * n if c.residual.slot != kc.NO_SLOT else 0
+        weights = c.k * n
+        if c.tiles.slot != kc.NO_SLOT:
+            t = words(c.tiles)
+            used = t[1:1 + t[0]]
+            m = call_work.pairs
+            outs = outs * m // c.m
+            weights *= len(set(used.tolist()))
+            name = f"grouped Linear {c.k} x {n}, {len(set(used.tolist()))} experts, {m} pairs"
+        elif c.a_pos.slot != kc.NO_SLOT:
+            m = min(c.m, pos + call_work.rows - max(0, pos - c.a_back))
+            outs = outs * m // c.m
+            name += f" over {m} cached rows"
+        kinds = {kc.LINEAR_ACT_RELU2: "relu2", kc.LINEAR_ACT_GELU_TANH: "gelu", kc.LINEAR_ACT_SILU: "silu", kc.LINEAR_ACT_SILU_GATE: "silu gate"}
+        extra = sorted({kinds[g.act] for g in segs if g.act}) + (["rotation"] if any(g.rot_head for g in segs) else []) + (["residual"] if res else [])
+        return name + (" (" + ", ".join(extra) + ")" if extra else ""), weights * b + m * c.k * b + outs + res, 2.0 * m * c.k * n, (k, c.m, c.k, n, c.nseg, tuple(extra))
+    if k == kc.K_RMS_NORM_MULTI:
+        c = u.rms_norm_multi
+        n = 2 if c.gamma1.slot != kc.NO_SLOT else 1
+        return "RmsNormMulti", c.rows * c.feature * (4 + n * es(c.dtype)), 0, (k, c.rows, c.feature, n)
+    if k == kc.K_RMS_NORM_PARTS:
+        c = u.rms_norm_parts
+        w = sum(p.width for p in list(c.part)[:c.nparts])
+        return f"RmsNormParts ({'norm' if c.part[0].norm else 'copy'})", c.rows * w * (4 + es(c.dtype)), 0, (k, c.rows, w)
+    if k == kc.K_ROTARY_TABLE:
+        c = u.rotary_table
+        return "RotaryTable", 8 * c.rows * c.half, 0, (k, c.rows, c.half)
+    if k == kc.K_HEAD_LINEAR:
+        c = u.head_linear
+        return f"HeadLinear {c.heads} x {c.k} x {c.n}", es(c.dtype) * (c.heads * c.k * c.n + c.rows * c.heads * (c.k + c.n)), 2.0 * c.rows * c.heads * c.k * c.n, (k, c.rows, c.heads, c.k, c.n)
+    if k == kc.K_WINDOW_ATTENTION:
+        c = u.window_attention
+        seen = sum(min(pos + i + 1, c.window or 1 << 30) for i in range(c.rows))
+        span = min(pos + c.rows, (c.window + c.rows - 1) if c.window else 1 << 30)
+        values = 0 if c.v.slot == c.k.slot and c.v.offset == c.k.offset else c.vdim
+        nbytes = es(c.dtype) * (c.rows * c.heads * (c.dim + c.dim2 + c.vdim) + span * (c.kv_heads * (c.dim + values) + c.dim2))
+        return f"WindowAttention {c.heads} heads, {c.dim}+{c.dim2} / {c.vdim}, window {c.window}", nbytes, 2.0 * c.heads * (c.dim + c.dim2 + c.vdim) * seen, (k, c.rows, c.heads, c.dim)
+    if k == kc.K_CAUSAL_ATTENTION:
+        c = u.causal_attention
+        seen = sum(pos + i + 1 for i in range(c.rows))
+        nbytes = es(c.dtype) * (c.rows * c.heads * (c.dim + c.vdim) + (pos + c.rows) * c.kv_heads * (c.dim + c.vdim))
+        return f"CausalAttention {c.heads} / {c.kv_heads} heads, {c.dim} / {c.vdim}", nbytes, 2.0 * c.heads * (c.dim + c.vdim) * seen, (k, c.rows, c.heads, c.dim)
+    if k == kc.K_RETENTION:
+        c = u.retention
+        return (f"Retention {c.heads} heads, {c.dim} x {c.vdim}", es(c.dtype) * c.rows * c.heads * (2 * c.dim + 3 * c.vdim) + 8 * c.heads * c.dim * c.vdim,
+                4.0 * c.rows * c.heads * c.dim * c.vdim, (k, c.rows, c.heads, c.dim))
+    if k == kc.K_MOE_PLAN:
+        c = u.moe_plan
+        return "MoePlan", 4 * c.rows * (c.experts + 3 * c.top), 0, (k, c.rows, c.experts)
+    if k == kc.K_MOE_COMBINE:
+        c = u.moe_combine
+        return "MoeCombine", c.rows * c.width * (8 + c.top * es(c.dtype)), 0, (k, c.rows, c.width)
+    if k == kc.K_GATHER:
+        c = u.gather
+        return "Gather", 2 * c.num_indices * c.inner * es(c.dtype), 0, (k, c.num_indices, c.inner)
+    if k == kc.K_CAST:
+        c = u.cast
+        return "Cast", c.element_count * (es(c.src_dtype) + es(c.dst_dtype)), 0, (k, c.element_count)
+    return f"call {k}", 0, 0, (k,)
+
+
+def bench_zisevik(be, torch, args, stream):
+    import hologram_b200 as hb
+    from hologram_b200 import decode, fokonex as fk, kernel_call as kc, safetensors_io as st, zisevik as zk
+    peaks = measured_peaks()
+    rows_prefill, cached = 2048, 4096
+    warm, iters = max(args.warmup, 3), max(args.steps, 20)
+    sizes = [x for x in os.environ.get("HOLO_BENCH_ZISEVIK", ",".join(ZISEVIK_SIZES)).split(",") if x]
+
+    def time_ms(run, n):
+        for i in range(warm):
+            run(i)
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(stream)
+        for i in range(n):
+            run(warm + i)
+        e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    def frac(nbytes, flops, ms, tensor):
+        return max(nbytes / peaks["hbm_gbs"] / 1e6, flops / tensor / 1e9) / ms
+
+    def make(model_class, cfg):
+        g = torch.Generator(device="cuda").manual_seed(0x21)
+        tensors = {}
+        for name, shape in cfg.tensor_shapes().items():
+            t = 1.0 + 0.1 * torch.randn(shape, generator=g, device="cuda") if len(shape) == 1 else torch.randn(shape, generator=g, device="cuda") / shape[-1] ** 0.5
+            tensors[name] = st.Tensor("BF16", t.to(torch.bfloat16).view(torch.int16).cpu().numpy().view(np.uint16))
+        model = model_class(cfg, tensors)
+        return model, decode.StepRunner(be, model, cached + rows_prefill + 64, max_rows=rows_prefill)
+
+    def kernels(model, runner, rows, pos):
+        """Every distinct call of a step alone, over copies of its operands (as the step left them) that exceed L2 together."""
+        writer = model.step_writer(rows, runner.cache.capacity, runner.max_rows, rows == 1)
+        session = runner._steps[rows][0]
+        call_work.rows = rows
+        out, seen = [], set()
+        for call in writer.calls:
+            if call.kind == kc.K_MOE_PLAN:
+                call_work.pairs = rows * call.u.moe_plan.top
+            name, nbytes, flops, key = call_work(kc, call, pos, lambda r: session.workspace.read(kc.rb(r.slot, r.offset, r.length), r.length, np.int32))
+            if key in seen:
+                continue
+            seen.add(key)
+            used = {}
+            for _, ref in call_refs(kc, call):
+                if ref.slot != kc.NO_SLOT and ref.slot not in used:
+                    used[ref.slot] = session.workspace.slot(ref.slot)
+            total = sum(n for _, n in used.values())
+            copies = max(1, min(48, -(-300_000_000 // total)))
+            sets = []
+            for i in range(copies):
+                ws, keep = hb.DeviceWorkspace(be, max(used) + 1), []
+                for slot, (ptr, n) in used.items():
+                    t = torch.as_tensor(DeviceBytes(ptr, n), device="cuda").clone()
+                    ws.bind(slot, t.data_ptr(), n)
+                    keep.append(t)
+                sets.append((ws, keep))
+            torch.cuda.synchronize()
+            ms = time_ms(lambda i: be.dispatch(call, sets[i % copies][0]), iters)
+            t_mem, t_mma = nbytes / peaks["hbm_gbs"] / 1e6, flops / peaks["bf16_tflops"] / 1e9
+            out.append({"kernel": name, "us": round(ms * 1e3, 2), "bound": "hbm" if t_mem >= t_mma else "tensor", "roofline_us": round(max(t_mem, t_mma) * 1e3, 2),
+                        "frac": round(max(t_mem, t_mma) / ms, 3)})
+            del sets
+        return out
+
+    def steps(model, runner, vocab):
+        """Prefill and decode throughput, device-resident and through the public step."""
+        res = {}
+        ids = np.random.default_rng(0).integers(0, vocab, size=rows_prefill).astype(np.int32)
+        for i in range(cached // rows_prefill):
+            runner.step("bench", ids, [])
+        pre = runner._steps[rows_prefill][0]
+        for base in (0, cached):
+            step_in = np.zeros(4 + rows_prefill, np.int32)
+            step_in[0], step_in[1], step_in[4:] = base, rows_prefill, ids
+            pre.write("step_in", step_in)
+            ms = time_ms(lambda i: pre.execute(), 10)
+            res[f"prefill_{rows_prefill}_at_{base}"] = {"ms": round(ms, 3), "tokens_per_s": round(rows_prefill / ms * 1e3)}
+        res["prefill kernels"] = kernels(model, runner, rows_prefill, cached)
+        one = runner._steps[1][0]
+        runner.step("bench", ids[:1])
+        step_in = np.zeros(5, np.int32)
+        step_in[0], step_in[1], step_in[4] = cached, 1, 1
+        one.write("step_in", step_in)
+        ms = time_ms(lambda i: one.execute(), 100)
+        res["decode_at_4096"] = {"ms": round(ms, 4), "tokens_per_s": round(1e3 / ms, 1), "launches": be.launch_count}
+        l0 = be.launch_count
+        one.execute()
+        res["decode_at_4096"]["launches"] = be.launch_count - l0
+        t0 = time.perf_counter()
+        for i in range(50):
+            runner.step("bench", ids[i:i + 1])
+        res["decode_e2e_tokens_per_s"] = round(50 / (time.perf_counter() - t0), 1)
+        res["decode kernels"] = kernels(model, runner, 1, cached)
+        # all of a decoded token's weights and caches once: what the step would take at the copy bandwidth
+        writer = model.step_writer(1, runner.cache.capacity, runner.max_rows, True)
+        call_work.rows, total = 1, 0
+        for call in writer.calls:
+            if call.kind == kc.K_MOE_PLAN:
+                call_work.pairs = call.u.moe_plan.top
+            total += call_work(kc, call, cached, lambda r: one.workspace.read(kc.rb(r.slot, r.offset, r.length), r.length, np.int32))[1]
+        res["decode_at_4096"]["frac"] = round(frac(total, 0, res["decode_at_4096"]["ms"], 1.0), 3)
+        return res
+
+    results = []
+    for size in sizes:
+        cfg = zisevik_config(size)
+        model, runner = make(zk.ZisevikModel, cfg)
+        res = {"size": size, "config": str(ZISEVIK_SIZES[size]), "layer_runs": len(cfg.runs())}
+        res.update(steps(model, runner, cfg.vocab))
+        runner.close()
+        del model, runner
+        fcfg = fokonex_config(size, len(cfg.runs()))
+        model, runner = make(fk.FokonexModel, fcfg)
+        res["fokonex"] = dict(steps(model, runner, fcfg.vocab), config=str(FOKONEX_SIZES[size]))
+        runner.close()
+        del model, runner
+        results.append(res)
+    return results
+
+
+def call_refs(kc, call):
+    """(field, BufferRef) of every operand of a call."""
+    fields = {kc.K_LINEAR: "linear", kc.K_LINEAR_EX: "linear", kc.K_GATHER: "gather", kc.K_CAST: "cast", kc.K_RMS_NORM_MULTI: "rms_norm_multi",
+              kc.K_CAUSAL_ATTENTION: "causal_attention", kc.K_ROTARY_TABLE: "rotary_table", kc.K_RMS_NORM_PARTS: "rms_norm_parts", kc.K_HEAD_LINEAR: "head_linear",
+              kc.K_WINDOW_ATTENTION: "window_attention", kc.K_RETENTION: "retention", kc.K_MOE_PLAN: "moe_plan", kc.K_MOE_COMBINE: "moe_combine"}
+    todo = [getattr(call.u, fields[call.kind])]
+    while todo:
+        x = todo.pop()
+        for name, kind in type(x)._fields_:
+            v = getattr(x, name)
+            if kind is kc.BufferRef:
+                yield name, v
+            elif name in ("seg", "part"):
+                todo += list(v)[:x.nseg if name == "seg" else x.nparts]
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -912,6 +1149,18 @@ def main():
         emit({"metric": "fokonex_decode_tokens_per_s", "value": big["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": 100, "warmup": args.warmup,
               "ms_per_step": big["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 (f32 residual)",
               "data": "synthetic (random weights)", "config": {"model": "Fokonex " + results[-1]["config"], "global_batch": 1, "seq_len": 4096,
+              "l2": "kernels alone rotate over copies that exceed L2; a step's weights exceed L2"}, "gpu_launches": be.launch_count, "clocks": clocks,
+              "peaks": measured_peaks(), "sizes": results})
+        return
+    if args.workload == "zisevik":
+        sampler = ClockSampler(local_rank)
+        sampler.start()
+        results = bench_zisevik(be, torch, args, stream)
+        clocks = sampler.stop()
+        big = results[-1]["decode_at_4096"]
+        emit({"metric": "zisevik_decode_tokens_per_s", "value": big["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": 100, "warmup": args.warmup,
+              "ms_per_step": big["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 (f32 residual and state)",
+              "data": "synthetic (random weights)", "config": {"model": "Zisevik " + results[-1]["config"], "global_batch": 1, "seq_len": 4096,
               "l2": "kernels alone rotate over copies that exceed L2; a step's weights exceed L2"}, "gpu_launches": be.launch_count, "clocks": clocks,
               "peaks": measured_peaks(), "sizes": results})
         return
