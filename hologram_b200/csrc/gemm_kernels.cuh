@@ -100,17 +100,18 @@ __device__ __forceinline__ uint32_t lin_segment(const GemmParams& p, uint32_t co
     while (si + 1 < p.nlin && col >= p.lin[si + 1].col_begin) ++si;
     return si;
 }
-// The A row behind row m0 of the product (m0 a multiple of the tile's rows).
-__device__ __forceinline__ uint32_t lin_a_row(const GemmParams& p, uint32_t m0) {
+// The first row of a product's window of A, and the A row behind row m0 of the product (m0 a multiple of the tile's rows).
+__device__ __forceinline__ uint32_t lin_a_start(const GemmParams& p) {
     const uint32_t pos = *p.a_pos;
-    return (((pos > p.a_back ? pos - p.a_back : 0u) & ~127u) + m0) % p.a_rows;
+    return (pos > p.a_back ? pos - p.a_back : 0u) & ~127u;
 }
+__device__ __forceinline__ uint32_t lin_a_row(const GemmParams& p, uint32_t start, uint32_t m0) { return (start + m0) % p.a_rows; }
 // What a CTA's tile of a Linear product reads and stores, once the dependency wait is over.
 struct LinTile {
     uint32_t a_row, b_row, m_end;   // first A row, first B row, end of the rows to store (m0 when the tile is not in use)
     bool used;
 };
-__device__ __forceinline__ LinTile lin_tile(const GemmParams& p, uint32_t tile, uint32_t m0) {
+__device__ __forceinline__ LinTile lin_tile(const GemmParams& p, uint32_t a_start, uint32_t tile, uint32_t m0) {
     LinTile t = {m0, 0u, p.m, true};
     if (p.tiles) {
         t.used = tile < (uint32_t)p.tiles[0];
@@ -118,7 +119,7 @@ __device__ __forceinline__ LinTile lin_tile(const GemmParams& p, uint32_t tile, 
         if (p.a_shared) t.a_row = 0;
         t.m_end = !t.used ? m0 : m0 + (p.a_shared ? p.a_shared : p.tile_rows);
     } else if (p.a_pos) {
-        t.a_row = lin_a_row(p, m0);
+        t.a_row = lin_a_row(p, a_start, m0);
     }
     return t;
 }
@@ -152,22 +153,46 @@ __device__ __forceinline__ bool lin_out_row(const GemmLin& g, uint32_t row, uint
     *out = r;
     return r < g.row_limit;
 }
-// Turn the pairs of N consecutive columns (N and the first column even) of one row.
+// Turn the pairs of N consecutive columns (N and the first column even) of one row. Every table entry is requested before the
+// first one is used; columns that do not turn read the row's first entry and ignore it.
 template <int N>
 __device__ __forceinline__ void lin_rotate(const GemmParams& p, const GemmLin& g, uint32_t row, uint32_t c, float (&v)[N]) {
     uint32_t cc = c % g.rot_head;
+    const uint32_t end = g.rot_begin + g.rot_dims;
+    if (cc + N <= g.rot_head && (cc >= end || cc + N <= g.rot_begin)) return;      // none of them turns
     const float2* table = p.rot + (uint64_t)row * (g.rot_dims >> 1);
+    if (N % 4 == 0 && cc >= g.rot_begin && cc + N <= end && (((cc - g.rot_begin) | g.rot_dims) & 3u) == 0 && ((uintptr_t)p.rot & 15u) == 0) {   // all of them do
+        const float4* t4 = reinterpret_cast<const float4*>(table + ((cc - g.rot_begin) >> 1));
+        float4 t[N / 4];
 #pragma unroll
-    for (int i = 0; i < N; i += 2) {
-        if (cc >= g.rot_begin && cc < g.rot_begin + g.rot_dims) {
-            const float2 t = table[(cc - g.rot_begin) >> 1];
-            const float a = v[i], b = v[i + 1];
-            v[i] = a * t.x - b * t.y;
-            v[i + 1] = b * t.x + a * t.y;
+        for (int i = 0; i < N / 4; ++i) t[i] = t4[i];
+#pragma unroll
+        for (int i = 0; i < N / 4; ++i) {
+            const float a0 = v[4 * i], b0 = v[4 * i + 1], a1 = v[4 * i + 2], b1 = v[4 * i + 3];
+            v[4 * i] = a0 * t[i].x - b0 * t[i].y;
+            v[4 * i + 1] = b0 * t[i].x + a0 * t[i].y;
+            v[4 * i + 2] = a1 * t[i].z - b1 * t[i].w;
+            v[4 * i + 3] = b1 * t[i].z + a1 * t[i].w;
         }
+        return;
+    }
+    float2 t[N / 2];
+    uint32_t turns = 0;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+        const bool in = cc >= g.rot_begin && cc < end;
+        t[i] = table[in ? (cc - g.rot_begin) >> 1 : 0u];
+        turns |= (in ? 1u : 0u) << i;
         cc += 2;
         if (cc >= g.rot_head) cc -= g.rot_head;
     }
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i)
+        if (turns >> i & 1u) {
+            const float a = v[2 * i], b = v[2 * i + 1];
+            v[2 * i] = a * t[i].x - b * t[i].y;
+            v[2 * i + 1] = b * t[i].x + a * t[i].y;
+        }
 }
 // Store N consecutive finished cells of one row, of which `left` exist.
 template <int N>
@@ -235,8 +260,20 @@ __device__ __forceinline__ void lin_store(const GemmParams& p, uint32_t row, uin
         return;
     }
     float v[N];
+    // one branch for all cells
+    if (act == HOLO_LINEAR_ACT_NONE) {
 #pragma unroll
-    for (int i = 0; i < N; ++i) v[i] = lin_act<true>(acc[i], act);
+        for (int i = 0; i < N; ++i) v[i] = acc[i];
+    } else if (act == HOLO_LINEAR_ACT_RELU2) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lin_act<true>(acc[i], HOLO_LINEAR_ACT_RELU2);
+    } else if (act == HOLO_LINEAR_ACT_GELU_TANH) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lin_act<true>(acc[i], HOLO_LINEAR_ACT_GELU_TANH);
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lin_act<true>(acc[i], HOLO_LINEAR_ACT_SILU);
+    }
     if (g.rot_head) lin_rotate<N>(p, g, row, c, v);
 #pragma unroll
     for (int i = 0; i < N; ++i) v[i] *= alpha;
@@ -438,7 +475,7 @@ matmul_bf16_umma_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
     holo_pdl_wait();  // barriers and TMEM were set up while the previous kernel drained
     uint32_t m_end = p.m, a_row = m0, b_row = 0;
     if (LIN) {
-        const LinTile t = lin_tile(p, blockIdx.y, m0);
+        const LinTile t = lin_tile(p, p.a_pos ? lin_a_start(p) : 0u, blockIdx.y, m0);
         m_end = t.m_end; a_row = t.a_row; b_row = t.b_row;
         if (!t.used) nkb = 0;    // the whole cluster of this tile idles through
     }
@@ -893,6 +930,7 @@ matmul_umma_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const _
         // ---------------- TMA producer ----------------
         if (lane == 0) {
             const uint32_t tx = S::A_BYTES + S::B_BYTES;
+            const uint32_t a_start = LIN && p.a_pos ? lin_a_start(p) : 0u;
             uint32_t it = 0;
             bool ok = true;
             for (uint32_t tile = blockIdx.x; tile < ntiles && ok; tile += gridDim.x) {
@@ -900,7 +938,7 @@ matmul_umma_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const _
                 const int a_k0 = LIN ? (int)p.lin[lin_segment(p, (uint32_t)n0)].k_offset : 0;
                 int a_row = m0, b_row = 0;
                 if (LIN) {
-                    const LinTile t = lin_tile(p, tile / tiles_n, (uint32_t)m0);
+                    const LinTile t = lin_tile(p, a_start, tile / tiles_n, (uint32_t)m0);
                     a_row = (int)t.a_row; b_row = (int)t.b_row;
                 }
                 for (uint32_t kb = 0; kb < p.kblocks; ++kb, ++it) {
@@ -1117,6 +1155,7 @@ matmul_umma_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
     if (warp == 0) {
         // ---------------- TMA producer (both CTAs) ----------------
         if (lane == 0) {
+            const uint32_t a_start = LIN && p.a_pos ? lin_a_start(p) : 0u;
             uint32_t it = 0;
             bool ok = true;
             for (uint32_t w = pair; w < p.n_items && ok; w += npairs) {
@@ -1124,7 +1163,7 @@ matmul_umma_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_
                 // this CTA's halves: rows [128 r, +128) of the A block, columns [bn/2 r, +bn/2) of the B block
                 const int m0 = (int)(item.m_tile * 256 + rank * 128), n0 = (int)(item.n0 + rank * (item.bn >> 1));
                 const int a_k0 = LIN ? (int)p.lin[lin_segment(p, item.n0)].k_offset : 0;
-                const int a_row = LIN && p.a_pos ? (int)lin_a_row(p, (uint32_t)m0) : m0;
+                const int a_row = LIN && p.a_pos ? (int)lin_a_row(p, a_start, (uint32_t)m0) : m0;
                 const uint32_t tx = 2u * (S::A_BYTES + (item.bn >> 1) * BK * 2);
                 for (uint32_t kb = 0; kb < p.kblocks; ++kb, ++it) {
                     const uint32_t s = it % QSTAGES, use = it / QSTAGES;

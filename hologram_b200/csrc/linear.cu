@@ -36,7 +36,7 @@ linear_cell_kernel(const T* __restrict__ a, const T* __restrict__ b, const GemmP
     for (int r = 0; r < CELL_ROWS; ++r) {
         uint32_t ar = row0 + min((uint32_t)r, rows - 1);
         if (p.tiles && p.a_shared) ar %= p.tile_rows;
-        else if (p.a_pos) ar = lin_a_row(p, ar);
+        else if (p.a_pos) ar = lin_a_row(p, lin_a_start(p), ar);
         arow[r] = a + (uint64_t)ar * lda + g.k_offset;
     }
     float acc[CELL_ROWS] = {};
@@ -270,45 +270,66 @@ __global__ void rotary_table_kernel(const uint32_t* __restrict__ pos, const floa
     out[i] = make_float2(c, s);
 }
 
-// One warp per (row, part).
-constexpr int PARTS_WARPS = 4, PARTS_HELD = 16;
-template <typename T>
-__global__ void __launch_bounds__(PARTS_WARPS * 32)
+// One CTA per (row, part). VEC: everything is a multiple of four wide and aligned; up to PARTS_HELD vectors per thread stay in
+// registers between the reduction and the scaling.
+constexpr int PARTS_THREADS = 128, PARTS_HELD = 4;
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(PARTS_THREADS)
 rms_norm_parts_kernel(const HoloNormPartsArgs a) {
+    __shared__ float s_part[PARTS_THREADS / 32];
     holo_pdl_trigger();
-    const uint32_t unit = blockIdx.x * PARTS_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (unit >= a.rows * a.nparts) return;
-    const uint32_t row = unit / a.nparts;
-    const HoloNormPartArgs& p = a.part[unit % a.nparts];
+    const uint32_t row = blockIdx.x, tid = threadIdx.x;
+    const HoloNormPartArgs& p = a.part[blockIdx.y];
+    constexpr int V = VEC ? 4 : 1;
+    const uint32_t nvec = p.width / V;
     holo_pdl_wait();
+    const float* x = a.x + (uint64_t)row * a.ld_in + p.in_col;
+    auto fetch = [&](uint32_t j) {
+        if constexpr (VEC) return reinterpret_cast<const float4*>(x)[j];
+        else return make_float4(x[j], 0.f, 0.f, 0.f);
+    };
+    auto square = [](const float4& v, float acc) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, acc)))); };
+    float4 held[PARTS_HELD];
+#pragma unroll
+    for (int i = 0; i < PARTS_HELD; ++i) {
+        const uint32_t j = tid + PARTS_THREADS * i;
+        held[i] = j < nvec ? fetch(j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     uint64_t orow = row;
     if (p.ring) {
         if (row >= a.step[1]) return;
         orow = (a.step[0] + row) % (uint32_t)p.row_limit;
     }
-    const float* x = a.x + (uint64_t)row * a.ld_in + p.in_col;
-    T* out = (T*)p.out + orow * p.ld;
-    float held[PARTS_HELD], acc = 0.0f;
-#pragma unroll
-    for (int i = 0; i < PARTS_HELD; ++i) {
-        const uint32_t j = lane + 32 * i;
-        held[i] = j < p.width ? x[j] : 0.0f;
-    }
     float inv = 1.0f;
     if (p.norm) {
+        float acc = 0.0f;
 #pragma unroll
-        for (int i = 0; i < PARTS_HELD; ++i) acc = fmaf(held[i], held[i], acc);
-        for (uint32_t j = lane + 32 * PARTS_HELD; j < p.width; j += 32) acc = fmaf(x[j], x[j], acc);
+        for (int i = 0; i < PARTS_HELD; ++i) acc = square(held[i], acc);
+        for (uint32_t j = tid + PARTS_THREADS * PARTS_HELD; j < nvec; j += PARTS_THREADS) acc = square(fetch(j), acc);
         for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if ((tid & 31u) == 0) s_part[tid >> 5] = acc;
+        __syncthreads();
+        acc = 0.0f;
+#pragma unroll
+        for (int w = 0; w < PARTS_THREADS / 32; ++w) acc += s_part[w];
         inv = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(acc, (float)p.width), a.eps)));
     }
+    T* out = (T*)p.out + orow * p.ld;
+    auto put = [&](uint32_t j, const float4& v) {
+        if constexpr (VEC) {
+            const float4 w = p.weight ? reinterpret_cast<const float4*>(p.weight)[j] : make_float4(1.f, 1.f, 1.f, 1.f);
+            store_norm4(out, 4 * j, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
+        } else {
+            store_norm(out, j, v.x * inv * (p.weight ? p.weight[j] : 1.0f));
+        }
+    };
 #pragma unroll
     for (int i = 0; i < PARTS_HELD; ++i) {
-        const uint32_t j = lane + 32 * i;
-        if (j < p.width) store_norm(out, j, held[i] * inv * (p.weight ? p.weight[j] : 1.0f));
+        const uint32_t j = tid + PARTS_THREADS * i;
+        if (j < nvec) put(j, held[i]);
     }
-    for (uint32_t j = lane + 32 * PARTS_HELD; j < p.width; j += 32) store_norm(out, j, x[j] * inv * (p.weight ? p.weight[j] : 1.0f));
-    for (uint32_t j = p.width + lane; j < p.out_width; j += 32) store_norm(out, j, 0.0f);
+    for (uint32_t j = tid + PARTS_THREADS * PARTS_HELD; j < nvec; j += PARTS_THREADS) put(j, fetch(j));
+    for (uint32_t j = p.width + tid; j < p.out_width; j += PARTS_THREADS) store_norm(out, j, 0.0f);
 }
 
 // A CTA takes HEAD_COLS columns of one head for up to R rows; its threads split k and add up through shared memory.
@@ -344,7 +365,7 @@ head_linear_kernel(const HoloHeadLinearArgs a, uint32_t vec) {
     holo_pdl_wait();
     if (left) {
         const bool whole = vec && left >= (uint32_t)N;
-#pragma unroll 4
+#pragma unroll 8
         for (uint32_t k = kg; k < a.k; k += KG) {
             float v[N];
             load_vec<T>(b + (uint64_t)k * a.b_ld, whole, left, v);
@@ -397,12 +418,21 @@ int32_t holo_launch_rotary_table(holo_b200_ctx* ctx, const uint32_t* pos, const 
     return HOLO_OK;
 }
 
-int32_t holo_launch_rms_norm_parts(holo_b200_ctx* ctx, const HoloNormPartsArgs& a) {
-    const uint32_t grid = (a.rows * a.nparts + PARTS_WARPS - 1) / PARTS_WARPS;
-    if (a.dtype == HOLO_DTYPE_F32) HOLO_CUDA(holo_launch_kernel(ctx, rms_norm_parts_kernel<float>, dim3(grid), dim3(PARTS_WARPS * 32), 0, 1, a));
-    else HOLO_CUDA(holo_launch_kernel(ctx, rms_norm_parts_kernel<__nv_bfloat16>, dim3(grid), dim3(PARTS_WARPS * 32), 0, 1, a));
+template <typename T>
+static int32_t launch_norm_parts(holo_b200_ctx* ctx, const HoloNormPartsArgs& a) {
+    bool vec = a.ld_in % 4 == 0 && ((uintptr_t)a.x & 15u) == 0;
+    for (uint32_t i = 0; i < a.nparts; ++i) {
+        const HoloNormPartArgs& p = a.part[i];
+        vec = vec && p.width % 4 == 0 && p.in_col % 4 == 0 && p.ld % 4 == 0 && (((uintptr_t)p.weight & 15u) | ((uintptr_t)p.out & (4 * sizeof(T) - 1))) == 0;
+    }
+    const dim3 grid(a.rows, a.nparts);
+    if (vec) HOLO_CUDA(holo_launch_kernel(ctx, rms_norm_parts_kernel<T, true>, grid, dim3(PARTS_THREADS), 0, 1, a));
+    else HOLO_CUDA(holo_launch_kernel(ctx, rms_norm_parts_kernel<T, false>, grid, dim3(PARTS_THREADS), 0, 1, a));
     ctx->launches++;
     return HOLO_OK;
+}
+int32_t holo_launch_rms_norm_parts(holo_b200_ctx* ctx, const HoloNormPartsArgs& a) {
+    return a.dtype == HOLO_DTYPE_F32 ? launch_norm_parts<float>(ctx, a) : launch_norm_parts<__nv_bfloat16>(ctx, a);
 }
 
 int32_t holo_launch_head_linear(holo_b200_ctx* ctx, const HoloHeadLinearArgs& a) {

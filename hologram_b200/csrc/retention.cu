@@ -30,52 +30,59 @@ __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.w
 // Grid (slices, heads). A thread owns four columns of the slice and every GROUPS-th key dimension; the state is read, advanced
 // and written once.
 constexpr int TOK_THREADS = 256;
-template <typename T>
+template <typename T, int HELD>   // a thread's share of the key dimensions, requested at once
 __global__ void __launch_bounds__(TOK_THREADS)
 retention_token_kernel(const HoloRetentionArgs a, uint32_t width) {
-    extern __shared__ __align__(16) float t_mem[];      // q [dim], k [dim], parts [groups][width], o [width]
+    extern __shared__ __align__(16) float t_mem[];      // parts [groups][width], o [width]
     __shared__ float s_sq[MAX_SLICES], s_part[TOK_THREADS / 32];
     const uint32_t slice = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, vecs = width / 4, groups = TOK_THREADS / vecs;
-    float *s_q = t_mem, *s_k = s_q + a.dim, *s_parts = s_k + a.dim, *s_o = s_parts + groups * width;
+    float *s_parts = t_mem, *s_o = s_parts + groups * width;
+    const uint32_t cv = tid % vecs, group = tid / vecs, e0 = slice * width + cv * 4;
+    float* state = a.state + (uint64_t)h * a.dim * a.vdim + e0;
+    const T *q = (const T*)a.q + (uint64_t)h * a.dim, *k = (const T*)a.k + (uint64_t)h * a.dim;
     holo_pdl_trigger();
     cluster_arrive();       // everyone has started: their shared memory may be written
     holo_pdl_wait();
     cluster_wait();
-    const bool run = a.step[1] != 0, fresh = a.step[0] == 0;     // the same for every thread of the cluster
-    const uint32_t cv = tid % vecs, group = tid / vecs, e0 = slice * width + cv * 4;
-    if (run) {
-        for (uint32_t i = tid; i < a.dim; i += TOK_THREADS) {
-            s_q[i] = (float)((const T*)a.q)[(uint64_t)h * a.dim + i];
-            s_k[i] = (float)((const T*)a.k)[(uint64_t)h * a.dim + i];
-        }
-        __syncthreads();
-        if (group < groups) {
-            const float decay = a.decay[h];
-            float v[4], acc[4] = {};
+    float4 s[HELD];
+    float qk[HELD][2], v[4] = {};
 #pragma unroll
-            for (int i = 0; i < 4; ++i) v[i] = (float)((const T*)a.v)[(uint64_t)h * a.vdim + e0 + i];
-            float* state = a.state + (uint64_t)h * a.dim * a.vdim + e0;
-#pragma unroll 8
-            for (uint32_t d = group; d < a.dim; d += groups) {
-                float4* at = reinterpret_cast<float4*>(state + (uint64_t)d * a.vdim);
-                float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *at;
-                const float k = s_k[d], q = s_q[d];
-                s.x = fmaf(decay, s.x, k * v[0]); s.y = fmaf(decay, s.y, k * v[1]);
-                s.z = fmaf(decay, s.z, k * v[2]); s.w = fmaf(decay, s.w, k * v[3]);
-                *at = s;
-                acc[0] = fmaf(s.x, q, acc[0]); acc[1] = fmaf(s.y, q, acc[1]);
-                acc[2] = fmaf(s.z, q, acc[2]); acc[3] = fmaf(s.w, q, acc[3]);
-            }
-            *reinterpret_cast<float4*>(s_parts + group * width + cv * 4) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+    for (int i = 0; i < HELD; ++i) {
+        const uint32_t d = group + groups * i;
+        const bool mine = group < groups && d < a.dim;
+        s[i] = mine ? *reinterpret_cast<const float4*>(state + (uint64_t)d * a.vdim) : make_float4(0.f, 0.f, 0.f, 0.f);
+        qk[i][0] = mine ? (float)q[d] : 0.0f;
+        qk[i][1] = mine ? (float)k[d] : 0.0f;
+    }
+    if (group < groups)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) v[i] = (float)((const T*)a.v)[(uint64_t)h * a.vdim + e0 + i];
+    float gate = 0.0f;      // of the column this thread finishes (width is at most the CTA's threads)
+    if (tid < width) gate = (float)((const T*)a.gate)[(uint64_t)h * a.vdim + slice * width + tid];
+    const bool run = a.step[1] != 0;     // the same for every thread of the cluster
+    const float decay = a.step[0] == 0 ? 0.0f : a.decay[h];
+    const bool fresh = a.step[0] == 0;
+    if (run) {
+        float acc[4] = {};
+#pragma unroll
+        for (int i = 0; i < HELD; ++i) {
+            const uint32_t d = group + groups * i;
+            if (fresh) s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            s[i].x = fmaf(decay, s[i].x, qk[i][1] * v[0]); s[i].y = fmaf(decay, s[i].y, qk[i][1] * v[1]);
+            s[i].z = fmaf(decay, s[i].z, qk[i][1] * v[2]); s[i].w = fmaf(decay, s[i].w, qk[i][1] * v[3]);
+            if (group < groups && d < a.dim) *reinterpret_cast<float4*>(state + (uint64_t)d * a.vdim) = s[i];
+            acc[0] = fmaf(s[i].x, qk[i][0], acc[0]); acc[1] = fmaf(s[i].y, qk[i][0], acc[1]);
+            acc[2] = fmaf(s[i].z, qk[i][0], acc[2]); acc[3] = fmaf(s[i].w, qk[i][0], acc[3]);
         }
+        if (group < groups) *reinterpret_cast<float4*>(s_parts + group * width + cv * 4) = make_float4(acc[0], acc[1], acc[2], acc[3]);
         __syncthreads();
         float sq = 0.0f;
-        for (uint32_t c = tid; c < width; c += TOK_THREADS) {
+        if (tid < width) {
             float o = 0.0f;
-            for (uint32_t g = 0; g < groups; ++g) o += s_parts[g * width + c];
+            for (uint32_t g = 0; g < groups; ++g) o += s_parts[g * width + tid];
             o *= a.scale;
-            s_o[c] = o;
-            if (slice * width + c < a.vmean) sq = fmaf(o, o, sq);
+            s_o[tid] = o;
+            if (slice * width + tid < a.vmean) sq = o * o;
         }
         for (int o = 16; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
         if ((tid & 31u) == 0) s_part[tid >> 5] = sq;
@@ -90,28 +97,35 @@ retention_token_kernel(const HoloRetentionArgs a, uint32_t width) {
     __syncwarp();
     cluster_arrive();
     cluster_wait();
-    if (!run) return;
+    if (!run || tid >= width) return;
     float total = 0.0f;
     for (uint32_t i = 0; i < gridDim.x; ++i) total += s_sq[i];
     const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
-    for (uint32_t c = tid; c < width; c += TOK_THREADS) {
-        const uint64_t e = (uint64_t)h * a.vdim + slice * width + c;
-        store_out((T*)a.out, e, s_o[c] * inv * (float)((const T*)a.gate)[e]);
-    }
+    store_out((T*)a.out, (uint64_t)h * a.vdim + slice * width + tid, s_o[tid] * inv * gate);
 }
 
+template <typename T, int HELD>
+int32_t launch_token_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a, uint32_t slices, uint32_t width) {
+    const size_t smem = ((TOK_THREADS / (width / 4)) * width + width) * sizeof(float);    // at most 5 KiB
+    HOLO_CUDA(holo_launch_kernel_cluster(ctx, retention_token_kernel<T, HELD>, dim3(slices, a.heads), dim3(TOK_THREADS), smem, slices, 1u, a, width));
+    ctx->launches++;
+    return HOLO_OK;
+}
+// Launches the one-row kernel, or returns with *taken false when the shape does not suit it.
 template <typename T>
-int32_t launch_token(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
+int32_t try_token(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
     *taken = false;
     uint32_t slices = MAX_SLICES;
     while (slices > 1 && (a.vdim % (4 * slices) != 0 || a.vdim / slices < 16)) slices /= 2;
     const uint32_t width = a.vdim / slices;
-    if (a.dim % 4 || a.vdim % 4 || width > 4 * TOK_THREADS) return HOLO_OK;
-    const size_t smem = (2 * a.dim + (TOK_THREADS / (width / 4)) * width + width) * sizeof(float);    // at most 16 KiB
-    HOLO_CUDA(holo_launch_kernel_cluster(ctx, retention_token_kernel<T>, dim3(slices, a.heads), dim3(TOK_THREADS), smem, slices, 1u, a, width));
-    ctx->launches++;
+    if (a.vdim % 4 || width > TOK_THREADS) return HOLO_OK;
+    const uint32_t groups = TOK_THREADS / (width / 4), share = (a.dim + groups - 1) / groups;
+    if (share > 32) return HOLO_OK;
     *taken = true;
-    return HOLO_OK;
+    if (share <= 4) return launch_token_as<T, 4>(ctx, a, slices, width);
+    if (share <= 8) return launch_token_as<T, 8>(ctx, a, slices, width);
+    if (share <= 16) return launch_token_as<T, 16>(ctx, a, slices, width);
+    return launch_token_as<T, 32>(ctx, a, slices, width);
 }
 
 // ---- several rows -----------------------------------------------------------------------------------------------------------
@@ -519,7 +533,7 @@ int32_t launch_sequence(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
 int32_t holo_launch_retention(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
     if (!getenv("HOLO_RETENTION_GENERAL")) {
         bool taken = false;
-        if (a.rows == 1) HOLO_TRY(a.dtype == HOLO_DTYPE_F32 ? launch_token<float>(ctx, a, &taken) : launch_token<__nv_bfloat16>(ctx, a, &taken));
+        if (a.rows == 1) HOLO_TRY(a.dtype == HOLO_DTYPE_F32 ? try_token<float>(ctx, a, &taken) : try_token<__nv_bfloat16>(ctx, a, &taken));
         else HOLO_TRY(try_chunk(ctx, a, &taken));
         if (taken) return HOLO_OK;
     }

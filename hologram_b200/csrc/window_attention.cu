@@ -320,29 +320,49 @@ latent_attention_kernel(const LatentParams p) {
     }
 }
 
-// One CTA per (pair, 128 value columns).
+// One CTA per (pair, 128 value columns). At most MERGE_SPLITS shares.
+constexpr uint32_t MERGE_SPLITS = 256;
 template <int KT>
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const LatentParams p) {
+    __shared__ float s_factor[MERGE_SPLITS], s_red[8];
     const HoloWindowArgs& a = p.a;
-    const uint32_t pair = blockIdx.x, tile = pair >> 4, row = pair / a.heads, head = pair % a.heads, c = blockIdx.y * 128 + threadIdx.x;
+    const uint32_t pair = blockIdx.x, tile = pair >> 4, row = pair / a.heads, head = pair % a.heads, tid = threadIdx.x, c = blockIdx.y * 128 + tid;
     holo_pdl_trigger();
     holo_pdl_wait();
     const LatentRange range = latent_range(a, tile, *a.pos);
     const uint32_t used = min(p.splits, (range.hi - range.lo + KT) / KT), ml = a.vdim + 2;
-    if (used < 2 || c >= a.vdim) return;
+    if (used < 2) return;
     const float* part = p.partials + (uint64_t)tile * p.splits * 16 * ml + (pair & 15u) * ml;
     const float sink = a.sink ? a.sink[head] * LOG2E : -INFINITY;
+    float2 mine[MERGE_SPLITS / 128];
     float top = sink;
-    for (uint32_t i = 0; i < used; ++i) top = fmaxf(top, part[(uint64_t)i * 16 * ml + a.vdim]);
-    float denom = exp2f(sink - top), acc = 0.0f;
-#pragma unroll 8
-    for (uint32_t i = 0; i < used; ++i) {
-        const float* share = part + (uint64_t)i * 16 * ml;
-        const float f = exp2f(share[a.vdim] - top);
-        denom = fmaf(share[a.vdim + 1], f, denom);
-        acc = fmaf(share[c], f, acc);
+#pragma unroll
+    for (uint32_t i = 0; i < MERGE_SPLITS / 128; ++i) {
+        const uint32_t share = tid + 128 * i;
+        mine[i] = share < used ? *reinterpret_cast<const float2*>(part + (uint64_t)share * 16 * ml + a.vdim) : make_float2(-INFINITY, 0.0f);
+        top = fmaxf(top, mine[i].x);
     }
+    for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+    if ((tid & 31u) == 0) s_red[tid >> 5] = top;
+    __syncthreads();
+    top = fmaxf(fmaxf(s_red[0], s_red[1]), fmaxf(s_red[2], s_red[3]));
+    float denom = 0.0f;
+#pragma unroll
+    for (uint32_t i = 0; i < MERGE_SPLITS / 128; ++i) {
+        const uint32_t share = tid + 128 * i;
+        const float f = exp2f(mine[i].x - top);
+        if (share < used) s_factor[share] = f;
+        denom = fmaf(mine[i].y, f, denom);
+    }
+    for (int o = 16; o > 0; o >>= 1) denom += __shfl_xor_sync(0xffffffffu, denom, o);
+    if ((tid & 31u) == 0) s_red[4 + (tid >> 5)] = denom;
+    __syncthreads();
+    if (c >= a.vdim) return;
+    denom = (s_red[4] + s_red[5]) + (s_red[6] + s_red[7]) + exp2f(sink - top);
+    float acc = 0.0f;
+#pragma unroll 16
+    for (uint32_t i = 0; i < used; ++i) acc = fmaf(part[(uint64_t)i * 16 * ml + c], s_factor[i], acc);
     ((__nv_bfloat16*)a.out)[(uint64_t)row * a.ld + (uint64_t)head * a.vdim + c] = __float2bfloat16_rn(acc / denom);
 }
 
@@ -359,6 +379,7 @@ int32_t launch_latent(holo_b200_ctx* ctx, LatentParams p, uint32_t pair_tiles) {
     uint64_t splits = std::max<uint64_t>(1, (uint64_t)ctx->sm_count / pair_tiles);
     splits = std::min<uint64_t>(splits, (keys + KT - 1) / KT);
     splits = std::min<uint64_t>(splits, LAT_PARTIAL_FLOATS / ((uint64_t)pair_tiles * 16 * (a.vdim + 2)));
+    splits = std::min<uint64_t>(splits, MERGE_SPLITS);
     p.splits = (uint32_t)std::max<uint64_t>(splits, 1);
     HOLO_CUDA(holo_launch_kernel(ctx, latent_attention_kernel<KT, UW>, dim3(p.splits, pair_tiles), dim3(LAT_WARPS * 32), LatentSmem<KT>(a.dim + a.dim2).total, 1, p));
     ctx->launches++;
@@ -392,7 +413,10 @@ int32_t try_latent(holo_b200_ctx* ctx, const HoloWindowArgs& a, bool* taken) {
     if (!ctx->latent_partials) HOLO_CUDA(cudaMalloc(&ctx->latent_partials, (size_t)LAT_PARTIAL_FLOATS * 4));
     p.partials = ctx->latent_partials;
     *taken = true;
-    return wide ? launch_latent_kt<64>(ctx, p, (uint32_t)pair_tiles) : launch_latent_kt<32>(ctx, p, (uint32_t)pair_tiles);
+    // tiles of 32 keys where those of 64 would not reach every SM
+    const uint64_t keys = a.window ? std::min<uint64_t>(a.window, a.kv_rows) : a.kv_rows;
+    return wide && pair_tiles * ((keys + 63) / 64) > (uint64_t)ctx->sm_count / 2 ? launch_latent_kt<64>(ctx, p, (uint32_t)pair_tiles)
+                                                                                : launch_latent_kt<32>(ctx, p, (uint32_t)pair_tiles);
 }
 
 // ---- many rows: 128-row tiles on tcgen05 ------------------------------------------------------------------------------
