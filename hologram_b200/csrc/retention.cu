@@ -1,12 +1,13 @@
 // Retention (linear attention with one fixed decay per head): S = decay S + k v^T, o = scale S^T q, every head's o divided by its
 // root mean square and multiplied by the gate. The state is f32 and stays in place between steps.
 //
-//   retention_chunk_kernel      bf16, several rows: chunks of 128 tokens on mma.sync, the state in registers from the first
-//                               chunk to the last
+//   retention_tile_kernel       bf16, many rows, heads of 128 or 256 key dimensions: chunks of 128 tokens on tcgen05, the state
+//                               in tensor memory from the first chunk to the last
+//   retention_chunk_kernel      bf16, several rows, other heads: the same chunks on mma.sync, the state in registers
 //   retention_token_kernel      one row
 //   retention_sequence_kernel   everything else: token by token, one CTA per head
 //
-// In the first two a cluster of CTAs shares a head, each with a slice of the value columns; they exchange the sums of squares.
+// In all but the last a cluster of CTAs shares a head, each with a slice of the value columns; they exchange the sums of squares.
 #include "attention_tile.cuh"
 
 #include <algorithm>
@@ -450,6 +451,446 @@ int32_t try_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
     return HOLO_OK;
 }
 
+// ---- many rows, heads of 128 or 256 key dimensions: tcgen05 ------------------------------------------------------------------
+// The same chunks of 128 tokens and the same sums, a slice of 64 value columns per CTA; all four products run on tcgen05 with
+// their f32 results in TMEM, where the state stays from the first chunk to the last.
+//   warp 0      TMA producer: q and k tiles (a ring of one or two chunks), v tiles
+//   warp 1      MMA issuer. Per chunk: scores = Q K^T; O1 = Q S (S as two bf16 parts in shared memory, 128 key dimensions at a
+//               time); S += K^T V' (V' the decayed values as two bf16 parts); O2 = P V (P the decayed scores as two bf16 parts in TMEM)
+//   warps 2-5   one thread per token: scores -> P over them; then o = scale (p(i + 1) O1 + O2), its sum of squares to every CTA of
+//               the head (distributed shared memory), and the normed, gated row
+//   warps 6-9   one thread per key dimension: S -> shared memory and p(L) S -> TMEM; and one thread per token: V -> V'
+// TMEM columns: scores 0 and 128 (by turns), O1 256, O2 320, S 384 (+ 64 for the upper 128 key dimensions). It is allocated
+// after the dependency wait, dependents are released after that. Every wait is bounded; the cluster barriers at the two ends
+// are reached after bounded waits only.
+constexpr int RT_THREADS = 320, RT_W = 64;
+
+struct RetentionTileParams {
+    HoloRetentionArgs a;
+    uint32_t* status;
+};
+
+// Like mbar_wait, for a barrier that other CTAs of the cluster arrive on after writing this CTA's shared memory.
+__device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity, volatile uint32_t* abort_flag, uint32_t* status) {
+    for (uint32_t it = 0; it < WAIT_LIMIT; ++it) {
+        uint32_t ok;
+        asm volatile(
+            "{\n.reg .pred p;\nmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}\n"
+            : "=r"(ok)
+            : "r"(bar), "r"(parity)
+            : "memory");
+        if (ok) return true;
+        if (*abort_flag) return false;
+        if (it > 64) __nanosleep(64);
+    }
+    *abort_flag = 1;
+    atomicOr(status, 4u);
+    return false;
+}
+__device__ __forceinline__ void mbar_arrive(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
+__device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
+
+template <int DT>   // dim = 128 DT
+__global__ void __launch_bounds__(RT_THREADS, 1)
+retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+                      const RetentionTileParams p) {
+    constexpr uint32_t NS = DT == 1 ? 2 : 1, QK = 2 * DT * TILE_CHUNK, STAGE = 2 * QK;      // q and k tiles of a chunk
+    constexpr uint32_t OFF_V = NS * STAGE, OFF_VBIG = OFF_V + TILE_CHUNK, OFF_VSMALL = OFF_VBIG + TILE_CHUNK, OFF_SBIG = OFF_VSMALL + TILE_CHUNK,
+                       OFF_SSMALL = OFF_SBIG + TILE_CHUNK, OFF_POWER = OFF_SSMALL + TILE_CHUNK, OFF_SUMS = OFF_POWER + 1024, OFF_BARS = OFF_SUMS + 2 * MAX_SLICES * 128 * 4;
+    extern __shared__ uint8_t smem_raw[];
+    const HoloRetentionArgs& a = p.a;
+    const uint32_t raw = smem_u32(smem_raw);
+    const uint32_t base = (raw + 1023u) & ~1023u;
+    uint8_t* sm = smem_raw + (base - raw);
+    const uint32_t bars = base + OFF_BARS, bar_qk_full = bars, bar_qk_empty = bars + 16, bar_sc = bars + 32, bar_sums = bars + 48, bar_sbuf = bars + 64, bar_m2 = bars + 80,
+                   bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_p = bars + 112, bar_ready = bars + 120, bar_o = bars + 128, bar_oread = bars + 136, bar_s4 = bars + 144;
+    uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + OFF_BARS + 160);
+    volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + OFF_BARS + 164);
+    float* s_power = reinterpret_cast<float*>(sm + OFF_POWER);      // [127 + n] = decay^n, 0 for n < 0
+    float* s_sums = reinterpret_cast<float*>(sm + OFF_SUMS);
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, slice = blockIdx.x, slices = gridDim.x, h = blockIdx.y;
+    if (tid == 0) {
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(bar_qk_full + 8 * i, 1);
+            mbar_init(bar_qk_empty + 8 * i, 1);
+            mbar_init(bar_sc + 8 * i, 1);
+            mbar_init(bar_sums + 8 * i, 4 * slices);   // the token warps of every slice
+            mbar_init(bar_sbuf + 8 * i, 4);
+            mbar_init(bar_m2 + 8 * i, 1);
+        }
+        mbar_init(bar_v_full, 1);
+        mbar_init(bar_v_empty, 5);                     // the product that read v, and the four warps that decayed it
+        mbar_init(bar_p, 4);
+        mbar_init(bar_ready, 4);
+        mbar_init(bar_o, 1);
+        mbar_init(bar_oread, 4);
+        mbar_init(bar_s4, 1);
+        *s_abort = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    holo_pdl_wait();
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(s_tmem)), "r"(512u) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    const float decay = a.decay[h];
+    if (tid < 256) s_power[tid] = tid < 127 ? 0.0f : tid == 127 ? 1.0f : powf(decay, (float)(tid - 127));
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    cluster_arrive();       // every CTA's barriers are set up before anyone arrives on them
+    cluster_wait();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    holo_pdl_trigger();
+    const uint32_t tmem = *s_tmem, tmem_o1 = tmem + 256, tmem_o2 = tmem + 320, tmem_s = tmem + 384;
+    const uint32_t count = min(a.rows, a.step[1]), chunks = (count + 127) / 128;
+
+    if (warp == 0) {
+        // ---------------- TMA producer ----------------
+        if (lane == 0) {
+            uint32_t issued = 0, vissued = 0;
+            for (uint32_t c = 0; c < chunks; ++c) {
+                const uint32_t s = c % NS, st = base + s * STAGE;
+                if (c >= NS && !mbar_wait(bar_qk_empty + 8 * s, (c / NS - 1) & 1, s_abort, p.status)) break;
+                mbar_arrive_expect_tx(bar_qk_full + 8 * s, STAGE);
+                for (uint32_t x = 0; x < 2 * DT; ++x) {
+                    tma_load_2d(st + x * TILE_CHUNK, &map_q, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_qk_full + 8 * s);
+                    tma_load_2d(st + QK + x * TILE_CHUNK, &map_k, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_qk_full + 8 * s);
+                }
+                ++issued;
+                if (c > 0 && !mbar_wait(bar_v_empty, (c - 1) & 1, s_abort, p.status)) break;
+                mbar_arrive_expect_tx(bar_v_full, TILE_CHUNK);
+                tma_load_2d(base + OFF_V, &map_v, (int)(h * a.vdim + slice * RT_W), (int)(c * 128), bar_v_full);
+                ++vissued;
+            }
+            // nothing may still be on its way into this CTA's shared memory when it ends
+            for (uint32_t c = issued > NS ? issued - NS : 0; c < issued; ++c)
+                for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_qk_full + 8 * (c % NS), (c / NS) & 1); ++it) __nanosleep(64);
+            for (uint32_t it = 0; vissued && it < WAIT_LIMIT && !mbar_try_wait(bar_v_full, (vissued - 1) & 1); ++it) __nanosleep(64);
+        }
+    } else if (warp == 1) {
+        // ---------------- MMA issuer ----------------
+        if (lane == 0) {
+            // D = f32, A = B = bf16, M = 128; scores: both operands K-major, N = 128; the others: B N-major, N = 64; the state's A is K^T (M-major)
+            constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 4) << 24);
+            constexpr uint32_t idesc_sc = idesc | ((128u >> 3) << 17), idesc_n = idesc | (1u << 16) | ((64u >> 3) << 17), idesc_st = idesc_n | (1u << 15);
+            const uint64_t d_v = smem_desc(base + OFF_V, TILE_CHUNK, 1024), d_vb = smem_desc(base + OFF_VBIG, TILE_CHUNK, 1024), d_sb = smem_desc(base + OFF_SBIG, TILE_CHUNK, 1024);
+            constexpr uint64_t PART = TILE_CHUNK >> 4;       // from a big part to its small one
+            bool ok = true;
+            for (uint32_t c = 0; c < chunks && ok; ++c) {
+                const uint32_t s = c % NS, st = base + s * STAGE, sc = tmem + (c & 1u) * 128;
+                const uint64_t d_q = smem_desc(st, 16, 1024), d_k = smem_desc(st + QK, 16, 1024), d_kt = smem_desc(st + QK, TILE_CHUNK, 1024);
+                // O1 of 128 key dimensions
+                auto inter = [&](uint32_t half) {
+#pragma unroll
+                    for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                        for (uint32_t k = 0; k < 8; ++k)
+                            umma_bf16(tmem_o1, d_q + (2 * half + (k >> 2)) * PART + 2 * (k & 3), d_sb + part * PART + 128 * k, idesc_n, (half | part | k) != 0);
+                    umma_commit(bar_m2 + 8 * half);
+                };
+                if (!(ok = mbar_wait(bar_qk_full + 8 * s, (c / NS) & 1, s_abort, p.status))) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(sc, d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
+                umma_commit(bar_sc + 8 * (c & 1u));
+                ok = (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status)) && mbar_wait(bar_ready, c & 1, s_abort, p.status);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                inter(0);
+#pragma unroll
+                for (uint32_t half = 0; half < DT; ++half)
+#pragma unroll
+                    for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                        for (uint32_t k = 0; k < 8; ++k) umma_bf16(tmem_s + 64 * half, d_kt + 2 * half * PART + 128 * k, d_vb + part * PART + 128 * k, idesc_st, 1u);
+                umma_commit(bar_s4);
+                if (DT == 2) {
+                    if (!(ok = mbar_wait(bar_sbuf + 8, c & 1, s_abort, p.status))) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    inter(1);
+                }
+                ok = mbar_wait(bar_v_full, c & 1, s_abort, p.status) && mbar_wait(bar_p, c & 1, s_abort, p.status);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+                for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                    for (uint32_t k = 0; k < 8; ++k)
+                        umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
+                umma_commit(bar_o);
+                umma_commit(bar_v_empty);
+                umma_commit(bar_qk_empty + 8 * s);
+            }
+        }
+    } else if (warp < 6) {
+        // ---------------- tokens (TMEM lane quarter = warp % 4) ----------------
+        const uint32_t quarter = warp & 3u, i = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
+        const float* power = s_power + 127;
+        bool ok = true;
+        for (uint32_t c = 0; c < chunks; ++c) {
+            const uint32_t row = c * 128 + i, sc = tmem + (c & 1u) * 128 + lanes;
+            ok = mbar_wait(bar_sc + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
+            ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+            for (uint32_t b2 = 0; b2 < 2; ++b2) {
+                uint32_t v[2][32];
+                const bool some = 64 * b2 < quarter * 32 + 32;      // else no token of this warp sees any of these
+                if (some) {
+                    tmem_ld32_request(sc + 64 * b2, v[0]);
+                    tmem_ld32_request(sc + 64 * b2 + 32, v[1]);
+                    tmem_ld32_wait(v[0]);
+                    tmem_ld32_pass(v[1]);
+                }
+#pragma unroll
+                for (uint32_t b = 0; b < 2; ++b) {
+                    uint32_t big[16], small[16];
+#pragma unroll
+                    for (uint32_t e = 0; e < 16; ++e) {
+                        big[e] = small[e] = 0;
+                        if (some) {
+                            const float* w = power + (int)i - (int)(64 * b2 + 32 * b + 2 * e);
+                            split_bf16(__uint_as_float(v[b][2 * e]) * w[0], __uint_as_float(v[b][2 * e + 1]) * w[-1], big[e], small[e]);
+                        }
+                    }
+                    tmem_st16(sc + 64 * b2 + 32 * b, big);          // over scores this warp has already read
+                    tmem_st16(sc + 64 * b2 + 32 * b + 16, small);
+                }
+            }
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_p);
+            uint4 gate[8];
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+                gate[x] = row < count ? reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim + slice * RT_W)[x]
+                                      : make_uint4(0, 0, 0, 0);
+            ok = mbar_wait(bar_o, c & 1, s_abort, p.status) && !*s_abort;
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            float o[2][32], sq = 0.0f;
+            const float f = a.scale * power[i + 1];
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                uint32_t v0[32], v1[32];
+                tmem_ld32_request(tmem_o1 + lanes + 32 * x, v0);
+                tmem_ld32_request(tmem_o2 + lanes + 32 * x, v1);
+                tmem_ld32_wait(v0);
+                tmem_ld32_pass(v1);
+#pragma unroll
+                for (int e = 0; e < 32; ++e) {
+                    o[x][e] = fmaf(f, __uint_as_float(v0[e]), a.scale * __uint_as_float(v1[e]));
+                    if (slice * RT_W + 32 * x + e < a.vmean) sq = fmaf(o[x][e], o[x][e], sq);
+                }
+            }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            // this row's sum of squares, to every CTA of the head
+            const uint32_t at = base + OFF_SUMS + (((c & 1u) * MAX_SLICES + slice) * 128 + i) * 4;
+            for (uint32_t to = 0; to < slices; ++to) store_remote(at, to, sq);
+            asm volatile("fence.acq_rel.cluster;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_oread);
+            if (lane < slices) {
+                uint32_t remote;
+                asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(bar_sums + 8 * (c & 1u)), "r"(lane));
+                asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(remote) : "memory");
+            }
+            __syncwarp();
+            ok = mbar_wait_cluster(bar_sums + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort && !(*reinterpret_cast<volatile uint32_t*>(p.status) & 4u);
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
+            float total = 0.0f;
+            for (uint32_t x = 0; x < slices; ++x) total += s_sums[((c & 1u) * MAX_SLICES + x) * 128 + i];
+            const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
+            if (row < count) {
+                uint4* out = reinterpret_cast<uint4*>((__nv_bfloat16*)a.out + (uint64_t)row * a.ld + (uint64_t)h * a.vdim + slice * RT_W);
+#pragma unroll
+                for (int x = 0; x < 8; ++x) {
+                    const uint32_t g[4] = {gate[x].x, gate[x].y, gate[x].z, gate[x].w};
+                    uint32_t w[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162*>(&g[e]);
+                        const float* oo = &o[x >> 2][8 * (x & 3) + 2 * e];
+                        w[e] = pack_bf16(oo[0] * inv * __low2float(gg), oo[1] * inv * __high2float(gg));
+                    }
+                    out[x] = make_uint4(w[0], w[1], w[2], w[3]);
+                }
+            }
+        }
+    } else {
+        // ---------------- state and values (TMEM lane quarter = warp % 4) ----------------
+        const uint32_t quarter = warp & 3u, r = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
+        const float* power = s_power + 127;
+        const bool fresh = a.step[0] == 0;
+        float* home = a.state + ((uint64_t)h * a.dim + r) * a.vdim + slice * RT_W;      // key dimension r; the upper 128 follow 128 rows later
+        if (chunks != 0) {
+#pragma unroll
+            for (int half = 0; half < DT; ++half)
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                    uint32_t v[16];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float4 f = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : reinterpret_cast<const float4*>(home + (uint64_t)half * 128 * a.vdim)[4 * x + e];
+                        v[4 * e] = __float_as_uint(f.x); v[4 * e + 1] = __float_as_uint(f.y); v[4 * e + 2] = __float_as_uint(f.z); v[4 * e + 3] = __float_as_uint(f.w);
+                    }
+                    tmem_st16(tmem_s + 64 * half + lanes + 16 * x, v);
+                }
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+        }
+        // a row of S as two bf16 parts, 16-byte units swizzled as the matrix descriptor says
+        auto stage_state = [&](const uint32_t (&v)[2][32]) {
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                uint32_t big[4], small[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    split_bf16(__uint_as_float(v[u >> 2][8 * (u & 3) + 2 * e]), __uint_as_float(v[u >> 2][8 * (u & 3) + 2 * e + 1]), big[e], small[e]);
+                const uint32_t at = r * 128 + (((uint32_t)u ^ (r & 7u)) << 4);
+                *reinterpret_cast<uint4*>(sm + OFF_SBIG + at) = make_uint4(big[0], big[1], big[2], big[3]);
+                *reinterpret_cast<uint4*>(sm + OFF_SSMALL + at) = make_uint4(small[0], small[1], small[2], small[3]);
+            }
+        };
+        auto load_state = [&](int half, uint32_t (&v)[2][32]) {
+            tmem_ld32_request(tmem_s + 64 * half + lanes, v[0]);
+            tmem_ld32_request(tmem_s + 64 * half + lanes + 32, v[1]);
+            tmem_ld32_wait(v[0]);
+            tmem_ld32_pass(v[1]);
+        };
+        auto keep_state = [&](int half, const uint32_t (&v)[2][32], float keep) {
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                uint32_t w[16];
+#pragma unroll
+                for (int e = 0; e < 16; ++e) w[e] = __float_as_uint(__uint_as_float(v[x >> 1][16 * (x & 1) + e]) * keep);
+                tmem_st16(tmem_s + 64 * half + lanes + 16 * x, w);
+            }
+        };
+        bool ok = true;
+        for (uint32_t c = 0; c < chunks; ++c) {
+            const uint32_t tokens = min(128u, count - c * 128);
+            const float keep = power[tokens], f = r < tokens ? power[tokens - 1 - r] : 0.0f;
+            // the last chunk's products have read V' and written S, and (for the first half) read S's parts
+            ok = (c == 0 || (mbar_wait(bar_s4, (c - 1) & 1, s_abort, p.status) && mbar_wait(bar_m2 + 8 * (DT - 1), (c - 1) & 1, s_abort, p.status))) &&
+                 mbar_wait(bar_v_full, c & 1, s_abort, p.status) && !*s_abort;
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            uint32_t v[2][32];
+            load_state(0, v);
+            stage_state(v);
+            keep_state(0, v, keep);
+            if (DT == 2) {
+                load_state(1, v);
+                keep_state(1, v, keep);
+            }
+            // one token's values, the same places in both parts (units taken in another order by every lane: no bank is asked twice)
+#pragma unroll
+            for (uint32_t u0 = 0; u0 < 8; ++u0) {
+                const uint32_t at = r * 128 + (((u0 + lane) & 7u) << 4);
+                const uint4 x = *reinterpret_cast<const uint4*>(sm + OFF_V + at);
+                const uint32_t in[4] = {x.x, x.y, x.z, x.w};
+                uint32_t big[4], small[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const __nv_bfloat162 y = *reinterpret_cast<const __nv_bfloat162*>(&in[e]);
+                    split_bf16(__low2float(y) * f, __high2float(y) * f, big[e], small[e]);
+                }
+                *reinterpret_cast<uint4*>(sm + OFF_VBIG + at) = make_uint4(big[0], big[1], big[2], big[3]);
+                *reinterpret_cast<uint4*>(sm + OFF_VSMALL + at) = make_uint4(small[0], small[1], small[2], small[3]);
+            }
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            fence_async_smem();
+            __syncwarp();
+            if (lane == 0) {
+                mbar_arrive(bar_v_empty);
+                mbar_arrive(bar_ready);
+            }
+            if (DT == 2) {
+                ok = mbar_wait(bar_m2, c & 1, s_abort, p.status);
+                ok = __all_sync(0xffffffffu, ok);
+                if (!ok) break;
+                stage_state(v);
+                fence_async_smem();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(bar_sbuf + 8);
+            }
+        }
+        ok = ok && (chunks == 0 || mbar_wait(bar_s4, (chunks - 1) & 1, s_abort, p.status));
+        ok = __all_sync(0xffffffffu, ok) && chunks != 0;
+        if (ok) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+            for (int half = 0; half < DT; ++half) {
+                uint32_t v[2][32];
+                load_state(half, v);
+                float4* to = reinterpret_cast<float4*>(home + (uint64_t)half * 128 * a.vdim);
+#pragma unroll
+                for (int x = 0; x < 16; ++x)
+                    to[x] = make_float4(__uint_as_float(v[x >> 3][4 * (x & 7)]), __uint_as_float(v[x >> 3][4 * (x & 7) + 1]), __uint_as_float(v[x >> 3][4 * (x & 7) + 2]),
+                                        __uint_as_float(v[x >> 3][4 * (x & 7) + 3]));
+            }
+        }
+    }
+    // everyone meets here, whatever happened above: TMEM is released, and no CTA leaves while another may still write its sums
+    __syncwarp();
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    cluster_arrive();
+    cluster_wait();
+    if (warp == 1) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
+    }
+}
+
+int32_t make_map_rows(CUtensorMap* map, const void* ptr, uint64_t cols, uint64_t rows, uint64_t ld) {
+    cuuint64_t dims[2] = {cols, rows};
+    cuuint64_t strides[1] = {ld * 2};
+    cuuint32_t box[2] = {64, 128};
+    cuuint32_t es[2] = {1, 1};
+    const CUresult r = encode_tiled_fn()(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS ? HOLO_OK : holo_fail(HOLO_ERR_DISPATCH, "dispatch failed: cuTensorMapEncodeTiled (retention) returned %d", (int)r);
+}
+
+template <int DT>
+int32_t launch_tile_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
+    constexpr uint32_t smem = (DT == 1 ? 2 : 1) * 4 * DT * TILE_CHUNK + 5 * TILE_CHUNK + 1024 + 2 * MAX_SLICES * 128 * 4 + 256 + 1024;
+    static_assert(smem <= 227 * 1024, "retention tile");
+    static thread_local int configured_device = -1;
+    if (configured_device != ctx->device) {
+        HOLO_CUDA(cudaFuncSetAttribute(retention_tile_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        configured_device = ctx->device;
+    }
+    CUtensorMap mq, mk, mv;
+    HOLO_TRY(make_map_rows(&mq, a.q, (uint64_t)a.heads * a.dim, a.rows, a.q_ld));
+    HOLO_TRY(make_map_rows(&mk, a.k, (uint64_t)a.heads * a.dim, a.rows, a.k_ld));
+    HOLO_TRY(make_map_rows(&mv, a.v, (uint64_t)a.heads * a.vdim, a.rows, a.v_ld));
+    RetentionTileParams p;
+    p.a = a;
+    p.status = ctx->dev_status;
+    const uint32_t slices = a.vdim / RT_W;
+    HOLO_CUDA(holo_launch_kernel_cluster(ctx, retention_tile_kernel<DT>, dim3(slices, a.heads), dim3(RT_THREADS), smem, slices, 1u, mq, mk, mv, p));
+    ctx->launches++;
+    return HOLO_OK;
+}
+// Launches the tile kernel, or returns with *taken false when the shape does not suit it.
+int32_t try_tile(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
+    *taken = false;
+    if (a.dtype != HOLO_DTYPE_BF16 || a.rows < 128 || (a.dim != 128 && a.dim != 256) || a.vdim % RT_W || a.vdim / RT_W > MAX_SLICES ||
+        (a.q_ld | a.k_ld | a.v_ld | a.gate_ld | a.ld) % 8 || (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.gate | (uintptr_t)a.out) & 15u) ||
+        encode_tiled_fn() == nullptr || getenv("HOLO_RETENTION_NO_TILE"))
+        return HOLO_OK;
+    *taken = true;
+    return a.dim == 128 ? launch_tile_as<1>(ctx, a) : launch_tile_as<2>(ctx, a);
+}
+
 // ---- general form: one CTA per head, token by token ---------------------------------------------------------------------
 // 64 value columns at a time, four threads per column over the key dimensions. The state sits in shared memory where it fits.
 constexpr int SEQ_THREADS = 256, SEQ_COLS = 64, SEQ_GROUPS = SEQ_THREADS / SEQ_COLS;
@@ -534,7 +975,8 @@ int32_t holo_launch_retention(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
     if (!getenv("HOLO_RETENTION_GENERAL")) {
         bool taken = false;
         if (a.rows == 1) HOLO_TRY(a.dtype == HOLO_DTYPE_F32 ? try_token<float>(ctx, a, &taken) : try_token<__nv_bfloat16>(ctx, a, &taken));
-        else HOLO_TRY(try_chunk(ctx, a, &taken));
+        else HOLO_TRY(try_tile(ctx, a, &taken));
+        if (!taken && a.rows > 1) HOLO_TRY(try_chunk(ctx, a, &taken));
         if (taken) return HOLO_OK;
     }
     return a.dtype == HOLO_DTYPE_F32 ? launch_sequence<float>(ctx, a) : launch_sequence<__nv_bfloat16>(ctx, a);

@@ -361,19 +361,30 @@ def test_retention_many_rows(backend, dtype, heads, dim, vdim, vmean, rows, coun
     check_retention(backend, dtype, rows, count, heads, dim, vdim, vmean, first)
 
 
+@pytest.mark.parametrize("heads,dim,vdim,vmean", [(3, 128, 64, 64), (2, 128, 192, 180), (5, 256, 512, 500), (1, 256, 64, 64), (2, 128, 512, 512)])
+@pytest.mark.parametrize("tile", [True, False])
+def test_retention_long_prompts_in_both_chunked_forms(backend, monkeypatch, heads, dim, vdim, vmean, tile):
+    if not tile:
+        monkeypatch.setenv("HOLO_RETENTION_NO_TILE", "1")
+    for rows, count, first in ((128, 128, 0), (1024, 1023, 3), (640, 1, 5)):
+        check_retention(backend, BF, rows, count, heads, dim, vdim, vmean, first, seed=rows, decay=[1 - 2.0 ** -(h + 1) for h in range(heads)])
+
+
 def test_retention_general_form_and_extreme_decays(backend, monkeypatch):
     for decay in ([1.0, 0.0, 0.5, 0.9999],):
         check_retention(backend, BF, 256, 200, 4, 32, 64, 64, 3, decay=decay)
+        check_retention(backend, BF, 256, 200, 4, 128, 64, 64, 3, decay=decay)
         check_retention(backend, BF, 1, 1, 4, 32, 64, 64, 3, decay=decay)
         monkeypatch.setenv("HOLO_RETENTION_GENERAL", "1")
         check_retention(backend, BF, 64, 50, 4, 32, 64, 64, 3, decay=decay)
         check_retention(backend, F32, 64, 50, 1, 256, 512, 500, 0, decay=[0.97])   # the state does not fit shared memory
 
 
-def test_retention_remembers_one_token_far_back(backend):
+@pytest.mark.parametrize("dim", [64, 128, 256])
+def test_retention_remembers_one_token_far_back(backend, dim):
     """A single loud key and value 300 tokens before a query that asks for it, everything between quiet."""
     rng = np.random.default_rng(8)
-    rows, dim, vdim = 512, 64, 64
+    rows, vdim = 512, 64
     q, k, v = (1e-3 * rng.standard_normal((rows, 1, n)) for n in (dim, dim, vdim))
     mark = rng.standard_normal(dim)
     k[77], v[77], q[377] = mark, rng.standard_normal(vdim), mark
