@@ -455,15 +455,17 @@ int32_t try_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
 // The same chunks of 128 tokens and the same sums, a slice of 64 value columns per CTA; all four products run on tcgen05 with
 // their f32 results in TMEM, where the state stays from the first chunk to the last.
 //   warp 0      TMA producer: q and k tiles (a ring of one or two chunks), v tiles
-//   warp 1      MMA issuer. Per chunk: scores = Q K^T; O1 = Q S (S as two bf16 parts in shared memory, 128 key dimensions at a
-//               time); S += K^T V' (V' the decayed values as two bf16 parts); O2 = P V (P the decayed scores as two bf16 parts in TMEM)
-//   warps 2-5   one thread per token: scores -> P over them; then o = scale (p(i + 1) O1 + O2), its sum of squares to every CTA of
-//               the head (distributed shared memory), and the normed, gated row
-//   warps 6-9   one thread per key dimension: S -> shared memory and p(L) S -> TMEM; and one thread per token: V -> V'
+//   warp 1      MMA issuer. Per chunk: scores = Q K^T; O2 = P V (P the decayed scores as two bf16 parts in TMEM); S += K^T V' (V'
+//               the decayed values as two bf16 parts); O1 = Q S (S as two bf16 parts in shared memory, 128 key dimensions at a
+//               time). What one chunk hands to the next is S alone: its product comes as early as it can
+//   warps 2-5   one thread per token: scores -> P over them, V -> V'
+//   warps 6-9   one thread per key dimension: S -> shared memory and p(L) S -> TMEM
+//   warps 10-13 one thread per token: o = scale (p(i + 1) O1 + O2), its sum of squares to every CTA of the head (asynchronous
+//               stores to distributed shared memory that count on the reader's barrier), and the normed, gated row
 // TMEM columns: scores 0 and 128 (by turns), O1 256, O2 320, S 384 (+ 64 for the upper 128 key dimensions). It is allocated
 // after the dependency wait, dependents are released after that. Every wait is bounded; the cluster barriers at the two ends
 // are reached after bounded waits only.
-constexpr int RT_THREADS = 320, RT_W = 64;
+constexpr int RT_THREADS = 448, RT_W = 64;
 
 struct RetentionTileParams {
     HoloRetentionArgs a;
@@ -487,6 +489,13 @@ __device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity,
     atomicOr(status, 4u);
     return false;
 }
+// Store to the shared memory of CTA `rank`, counted as four bytes on its barrier.
+__device__ __forceinline__ void store_async(uint32_t addr, uint32_t bar, uint32_t rank, float v) {
+    uint32_t ra, rb;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(addr), "r"(rank));
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(rb) : "r"(bar), "r"(rank));
+    asm volatile("st.async.weak.shared::cluster.mbarrier::complete_tx::bytes.b32 [%0], %1, [%2];" ::"r"(ra), "r"(__float_as_uint(v)), "r"(rb) : "memory");
+}
 __device__ __forceinline__ void mbar_arrive(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
 __device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 
@@ -502,7 +511,7 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
     uint8_t* sm = smem_raw + (base - raw);
-    const uint32_t bars = base + OFF_BARS, bar_qk_full = bars, bar_qk_empty = bars + 16, bar_sc = bars + 32, bar_sums = bars + 48, bar_sbuf = bars + 64, bar_m2 = bars + 80,
+    const uint32_t bars = base + OFF_BARS, bar_q_full = bars, bar_q_empty = bars + 16, bar_k_full = bars + 168, bar_k_empty = bars + 184, bar_vready = bars + 200, bar_sc = bars + 32, bar_sums = bars + 48, bar_sbuf = bars + 64, bar_m2 = bars + 80,
                    bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_p = bars + 112, bar_ready = bars + 120, bar_o = bars + 128, bar_oread = bars + 136, bar_s4 = bars + 144;
     uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + OFF_BARS + 160);
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + OFF_BARS + 164);
@@ -511,10 +520,12 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, slice = blockIdx.x, slices = gridDim.x, h = blockIdx.y;
     if (tid == 0) {
         for (int i = 0; i < 2; ++i) {
-            mbar_init(bar_qk_full + 8 * i, 1);
-            mbar_init(bar_qk_empty + 8 * i, 1);
+            mbar_init(bar_q_full + 8 * i, 1);
+            mbar_init(bar_q_empty + 8 * i, 1);
+            mbar_init(bar_k_full + 8 * i, 1);
+            mbar_init(bar_k_empty + 8 * i, 1);
             mbar_init(bar_sc + 8 * i, 1);
-            mbar_init(bar_sums + 8 * i, 4 * slices);   // the token warps of every slice
+            mbar_init(bar_sums + 8 * i, 1);            // and 512 bytes from every slice
             mbar_init(bar_sbuf + 8 * i, 4);
             mbar_init(bar_m2 + 8 * i, 1);
         }
@@ -522,6 +533,7 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         mbar_init(bar_v_empty, 5);                     // the product that read v, and the four warps that decayed it
         mbar_init(bar_p, 4);
         mbar_init(bar_ready, 4);
+        mbar_init(bar_vready, 4);
         mbar_init(bar_o, 1);
         mbar_init(bar_oread, 4);
         mbar_init(bar_s4, 1);
@@ -547,25 +559,28 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     if (warp == 0) {
         // ---------------- TMA producer ----------------
         if (lane == 0) {
-            uint32_t issued = 0, vissued = 0;
+            uint32_t nk = 0, nq = 0, nv = 0;       // loads requested
             for (uint32_t c = 0; c < chunks; ++c) {
                 const uint32_t s = c % NS, st = base + s * STAGE;
-                if (c >= NS && !mbar_wait(bar_qk_empty + 8 * s, (c / NS - 1) & 1, s_abort, p.status)) break;
-                mbar_arrive_expect_tx(bar_qk_full + 8 * s, STAGE);
-                for (uint32_t x = 0; x < 2 * DT; ++x) {
-                    tma_load_2d(st + x * TILE_CHUNK, &map_q, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_qk_full + 8 * s);
-                    tma_load_2d(st + QK + x * TILE_CHUNK, &map_k, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_qk_full + 8 * s);
-                }
-                ++issued;
+                if (c >= NS && !mbar_wait(bar_k_empty + 8 * s, (c / NS - 1) & 1, s_abort, p.status)) break;
+                mbar_arrive_expect_tx(bar_k_full + 8 * s, QK);
+                for (uint32_t x = 0; x < 2 * DT; ++x) tma_load_2d(st + QK + x * TILE_CHUNK, &map_k, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_k_full + 8 * s);
+                ++nk;
                 if (c > 0 && !mbar_wait(bar_v_empty, (c - 1) & 1, s_abort, p.status)) break;
                 mbar_arrive_expect_tx(bar_v_full, TILE_CHUNK);
                 tma_load_2d(base + OFF_V, &map_v, (int)(h * a.vdim + slice * RT_W), (int)(c * 128), bar_v_full);
-                ++vissued;
+                ++nv;
+                if (c >= NS && !mbar_wait(bar_q_empty + 8 * s, (c / NS - 1) & 1, s_abort, p.status)) break;
+                mbar_arrive_expect_tx(bar_q_full + 8 * s, QK);
+                for (uint32_t x = 0; x < 2 * DT; ++x) tma_load_2d(st + x * TILE_CHUNK, &map_q, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_q_full + 8 * s);
+                ++nq;
             }
             // nothing may still be on its way into this CTA's shared memory when it ends
-            for (uint32_t c = issued > NS ? issued - NS : 0; c < issued; ++c)
-                for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_qk_full + 8 * (c % NS), (c / NS) & 1); ++it) __nanosleep(64);
-            for (uint32_t it = 0; vissued && it < WAIT_LIMIT && !mbar_try_wait(bar_v_full, (vissued - 1) & 1); ++it) __nanosleep(64);
+            for (uint32_t c = nk > NS ? nk - NS : 0; c < nk; ++c)
+                for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_k_full + 8 * (c % NS), (c / NS) & 1); ++it) __nanosleep(64);
+            for (uint32_t c = nq > NS ? nq - NS : 0; c < nq; ++c)
+                for (uint32_t it = 0; it < WAIT_LIMIT && !mbar_try_wait(bar_q_full + 8 * (c % NS), (c / NS) & 1); ++it) __nanosleep(64);
+            for (uint32_t it = 0; nv && it < WAIT_LIMIT && !mbar_try_wait(bar_v_full, (nv - 1) & 1); ++it) __nanosleep(64);
         }
     } else if (warp == 1) {
         // ---------------- MMA issuer ----------------
@@ -575,10 +590,21 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             constexpr uint32_t idesc_sc = idesc | ((128u >> 3) << 17), idesc_n = idesc | (1u << 16) | ((64u >> 3) << 17), idesc_st = idesc_n | (1u << 15);
             const uint64_t d_v = smem_desc(base + OFF_V, TILE_CHUNK, 1024), d_vb = smem_desc(base + OFF_VBIG, TILE_CHUNK, 1024), d_sb = smem_desc(base + OFF_SBIG, TILE_CHUNK, 1024);
             constexpr uint64_t PART = TILE_CHUNK >> 4;       // from a big part to its small one
-            bool ok = true;
+            // the scores of a chunk, into the buffer whose weights the product two chunks before has read
+            auto scores = [&](uint32_t c) {
+                const uint32_t s = c % NS, st = base + s * STAGE;
+                if (!mbar_wait(bar_k_full + 8 * s, (c / NS) & 1, s_abort, p.status) || !mbar_wait(bar_q_full + 8 * s, (c / NS) & 1, s_abort, p.status)) return false;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                const uint64_t d_q = smem_desc(st, 16, 1024), d_k = smem_desc(st + QK, 16, 1024);
+#pragma unroll
+                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(tmem + (c & 1u) * 128, d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
+                umma_commit(bar_sc + 8 * (c & 1u));
+                return true;
+            };
+            bool ok = chunks == 0 || scores(0);
             for (uint32_t c = 0; c < chunks && ok; ++c) {
                 const uint32_t s = c % NS, st = base + s * STAGE, sc = tmem + (c & 1u) * 128;
-                const uint64_t d_q = smem_desc(st, 16, 1024), d_k = smem_desc(st + QK, 16, 1024), d_kt = smem_desc(st + QK, TILE_CHUNK, 1024);
+                const uint64_t d_q = smem_desc(st, 16, 1024), d_kt = smem_desc(st + QK, TILE_CHUNK, 1024);
                 // O1 of 128 key dimensions
                 auto inter = [&](uint32_t half) {
 #pragma unroll
@@ -588,28 +614,8 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                             umma_bf16(tmem_o1, d_q + (2 * half + (k >> 2)) * PART + 2 * (k & 3), d_sb + part * PART + 128 * k, idesc_n, (half | part | k) != 0);
                     umma_commit(bar_m2 + 8 * half);
                 };
-                if (!(ok = mbar_wait(bar_qk_full + 8 * s, (c / NS) & 1, s_abort, p.status))) break;
-                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-#pragma unroll
-                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(sc, d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
-                umma_commit(bar_sc + 8 * (c & 1u));
-                ok = (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status)) && mbar_wait(bar_ready, c & 1, s_abort, p.status);
-                if (!ok) break;
-                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                inter(0);
-#pragma unroll
-                for (uint32_t half = 0; half < DT; ++half)
-#pragma unroll
-                    for (uint32_t part = 0; part < 2; ++part)
-#pragma unroll
-                        for (uint32_t k = 0; k < 8; ++k) umma_bf16(tmem_s + 64 * half, d_kt + 2 * half * PART + 128 * k, d_vb + part * PART + 128 * k, idesc_st, 1u);
-                umma_commit(bar_s4);
-                if (DT == 2) {
-                    if (!(ok = mbar_wait(bar_sbuf + 8, c & 1, s_abort, p.status))) break;
-                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                    inter(1);
-                }
-                ok = mbar_wait(bar_v_full, c & 1, s_abort, p.status) && mbar_wait(bar_p, c & 1, s_abort, p.status);
+                ok = mbar_wait(bar_v_full, c & 1, s_abort, p.status) && mbar_wait(bar_p, c & 1, s_abort, p.status) &&
+                     (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status));
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
@@ -617,18 +623,37 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
                     for (uint32_t k = 0; k < 8; ++k)
                         umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
-                umma_commit(bar_o);
                 umma_commit(bar_v_empty);
-                umma_commit(bar_qk_empty + 8 * s);
+                ok = mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+                for (uint32_t half = 0; half < DT; ++half)
+#pragma unroll
+                    for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                        for (uint32_t k = 0; k < 8; ++k) umma_bf16(tmem_s + 64 * half, d_kt + 2 * half * PART + 128 * k, d_vb + part * PART + 128 * k, idesc_st, 1u);
+                umma_commit(bar_s4);
+                umma_commit(bar_k_empty + 8 * s);
+                inter(0);
+                if (NS == 2 && c + 1 < chunks && !(ok = scores(c + 1))) break;
+                if (DT == 2) {
+                    if (!(ok = mbar_wait(bar_sbuf + 8, c & 1, s_abort, p.status))) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    inter(1);
+                }
+                umma_commit(bar_o);
+                umma_commit(bar_q_empty + 8 * s);
+                if (NS == 1 && c + 1 < chunks) ok = scores(c + 1);
             }
         }
     } else if (warp < 6) {
-        // ---------------- tokens (TMEM lane quarter = warp % 4) ----------------
+        // ---------------- scores (TMEM lane quarter = warp % 4) ----------------
         const uint32_t quarter = warp & 3u, i = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
         const float* power = s_power + 127;
         bool ok = true;
         for (uint32_t c = 0; c < chunks; ++c) {
-            const uint32_t row = c * 128 + i, sc = tmem + (c & 1u) * 128 + lanes;
+            const uint32_t sc = tmem + (c & 1u) * 128 + lanes;
             ok = mbar_wait(bar_sc + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
             ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
             if (!ok) break;
@@ -662,66 +687,35 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
             if (lane == 0) mbar_arrive(bar_p);
-            uint4 gate[8];
-#pragma unroll
-            for (int x = 0; x < 8; ++x)
-                gate[x] = row < count ? reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim + slice * RT_W)[x]
-                                      : make_uint4(0, 0, 0, 0);
-            ok = mbar_wait(bar_o, c & 1, s_abort, p.status) && !*s_abort;
+            // the last chunk's product has read V'
+            ok = (c == 0 || mbar_wait(bar_s4, (c - 1) & 1, s_abort, p.status)) && mbar_wait(bar_v_full, c & 1, s_abort, p.status);
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
-            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            float o[2][32], sq = 0.0f;
-            const float f = a.scale * power[i + 1];
+            const uint32_t tokens = min(128u, count - c * 128);
+            const float f = i < tokens ? power[tokens - 1 - i] : 0.0f;
+            // one token's values, the same places in both parts (units taken in another order by every lane: no bank is asked twice)
 #pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                uint32_t v0[32], v1[32];
-                tmem_ld32_request(tmem_o1 + lanes + 32 * x, v0);
-                tmem_ld32_request(tmem_o2 + lanes + 32 * x, v1);
-                tmem_ld32_wait(v0);
-                tmem_ld32_pass(v1);
+            for (uint32_t u0 = 0; u0 < 8; ++u0) {
+                const uint32_t at = i * 128 + (((u0 + lane) & 7u) << 4);
+                const uint4 x = *reinterpret_cast<const uint4*>(sm + OFF_V + at);
+                const uint32_t in[4] = {x.x, x.y, x.z, x.w};
+                uint32_t big[4], small[4];
 #pragma unroll
-                for (int e = 0; e < 32; ++e) {
-                    o[x][e] = fmaf(f, __uint_as_float(v0[e]), a.scale * __uint_as_float(v1[e]));
-                    if (slice * RT_W + 32 * x + e < a.vmean) sq = fmaf(o[x][e], o[x][e], sq);
+                for (int e = 0; e < 4; ++e) {
+                    const __nv_bfloat162 y = *reinterpret_cast<const __nv_bfloat162*>(&in[e]);
+                    split_bf16(__low2float(y) * f, __high2float(y) * f, big[e], small[e]);
                 }
+                *reinterpret_cast<uint4*>(sm + OFF_VBIG + at) = make_uint4(big[0], big[1], big[2], big[3]);
+                *reinterpret_cast<uint4*>(sm + OFF_VSMALL + at) = make_uint4(small[0], small[1], small[2], small[3]);
             }
-            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            // this row's sum of squares, to every CTA of the head
-            const uint32_t at = base + OFF_SUMS + (((c & 1u) * MAX_SLICES + slice) * 128 + i) * 4;
-            for (uint32_t to = 0; to < slices; ++to) store_remote(at, to, sq);
-            asm volatile("fence.acq_rel.cluster;" ::: "memory");
+            fence_async_smem();
             __syncwarp();
-            if (lane == 0) mbar_arrive(bar_oread);
-            if (lane < slices) {
-                uint32_t remote;
-                asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(bar_sums + 8 * (c & 1u)), "r"(lane));
-                asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(remote) : "memory");
-            }
-            __syncwarp();
-            ok = mbar_wait_cluster(bar_sums + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort && !(*reinterpret_cast<volatile uint32_t*>(p.status) & 4u);
-            ok = __all_sync(0xffffffffu, ok);
-            if (!ok) break;
-            float total = 0.0f;
-            for (uint32_t x = 0; x < slices; ++x) total += s_sums[((c & 1u) * MAX_SLICES + x) * 128 + i];
-            const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
-            if (row < count) {
-                uint4* out = reinterpret_cast<uint4*>((__nv_bfloat16*)a.out + (uint64_t)row * a.ld + (uint64_t)h * a.vdim + slice * RT_W);
-#pragma unroll
-                for (int x = 0; x < 8; ++x) {
-                    const uint32_t g[4] = {gate[x].x, gate[x].y, gate[x].z, gate[x].w};
-                    uint32_t w[4];
-#pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162*>(&g[e]);
-                        const float* oo = &o[x >> 2][8 * (x & 3) + 2 * e];
-                        w[e] = pack_bf16(oo[0] * inv * __low2float(gg), oo[1] * inv * __high2float(gg));
-                    }
-                    out[x] = make_uint4(w[0], w[1], w[2], w[3]);
-                }
+            if (lane == 0) {
+                mbar_arrive(bar_v_empty);
+                mbar_arrive(bar_vready);
             }
         }
-    } else {
+    } else if (warp < 10) {
         // ---------------- state and values (TMEM lane quarter = warp % 4) ----------------
         const uint32_t quarter = warp & 3u, r = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
         const float* power = s_power + 127;
@@ -772,11 +766,9 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         };
         bool ok = true;
         for (uint32_t c = 0; c < chunks; ++c) {
-            const uint32_t tokens = min(128u, count - c * 128);
-            const float keep = power[tokens], f = r < tokens ? power[tokens - 1 - r] : 0.0f;
-            // the last chunk's products have read V' and written S, and (for the first half) read S's parts
-            ok = (c == 0 || (mbar_wait(bar_s4, (c - 1) & 1, s_abort, p.status) && mbar_wait(bar_m2 + 8 * (DT - 1), (c - 1) & 1, s_abort, p.status))) &&
-                 mbar_wait(bar_v_full, c & 1, s_abort, p.status) && !*s_abort;
+            const float keep = power[min(128u, count - c * 128)];
+            // the last chunk's products have written S and read its parts
+            ok = (c == 0 || (mbar_wait(bar_s4, (c - 1) & 1, s_abort, p.status) && mbar_wait(bar_m2 + 8 * (DT - 1), (c - 1) & 1, s_abort, p.status))) && !*s_abort;
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -788,29 +780,11 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 load_state(1, v);
                 keep_state(1, v, keep);
             }
-            // one token's values, the same places in both parts (units taken in another order by every lane: no bank is asked twice)
-#pragma unroll
-            for (uint32_t u0 = 0; u0 < 8; ++u0) {
-                const uint32_t at = r * 128 + (((u0 + lane) & 7u) << 4);
-                const uint4 x = *reinterpret_cast<const uint4*>(sm + OFF_V + at);
-                const uint32_t in[4] = {x.x, x.y, x.z, x.w};
-                uint32_t big[4], small[4];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const __nv_bfloat162 y = *reinterpret_cast<const __nv_bfloat162*>(&in[e]);
-                    split_bf16(__low2float(y) * f, __high2float(y) * f, big[e], small[e]);
-                }
-                *reinterpret_cast<uint4*>(sm + OFF_VBIG + at) = make_uint4(big[0], big[1], big[2], big[3]);
-                *reinterpret_cast<uint4*>(sm + OFF_VSMALL + at) = make_uint4(small[0], small[1], small[2], small[3]);
-            }
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             fence_async_smem();
             __syncwarp();
-            if (lane == 0) {
-                mbar_arrive(bar_v_empty);
-                mbar_arrive(bar_ready);
-            }
+            if (lane == 0) mbar_arrive(bar_ready);
             if (DT == 2) {
                 ok = mbar_wait(bar_m2, c & 1, s_abort, p.status);
                 ok = __all_sync(0xffffffffu, ok);
@@ -834,6 +808,72 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 for (int x = 0; x < 16; ++x)
                     to[x] = make_float4(__uint_as_float(v[x >> 3][4 * (x & 7)]), __uint_as_float(v[x >> 3][4 * (x & 7) + 1]), __uint_as_float(v[x >> 3][4 * (x & 7) + 2]),
                                         __uint_as_float(v[x >> 3][4 * (x & 7) + 3]));
+            }
+        }
+    } else {
+        // ---------------- outputs (TMEM lane quarter = warp % 4) ----------------
+        const uint32_t quarter = warp & 3u, i = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
+        const float* power = s_power + 127;
+        bool ok = true;
+        if (chunks != 0 && (*reinterpret_cast<volatile uint32_t*>(p.status) & 4u)) *s_abort = 1;      // an earlier launch gave up: store nothing
+        for (uint32_t c = 0; c < chunks; ++c) {
+            const uint32_t row = c * 128 + i;
+            uint4 gate[8];
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+                gate[x] = row < count ? reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim + slice * RT_W)[x]
+                                      : make_uint4(0, 0, 0, 0);
+            ok = mbar_wait(bar_o, c & 1, s_abort, p.status) && !*s_abort;
+            ok = __all_sync(0xffffffffu, ok);
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            float o[2][32], sq = 0.0f;
+            const float f = a.scale * power[i + 1];
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                uint32_t v0[32], v1[32];
+                tmem_ld32_request(tmem_o1 + lanes + 32 * x, v0);
+                tmem_ld32_request(tmem_o2 + lanes + 32 * x, v1);
+                tmem_ld32_wait(v0);
+                tmem_ld32_pass(v1);
+#pragma unroll
+                for (int e = 0; e < 32; ++e) {
+                    o[x][e] = fmaf(f, __uint_as_float(v0[e]), a.scale * __uint_as_float(v1[e]));
+                    if (slice * RT_W + 32 * x + e < a.vmean) sq = fmaf(o[x][e], o[x][e], sq);
+                }
+            }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_oread);
+            float total = sq;
+            if (slices > 1) {
+                // this row's sum of squares, to every CTA of the head. Asynchronous stores need a launch with clusters: a head of one
+                // slice is launched without and has nothing to exchange.
+                const uint32_t at = base + OFF_SUMS + (((c & 1u) * MAX_SLICES + slice) * 128 + i) * 4;
+                if (warp == 10 && lane == 0) mbar_arrive_expect_tx(bar_sums + 8 * (c & 1u), slices * 512);
+                for (uint32_t to = 0; to < slices; ++to) store_async(at, bar_sums + 8 * (c & 1u), to, sq);
+                __syncwarp();
+                ok = mbar_wait_cluster(bar_sums + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
+                ok = __all_sync(0xffffffffu, ok);
+                if (!ok) break;
+                total = 0.0f;
+                for (uint32_t x = 0; x < slices; ++x) total += s_sums[((c & 1u) * MAX_SLICES + x) * 128 + i];
+            }
+            const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
+            if (row < count) {
+                uint4* out = reinterpret_cast<uint4*>((__nv_bfloat16*)a.out + (uint64_t)row * a.ld + (uint64_t)h * a.vdim + slice * RT_W);
+#pragma unroll
+                for (int x = 0; x < 8; ++x) {
+                    const uint32_t g[4] = {gate[x].x, gate[x].y, gate[x].z, gate[x].w};
+                    uint32_t w[4];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162*>(&g[e]);
+                        const float* oo = &o[x >> 2][8 * (x & 3) + 2 * e];
+                        w[e] = pack_bf16(oo[0] * inv * __low2float(gg), oo[1] * inv * __high2float(gg));
+                    }
+                    out[x] = make_uint4(w[0], w[1], w[2], w[3]);
+                }
             }
         }
     }
