@@ -455,15 +455,16 @@ int32_t try_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
 // The same chunks of 128 tokens and the same sums, a slice of 64 value columns per CTA; all four products run on tcgen05 with
 // their f32 results in TMEM, where the state stays from the first chunk to the last.
 //   warp 0      TMA producer: q and k tiles (a ring of one or two chunks), v tiles
-//   warp 1      MMA issuer. Per chunk: scores = Q K^T; O2 = P V (P the decayed scores as two bf16 parts in TMEM); S += K^T V' (V'
-//               the decayed values as two bf16 parts); O1 = Q S (S as two bf16 parts in shared memory, 128 key dimensions at a
-//               time). What one chunk hands to the next is S alone: its product comes as early as it can
+//   warp 1      MMA issuer. Per chunk: scores = Q K^T; S += K^T V' (V' the decayed values as two bf16 parts); O1 = Q S (S as two
+//               bf16 parts side by side in shared memory, 128 key dimensions at a time; their products stay side by side as
+//               well); O2 = P V (P the decayed scores as two bf16 parts in TMEM). Where two chunks of q and k fit, the next chunk's
+//               scores come first, so that their weights are ready in time
 //   warps 2-5   one thread per token: scores -> P over them, V -> V'
 //   warps 6-9   one thread per key dimension: S -> shared memory and p(L) S -> TMEM
 //   warps 10-13 one thread per token: o = scale (p(i + 1) O1 + O2), its sum of squares to every CTA of the head (asynchronous
 //               stores to distributed shared memory that count on the reader's barrier), and the normed, gated row
-// TMEM columns: scores 0 and 128 (by turns), O1 256, O2 320, S 384 (+ 64 for the upper 128 key dimensions). It is allocated
-// after the dependency wait, dependents are released after that. Every wait is bounded; the cluster barriers at the two ends
+// TMEM columns: O1 0 (and 64), O2 128, S 192 (+ 64 for the upper 128 key dimensions), scores 256 and 384 by turns (384 alone
+// where one chunk of q and k fits). It is allocated after the dependency wait, dependents are released after that. Every wait is bounded; the cluster barriers at the two ends
 // are reached after bounded waits only.
 constexpr int RT_THREADS = 448, RT_W = 64;
 
@@ -512,7 +513,7 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const uint32_t base = (raw + 1023u) & ~1023u;
     uint8_t* sm = smem_raw + (base - raw);
     const uint32_t bars = base + OFF_BARS, bar_q_full = bars, bar_q_empty = bars + 16, bar_k_full = bars + 168, bar_k_empty = bars + 184, bar_vready = bars + 200, bar_sc = bars + 32, bar_sums = bars + 48, bar_sbuf = bars + 64, bar_m2 = bars + 80,
-                   bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_p = bars + 112, bar_ready = bars + 120, bar_o = bars + 128, bar_oread = bars + 136, bar_s4 = bars + 144;
+                   bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_p = bars + 208, bar_ready = bars + 120, bar_o = bars + 128, bar_oread = bars + 136, bar_s4 = bars + 144;
     uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + OFF_BARS + 160);
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + OFF_BARS + 164);
     float* s_power = reinterpret_cast<float*>(sm + OFF_POWER);      // [127 + n] = decay^n, 0 for n < 0
@@ -525,13 +526,13 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             mbar_init(bar_k_full + 8 * i, 1);
             mbar_init(bar_k_empty + 8 * i, 1);
             mbar_init(bar_sc + 8 * i, 1);
+            mbar_init(bar_p + 8 * i, 4);               // two: weights may be ready a chunk before they are asked for
             mbar_init(bar_sums + 8 * i, 1);            // and 512 bytes from every slice
             mbar_init(bar_sbuf + 8 * i, 4);
             mbar_init(bar_m2 + 8 * i, 1);
         }
         mbar_init(bar_v_full, 1);
         mbar_init(bar_v_empty, 5);                     // the product that read v, and the four warps that decayed it
-        mbar_init(bar_p, 4);
         mbar_init(bar_ready, 4);
         mbar_init(bar_vready, 4);
         mbar_init(bar_o, 1);
@@ -553,7 +554,8 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     cluster_wait();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     holo_pdl_trigger();
-    const uint32_t tmem = *s_tmem, tmem_o1 = tmem + 256, tmem_o2 = tmem + 320, tmem_s = tmem + 384;
+    const uint32_t tmem = *s_tmem, tmem_o1 = tmem, tmem_o2 = tmem + 128, tmem_s = tmem + 192;
+    auto tmem_sc = [&](uint32_t c) { return tmem + (NS == 2 && (c & 1u) == 0 ? 256u : 384u); };
     const uint32_t count = min(a.rows, a.step[1]), chunks = (count + 127) / 128;
 
     if (warp == 0) {
@@ -566,14 +568,15 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 mbar_arrive_expect_tx(bar_k_full + 8 * s, QK);
                 for (uint32_t x = 0; x < 2 * DT; ++x) tma_load_2d(st + QK + x * TILE_CHUNK, &map_k, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_k_full + 8 * s);
                 ++nk;
-                if (c > 0 && !mbar_wait(bar_v_empty, (c - 1) & 1, s_abort, p.status)) break;
-                mbar_arrive_expect_tx(bar_v_full, TILE_CHUNK);
-                tma_load_2d(base + OFF_V, &map_v, (int)(h * a.vdim + slice * RT_W), (int)(c * 128), bar_v_full);
-                ++nv;
+                // (the values last: their buffer is free only after the product that follows the next chunk's scores)
                 if (c >= NS && !mbar_wait(bar_q_empty + 8 * s, (c / NS - 1) & 1, s_abort, p.status)) break;
                 mbar_arrive_expect_tx(bar_q_full + 8 * s, QK);
                 for (uint32_t x = 0; x < 2 * DT; ++x) tma_load_2d(st + x * TILE_CHUNK, &map_q, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_q_full + 8 * s);
                 ++nq;
+                if (c > 0 && !mbar_wait(bar_v_empty, (c - 1) & 1, s_abort, p.status)) break;
+                mbar_arrive_expect_tx(bar_v_full, TILE_CHUNK);
+                tma_load_2d(base + OFF_V, &map_v, (int)(h * a.vdim + slice * RT_W), (int)(c * 128), bar_v_full);
+                ++nv;
             }
             // nothing may still be on its way into this CTA's shared memory when it ends
             for (uint32_t c = nk > NS ? nk - NS : 0; c < nk; ++c)
@@ -587,44 +590,35 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (lane == 0) {
             // D = f32, A = B = bf16, M = 128; scores: both operands K-major, N = 128; the others: B N-major, N = 64; the state's A is K^T (M-major)
             constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 4) << 24);
-            constexpr uint32_t idesc_sc = idesc | ((128u >> 3) << 17), idesc_n = idesc | (1u << 16) | ((64u >> 3) << 17), idesc_st = idesc_n | (1u << 15);
+            constexpr uint32_t idesc_sc = idesc | ((128u >> 3) << 17), idesc_n = idesc | (1u << 16) | ((64u >> 3) << 17), idesc_st = idesc_n | (1u << 15),
+                               idesc_o1 = idesc | (1u << 16) | ((128u >> 3) << 17);
             const uint64_t d_v = smem_desc(base + OFF_V, TILE_CHUNK, 1024), d_vb = smem_desc(base + OFF_VBIG, TILE_CHUNK, 1024), d_sb = smem_desc(base + OFF_SBIG, TILE_CHUNK, 1024);
             constexpr uint64_t PART = TILE_CHUNK >> 4;       // from a big part to its small one
-            // the scores of a chunk, into the buffer whose weights the product two chunks before has read
+            // the scores of a chunk, over weights that an earlier product has read
             auto scores = [&](uint32_t c) {
                 const uint32_t s = c % NS, st = base + s * STAGE;
                 if (!mbar_wait(bar_k_full + 8 * s, (c / NS) & 1, s_abort, p.status) || !mbar_wait(bar_q_full + 8 * s, (c / NS) & 1, s_abort, p.status)) return false;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint64_t d_q = smem_desc(st, 16, 1024), d_k = smem_desc(st + QK, 16, 1024);
 #pragma unroll
-                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(tmem + (c & 1u) * 128, d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
+                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(tmem_sc(c), d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
                 umma_commit(bar_sc + 8 * (c & 1u));
                 return true;
             };
             bool ok = chunks == 0 || scores(0);
             for (uint32_t c = 0; c < chunks && ok; ++c) {
-                const uint32_t s = c % NS, st = base + s * STAGE, sc = tmem + (c & 1u) * 128;
+                const uint32_t s = c % NS, st = base + s * STAGE, sc = tmem_sc(c);
                 const uint64_t d_q = smem_desc(st, 16, 1024), d_kt = smem_desc(st + QK, TILE_CHUNK, 1024);
                 // O1 of 128 key dimensions
                 auto inter = [&](uint32_t half) {
 #pragma unroll
-                    for (uint32_t part = 0; part < 2; ++part)
-#pragma unroll
-                        for (uint32_t k = 0; k < 8; ++k)
-                            umma_bf16(tmem_o1, d_q + (2 * half + (k >> 2)) * PART + 2 * (k & 3), d_sb + part * PART + 128 * k, idesc_n, (half | part | k) != 0);
+                    for (uint32_t k = 0; k < 8; ++k)
+                        umma_bf16(tmem_o1, d_q + (2 * half + (k >> 2)) * PART + 2 * (k & 3), d_sb + 128 * k, idesc_o1, (half | k) != 0);
                     umma_commit(bar_m2 + 8 * half);
                 };
-                ok = mbar_wait(bar_v_full, c & 1, s_abort, p.status) && mbar_wait(bar_p, c & 1, s_abort, p.status) &&
+                if (NS == 2 && c + 1 < chunks && !(ok = scores(c + 1))) break;
+                ok = mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status) &&
                      (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status));
-                if (!ok) break;
-                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-#pragma unroll
-                for (uint32_t part = 0; part < 2; ++part)
-#pragma unroll
-                    for (uint32_t k = 0; k < 8; ++k)
-                        umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
-                umma_commit(bar_v_empty);
-                ok = mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
@@ -636,69 +630,82 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 umma_commit(bar_s4);
                 umma_commit(bar_k_empty + 8 * s);
                 inter(0);
-                if (NS == 2 && c + 1 < chunks && !(ok = scores(c + 1))) break;
                 if (DT == 2) {
                     if (!(ok = mbar_wait(bar_sbuf + 8, c & 1, s_abort, p.status))) break;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                     inter(1);
                 }
-                umma_commit(bar_o);
                 umma_commit(bar_q_empty + 8 * s);
+                ok = mbar_wait(bar_v_full, c & 1, s_abort, p.status) && mbar_wait(bar_p + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status);
+                if (!ok) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+                for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                    for (uint32_t k = 0; k < 8; ++k)
+                        umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
+                umma_commit(bar_o);
+                umma_commit(bar_v_empty);
                 if (NS == 1 && c + 1 < chunks) ok = scores(c + 1);
             }
         }
     } else if (warp < 6) {
-        // ---------------- scores (TMEM lane quarter = warp % 4) ----------------
+        // ---------------- weights and decayed values (TMEM lane quarter = warp % 4) ----------------
         const uint32_t quarter = warp & 3u, i = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
         const float* power = s_power + 127;
-        bool ok = true;
-        for (uint32_t c = 0; c < chunks; ++c) {
-            const uint32_t sc = tmem + (c & 1u) * 128 + lanes;
-            ok = mbar_wait(bar_sc + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
-            ok = __all_sync(0xffffffffu, ok);   // the TMEM accesses below are whole-warp instructions
-            if (!ok) break;
+        float diagonal[32];      // the decays among this warp's own 32 tokens
+#pragma unroll
+        for (int e = 0; e < 32; ++e) diagonal[e] = power[(int)lane - e];
+        // scores -> weights, 32 tokens at a time: token 32 b + e is p(i - 32 b - 31) p(31 - e) away from the tokens of later blocks
+        auto weights = [&](uint32_t c) {
+            const uint32_t sc = tmem_sc(c) + lanes;
+            bool ok = mbar_wait(bar_sc + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
+            if (!__all_sync(0xffffffffu, ok)) return false;   // the TMEM accesses below are whole-warp instructions
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll 1
+            for (uint32_t b = 0; b < 4; ++b) {
+                uint32_t big[16], small[16];
+                if (b > quarter) {
 #pragma unroll
-            for (uint32_t b2 = 0; b2 < 2; ++b2) {
-                uint32_t v[2][32];
-                const bool some = 64 * b2 < quarter * 32 + 32;      // else no token of this warp sees any of these
-                if (some) {
-                    tmem_ld32_request(sc + 64 * b2, v[0]);
-                    tmem_ld32_request(sc + 64 * b2 + 32, v[1]);
-                    tmem_ld32_wait(v[0]);
-                    tmem_ld32_pass(v[1]);
-                }
+                    for (int e = 0; e < 16; ++e) big[e] = small[e] = 0;
+                } else {
+                    uint32_t v[32];
+                    tmem_ld32_request(sc + 32 * b, v);
+                    const float far = b < quarter ? power[(int)i - (int)(32 * b) - 31] : 1.0f;
+                    float4 w[8];
 #pragma unroll
-                for (uint32_t b = 0; b < 2; ++b) {
-                    uint32_t big[16], small[16];
+                    for (int e = 0; e < 8; ++e)
+                        w[e] = b < quarter ? make_float4(power[31 - 4 * e], power[30 - 4 * e], power[29 - 4 * e], power[28 - 4 * e])
+                                           : make_float4(diagonal[4 * e], diagonal[4 * e + 1], diagonal[4 * e + 2], diagonal[4 * e + 3]);
+                    tmem_ld32_wait(v);
 #pragma unroll
-                    for (uint32_t e = 0; e < 16; ++e) {
-                        big[e] = small[e] = 0;
-                        if (some) {
-                            const float* w = power + (int)i - (int)(64 * b2 + 32 * b + 2 * e);
-                            split_bf16(__uint_as_float(v[b][2 * e]) * w[0], __uint_as_float(v[b][2 * e + 1]) * w[-1], big[e], small[e]);
-                        }
+                    for (int e = 0; e < 8; ++e) {
+                        split_bf16(__uint_as_float(v[4 * e]) * (w[e].x * far), __uint_as_float(v[4 * e + 1]) * (w[e].y * far), big[2 * e], small[2 * e]);
+                        split_bf16(__uint_as_float(v[4 * e + 2]) * (w[e].z * far), __uint_as_float(v[4 * e + 3]) * (w[e].w * far), big[2 * e + 1], small[2 * e + 1]);
                     }
-                    tmem_st16(sc + 64 * b2 + 32 * b, big);          // over scores this warp has already read
-                    tmem_st16(sc + 64 * b2 + 32 * b + 16, small);
                 }
+                tmem_st16(sc + 32 * b, big);          // over scores this warp has already read
+                tmem_st16(sc + 32 * b + 16, small);
             }
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             __syncwarp();
-            if (lane == 0) mbar_arrive(bar_p);
-            // the last chunk's product has read V'
-            ok = (c == 0 || mbar_wait(bar_s4, (c - 1) & 1, s_abort, p.status)) && mbar_wait(bar_v_full, c & 1, s_abort, p.status);
-            ok = __all_sync(0xffffffffu, ok);
-            if (!ok) break;
+            if (lane == 0) mbar_arrive(bar_p + 8 * (c & 1u));
+            return true;
+        };
+        // one token's values, the same places in both parts (units taken in another order by every lane: no bank is asked twice)
+        auto values = [&](uint32_t c) {
+            bool ok = (c == 0 || mbar_wait(bar_s4, (c - 1) & 1, s_abort, p.status)) && mbar_wait(bar_v_full, c & 1, s_abort, p.status);   // the last product has read V'
+            if (!__all_sync(0xffffffffu, ok)) return false;
             const uint32_t tokens = min(128u, count - c * 128);
             const float f = i < tokens ? power[tokens - 1 - i] : 0.0f;
-            // one token's values, the same places in both parts (units taken in another order by every lane: no bank is asked twice)
+            uint4 x[8];
+#pragma unroll
+            for (uint32_t u0 = 0; u0 < 8; ++u0) x[u0] = *reinterpret_cast<const uint4*>(sm + OFF_V + i * 128 + (((u0 + lane) & 7u) << 4));
 #pragma unroll
             for (uint32_t u0 = 0; u0 < 8; ++u0) {
                 const uint32_t at = i * 128 + (((u0 + lane) & 7u) << 4);
-                const uint4 x = *reinterpret_cast<const uint4*>(sm + OFF_V + at);
-                const uint32_t in[4] = {x.x, x.y, x.z, x.w};
+                const uint32_t in[4] = {x[u0].x, x[u0].y, x[u0].z, x[u0].w};
                 uint32_t big[4], small[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
@@ -714,7 +721,11 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 mbar_arrive(bar_v_empty);
                 mbar_arrive(bar_vready);
             }
-        }
+            return true;
+        };
+        // with two chunks of q and k in flight a chunk's scores are there before the state's last product is through, else after
+        for (uint32_t c = 0; c < chunks; ++c)
+            if (NS == 2 ? !(weights(c) && values(c)) : !(values(c) && weights(c))) break;
     } else if (warp < 10) {
         // ---------------- state and values (TMEM lane quarter = warp % 4) ----------------
         const uint32_t quarter = warp & 3u, r = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
@@ -818,28 +829,20 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (chunks != 0 && (*reinterpret_cast<volatile uint32_t*>(p.status) & 4u)) *s_abort = 1;      // an earlier launch gave up: store nothing
         for (uint32_t c = 0; c < chunks; ++c) {
             const uint32_t row = c * 128 + i;
-            uint4 gate[8];
-#pragma unroll
-            for (int x = 0; x < 8; ++x)
-                gate[x] = row < count ? reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim + slice * RT_W)[x]
-                                      : make_uint4(0, 0, 0, 0);
             ok = mbar_wait(bar_o, c & 1, s_abort, p.status) && !*s_abort;
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            float o[2][32], sq = 0.0f;
+            float o[64], sq = 0.0f;
             const float f = a.scale * power[i + 1];
 #pragma unroll
-            for (int x = 0; x < 2; ++x) {
-                uint32_t v0[32], v1[32];
-                tmem_ld32_request(tmem_o1 + lanes + 32 * x, v0);
-                tmem_ld32_request(tmem_o2 + lanes + 32 * x, v1);
-                tmem_ld32_wait(v0);
-                tmem_ld32_pass(v1);
+            for (int x = 0; x < 4; ++x) {
+                uint32_t big[16], small[16], near[16];
+                tmem_ld16x3(tmem_o1 + lanes + 16 * x, tmem_o1 + lanes + 64 + 16 * x, tmem_o2 + lanes + 16 * x, big, small, near);
 #pragma unroll
-                for (int e = 0; e < 32; ++e) {
-                    o[x][e] = fmaf(f, __uint_as_float(v0[e]), a.scale * __uint_as_float(v1[e]));
-                    if (slice * RT_W + 32 * x + e < a.vmean) sq = fmaf(o[x][e], o[x][e], sq);
+                for (int e = 0; e < 16; ++e) {
+                    o[16 * x + e] = fmaf(f, __uint_as_float(big[e]) + __uint_as_float(small[e]), a.scale * __uint_as_float(near[e]));
+                    if (slice * RT_W + 16 * x + e < a.vmean) sq = fmaf(o[16 * x + e], o[16 * x + e], sq);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -853,6 +856,13 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 if (warp == 10 && lane == 0) mbar_arrive_expect_tx(bar_sums + 8 * (c & 1u), slices * 512);
                 for (uint32_t to = 0; to < slices; ++to) store_async(at, bar_sums + 8 * (c & 1u), to, sq);
                 __syncwarp();
+            }
+            uint4 gate[8];
+#pragma unroll
+            for (int x = 0; x < 8; ++x)
+                gate[x] = row < count ? reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim + slice * RT_W)[x]
+                                      : make_uint4(0, 0, 0, 0);
+            if (slices > 1) {
                 ok = mbar_wait_cluster(bar_sums + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
                 ok = __all_sync(0xffffffffu, ok);
                 if (!ok) break;
@@ -869,7 +879,7 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162*>(&g[e]);
-                        const float* oo = &o[x >> 2][8 * (x & 3) + 2 * e];
+                        const float* oo = &o[8 * x + 2 * e];
                         w[e] = pack_bf16(oo[0] * inv * __low2float(gg), oo[1] * inv * __high2float(gg));
                     }
                     out[x] = make_uint4(w[0], w[1], w[2], w[3]);
