@@ -1226,6 +1226,13 @@ int32_t do_retention(holo_b200_ctx* ctx, const HoloRetentionCall& c, holo_b200_w
     HOLO_TRY(resolve_words(ws, c.step, 2, &step));
     HOLO_TRY(holo_resolve(ws, c.state, sb, &state, nullptr));
     if (((uintptr_t)state & 15u) != 0) return holo_fail_slot(c.state.slot, "the retention state must be 16-byte aligned on the device");
+    if (c.work.slot != HOLO_NO_SLOT) {
+        const uint64_t wb = 4ull * c.rows * c.heads * c.vdim;
+        uint8_t* work;
+        HOLO_TRY(holo_resolve(ws, c.work, wb, &work, nullptr));
+        HOLO_TRY(check_disjoint({work, wb}, c.work.slot, {rq, rk, rv, rg, ro, {decay, 4ull * c.heads}, {step, 8}, {state, sb}}));
+        a.work = (float*)work;
+    }
     HOLO_TRY(check_disjoint(ro, c.output.slot, {rq, rk, rv, rg, {decay, 4ull * c.heads}, {step, 8}, {state, sb}}));
     HOLO_TRY(check_disjoint({state, sb}, c.state.slot, {rq, rk, rv, rg, {decay, 4ull * c.heads}, {step, 8}}));
     a.q = q; a.k = k; a.v = v; a.gate = gate; a.decay = (const float*)decay; a.step = (const uint32_t*)step; a.state = (float*)state; a.out = out;
@@ -1570,6 +1577,7 @@ bool holo_collect_refs(HoloKernelCall* c, HoloRefList* l) {
             l->in(&q.q); l->in(&q.k); l->in(&q.v); l->in(&q.gate); l->in(&q.decay); l->in(&q.step);
             l->out(&q.state, 4ull * q.heads * q.dim * q.vdim);
             l->out(&q.output, ((uint64_t)(q.rows - 1) * q.ld + (uint64_t)q.heads * q.vdim) * holo_dtype_size(q.dtype));
+            l->out(&q.work, 4ull * q.rows * q.heads * q.vdim);
             return true;
         }
         case HOLO_K_MOE_PLAN: {

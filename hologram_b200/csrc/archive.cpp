@@ -283,7 +283,7 @@ int32_t decode_call(Reader& r, HoloKernelCall* out) {
         }
         case HOLO_K_RETENTION: {
             HoloRetentionCall& c = out->u.retention;
-            for (HoloBufferRef* b : {&c.q, &c.k, &c.v, &c.gate, &c.decay, &c.step, &c.state, &c.output}) *b = r.buf();
+            for (HoloBufferRef* b : {&c.q, &c.k, &c.v, &c.gate, &c.decay, &c.step, &c.state, &c.output, &c.work}) *b = r.buf();
             for (uint32_t* f : {&c.rows, &c.heads, &c.dim, &c.vdim, &c.vmean, &c.q_ld, &c.k_ld, &c.v_ld, &c.gate_ld, &c.ld, &c.scale_bits, &c.epsilon_bits}) *f = r.u32();
             c.dtype = r.u8();
             if (c.rows == 0) return holo_fail(HOLO_ERR_INIT, "backend init failed: retention over no rows");

@@ -345,7 +345,7 @@ struct HoloRetentionArgs {
     const void *q, *k, *v, *gate;
     const float* decay;
     const uint32_t* step;
-    float* state;
+    float *state, *work;         // work: null, or [rows, heads * vdim]
     void* out;
     uint32_t rows, heads, dim, vdim, vmean, q_ld, k_ld, v_ld, gate_ld, ld;
     float scale, eps;

@@ -7,7 +7,8 @@
 //   retention_token_kernel      one row
 //   retention_sequence_kernel   everything else: token by token, one CTA per head
 //
-// In all but the last a cluster of CTAs shares a head, each with a slice of the value columns; they exchange the sums of squares.
+// In all but the last the CTAs of a head have a slice of the value columns each; for one row and for other heads they are a
+// cluster and exchange the sums of squares.
 #include "attention_tile.cuh"
 
 #include <algorithm>
@@ -461,11 +462,12 @@ int32_t try_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
 //               scores come first, so that their weights are ready in time
 //   warps 2-5   one thread per token: scores -> P over them, V -> V'
 //   warps 6-9   one thread per key dimension: S -> shared memory and p(L) S -> TMEM
-//   warps 10-13 one thread per token: o = scale (p(i + 1) O1 + O2), its sum of squares to every CTA of the head (asynchronous
-//               stores to distributed shared memory that count on the reader's barrier), and the normed, gated row
+//   warps 10-13 one thread per token: o = scale (p(i + 1) O1 + O2), f32, to the call's work buffer
+// A second launch divides every head's o by its root mean square and applies the gate. (A cluster per head that exchanged its
+// sums of squares needed no second launch, but eight CTAs of this size rarely find room in one GPC: half the chip stood idle.)
 // TMEM columns: O1 0 (and 64), O2 128, S 192 (+ 64 for the upper 128 key dimensions), scores 256 and 384 by turns (384 alone
-// where one chunk of q and k fits). It is allocated after the dependency wait, dependents are released after that. Every wait is bounded; the cluster barriers at the two ends
-// are reached after bounded waits only.
+// where one chunk of q and k fits). It is allocated after the dependency wait, dependents are released after that.
+// Every wait is bounded.
 constexpr int RT_THREADS = 448, RT_W = 64;
 
 struct RetentionTileParams {
@@ -473,29 +475,8 @@ struct RetentionTileParams {
     uint32_t* status;
 };
 
-// Like mbar_wait, for a barrier that other CTAs of the cluster arrive on after writing this CTA's shared memory.
-__device__ __forceinline__ bool mbar_wait_cluster(uint32_t bar, uint32_t parity, volatile uint32_t* abort_flag, uint32_t* status) {
-    for (uint32_t it = 0; it < WAIT_LIMIT; ++it) {
-        uint32_t ok;
-        asm volatile(
-            "{\n.reg .pred p;\nmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}\n"
-            : "=r"(ok)
-            : "r"(bar), "r"(parity)
-            : "memory");
-        if (ok) return true;
-        if (*abort_flag) return false;
-        if (it > 64) __nanosleep(64);
-    }
-    *abort_flag = 1;
-    atomicOr(status, 4u);
-    return false;
-}
-// Store to the shared memory of CTA `rank`, counted as four bytes on its barrier.
-__device__ __forceinline__ void store_async(uint32_t addr, uint32_t bar, uint32_t rank, float v) {
-    uint32_t ra, rb;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(ra) : "r"(addr), "r"(rank));
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(rb) : "r"(bar), "r"(rank));
-    asm volatile("st.async.weak.shared::cluster.mbarrier::complete_tx::bytes.b32 [%0], %1, [%2];" ::"r"(ra), "r"(__float_as_uint(v)), "r"(rb) : "memory");
+__device__ __forceinline__ void tma_prefetch_2d(const CUtensorMap* map, int x, int y) {
+    asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global.tile [%0, {%1, %2}];" ::"l"(map), "r"(x), "r"(y) : "memory");
 }
 __device__ __forceinline__ void mbar_arrive(uint32_t bar) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory"); }
 __device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
@@ -506,18 +487,17 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                       const RetentionTileParams p) {
     constexpr uint32_t NS = DT == 1 ? 2 : 1, QK = 2 * DT * TILE_CHUNK, STAGE = 2 * QK;      // q and k tiles of a chunk
     constexpr uint32_t OFF_V = NS * STAGE, OFF_VBIG = OFF_V + TILE_CHUNK, OFF_VSMALL = OFF_VBIG + TILE_CHUNK, OFF_SBIG = OFF_VSMALL + TILE_CHUNK,
-                       OFF_SSMALL = OFF_SBIG + TILE_CHUNK, OFF_POWER = OFF_SSMALL + TILE_CHUNK, OFF_SUMS = OFF_POWER + 1024, OFF_BARS = OFF_SUMS + 2 * MAX_SLICES * 128 * 4;
+                       OFF_SSMALL = OFF_SBIG + TILE_CHUNK, OFF_POWER = OFF_SSMALL + TILE_CHUNK, OFF_BARS = OFF_POWER + 1024;
     extern __shared__ uint8_t smem_raw[];
     const HoloRetentionArgs& a = p.a;
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
     uint8_t* sm = smem_raw + (base - raw);
-    const uint32_t bars = base + OFF_BARS, bar_q_full = bars, bar_q_empty = bars + 16, bar_k_full = bars + 168, bar_k_empty = bars + 184, bar_vready = bars + 200, bar_sc = bars + 32, bar_sums = bars + 48, bar_sbuf = bars + 64, bar_m2 = bars + 80,
+    const uint32_t bars = base + OFF_BARS, bar_q_full = bars, bar_q_empty = bars + 16, bar_k_full = bars + 168, bar_k_empty = bars + 184, bar_vready = bars + 200, bar_sc = bars + 32, bar_sbuf = bars + 64, bar_m2 = bars + 80,
                    bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_p = bars + 208, bar_ready = bars + 120, bar_o = bars + 128, bar_oread = bars + 136, bar_s4 = bars + 144;
     uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + OFF_BARS + 160);
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + OFF_BARS + 164);
     float* s_power = reinterpret_cast<float*>(sm + OFF_POWER);      // [127 + n] = decay^n, 0 for n < 0
-    float* s_sums = reinterpret_cast<float*>(sm + OFF_SUMS);
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, slice = blockIdx.x, slices = gridDim.x, h = blockIdx.y;
     if (tid == 0) {
         for (int i = 0; i < 2; ++i) {
@@ -527,7 +507,6 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             mbar_init(bar_k_empty + 8 * i, 1);
             mbar_init(bar_sc + 8 * i, 1);
             mbar_init(bar_p + 8 * i, 4);               // two: weights may be ready a chunk before they are asked for
-            mbar_init(bar_sums + 8 * i, 1);            // and 512 bytes from every slice
             mbar_init(bar_sbuf + 8 * i, 4);
             mbar_init(bar_m2 + 8 * i, 1);
         }
@@ -550,8 +529,6 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     if (tid < 256) s_power[tid] = tid < 127 ? 0.0f : tid == 127 ? 1.0f : powf(decay, (float)(tid - 127));
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
-    cluster_arrive();       // every CTA's barriers are set up before anyone arrives on them
-    cluster_wait();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     holo_pdl_trigger();
     const uint32_t tmem = *s_tmem, tmem_o1 = tmem, tmem_o2 = tmem + 128, tmem_s = tmem + 192;
@@ -564,6 +541,14 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             uint32_t nk = 0, nq = 0, nv = 0;       // loads requested
             for (uint32_t c = 0; c < chunks; ++c) {
                 const uint32_t s = c % NS, st = base + s * STAGE;
+                // two chunks ahead, into L2 (every slice of the head asks for its share of q and k)
+                for (uint32_t f = c == 0 ? 1 : c + 2; f <= c + 2 && f < chunks; ++f) {
+                    tma_prefetch_2d(&map_v, (int)(h * a.vdim + slice * RT_W), (int)(f * 128));
+                    for (uint32_t x = slice; x < 2 * DT; x += slices) {
+                        tma_prefetch_2d(&map_k, (int)(h * a.dim + 64 * x), (int)(f * 128));
+                        tma_prefetch_2d(&map_q, (int)(h * a.dim + 64 * x), (int)(f * 128));
+                    }
+                }
                 if (c >= NS && !mbar_wait(bar_k_empty + 8 * s, (c / NS - 1) & 1, s_abort, p.status)) break;
                 mbar_arrive_expect_tx(bar_k_full + 8 * s, QK);
                 for (uint32_t x = 0; x < 2 * DT; ++x) tma_load_2d(st + QK + x * TILE_CHUNK, &map_k, (int)(h * a.dim + 64 * x), (int)(c * 128), bar_k_full + 8 * s);
@@ -617,8 +602,21 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                     umma_commit(bar_m2 + 8 * half);
                 };
                 if (NS == 2 && c + 1 < chunks && !(ok = scores(c + 1))) break;
-                ok = mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status) &&
-                     (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status));
+                // O2 = P V
+                auto near = [&]() {
+                    if (!mbar_wait(bar_v_full, c & 1, s_abort, p.status) || !mbar_wait(bar_p + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status)) return false;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+#pragma unroll
+                    for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                        for (uint32_t k = 0; k < 8; ++k)
+                            umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
+                    umma_commit(bar_v_empty);
+                    return true;
+                };
+                // with two chunks in flight the weights are there already: their product first gives the value buffer back early
+                ok = (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status)) && (NS == 1 || near()) &&
+                     mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
@@ -636,16 +634,8 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                     inter(1);
                 }
                 umma_commit(bar_q_empty + 8 * s);
-                ok = mbar_wait(bar_v_full, c & 1, s_abort, p.status) && mbar_wait(bar_p + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status);
-                if (!ok) break;
-                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-#pragma unroll
-                for (uint32_t part = 0; part < 2; ++part)
-#pragma unroll
-                    for (uint32_t k = 0; k < 8; ++k)
-                        umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
+                if (NS == 1 && !(ok = near())) break;
                 umma_commit(bar_o);
-                umma_commit(bar_v_empty);
                 if (NS == 1 && c + 1 < chunks) ok = scores(c + 1);
             }
         }
@@ -833,66 +823,47 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            float o[64], sq = 0.0f;
+            float4* out = reinterpret_cast<float4*>(a.work + ((uint64_t)row * a.heads + h) * a.vdim + slice * RT_W);
             const float f = a.scale * power[i + 1];
+            uint32_t big[2][16], small[2][16], near[2][16];
 #pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                uint32_t big[16], small[16], near[16];
-                tmem_ld16x3(tmem_o1 + lanes + 16 * x, tmem_o1 + lanes + 64 + 16 * x, tmem_o2 + lanes + 16 * x, big, small, near);
+            for (int y = 0; y < 2; ++y) {
 #pragma unroll
-                for (int e = 0; e < 16; ++e) {
-                    o[16 * x + e] = fmaf(f, __uint_as_float(big[e]) + __uint_as_float(small[e]), a.scale * __uint_as_float(near[e]));
-                    if (slice * RT_W + 16 * x + e < a.vmean) sq = fmaf(o[16 * x + e], o[16 * x + e], sq);
+                for (int x = 0; x < 2; ++x) {
+                    tmem_ld16_request(tmem_o1 + lanes + 32 * y + 16 * x, big[x]);
+                    tmem_ld16_request(tmem_o1 + lanes + 64 + 32 * y + 16 * x, small[x]);
+                    tmem_ld16_request(tmem_o2 + lanes + 32 * y + 16 * x, near[x]);
                 }
-            }
-            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-            __syncwarp();
-            if (lane == 0) mbar_arrive(bar_oread);
-            float total = sq;
-            if (slices > 1) {
-                // this row's sum of squares, to every CTA of the head. Asynchronous stores need a launch with clusters: a head of one
-                // slice is launched without and has nothing to exchange.
-                const uint32_t at = base + OFF_SUMS + (((c & 1u) * MAX_SLICES + slice) * 128 + i) * 4;
-                if (warp == 10 && lane == 0) mbar_arrive_expect_tx(bar_sums + 8 * (c & 1u), slices * 512);
-                for (uint32_t to = 0; to < slices; ++to) store_async(at, bar_sums + 8 * (c & 1u), to, sq);
-                __syncwarp();
-            }
-            uint4 gate[8];
+                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-            for (int x = 0; x < 8; ++x)
-                gate[x] = row < count ? reinterpret_cast<const uint4*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim + slice * RT_W)[x]
-                                      : make_uint4(0, 0, 0, 0);
-            if (slices > 1) {
-                ok = mbar_wait_cluster(bar_sums + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
-                ok = __all_sync(0xffffffffu, ok);
-                if (!ok) break;
-                total = 0.0f;
-                for (uint32_t x = 0; x < slices; ++x) total += s_sums[((c & 1u) * MAX_SLICES + x) * 128 + i];
-            }
-            const float inv = 1.0f / sqrtf(total / (float)a.vmean + a.eps);
-            if (row < count) {
-                uint4* out = reinterpret_cast<uint4*>((__nv_bfloat16*)a.out + (uint64_t)row * a.ld + (uint64_t)h * a.vdim + slice * RT_W);
+                for (int x = 0; x < 2; ++x) {
+                    tmem_ld16_pass(big[x]);
+                    tmem_ld16_pass(small[x]);
+                    tmem_ld16_pass(near[x]);
+                }
+                if (y == 1) {
+                    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+                    __syncwarp();
+                    if (lane == 0) mbar_arrive(bar_oread);
+                }
+                if (row < count)
 #pragma unroll
-                for (int x = 0; x < 8; ++x) {
-                    const uint32_t g[4] = {gate[x].x, gate[x].y, gate[x].z, gate[x].w};
-                    uint32_t w[4];
+                    for (int e = 0; e < 8; ++e) {
+                        float v[4];
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) {
-                        const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162*>(&g[e]);
-                        const float* oo = &o[8 * x + 2 * e];
-                        w[e] = pack_bf16(oo[0] * inv * __low2float(gg), oo[1] * inv * __high2float(gg));
+                        for (int n = 0; n < 4; ++n) {
+                            const int at = (4 * e + n) & 15, x = e >> 2;
+                            v[n] = fmaf(f, __uint_as_float(big[x][at]) + __uint_as_float(small[x][at]), a.scale * __uint_as_float(near[x][at]));
+                        }
+                        out[8 * y + e] = make_float4(v[0], v[1], v[2], v[3]);
                     }
-                    out[x] = make_uint4(w[0], w[1], w[2], w[3]);
-                }
             }
         }
     }
-    // everyone meets here, whatever happened above: TMEM is released, and no CTA leaves while another may still write its sums
+    // everyone meets here, whatever happened above, so that TMEM is always released
     __syncwarp();
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
-    cluster_arrive();
-    cluster_wait();
     if (warp == 1) {
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
@@ -909,9 +880,48 @@ int32_t make_map_rows(CUtensorMap* map, const void* ptr, uint64_t cols, uint64_t
     return r == CUDA_SUCCESS ? HOLO_OK : holo_fail(HOLO_ERR_DISPATCH, "dispatch failed: cuTensorMapEncodeTiled (retention) returned %d", (int)r);
 }
 
+// One warp per (row, head): o over its root mean square, times the gate.
+template <int PL>   // vdim <= 128 PL
+__global__ void __launch_bounds__(256)
+retention_finish_kernel(const HoloRetentionArgs a) {
+    holo_pdl_trigger();
+    const uint32_t unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, row = unit / a.heads, h = unit % a.heads;
+    holo_pdl_wait();
+    if (row >= min(a.rows, a.step[1])) return;
+    const float4* o = reinterpret_cast<const float4*>(a.work + (uint64_t)unit * a.vdim);
+    const uint2* gate = reinterpret_cast<const uint2*>((const __nv_bfloat16*)a.gate + (uint64_t)row * a.gate_ld + (uint64_t)h * a.vdim);
+    float4 v[PL];
+    uint2 g[PL];
+    float sq = 0.0f;
+#pragma unroll
+    for (int x = 0; x < PL; ++x) {
+        const uint32_t j = lane + 32 * x;
+        v[x] = 4 * j < a.vdim ? o[j] : make_float4(0.f, 0.f, 0.f, 0.f);
+        g[x] = 4 * j < a.vdim ? gate[j] : make_uint2(0, 0);
+    }
+#pragma unroll
+    for (int x = 0; x < PL; ++x) {
+        const uint32_t j = 4 * (lane + 32 * x);
+        const float e[4] = {v[x].x, v[x].y, v[x].z, v[x].w};
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+            if (j + n < a.vmean) sq = fmaf(e[n], e[n], sq);
+    }
+    for (int off = 16; off > 0; off >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, off);
+    const float inv = 1.0f / sqrtf(sq / (float)a.vmean + a.eps);
+    uint2* out = reinterpret_cast<uint2*>((__nv_bfloat16*)a.out + (uint64_t)row * a.ld + (uint64_t)h * a.vdim);
+#pragma unroll
+    for (int x = 0; x < PL; ++x) {
+        const uint32_t j = lane + 32 * x;
+        if (4 * j >= a.vdim) continue;
+        const __nv_bfloat162 g0 = *reinterpret_cast<const __nv_bfloat162*>(&g[x].x), g1 = *reinterpret_cast<const __nv_bfloat162*>(&g[x].y);
+        out[j] = make_uint2(pack_bf16(v[x].x * inv * __low2float(g0), v[x].y * inv * __high2float(g0)), pack_bf16(v[x].z * inv * __low2float(g1), v[x].w * inv * __high2float(g1)));
+    }
+}
+
 template <int DT>
 int32_t launch_tile_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
-    constexpr uint32_t smem = (DT == 1 ? 2 : 1) * 4 * DT * TILE_CHUNK + 5 * TILE_CHUNK + 1024 + 2 * MAX_SLICES * 128 * 4 + 256 + 1024;
+    constexpr uint32_t smem = (DT == 1 ? 2 : 1) * 4 * DT * TILE_CHUNK + 5 * TILE_CHUNK + 1024 + 256 + 1024;
     static_assert(smem <= 227 * 1024, "retention tile");
     static thread_local int configured_device = -1;
     if (configured_device != ctx->device) {
@@ -925,15 +935,19 @@ int32_t launch_tile_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
     RetentionTileParams p;
     p.a = a;
     p.status = ctx->dev_status;
-    const uint32_t slices = a.vdim / RT_W;
-    HOLO_CUDA(holo_launch_kernel_cluster(ctx, retention_tile_kernel<DT>, dim3(slices, a.heads), dim3(RT_THREADS), smem, slices, 1u, mq, mk, mv, p));
-    ctx->launches++;
+    HOLO_CUDA(holo_launch_kernel(ctx, retention_tile_kernel<DT>, dim3(a.vdim / RT_W, a.heads), dim3(RT_THREADS), smem, 1, mq, mk, mv, p));
+    const dim3 grid((a.rows * a.heads + 7) / 8);
+    if (a.vdim <= 128) HOLO_CUDA(holo_launch_kernel(ctx, retention_finish_kernel<1>, grid, dim3(256), 0, 1, a));
+    else if (a.vdim <= 256) HOLO_CUDA(holo_launch_kernel(ctx, retention_finish_kernel<2>, grid, dim3(256), 0, 1, a));
+    else if (a.vdim <= 512) HOLO_CUDA(holo_launch_kernel(ctx, retention_finish_kernel<4>, grid, dim3(256), 0, 1, a));
+    else HOLO_CUDA(holo_launch_kernel(ctx, retention_finish_kernel<8>, grid, dim3(256), 0, 1, a));
+    ctx->launches += 2;
     return HOLO_OK;
 }
 // Launches the tile kernel, or returns with *taken false when the shape does not suit it.
 int32_t try_tile(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
     *taken = false;
-    if (a.dtype != HOLO_DTYPE_BF16 || a.rows < 128 || (a.dim != 128 && a.dim != 256) || a.vdim % RT_W || a.vdim / RT_W > MAX_SLICES ||
+    if (a.dtype != HOLO_DTYPE_BF16 || a.rows < 128 || (a.dim != 128 && a.dim != 256) || a.vdim % RT_W || !a.work || ((uintptr_t)a.work & 15u) || a.heads > 65535 ||
         (a.q_ld | a.k_ld | a.v_ld | a.gate_ld | a.ld) % 8 || (((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.gate | (uintptr_t)a.out) & 15u) ||
         encode_tiled_fn() == nullptr || getenv("HOLO_RETENTION_NO_TILE"))
         return HOLO_OK;

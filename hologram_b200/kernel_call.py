@@ -373,7 +373,7 @@ class WindowAttentionCall(C.Structure):
 
 class RetentionCall(C.Structure):
     """Extension: linear attention with one decay per head, an f32 state, and a normed, gated output."""
-    _fields_ = [(n, BufferRef) for n in ("q", "k", "v", "gate", "decay", "step", "state", "output")] + [(n, C.c_uint32) for n in (
+    _fields_ = [(n, BufferRef) for n in ("q", "k", "v", "gate", "decay", "step", "state", "output", "work")] + [(n, C.c_uint32) for n in (
         "rows", "heads", "dim", "vdim", "vmean", "q_ld", "k_ld", "v_ld", "gate_ld", "ld", "scale_bits", "epsilon_bits")] + [("dtype", C.c_uint8)]
 
 

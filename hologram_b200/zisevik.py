@@ -508,8 +508,9 @@ class ZisevikModel(StepModel):
             kc.LinearSeg.make(sl.ref(q), ldk, ldk, dt, cq, rotate=rotate), kc.LinearSeg.make(sl.ref(k), ldk, ldk, dt, ck, rotate=rotate),
             kc.LinearSeg.make(sl.ref(v), ldv, ldv, dt, cv), kc.LinearSeg.make(sl.ref(g), ldv, ldv, dt, cg, act=kc.LINEAR_ACT_SILU)], c.width_p, cols, rot=table)
         out = s.buffer("context", rows * ldv * es)
+        work = sl.ref(s.buffer("retention work", 4 * rows * ldv)) if dt == BF and rows > 1 else kc.NONE
         s.call(kc.KernelCall.Retention(kc.RetentionCall(
-            sl.ref(q), sl.ref(k), sl.ref(v), sl.ref(g), s.const(p + "decay"), s.step, sl.ref(state), sl.ref(out), rows, a.heads, a.dim_p, a.vdim_p, a.vdim,
+            sl.ref(q), sl.ref(k), sl.ref(v), sl.ref(g), s.const(p + "decay"), s.step, sl.ref(state), sl.ref(out), work, rows, a.heads, a.dim_p, a.vdim_p, a.vdim,
             ldk, ldk, ldv, ldv, ldv, kc.f32_bits(a.dim ** -0.5), kc.f32_bits(c.eps), dt)))
         self._add_to_residual(s, sl.ref(out), p + "o", ldv, x)
 

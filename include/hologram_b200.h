@@ -533,9 +533,10 @@ typedef struct HoloWindowAttentionCall {
  * where first is 0:   S = decay_h S + k_i v_i^T,   o_i = scale * S^T q_i
  *   output[i, h * vdim + e] = o_i[e] / sqrt(mean_{e < vmean}(o_i^2) + eps) * gate[i, h * vdim + e]
  * q, k [rows, heads * dim], v, gate [rows, heads * vdim] with pitches of their own; vmean <= vdim columns carry values (the
- * rest are zero). Rows from count on are not stored. */
+ * rest are zero). Rows from count on are not stored. work: optional f32 [rows, heads * vdim] that the call may overwrite (the
+ * fastest form for many rows needs it). */
 typedef struct HoloRetentionCall {
-    HoloBufferRef q, k, v, gate, decay, step, state, output;
+    HoloBufferRef q, k, v, gate, decay, step, state, output, work;
     uint32_t rows, heads, dim, vdim, vmean, q_ld, k_ld, v_ld, gate_ld, ld, scale_bits, epsilon_bits;
     uint8_t dtype;
 } HoloRetentionCall;

@@ -316,8 +316,8 @@ def retention_case(backend, dtype, rows, count, heads, dim, vdim, vmean, first, 
         out[:, :x[0].size] = x.reshape(rows, -1)
         return store(out, dtype)
     ws = workspace(backend, [padded(q, ldq), padded(k, ldq), padded(v, ldv), padded(gate, ldv), decay, words(first, count), np.asarray(state, np.float32),
-                             store(np.full((rows, ldv), 5.0), dtype)])
-    backend.dispatch(kc.KernelCall.Retention(kc.RetentionCall(*[rb(i) for i in range(8)], rows, heads, dim, vdim, vmean, ldq, ldq, ldv, ldv, ldv,
+                             store(np.full((rows, ldv), 5.0), dtype)], [4 * rows * heads * vdim])
+    backend.dispatch(kc.KernelCall.Retention(kc.RetentionCall(*[rb(i) for i in range(9)], rows, heads, dim, vdim, vmean, ldq, ldq, ldv, ldv, ldv,
                                                               kc.f32_bits(scale), kc.f32_bits(eps), dtype)), ws)
     got = load(ws.read(rb(7), rows * ldv * es), dtype).reshape(rows, ldv)[:, :heads * vdim].reshape(rows, heads, vdim)
     after = ws.read(rb(6), 4 * heads * dim * vdim, np.float32).reshape(heads, dim, vdim)
@@ -390,8 +390,8 @@ def test_retention_remembers_one_token_far_back(backend, dim):
     k[77], v[77], q[377] = mark, rng.standard_normal(vdim), mark
     q, k, v = ref.bf16(q), ref.bf16(k), ref.bf16(v)
     ones = np.ones((rows, 1, vdim))
-    ws = workspace(backend, [store(t, BF) for t in (q, k, v, ones)] + [np.array([0.995], np.float32), words(0, rows), np.zeros((dim, vdim), np.float32)], [rows * vdim * 2])
-    backend.dispatch(kc.KernelCall.Retention(kc.RetentionCall(*[rb(i) for i in range(8)], rows, 1, dim, vdim, vdim, dim, dim, vdim, vdim, vdim, kc.f32_bits(1.0), kc.f32_bits(1e-6), BF)), ws)
+    ws = workspace(backend, [store(t, BF) for t in (q, k, v, ones)] + [np.array([0.995], np.float32), words(0, rows), np.zeros((dim, vdim), np.float32)], [rows * vdim * 2, rows * vdim * 4])
+    backend.dispatch(kc.KernelCall.Retention(kc.RetentionCall(*[rb(i) for i in range(9)], rows, 1, dim, vdim, vdim, dim, dim, vdim, vdim, vdim, kc.f32_bits(1.0), kc.f32_bits(1e-6), BF)), ws)
     got = load(ws.read(rb(7), rows * vdim * 2), BF).reshape(rows, vdim)
     want = ref.rms(ref.retain(q.astype(np.float64), k.astype(np.float64), v.astype(np.float64), [0.995], np.zeros((1, dim, vdim)))[:, 0], 1e-6)
     close(got[377], want[377], BF)
