@@ -454,20 +454,20 @@ int32_t try_chunk(holo_b200_ctx* ctx, const HoloRetentionArgs& a, bool* taken) {
 
 // ---- many rows, heads of 128 or 256 key dimensions: tcgen05 ------------------------------------------------------------------
 // The same chunks of 128 tokens and the same sums, a slice of 64 value columns per CTA; all four products run on tcgen05 with
-// their f32 results in TMEM, where the state stays from the first chunk to the last.
+// their f32 results in TMEM, where the state stays from the first chunk to the last. S and the decayed values enter their
+// products as two bf16 parts; the decayed scores P, which touch nothing but their own token's output, as one, like the softmax
+// weights of the attention kernels.
 //   warp 0      TMA producer: q and k tiles (a ring of one or two chunks), v tiles
-//   warp 1      MMA issuer. Per chunk: scores = Q K^T; S += K^T V' (V' the decayed values as two bf16 parts); O1 = Q S (S as two
-//               bf16 parts side by side in shared memory, 128 key dimensions at a time; their products stay side by side as
-//               well); O2 = P V (P the decayed scores as two bf16 parts in TMEM). Where two chunks of q and k fit, the next chunk's
-//               scores come first, so that their weights are ready in time
+//   warp 1      MMA issuer. Per chunk: scores = Q K^T; O2 = P V; S += K^T V'; O1 = Q S (128 key dimensions at a time). Where two
+//               chunks of q and k fit, P V and the next chunk's scores come first (the weights are ready by then, and v can be
+//               replaced early), else last (the scores wait for their chunk)
 //   warps 2-5   one thread per token: scores -> P over them, V -> V'
 //   warps 6-9   one thread per key dimension: S -> shared memory and p(L) S -> TMEM
-//   warps 10-13 one thread per token: o = scale (p(i + 1) O1 + O2), f32, to the call's work buffer
+//   warps 10-13 one thread per token: o = scale (p(i + 1) O1 + O2), f32, through shared memory to the call's work buffer (TMA)
 // A second launch divides every head's o by its root mean square and applies the gate. (A cluster per head that exchanged its
 // sums of squares needed no second launch, but eight CTAs of this size rarely find room in one GPC: half the chip stood idle.)
-// TMEM columns: O1 0 (and 64), O2 128, S 192 (+ 64 for the upper 128 key dimensions), scores 256 and 384 by turns (384 alone
-// where one chunk of q and k fits). It is allocated after the dependency wait, dependents are released after that.
-// Every wait is bounded.
+// TMEM columns: O1 0 and 64, O2 128 and 192 (by turns), S 256 (+ 64 for the upper 128 key dimensions), scores 384. It is
+// allocated after the dependency wait, dependents are released after that. Every wait is bounded.
 constexpr int RT_THREADS = 448, RT_W = 64;
 
 struct RetentionTileParams {
@@ -484,17 +484,18 @@ __device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.a
 template <int DT>   // dim = 128 DT
 __global__ void __launch_bounds__(RT_THREADS, 1)
 retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
-                      const RetentionTileParams p) {
+                      const __grid_constant__ CUtensorMap map_work, const RetentionTileParams p) {
     constexpr uint32_t NS = DT == 1 ? 2 : 1, QK = 2 * DT * TILE_CHUNK, STAGE = 2 * QK;      // q and k tiles of a chunk
     constexpr uint32_t OFF_V = NS * STAGE, OFF_VBIG = OFF_V + TILE_CHUNK, OFF_VSMALL = OFF_VBIG + TILE_CHUNK, OFF_SBIG = OFF_VSMALL + TILE_CHUNK,
-                       OFF_SSMALL = OFF_SBIG + TILE_CHUNK, OFF_POWER = OFF_SSMALL + TILE_CHUNK, OFF_BARS = OFF_POWER + 1024;
+                       OFF_SSMALL = OFF_SBIG + TILE_CHUNK, OFF_OUT = OFF_SSMALL + TILE_CHUNK, OFF_POWER = OFF_OUT + TILE_CHUNK, OFF_BARS = OFF_POWER + 1024;
     extern __shared__ uint8_t smem_raw[];
     const HoloRetentionArgs& a = p.a;
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
     uint8_t* sm = smem_raw + (base - raw);
-    const uint32_t bars = base + OFF_BARS, bar_q_full = bars, bar_q_empty = bars + 16, bar_k_full = bars + 168, bar_k_empty = bars + 184, bar_vready = bars + 200, bar_sc = bars + 32, bar_sbuf = bars + 64, bar_m2 = bars + 80,
-                   bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_p = bars + 208, bar_ready = bars + 120, bar_o = bars + 128, bar_oread = bars + 136, bar_s4 = bars + 144;
+    const uint32_t bars = base + OFF_BARS, bar_q_full = bars, bar_q_empty = bars + 16, bar_sc = bars + 32, bar_o = bars + 48, bar_sbuf = bars + 64, bar_m2 = bars + 80,
+                   bar_v_full = bars + 96, bar_v_empty = bars + 104, bar_ready = bars + 112, bar_vready = bars + 120, bar_oread = bars + 128, bar_s4 = bars + 144,
+                   bar_k_full = bars + 168, bar_k_empty = bars + 184, bar_p = bars + 200;
     uint32_t* s_tmem = reinterpret_cast<uint32_t*>(sm + OFF_BARS + 160);
     volatile uint32_t* s_abort = reinterpret_cast<volatile uint32_t*>(sm + OFF_BARS + 164);
     float* s_power = reinterpret_cast<float*>(sm + OFF_POWER);      // [127 + n] = decay^n, 0 for n < 0
@@ -506,7 +507,9 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             mbar_init(bar_k_full + 8 * i, 1);
             mbar_init(bar_k_empty + 8 * i, 1);
             mbar_init(bar_sc + 8 * i, 1);
-            mbar_init(bar_p + 8 * i, 4);               // two: weights may be ready a chunk before they are asked for
+            mbar_init(bar_p + 8 * i, 4);
+            mbar_init(bar_o + 8 * i, 1);
+            mbar_init(bar_oread + 8 * i, 4);
             mbar_init(bar_sbuf + 8 * i, 4);
             mbar_init(bar_m2 + 8 * i, 1);
         }
@@ -514,8 +517,6 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         mbar_init(bar_v_empty, 5);                     // the product that read v, and the four warps that decayed it
         mbar_init(bar_ready, 4);
         mbar_init(bar_vready, 4);
-        mbar_init(bar_o, 1);
-        mbar_init(bar_oread, 4);
         mbar_init(bar_s4, 1);
         *s_abort = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -531,8 +532,7 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     holo_pdl_trigger();
-    const uint32_t tmem = *s_tmem, tmem_o1 = tmem, tmem_o2 = tmem + 128, tmem_s = tmem + 192;
-    auto tmem_sc = [&](uint32_t c) { return tmem + (NS == 2 && (c & 1u) == 0 ? 256u : 384u); };
+    const uint32_t tmem = *s_tmem, tmem_o1 = tmem, tmem_o2 = tmem + 128, tmem_s = tmem + 256, tmem_sc = tmem + 384;
     const uint32_t count = min(a.rows, a.step[1]), chunks = (count + 127) / 128;
 
     if (warp == 0) {
@@ -575,48 +575,44 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (lane == 0) {
             // D = f32, A = B = bf16, M = 128; scores: both operands K-major, N = 128; the others: B N-major, N = 64; the state's A is K^T (M-major)
             constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((128u >> 4) << 24);
-            constexpr uint32_t idesc_sc = idesc | ((128u >> 3) << 17), idesc_n = idesc | (1u << 16) | ((64u >> 3) << 17), idesc_st = idesc_n | (1u << 15),
-                               idesc_o1 = idesc | (1u << 16) | ((128u >> 3) << 17);
+            constexpr uint32_t idesc_sc = idesc | ((128u >> 3) << 17), idesc_n = idesc | (1u << 16) | ((64u >> 3) << 17), idesc_st = idesc_n | (1u << 15);
             const uint64_t d_v = smem_desc(base + OFF_V, TILE_CHUNK, 1024), d_vb = smem_desc(base + OFF_VBIG, TILE_CHUNK, 1024), d_sb = smem_desc(base + OFF_SBIG, TILE_CHUNK, 1024);
             constexpr uint64_t PART = TILE_CHUNK >> 4;       // from a big part to its small one
-            // the scores of a chunk, over weights that an earlier product has read
+            // the scores of a chunk, over weights that the product before has read
             auto scores = [&](uint32_t c) {
                 const uint32_t s = c % NS, st = base + s * STAGE;
                 if (!mbar_wait(bar_k_full + 8 * s, (c / NS) & 1, s_abort, p.status) || !mbar_wait(bar_q_full + 8 * s, (c / NS) & 1, s_abort, p.status)) return false;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint64_t d_q = smem_desc(st, 16, 1024), d_k = smem_desc(st + QK, 16, 1024);
 #pragma unroll
-                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(tmem_sc(c), d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
+                for (uint32_t k = 0; k < 8 * DT; ++k) umma_bf16(tmem_sc, d_q + (k >> 2) * PART + 2 * (k & 3), d_k + (k >> 2) * PART + 2 * (k & 3), idesc_sc, k != 0);
                 umma_commit(bar_sc + 8 * (c & 1u));
                 return true;
             };
             bool ok = chunks == 0 || scores(0);
             for (uint32_t c = 0; c < chunks && ok; ++c) {
-                const uint32_t s = c % NS, st = base + s * STAGE, sc = tmem_sc(c);
+                const uint32_t s = c % NS, st = base + s * STAGE, o = (c & 1u) * 64;
                 const uint64_t d_q = smem_desc(st, 16, 1024), d_kt = smem_desc(st + QK, TILE_CHUNK, 1024);
                 // O1 of 128 key dimensions
                 auto inter = [&](uint32_t half) {
 #pragma unroll
-                    for (uint32_t k = 0; k < 8; ++k)
-                        umma_bf16(tmem_o1, d_q + (2 * half + (k >> 2)) * PART + 2 * (k & 3), d_sb + 128 * k, idesc_o1, (half | k) != 0);
+                    for (uint32_t part = 0; part < 2; ++part)
+#pragma unroll
+                        for (uint32_t k = 0; k < 8; ++k)
+                            umma_bf16(tmem_o1 + o, d_q + (2 * half + (k >> 2)) * PART + 2 * (k & 3), d_sb + part * PART + 128 * k, idesc_n, (half | part | k) != 0);
                     umma_commit(bar_m2 + 8 * half);
                 };
-                if (NS == 2 && c + 1 < chunks && !(ok = scores(c + 1))) break;
                 // O2 = P V
                 auto near = [&]() {
                     if (!mbar_wait(bar_v_full, c & 1, s_abort, p.status) || !mbar_wait(bar_p + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status)) return false;
                     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
-                    for (uint32_t part = 0; part < 2; ++part)
-#pragma unroll
-                        for (uint32_t k = 0; k < 8; ++k)
-                            umma_bf16_ts(tmem_o2, sc + 32 * (k >> 1) + 8 * (k & 1) + 16 * part, d_v + 128 * k, idesc_n, (part | k) != 0);
+                    for (uint32_t k = 0; k < 8; ++k) umma_bf16_ts(tmem_o2 + o, tmem_sc + 8 * k, d_v + 128 * k, idesc_n, k != 0);
                     umma_commit(bar_v_empty);
                     return true;
                 };
-                // with two chunks in flight the weights are there already: their product first gives the value buffer back early
-                ok = (c == 0 || mbar_wait(bar_oread, (c - 1) & 1, s_abort, p.status)) && (NS == 1 || near()) &&
-                     mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status);
+                ok = (c < 2 || mbar_wait(bar_oread + 8 * (c & 1u), ((c >> 1) - 1) & 1, s_abort, p.status)) &&
+                     (NS == 1 || (near() && (c + 1 == chunks || scores(c + 1)))) && mbar_wait(bar_ready, c & 1, s_abort, p.status) && mbar_wait(bar_vready, c & 1, s_abort, p.status);
                 if (!ok) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
@@ -635,7 +631,7 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 }
                 umma_commit(bar_q_empty + 8 * s);
                 if (NS == 1 && !(ok = near())) break;
-                umma_commit(bar_o);
+                umma_commit(bar_o + 8 * (c & 1u));
                 if (NS == 1 && c + 1 < chunks) ok = scores(c + 1);
             }
         }
@@ -648,34 +644,37 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         for (int e = 0; e < 32; ++e) diagonal[e] = power[(int)lane - e];
         // scores -> weights, 32 tokens at a time: token 32 b + e is p(i - 32 b - 31) p(31 - e) away from the tokens of later blocks
         auto weights = [&](uint32_t c) {
-            const uint32_t sc = tmem_sc(c) + lanes;
+            const uint32_t sc = tmem_sc + lanes;
             bool ok = mbar_wait(bar_sc + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
             if (!__all_sync(0xffffffffu, ok)) return false;   // the TMEM accesses below are whole-warp instructions
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-#pragma unroll 1
-            for (uint32_t b = 0; b < 4; ++b) {
-                uint32_t big[16], small[16];
-                if (b > quarter) {
 #pragma unroll
-                    for (int e = 0; e < 16; ++e) big[e] = small[e] = 0;
-                } else {
-                    uint32_t v[32];
-                    tmem_ld32_request(sc + 32 * b, v);
-                    const float far = b < quarter ? power[(int)i - (int)(32 * b) - 31] : 1.0f;
-                    float4 w[8];
-#pragma unroll
-                    for (int e = 0; e < 8; ++e)
-                        w[e] = b < quarter ? make_float4(power[31 - 4 * e], power[30 - 4 * e], power[29 - 4 * e], power[28 - 4 * e])
-                                           : make_float4(diagonal[4 * e], diagonal[4 * e + 1], diagonal[4 * e + 2], diagonal[4 * e + 3]);
-                    tmem_ld32_wait(v);
-#pragma unroll
-                    for (int e = 0; e < 8; ++e) {
-                        split_bf16(__uint_as_float(v[4 * e]) * (w[e].x * far), __uint_as_float(v[4 * e + 1]) * (w[e].y * far), big[2 * e], small[2 * e]);
-                        split_bf16(__uint_as_float(v[4 * e + 2]) * (w[e].z * far), __uint_as_float(v[4 * e + 3]) * (w[e].w * far), big[2 * e + 1], small[2 * e + 1]);
-                    }
+            for (uint32_t b2 = 0; b2 < 2; ++b2) {
+                uint32_t v[2][32];
+                if (2 * b2 <= quarter) {
+                    tmem_ld32_request(sc + 64 * b2, v[0]);
+                    tmem_ld32_request(sc + 64 * b2 + 32, v[1]);
+                    tmem_ld32_wait(v[0]);
+                    tmem_ld32_pass(v[1]);
                 }
-                tmem_st16(sc + 32 * b, big);          // over scores this warp has already read
-                tmem_st16(sc + 32 * b + 16, small);
+#pragma unroll
+                for (uint32_t x = 0; x < 2; ++x) {
+                    const uint32_t b = 2 * b2 + x;
+                    uint32_t w[16];
+                    if (b < quarter) {
+                        const float far = power[(int)i - (int)(32 * b) - 31];
+#pragma unroll
+                        for (int e = 0; e < 16; ++e)
+                            w[e] = pack_bf16(__uint_as_float(v[x][2 * e]) * (power[31 - 2 * e] * far), __uint_as_float(v[x][2 * e + 1]) * (power[30 - 2 * e] * far));
+                    } else if (b == quarter) {
+#pragma unroll
+                        for (int e = 0; e < 16; ++e) w[e] = pack_bf16(__uint_as_float(v[x][2 * e]) * diagonal[2 * e], __uint_as_float(v[x][2 * e + 1]) * diagonal[2 * e + 1]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 16; ++e) w[e] = 0;
+                    }
+                    tmem_st16(sc + 16 * b, w);          // over scores this warp has already read
+                }
             }
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -816,49 +815,55 @@ retention_tile_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const uint32_t quarter = warp & 3u, i = quarter * 32 + lane, lanes = (quarter * 32u) << 16;
         const float* power = s_power + 127;
         bool ok = true;
+        uint32_t together = 1;
         if (chunks != 0 && (*reinterpret_cast<volatile uint32_t*>(p.status) & 4u)) *s_abort = 1;      // an earlier launch gave up: store nothing
         for (uint32_t c = 0; c < chunks; ++c) {
-            const uint32_t row = c * 128 + i;
-            ok = mbar_wait(bar_o, c & 1, s_abort, p.status) && !*s_abort;
-            ok = __all_sync(0xffffffffu, ok);
-            if (!ok) break;
+            ok = mbar_wait(bar_o + 8 * (c & 1u), (c >> 1) & 1, s_abort, p.status) && !*s_abort;
+            // the four warps go on together: they share the staging tile
+            __syncwarp();
+            asm volatile("{\n.reg .pred p, q;\nsetp.ne.b32 p, %1, 0;\nbarrier.red.and.pred.aligned q, 2, 128, p;\nselp.u32 %0, 1, 0, q;\n}\n"
+                         : "=r"(together)
+                         : "r"((uint32_t)ok)
+                         : "memory");
+            if (!together) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            float4* out = reinterpret_cast<float4*>(a.work + ((uint64_t)row * a.heads + h) * a.vdim + slice * RT_W);
             const float f = a.scale * power[i + 1];
-            uint32_t big[2][16], small[2][16], near[2][16];
+            const uint32_t turn = (c & 1u) * 64 + lanes;
 #pragma unroll
-            for (int y = 0; y < 2; ++y) {
-#pragma unroll
-                for (int x = 0; x < 2; ++x) {
-                    tmem_ld16_request(tmem_o1 + lanes + 32 * y + 16 * x, big[x]);
-                    tmem_ld16_request(tmem_o1 + lanes + 64 + 32 * y + 16 * x, small[x]);
-                    tmem_ld16_request(tmem_o2 + lanes + 32 * y + 16 * x, near[x]);
-                }
-                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-                for (int x = 0; x < 2; ++x) {
-                    tmem_ld16_pass(big[x]);
-                    tmem_ld16_pass(small[x]);
-                    tmem_ld16_pass(near[x]);
-                }
+            for (uint32_t y = 0; y < 2; ++y) {
+                uint32_t far[32], near[32];
+                tmem_ld32_request(tmem_o1 + turn + 32 * y, far);
+                tmem_ld32_request(tmem_o2 + turn + 32 * y, near);
+                tmem_ld32_wait(far);
+                tmem_ld32_pass(near);
                 if (y == 1) {
                     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
                     __syncwarp();
-                    if (lane == 0) mbar_arrive(bar_oread);
+                    if (lane == 0) mbar_arrive(bar_oread + 8 * (c & 1u));
                 }
-                if (row < count)
+                // the store before has read the staging tile
+                if (tid == 320) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
+                __syncwarp();
+                asm volatile("bar.sync 2, 128;" ::: "memory");
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) {
-                        float v[4];
+                for (uint32_t u = 0; u < 8; ++u) {
+                    float v[4];
 #pragma unroll
-                        for (int n = 0; n < 4; ++n) {
-                            const int at = (4 * e + n) & 15, x = e >> 2;
-                            v[n] = fmaf(f, __uint_as_float(big[x][at]) + __uint_as_float(small[x][at]), a.scale * __uint_as_float(near[x][at]));
-                        }
-                        out[8 * y + e] = make_float4(v[0], v[1], v[2], v[3]);
-                    }
+                    for (int n = 0; n < 4; ++n) v[n] = fmaf(f, __uint_as_float(far[4 * u + n]), a.scale * __uint_as_float(near[4 * u + n]));
+                    *reinterpret_cast<float4*>(sm + OFF_OUT + i * 128 + ((u ^ (i & 7u)) << 4)) = make_float4(v[0], v[1], v[2], v[3]);
+                }
+                fence_async_smem();
+                asm volatile("bar.sync 2, 128;" ::: "memory");
+                if (tid == 320) {
+                    asm volatile("cp.async.bulk.tensor.2d.global.shared::cta.tile.bulk_group [%0, {%1, %2}], [%3];" ::"l"(&map_work), "r"((int)(h * a.vdim + slice * RT_W + 32 * y)),
+                                 "r"((int)(c * 128)), "r"(base + OFF_OUT)
+                                 : "memory");
+                    asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+                }
+                __syncwarp();
             }
         }
+        if (tid == 320) asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
     }
     // everyone meets here, whatever happened above, so that TMEM is always released
     __syncwarp();
@@ -921,7 +926,7 @@ retention_finish_kernel(const HoloRetentionArgs a) {
 
 template <int DT>
 int32_t launch_tile_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
-    constexpr uint32_t smem = (DT == 1 ? 2 : 1) * 4 * DT * TILE_CHUNK + 5 * TILE_CHUNK + 1024 + 256 + 1024;
+    constexpr uint32_t smem = (DT == 1 ? 2 : 1) * 4 * DT * TILE_CHUNK + 6 * TILE_CHUNK + 1024 + 256 + 1024;
     static_assert(smem <= 227 * 1024, "retention tile");
     static thread_local int configured_device = -1;
     if (configured_device != ctx->device) {
@@ -932,10 +937,20 @@ int32_t launch_tile_as(holo_b200_ctx* ctx, const HoloRetentionArgs& a) {
     HOLO_TRY(make_map_rows(&mq, a.q, (uint64_t)a.heads * a.dim, a.rows, a.q_ld));
     HOLO_TRY(make_map_rows(&mk, a.k, (uint64_t)a.heads * a.dim, a.rows, a.k_ld));
     HOLO_TRY(make_map_rows(&mv, a.v, (uint64_t)a.heads * a.vdim, a.rows, a.v_ld));
+    CUtensorMap mw;
+    {   // stores of 32 f32 columns of 128 rows
+        cuuint64_t dims[2] = {(cuuint64_t)a.heads * a.vdim, a.rows};
+        cuuint64_t strides[1] = {(cuuint64_t)a.heads * a.vdim * 4};
+        cuuint32_t box[2] = {32, 128};
+        cuuint32_t es[2] = {1, 1};
+        const CUresult r = encode_tiled_fn()(&mw, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 2, a.work, dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+        if (r != CUDA_SUCCESS) return holo_fail(HOLO_ERR_DISPATCH, "dispatch failed: cuTensorMapEncodeTiled (retention) returned %d", (int)r);
+    }
     RetentionTileParams p;
     p.a = a;
     p.status = ctx->dev_status;
-    HOLO_CUDA(holo_launch_kernel(ctx, retention_tile_kernel<DT>, dim3(a.vdim / RT_W, a.heads), dim3(RT_THREADS), smem, 1, mq, mk, mv, p));
+    HOLO_CUDA(holo_launch_kernel(ctx, retention_tile_kernel<DT>, dim3(a.vdim / RT_W, a.heads), dim3(RT_THREADS), smem, 1, mq, mk, mv, mw, p));
     const dim3 grid((a.rows * a.heads + 7) / 8);
     if (a.vdim <= 128) HOLO_CUDA(holo_launch_kernel(ctx, retention_finish_kernel<1>, grid, dim3(256), 0, 1, a));
     else if (a.vdim <= 256) HOLO_CUDA(holo_launch_kernel(ctx, retention_finish_kernel<2>, grid, dim3(256), 0, 1, a));
