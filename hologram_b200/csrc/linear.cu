@@ -224,6 +224,12 @@ int32_t holo_launch_linear(holo_b200_ctx* ctx, const HoloLinearArgs& a) {
     // a group is weight streaming like one product as wide as all its tiles together
     if (a.tiles) tile_choice(ctx, a.tile_rows, a.n * gtiles, kblocks, &bn, &splits);
     else tile_choice(ctx, a.m, a.n, kblocks, &bn, &splits);
+    if (!a.tiles && mtiles > 1 && splits == 1) {      // many rows, few columns (a router): K slices fill the chip
+        const uint32_t tiles = mtiles * ((a.n + bn - 1) / bn);
+        splits = (uint32_t)ctx->sm_count / tiles;
+        if (splits > kblocks / 4) splits = kblocks / 4;
+        if (splits < 1) splits = 1;
+    }
     if (const char* e = getenv("HOLO_GEMM_BN")) bn = atoi(e) == 64 ? 64 : 128;
     if (const char* e = getenv("HOLO_GEMM_SPLITS")) splits = (uint32_t)atoi(e) > 0 ? (uint32_t)atoi(e) : 1;
     if (splits > kblocks) splits = kblocks;
