@@ -87,27 +87,6 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
         : "r"(taddr));
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
-// Three times 16 columns, one wait.
-__device__ __forceinline__ void tmem_ld16_request(uint32_t taddr, uint32_t (&v)[16]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
-        : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_ld16_pass(uint32_t (&v)[16]) {
-    asm volatile("" : "+r"(v[0]), "+r"(v[1]), "+r"(v[2]), "+r"(v[3]), "+r"(v[4]), "+r"(v[5]), "+r"(v[6]), "+r"(v[7]), "+r"(v[8]),
-                   "+r"(v[9]), "+r"(v[10]), "+r"(v[11]), "+r"(v[12]), "+r"(v[13]), "+r"(v[14]), "+r"(v[15])::"memory");
-}
-__device__ __forceinline__ void tmem_ld16x3(uint32_t t0, uint32_t t1, uint32_t t2, uint32_t (&v0)[16], uint32_t (&v1)[16], uint32_t (&v2)[16]) {
-    tmem_ld16_request(t0, v0);
-    tmem_ld16_request(t1, v1);
-    tmem_ld16_request(t2, v2);
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-    tmem_ld16_pass(v0);
-    tmem_ld16_pass(v1);
-    tmem_ld16_pass(v2);
-}
 // The two halves of tmem_ld32: request 32 columns; wait for everything requested (the values pass through the wait, so that
 // no use of them can be scheduled before it).
 __device__ __forceinline__ void tmem_ld32_request(uint32_t taddr, uint32_t (&v)[32]) {
